@@ -32,6 +32,9 @@ class RopeSpec:
     exact_table: bool = False      # the frequency table is formed in 64-bit and rounded once (else in 32-bit)
     scaling_factor: float = 1.0    # linear scaling: every frequency is divided by this number
     layout: str = "halves"         # pairs of the rotation: "halves" (i with i + dim/2) or "interleaved" (2i with 2i + 1)
+    # scaling by wavelength, (factor, low, high, original): a frequency whose wavelength is below original/high stays, one
+    # above original/low is divided by the factor, those between are a straight mixture of both
+    bands: Optional[tuple] = None
 
 
 @dataclass(frozen=True)
@@ -94,9 +97,14 @@ class GeneralAttentionSpec:
     # row count, the distance from which the last bucket serves); see parts.general_attention.distance_buckets
     distance_bias: Optional[tuple] = None
     sink: bool = False                      # exp(a learned number per head) counts once in the softmax's denominator
+    sink_score: Optional[float] = None      # the same with one fixed number for all heads (0: one is added)
+    # the heads' scaled scores mixed before the softmax: score_h <- sum_g T[h, g] score_g, T a tensor [heads, heads]
+    talk: bool = False
+    output_scale: float = 1.0               # multiplies every head before the output product
     # RMSNorm of every query and key head with ONE weight vector of the key size that all heads share (the norms'
     # names serve both kinds; a layer has the whole-projection norm or this one)
     head_norm_eps: Optional[float] = None
+    head_norm_weight: bool = True           # False: the heads' norm has no weight (a head divided by its root mean square)
     value_norm_eps: Optional[float] = None  # every value head divided by its root mean square (no weight); cached so
     # values rotated by their own position over their whole size (frequencies theta^(-2m/value_dim), never scaled, the
     # position encoding's theta and layout), cached so; every head's output turned back by the query's position
@@ -105,8 +113,8 @@ class GeneralAttentionSpec:
     chunk: Optional[int] = None             # a query sees the earlier positions of its chunk, chunks counted from 0
     prefix: str = "mix"
     # tensor names below the prefix: queries, keys, values, gate, output, whole-projection norms, score bias,
-    # temperature, distance bias, sink
-    names: tuple = ("q", "k", "v", "g", "o", "q.norm", "k.norm", "pb", "temp", "rel", "sink")
+    # temperature, distance bias, sink, score mixing
+    names: tuple = ("q", "k", "v", "g", "o", "q.norm", "k.norm", "pb", "temp", "rel", "sink", "talk")
     kind: str = "general_attention"
 
 
@@ -164,16 +172,32 @@ class MatrixMemorySpec:
 
 
 @dataclass(frozen=True)
+class MinGRUSpec:
+    """A gated recurrence whose gates read only the current token: z = sigmoid(W_z x + b_z), y = W_x x + b_x, candidate
+    y + 1/2 where y >= 0 and sigmoid(y) elsewhere; element by element S <- (1 - z) S + z * candidate; output
+    W_o (output_scale * S * silu(W_g x))."""
+    hidden_size: int
+    width: int                     # elements of the state
+    output_scale: float = 1.0
+    prefix: str = "mix"
+    # update gate and its bias, candidate and its bias, output gate, output product
+    names: tuple = ("z", "z.b", "x", "x.b", "g", "o")
+    kind: str = "min_gru"
+
+
+@dataclass(frozen=True)
 class MixerPairSpec:
-    """Two mixers that read the same input; the result is coef * (rms(left) * w_left + rms(right) * w_right) with a
-    plain RMSNorm over the model width on each output."""
+    """Two mixers that read the same input.  `combine` "norm_mean": the result is coef * (rms(left) * w_left +
+    rms(right) * w_right) with a plain RMSNorm over the model width on each output (weights `names`); "sum": the sum of
+    the two outputs (a factor on a side is that side's `output_scale`)."""
     hidden_size: int
     left: Any
     right: Any
-    eps: float
+    eps: float = 0.0
     coef: float = 0.5
     prefix: str = "mix"
     names: tuple = ("left.out", "right.out")
+    combine: str = "norm_mean"
     kind: str = "mixer_pair"
 
 
@@ -182,9 +206,12 @@ class DenseMLPSpec:
     """A feed-forward without a gate: down(act(up(x)))."""
     hidden_size: int
     intermediate_size: int
-    activation: str = "relu2"               # "relu2": relu(z)^2; "gelu": the exact (erf) gelu; "tanh"
+    # "relu2": relu(z)^2; "gelu": the exact (erf) gelu; "tanh"; "poly_norm": a N(z) + b N(z^2) + c N(z^3) + e with the four
+    # numbers of a tensor, powers element by element and N dividing a token's whole vector by its root mean square
+    activation: str = "relu2"
     prefix: str = "mlp"
-    names: tuple = ("up", "down")
+    names: tuple = ("up", "down", "act")    # the third: the numbers of "poly_norm"
+    norm_eps: float = 0.0                   # of N
     kind: str = "dense_mlp"
 
 
@@ -220,7 +247,8 @@ class LatentAttentionSpec:
 @dataclass(frozen=True)
 class RoutedExpertsSpec:
     """A mixture of small feed-forward experts down(act(up(x))): each token uses the `top_k` experts with the
-    largest router scores; with `n_groups` > 1 the experts form equal groups of neighbours, a group scores as
+    largest router scores, or those that a table names for its token id (`scoring` "table", each with the weight
+    1 / top_k); with `n_groups` > 1 the experts form equal groups of neighbours, a group scores as
     its best expert, and only experts of the `keep_groups` best groups can be chosen."""
     hidden_size: int
     num_experts: int
@@ -228,14 +256,17 @@ class RoutedExpertsSpec:
     expert_size: int
     n_groups: int = 1
     keep_groups: int = 1
-    scoring: str = "softmax"       # router scores: "softmax" over all experts, or "sigmoid" of each logit
+    scoring: str = "softmax"       # router scores: "softmax" over all experts, "sigmoid" of each logit, or "table": no
+                                   #   router, an integer tensor `table` [vocab_size, top_k] holds each token id's experts
     renormalize: bool = False      # whether the chosen scores are made to sum to one
     activation: str = "gelu"       # "gelu": down(gelu(up x)), exact (erf) gelu; "clamped_glu": experts with a gate
-                                   #   matrix, g = min(gate x, limit), u = clamp(up x, +-limit), down(g sigmoid(1.702 g) (u + 1))
+                                   #   matrix, g = min(gate x, limit), u = clamp(up x, +-limit), down(g sigmoid(1.702 g) (u + 1));
+                                   #   "swiglu": down(silu(gate x) * (up x))
     group_score: str = "max"       # a group's score: its best expert's ("max") or the sum of its two best ("top2_sum")
     renorm_eps: float = 0.0        # added to the chosen scores' sum before the division
     weight_scale: float = 1.0      # multiplies the weights at the end
     limit: float = 0.0             # of the clamped activation
+    vocab_size: int = 0            # rows of the table (scoring "table")
     prefix: str = "mlp"
     kind: str = "routed_experts"
 

@@ -3,7 +3,10 @@
 // the key size KD and the value size VD as compile-time constants of the LIBRARY (-DJV_KEY_DIM, -DJV_VALUE_DIM:
 // one library per pair of sizes that a model needs, built when it is first asked for), and with these options:
 //
-//   value heads    the value cache is [pages, page, n_v_heads, VD]; key head g reads value head g % n_v_heads
+//   value heads    the value cache is [pages, page, n_v_heads, VD]; group g of query heads reads value head g % n_v_heads
+//   key heads      the key cache is [pages, page, n_k_heads, KD]; group g reads key head g % n_k_heads (one key head under
+//                  several value heads: queries that already mix the heads of a wider key row, see talk_prepare.cu)
+//   output scale   the heads' outputs are multiplied by one number
 //   score cap      s <- cap * tanh(s / cap) on the scaled score
 //   sigmoid        the weight of a visible key is sigmoid(s + bias[query head]); no maximum, no sum, no division
 //   float output   two score maps are subtracted by the caller in 32-bit
@@ -54,7 +57,8 @@ struct Params {
   int n_dist;                  //   (distances of n_dist - 1 and more share the last column)
   const float* sink;           // [n_q_heads] or null (softmax only)
   int out_f32;                 // `out` is float
-  int n_v_heads;
+  int n_v_heads, n_k_heads;
+  float out_scale;
   int tokens_per_tile, heads_per_tile, n_head_groups, split_size, n_splits;
   int* status;
   int* counters;               // decode: one per (work item, kv head, head group), zero between launches
@@ -128,7 +132,7 @@ __device__ __forceinline__ void issue_tile(__nv_bfloat16* ks, __nv_bfloat16* vs,
   __nv_bfloat16* dst = is_v ? vs + n * Tile<VD>::STRIDE : ks + n * Tile<KD>::STRIDE;
   if (slot >= 0) {
     const __nv_bfloat16* src = is_v ? p.v_cache + (slot * p.n_v_heads + kv_head % p.n_v_heads) * VD
-                                    : p.k_cache + (slot * p.n_kv_heads + kv_head) * KD;
+                                    : p.k_cache + (slot * p.n_k_heads + kv_head % p.n_k_heads) * KD;
     mbar_expect_tx(bar, dim * 2);
     bulk_copy(dst, src, dim * 2, bar);
   } else {
@@ -423,6 +427,7 @@ __global__ void __launch_bounds__(THREADS) attn_prefill_general_kernel(const Par
       const float e = __expf(m[h] - mx);
       inv = e / (l[h] * e + __expf(sk - mx));
     }
+    inv *= p.out_scale;
 #pragma unroll
     for (int db = 0; db < VD / 8; ++db) {
       const int d = db * 8 + (lane & 3) * 2;
@@ -625,7 +630,7 @@ __global__ void __launch_bounds__(THREADS) attn_decode_general_kernel(const Para
       l_all += f * __ldcg(p.part_ml + (base + sp) * 2 + 1);
       o += f * __ldcg(p.part_o + (base + sp) * D + d);
     }
-    const float res = sigmoid ? o : o / l_all;
+    const float res = (sigmoid ? o : o / l_all) * p.out_scale;
     if (p.out_f32) ((float*)p.out)[(size_t)token * p.out_stride + (size_t)head * D + d] = res;
     else ((__nv_bfloat16*)p.out)[(size_t)token * p.out_stride + (size_t)head * D + d] = __float2bfloat16_rn(res);
   }
@@ -674,7 +679,7 @@ JV_EXPORT int jv_attn_general_tokens_per_tile(int n_q_heads, int n_kv_heads) {
 }
 
 // Arguments as for jv_attn_simt_ex (csrc/attn_simt.cu), bfloat16 only, for the key and value sizes of this library.
-// v_cache: [num_pages, page_size, n_v_heads, VD].  n_splits == 0: prompt portions, work = (entry, first token of the
+// k_cache: [num_pages, page_size, n_k_heads, KD], v_cache: [num_pages, page_size, n_v_heads, VD].  n_splits == 0: prompt portions, work = (entry, first token of the
 // tile).  n_splits > 0: single tokens, part_o [n_work*Hq*n_splits*VD] and part_ml [n_work*Hq*n_splits*2] floats of
 // scratch, and `counters`, n_work * n_kv_heads * ceil(G/16) ints that are zero before the launch (the kernel leaves
 // them zero).
@@ -684,11 +689,12 @@ JV_EXPORT int jv_attn_general_mma(const void* q, int q_stride, void* out, int ou
                                   const int* work, int n_work, int n_q_heads, int n_kv_heads, int n_v_heads, int key_dim,
                                   int value_dim, int page_size, int num_pages, int window, float scale, float score_cap,
                                   int sigmoid, const float* bias, const float* head_scale, const float* dist_bias,
-                                  int n_dist, const float* sink, int split_size, int n_splits, int* status,
-                                  cudaStream_t stream) {
+                                  int n_dist, const float* sink, int split_size, int n_splits, int n_k_heads,
+                                  float out_scale, int* status, cudaStream_t stream) {
   if (n_work == 0) return JV_OK;
   if ((dist_bias != nullptr && n_dist < 1) || (sink != nullptr && sigmoid)) return JV_ERR_UNSUPPORTED;
-  if (key_dim != KD || value_dim != VD || n_kv_heads < 1 || n_v_heads < 1 || n_q_heads % n_kv_heads != 0)
+  if (key_dim != KD || value_dim != VD || n_kv_heads < 1 || n_v_heads < 1 || n_k_heads < 1 ||
+      n_q_heads % n_kv_heads != 0)
     return JV_ERR_UNSUPPORTED;
   if ((q_stride % 8) || (out_stride % 2) || ((uintptr_t)q % 16) || ((uintptr_t)out % 8) || ((uintptr_t)k_cache % 16) ||
       ((uintptr_t)v_cache % 16))
@@ -703,6 +709,7 @@ JV_EXPORT int jv_attn_general_mma(const void* q, int q_stride, void* out, int ou
   p.num_pages = num_pages; p.window = window; p.scale = scale; p.score_cap = score_cap; p.sigmoid = sigmoid ? 1 : 0;
   p.bias = bias; p.status = status;
   p.head_scale = head_scale; p.dist_bias = dist_bias; p.n_dist = n_dist; p.sink = sink;
+  p.n_k_heads = n_k_heads; p.out_scale = out_scale;
   const int G = n_q_heads / n_kv_heads;
   p.heads_per_tile = G < 16 ? G : 16;
   p.n_head_groups = (G + p.heads_per_tile - 1) / p.heads_per_tile;

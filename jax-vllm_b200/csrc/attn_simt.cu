@@ -9,7 +9,8 @@
 // group: row m -> token q_off + m / heads_per_tile, head kv*G + hg*heads_per_tile +
 // m % heads_per_tile.  Keys run over the entry's block table; key j is visible to a
 // query at position p iff j <= p and (window == 0 or j > p - window).  Softmax is the
-// running (max, sum) form; scores, probabilities and the output sum are float.
+// running (max, sum) form; scores, probabilities and the output sum are float.  Key rows (and queries) longer than
+// `d_chunk` elements come through shared memory in pieces.
 //
 // SPLIT: split s covers key positions [s*split_size, (s+1)*split_size) of the visible
 // range; it writes its unnormalised output sum and (max, sum) to `part_o`/`part_ml`;
@@ -34,7 +35,10 @@ struct AttnParams {
   int n_q_heads, n_kv_heads, head_dim, v_dim, page_size, num_pages, window;
   float scale;
   int tokens_per_tile, heads_per_tile, n_head_groups, split_size, n_splits;
-  int n_v_heads, v_row;      // value heads (key head kv reads value head kv % n_v_heads) and elements of a cached value row
+  int n_v_heads, v_row;      // value heads (group kv reads value head kv % n_v_heads) and elements of a cached value row
+  int n_k_heads;             // key heads (group kv reads key head kv % n_k_heads)
+  int d_chunk;               // elements of the key rows that are in shared memory at a time
+  float out_scale;           // multiplies the heads' outputs
   float score_cap;           // > 0: score <- cap * tanh(score / cap), after the scale
   int sigmoid;               // 1: the weight of a visible key is sigmoid(score + bias[query head]), not normalised over keys
   const float* bias;         // [n_q_heads] or null
@@ -49,11 +53,11 @@ struct AttnParams {
 template <typename T, bool SPLIT>
 __global__ void __launch_bounds__(THREADS) attn_simt_kernel(const AttnParams p) {
   extern __shared__ float smem[];
-  const int D = p.head_dim;
+  const int D = p.head_dim, DCH = p.d_chunk;
   const int DV = p.v_dim;                          // leading elements of a value row that are used (<= v_row)
-  float* Qs = smem;                                // [BLOCK_M][D]
-  float* Ks = Qs + BLOCK_M * D;                    // [BLOCK_N][D+1]
-  float* Vs = Ks + BLOCK_N * (D + 1);              // [BLOCK_N][DV]
+  float* Qs = smem;                                // [BLOCK_M][DCH]
+  float* Ks = Qs + BLOCK_M * DCH;                  // [BLOCK_N][DCH+1]
+  float* Vs = Ks + BLOCK_N * (DCH + 1);            // [BLOCK_N][DV]
   float* Ss = Vs + BLOCK_N * DV;                   // [BLOCK_M][BLOCK_N]
   float* row_m = Ss + BLOCK_M * BLOCK_N;           // [BLOCK_M]
   float* row_l = row_m + BLOCK_M;                  // [BLOCK_M]
@@ -92,14 +96,17 @@ __global__ void __launch_bounds__(THREADS) attn_simt_kernel(const AttnParams p) 
     row_l[tid] = p.sigmoid ? 1.f : 0.f;
     row_alpha[tid] = 1.f;
   }
-  for (int idx = tid; idx < BLOCK_M * D; idx += THREADS) {
-    const int m = idx / D, d = idx - m * D;
-    const int t = m / p.heads_per_tile, hh = hg * p.heads_per_tile + m % p.heads_per_tile;
-    float v = 0.f;
-    if (t < tokens_here && hh < G)
-      v = to_f32(q[(size_t)(q_begin + q_off + t) * p.q_stride + (size_t)(kv_head * G + hh) * D + d]);
-    Qs[idx] = v;
-  }
+  auto load_q = [&](int d0, int dn) {                // elements [d0, d0 + dn) of the tile's queries
+    for (int idx = tid; idx < BLOCK_M * dn; idx += THREADS) {
+      const int m = idx / dn, d = idx - m * dn;
+      const int t = m / p.heads_per_tile, hh = hg * p.heads_per_tile + m % p.heads_per_tile;
+      float v = 0.f;
+      if (t < tokens_here && hh < G)
+        v = to_f32(q[(size_t)(q_begin + q_off + t) * p.q_stride + (size_t)(kv_head * G + hh) * D + d0 + d]);
+      Qs[m * DCH + d] = v;
+    }
+  };
+  if (D <= DCH) load_q(0, D);                        // whole rows fit: once for all keys
 
   constexpr int DC = 4;  // output columns per thread: d = tid, tid + THREADS, ...  (v_dim <= 512)
   float acc[BLOCK_M][DC];
@@ -110,37 +117,42 @@ __global__ void __launch_bounds__(THREADS) attn_simt_kernel(const AttnParams p) 
   __syncthreads();
 
   for (int j0 = j_lo; j0 < j_hi; j0 += BLOCK_N) {
-    // ---- keys and values of this chunk into shared memory (one warp per key row)
-    for (int n = warp; n < BLOCK_N; n += THREADS / 32) {
-      const int j = j0 + n;
-      const T* krow = nullptr;
-      const T* vrow = nullptr;
-      if (j < j_hi) {
-        const int pi = j / p.page_size;
-        const int page = pi < p.table_width ? p.block_table[(size_t)entry * p.table_width + pi] : -1;
-        if (page < 0 || page >= p.num_pages) {
-          if (lane == 0) atomicOr(p.status, JV_STATUS_BAD_PAGE);
-        } else {
-          const size_t slot = (size_t)page * p.page_size + (j % p.page_size);
-          krow = kc + (slot * p.n_kv_heads + kv_head) * D;
-          vrow = vc + (slot * p.n_v_heads + kv_head % p.n_v_heads) * p.v_row;
+    float s[4] = {0.f, 0.f, 0.f, 0.f};               // scores: thread (n = lane, rows warp*4 .. warp*4+3)
+    for (int d0 = 0; d0 < D; d0 += DCH) {
+      const int dn = min(DCH, D - d0);
+      if (d0 > 0) __syncthreads();                     // the piece before has been read
+      if (D > DCH) load_q(d0, dn);
+      // ---- keys and values of this chunk into shared memory (one warp per key row)
+      for (int n = warp; n < BLOCK_N; n += THREADS / 32) {
+        const int j = j0 + n;
+        const T* krow = nullptr;
+        const T* vrow = nullptr;
+        if (j < j_hi) {
+          const int pi = j / p.page_size;
+          const int page = pi < p.table_width ? p.block_table[(size_t)entry * p.table_width + pi] : -1;
+          if (page < 0 || page >= p.num_pages) {
+            if (lane == 0) atomicOr(p.status, JV_STATUS_BAD_PAGE);
+          } else {
+            const size_t slot = (size_t)page * p.page_size + (j % p.page_size);
+            krow = kc + (slot * p.n_k_heads + kv_head % p.n_k_heads) * D + d0;
+            vrow = vc + (slot * p.n_v_heads + kv_head % p.n_v_heads) * p.v_row;
+          }
         }
+        for (int d = lane; d < dn; d += 32) Ks[n * (DCH + 1) + d] = krow ? to_f32(krow[d]) : 0.f;
+        if (d0 == 0)
+          for (int d = lane; d < DV; d += 32) Vs[n * DV + d] = vrow ? to_f32(vrow[d]) : 0.f;
       }
-      for (int d = lane; d < D; d += 32) Ks[n * (D + 1) + d] = krow ? to_f32(krow[d]) : 0.f;
-      for (int d = lane; d < DV; d += 32) Vs[n * DV + d] = vrow ? to_f32(vrow[d]) : 0.f;
-    }
-    __syncthreads();
-
-    // ---- scores: thread (n = lane, rows warp*4 .. warp*4+3)
-    {
-      float s[4] = {0.f, 0.f, 0.f, 0.f};
-      const float* kr = Ks + lane * (D + 1);
-      const float* q0 = Qs + (warp * 4) * D;
-      for (int d = 0; d < D; ++d) {
+      __syncthreads();
+      const float* kr = Ks + lane * (DCH + 1);
+      const float* q0 = Qs + (warp * 4) * DCH;
+      for (int d = 0; d < dn; ++d) {
         const float kv = kr[d];
 #pragma unroll
-        for (int r = 0; r < 4; ++r) s[r] = fmaf(q0[r * D + d], kv, s[r]);
+        for (int r = 0; r < 4; ++r) s[r] = fmaf(q0[r * DCH + d], kv, s[r]);
       }
+    }
+
+    {
       const int j = j0 + lane;
 #pragma unroll
       for (int r = 0; r < 4; ++r) {
@@ -225,6 +237,7 @@ __global__ void __launch_bounds__(THREADS) attn_simt_kernel(const AttnParams p) 
           const float e = expf(row_m[m] - mx);
           o = acc[m][c] * e / (row_l[m] * e + expf(sk - mx));
         }
+        o *= p.out_scale;
         if (p.out_f32) ((float*)p.out)[token * p.out_stride + (size_t)head * DV + d] = o;
         else ((T*)p.out)[token * p.out_stride + (size_t)head * DV + d] = from_f32<T>(o);
       }
@@ -253,6 +266,7 @@ __global__ void attn_combine_kernel(const AttnParams p) {
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
       float o = 0.f;
       for (int s = s_first; s <= s_last; ++s) o += p.part_o[(base + s) * D + d];
+      o *= p.out_scale;
       if (p.out_f32) ((float*)p.out)[tok * p.out_stride + (size_t)head * D + d] = o;
       else ((T*)p.out)[tok * p.out_stride + (size_t)head * D + d] = from_f32<T>(o);
     }
@@ -268,8 +282,9 @@ __global__ void attn_combine_kernel(const AttnParams p) {
     float o = 0.f;
     for (int s = s_first; s <= s_last; ++s)
       o += expf(p.part_ml[(base + s) * 2] - m_all) * p.part_o[(base + s) * D + d];
-    if (p.out_f32) ((float*)p.out)[token * p.out_stride + (size_t)head * D + d] = o / l_all;
-    else ((T*)p.out)[token * p.out_stride + (size_t)head * D + d] = from_f32<T>(o / l_all);
+    const float r = o / l_all * p.out_scale;
+    if (p.out_f32) ((float*)p.out)[token * p.out_stride + (size_t)head * D + d] = r;
+    else ((T*)p.out)[token * p.out_stride + (size_t)head * D + d] = from_f32<T>(r);
   }
 }
 
@@ -293,7 +308,8 @@ JV_EXPORT int jv_attn_simt_tokens_per_tile(int n_q_heads, int n_kv_heads) {
 // v_dim: how many leading elements of a value row are used (0: all head_dim); out and part_o then have v_dim
 // elements per head.  A cache whose values are the leading part of its keys passes the same tensor twice.
 // jv_attn_simt_ex: keys and values of different sizes and head counts, capped scores, sigmoid weights, float output
-// a temperature per head, a bias by distance, a sink in the softmax's denominator
+// a temperature per head, a bias by distance, a sink in the softmax's denominator, fewer key heads than groups, an output
+// scale
 // (see AttnParams); jv_attn_simt is the plain softmax form with values shaped like the keys.
 // n_splits == 0: every work item attends to its whole visible range and writes `out`.
 // n_splits > 0: work items are single tokens; part_o [n_work*Hq*n_splits*D] and part_ml
@@ -305,19 +321,22 @@ JV_EXPORT int jv_attn_simt_ex(const void* q, int q_stride, void* out, int out_st
                               int n_kv_heads, int head_dim, int page_size, int num_pages, int window,
                               float scale, int split_size, int n_splits, int v_dim, int n_v_heads, int v_row,
                               float score_cap, int sigmoid, const float* bias, int out_f32, const float* head_scale,
-                              const float* dist_bias, int n_dist, const float* sink, int* status,
-                              cudaStream_t stream) {
+                              const float* dist_bias, int n_dist, const float* sink, int n_k_heads, float out_scale,
+                              int* status, cudaStream_t stream) {
   if (n_work == 0) return JV_OK;
   if ((dist_bias != nullptr && n_dist < 1) || (sink != nullptr && sigmoid)) return JV_ERR_UNSUPPORTED;
   if (v_row <= 0) v_row = head_dim;
   if (n_v_heads <= 0) n_v_heads = n_kv_heads;
   if (v_dim <= 0) v_dim = v_row;
-  if (head_dim < 1 || v_dim > v_row || v_dim > 512 || smem_bytes(head_dim, v_dim) > 227 * 1024 || n_kv_heads < 1 ||
+  if (n_k_heads <= 0) n_k_heads = n_kv_heads;
+  // whole key rows where they fit in shared memory beside the values, else pieces of 256 elements
+  const int d_chunk = smem_bytes(head_dim, v_dim) <= 200 * 1024 ? head_dim : 256;
+  if (head_dim < 1 || v_dim > v_row || v_dim > 512 || smem_bytes(d_chunk, v_dim) > 227 * 1024 || n_kv_heads < 1 ||
       n_q_heads % n_kv_heads != 0)
     return JV_ERR_UNSUPPORTED;
   AttnParams p;
   p.n_v_heads = n_v_heads; p.v_row = v_row; p.score_cap = score_cap; p.sigmoid = sigmoid ? 1 : 0; p.bias = bias;
-  p.out_f32 = out_f32 ? 1 : 0;
+  p.out_f32 = out_f32 ? 1 : 0; p.n_k_heads = n_k_heads; p.d_chunk = d_chunk; p.out_scale = out_scale;
   p.head_scale = head_scale; p.dist_bias = dist_bias; p.n_dist = n_dist; p.sink = sink;
   p.q = q; p.q_stride = q_stride; p.out = out; p.out_stride = out_stride;
   p.part_o = part_o; p.part_ml = part_ml; p.k_cache = k_cache; p.v_cache = v_cache;
@@ -331,7 +350,7 @@ JV_EXPORT int jv_attn_simt_ex(const void* q, int q_stride, void* out, int out_st
   p.n_head_groups = (G + p.heads_per_tile - 1) / p.heads_per_tile;
   p.split_size = split_size > 0 ? split_size : 1;
   p.n_splits = n_splits;
-  const size_t smem = smem_bytes(head_dim, v_dim);
+  const size_t smem = smem_bytes(d_chunk, v_dim);
   dim3 grid(n_work, n_kv_heads * p.n_head_groups, n_splits > 0 ? n_splits : 1);
   int rc = JV_OK;
   JV_DISPATCH_DTYPE(dtype, T, {
@@ -375,5 +394,5 @@ JV_EXPORT int jv_attn_simt(const void* q, int q_stride, void* out, int out_strid
   return jv_attn_simt_ex(q, q_stride, out, out_stride, dtype, part_o, part_ml, k_cache, v_cache, block_table,
                          table_width, cu_seqlens, start_pos, work, n_work, n_q_heads, n_kv_heads, head_dim, page_size,
                          num_pages, window, scale, split_size, n_splits, v_dim, n_kv_heads, head_dim, 0.f, 0, nullptr,
-                         0, nullptr, nullptr, 0, nullptr, status, stream);
+                         0, nullptr, nullptr, 0, nullptr, n_kv_heads, 1.f, status, stream);
 }

@@ -3,7 +3,7 @@
 // v_off; element offsets).  Every step is optional and all arithmetic is 32-bit (sums of squares, angles, cosines,
 // sines):
 //
-//   queries, keys   u <- u * rsqrt(mean(u^2) + eps) * weight[D]          one weight vector shared by all heads
+//   queries, keys   u <- u * rsqrt(mean(u^2) + eps) * weight[D]          one weight vector shared by all heads (or none)
 //                   rotation of the first rot_dim elements of the head by position * freq[j]; the rest passes
 //   values          v <- v * rsqrt(mean(v^2) + eps)                      no weight
 //                   rotation of the first v_rot_dim elements by position * v_freq[j]: a value that carries its own
@@ -30,7 +30,7 @@ struct HeadPrepareParams {
   const float* v_freq; int v_rot_dim;
   int interleaved;
   const void* q_norm_w; const void* k_norm_w; float eps;
-  int v_norm;
+  int v_norm, qk_unit;               // values, and queries and keys without a weight, divided by their root mean square
   void* k_cache; void* v_cache;
   int n, n_q_heads, n_k_heads, n_v_heads, key_dim, value_dim, page_size, num_pages;
   int* status;
@@ -81,8 +81,8 @@ __global__ void __launch_bounds__(32 * WARPS) head_prepare_kernel(const HeadPrep
   const T* row = (const T*)p.proj + (size_t)t * p.row_stride;
   if (h < p.n_q_heads) {
     prepare_head<T, TW>(row + p.q_off + (size_t)h * p.key_dim, (T*)p.q_out + ((size_t)t * p.n_q_heads + h) * p.key_dim,
-                        p.key_dim, p.q_norm_w != nullptr, (const TW*)p.q_norm_w, p.eps, p.freq, p.rot_dim, p.interleaved,
-                        pos, lane);
+                        p.key_dim, p.q_norm_w != nullptr || p.qk_unit != 0, (const TW*)p.q_norm_w, p.eps, p.freq, p.rot_dim,
+                        p.interleaved, pos, lane);
     return;
   }
   h -= p.n_q_heads;
@@ -96,8 +96,8 @@ __global__ void __launch_bounds__(32 * WARPS) head_prepare_kernel(const HeadPrep
   const size_t slot = (size_t)page * p.page_size + (posi - page_idx * p.page_size);
   if (h < p.n_k_heads) {
     prepare_head<T, TW>(row + p.k_off + (size_t)h * p.key_dim, (T*)p.k_cache + (slot * p.n_k_heads + h) * p.key_dim,
-                        p.key_dim, p.k_norm_w != nullptr, (const TW*)p.k_norm_w, p.eps, p.freq, p.rot_dim, p.interleaved,
-                        pos, lane);
+                        p.key_dim, p.k_norm_w != nullptr || p.qk_unit != 0, (const TW*)p.k_norm_w, p.eps, p.freq, p.rot_dim,
+                        p.interleaved, pos, lane);
     return;
   }
   h -= p.n_k_heads;
@@ -153,12 +153,13 @@ __global__ void __launch_bounds__(128) rms_rows_kernel(const T* __restrict__ in,
 
 // proj: [n, row_stride] of `dtype`; q_out: [n, n_q_heads*key_dim] of `dtype`; q_norm_w, k_norm_w: [key_dim] of
 // `w_dtype` or null; freq: [rot_dim/2] float or null (rot_dim 0); v_freq: [v_rot_dim/2] or null; v_norm: values
-// are unit-normed (no weight); caches as for jv_attn_prepare, both null: queries only.
+// are unit-normed (no weight); qk_unit: so are queries and keys where they have no weight; caches as for
+// jv_attn_prepare, both null: queries only.
 JV_EXPORT int jv_head_prepare(const void* proj, int dtype, long long row_stride, int q_off, int k_off, int v_off,
                               void* q_out, const int* positions, const int* token_entry, const int* block_table,
                               int table_width, const float* freq, int rot_dim, const float* v_freq, int v_rot_dim,
                               int interleaved, const void* q_norm_w, const void* k_norm_w, int w_dtype, float eps,
-                              int v_norm, void* k_cache, void* v_cache, int n, int n_q_heads, int n_k_heads,
+                              int v_norm, int qk_unit, void* k_cache, void* v_cache, int n, int n_q_heads, int n_k_heads,
                               int n_v_heads, int key_dim, int value_dim, int page_size, int num_pages, int* status,
                               cudaStream_t stream) {
   if (n == 0) return JV_OK;
@@ -170,8 +171,8 @@ JV_EXPORT int jv_head_prepare(const void* proj, int dtype, long long row_stride,
   p.proj = proj; p.row_stride = row_stride; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.q_out = q_out;
   p.positions = positions; p.token_entry = token_entry; p.block_table = block_table; p.table_width = table_width;
   p.freq = freq; p.rot_dim = rot_dim; p.v_freq = v_freq; p.v_rot_dim = v_rot_dim; p.interleaved = interleaved ? 1 : 0;
-  p.q_norm_w = q_norm_w; p.k_norm_w = k_norm_w; p.eps = eps; p.v_norm = v_norm ? 1 : 0; p.k_cache = k_cache;
-  p.v_cache = v_cache; p.n = n; p.n_q_heads = n_q_heads; p.n_k_heads = n_k_heads; p.n_v_heads = n_v_heads;
+  p.q_norm_w = q_norm_w; p.k_norm_w = k_norm_w; p.eps = eps; p.v_norm = v_norm ? 1 : 0; p.qk_unit = qk_unit ? 1 : 0;
+  p.k_cache = k_cache; p.v_cache = v_cache; p.n = n; p.n_q_heads = n_q_heads; p.n_k_heads = n_k_heads; p.n_v_heads = n_v_heads;
   p.key_dim = key_dim; p.value_dim = value_dim; p.page_size = page_size; p.num_pages = num_pages; p.status = status;
   const long long items = (long long)n * (n_q_heads + (k_cache != nullptr ? n_k_heads + n_v_heads : 0));
   const dim3 grid((unsigned)((items + WARPS - 1) / WARPS));

@@ -1,0 +1,163 @@
+// A gated recurrence whose gates read only the current token ("minimal GRU"), element by element over C channels:
+//
+//   z = sigmoid(zl + zb),  y = yl + yb,  candidate = y + 1/2 where y >= 0, sigmoid(y) elsewhere
+//   S <- (1 - z) S + z * candidate,      out = scale * S * silu(g)
+//
+// zl, yl and g are column ranges of the packed projection; everything from them on is 32-bit, the state is a row of
+// floats in the request's state slot.  Since the gates do not read the state, a run of tokens is one affine map of it:
+// S -> A S + B with A the product of the (1 - z) and B what the run makes of a zero state.  A block takes CB channels of
+// one entry in tiles of tokens: every thread reads TPT tokens of one channel (the loads of the next tile fly while this
+// one is computed), forms their (a, b) pairs in registers and the pair (A, B) of its run, the runs of a tile are chained
+// through shared memory from the state that the tile before left, and every thread goes through its tokens again from
+// its true start.  One pass over memory, one launch; the order of the sums differs from token by token by 32-bit
+// rounding only.  A step of single tokens is a flat kernel, one thread a channel.
+#include "common.cuh"
+#include <math.h>
+
+namespace {
+constexpr int TPT = 8;            // tokens of a thread per tile
+constexpr int THREADS = 1024;
+
+struct GruParams {
+  const void* proj; long long stride; int z_off, x_off, g_off;
+  const void* z_bias; const void* x_bias;
+  void* out; long long out_stride;
+  float* state; long long slot_stride;
+  const int* cu_seqlens; const int* slots;
+  int n_slots, channels;
+  float scale;
+  int* status;
+};
+
+// EXACT (32-bit projections): library exponentials and divisions; else the short forms, whose error is far below the
+// 16-bit rounding of what they are given.
+template <bool EXACT> __device__ __forceinline__ float exp_of(float x) { return EXACT ? expf(x) : __expf(x); }
+template <bool EXACT> __device__ __forceinline__ float recip(float x) { return EXACT ? 1.f / x : __fdividef(1.f, x); }
+
+// (a, b) of one token: S <- a S + b.
+template <bool EXACT>
+__device__ __forceinline__ void gru_pair(float zl, float y, float& a, float& b) {
+  const float e = exp_of<EXACT>(fminf(zl, 80.f));          // e^zl, kept finite
+  a = recip<EXACT>(1.f + e);                               // 1 - z
+  const float c = y >= 0.f ? y + 0.5f : recip<EXACT>(1.f + exp_of<EXACT>(fminf(-y, 80.f)));
+  b = e * a * c;                                           // z * candidate
+}
+template <bool EXACT>
+__device__ __forceinline__ float silu_of(float g) { return g * recip<EXACT>(1.f + exp_of<EXACT>(fminf(-g, 80.f))); }
+
+// CB channels a block, THREADS / CB runs of TPT tokens a tile.
+template <typename T, typename W, int CB>
+__global__ void __launch_bounds__(THREADS, 1) gru_scan_kernel(const GruParams p) {
+  constexpr int RUNS = THREADS / CB, TILE = RUNS * TPT;
+  constexpr bool EXACT = sizeof(T) == 4;
+  __shared__ float As[RUNS][CB], Bs[RUNS][CB];
+  __shared__ float carry[2][CB];
+  pdl_trigger();
+  const int cl = threadIdx.x % CB, run = threadIdx.x / CB;
+  const int c = blockIdx.y * CB + cl;
+  const bool live = c < p.channels;
+  const float zb = live ? to_f32(((const W*)p.z_bias)[c]) : 0.f, xb = live ? to_f32(((const W*)p.x_bias)[c]) : 0.f;
+  pdl_wait();
+  const int entry = blockIdx.x;
+  const int t0 = p.cu_seqlens[entry], t1 = p.cu_seqlens[entry + 1];
+  const int slot = p.slots[entry];
+  if (slot < 0 || slot >= p.n_slots) {
+    if (threadIdx.x == 0) atomicOr(p.status, JV_STATUS_BAD_ROW);
+    return;
+  }
+  float* S_g = p.state + (size_t)slot * p.slot_stride + c;
+  if (run == 0) carry[0][cl] = live ? *S_g : 0.f;
+  const T* zp = (const T*)p.proj + p.z_off + c;
+  const T* xp = (const T*)p.proj + p.x_off + c;
+  const T* gp = (const T*)p.proj + p.g_off + c;
+  T zr[TPT], xr[TPT], gr[TPT];
+  auto fetch = [&](int tile0) {
+#pragma unroll
+    for (int i = 0; i < TPT; ++i) {
+      const int t = tile0 + run * TPT + i;
+      if (live && t < t1) {
+        const size_t at = (size_t)t * p.stride;
+        zr[i] = zp[at]; xr[i] = xp[at]; gr[i] = gp[at];
+      } else {
+        zr[i] = xr[i] = gr[i] = from_f32<T>(0.f);
+      }
+    }
+  };
+  fetch(t0);
+  int which = 0;
+  for (int tile0 = t0; tile0 < t1; tile0 += TILE, which ^= 1) {
+    float a[TPT], b[TPT], g[TPT];
+    float A = 1.f, B = 0.f;
+#pragma unroll
+    for (int i = 0; i < TPT; ++i) {
+      gru_pair<EXACT>(to_f32(zr[i]) + zb, to_f32(xr[i]) + xb, a[i], b[i]);
+      g[i] = to_f32(gr[i]);
+      if (tile0 + run * TPT + i >= t1) { a[i] = 1.f; b[i] = 0.f; }      // no token: the state passes
+      A *= a[i];
+      B = fmaf(a[i], B, b[i]);
+    }
+    if (tile0 + TILE < t1) fetch(tile0 + TILE);
+    As[run][cl] = A;
+    Bs[run][cl] = B;
+    __syncthreads();
+    float S = carry[which][cl];
+    for (int r = 0; r < run; ++r) S = fmaf(As[r][cl], S, Bs[r][cl]);
+    if (run == RUNS - 1) carry[which ^ 1][cl] = fmaf(A, S, B);
+#pragma unroll
+    for (int i = 0; i < TPT; ++i) {
+      const int t = tile0 + run * TPT + i;
+      S = fmaf(a[i], S, b[i]);
+      if (live && t < t1) ((T*)p.out)[(size_t)t * p.out_stride + c] = from_f32<T>(p.scale * S * silu_of<EXACT>(g[i]));
+    }
+    __syncthreads();                                       // the runs' pairs have been read; the carry is there
+  }
+  if (run == 0 && live && t1 > t0) *S_g = carry[which][cl];
+}
+
+template <typename T, typename W>
+__global__ void __launch_bounds__(128) gru_single_kernel(const GruParams p) {
+  constexpr bool EXACT = sizeof(T) == 4;
+  pdl_trigger();
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= p.channels) return;
+  const float zb = to_f32(((const W*)p.z_bias)[c]), xb = to_f32(((const W*)p.x_bias)[c]);
+  pdl_wait();
+  const int t = p.cu_seqlens[blockIdx.x];
+  const int slot = p.slots[blockIdx.x];
+  if (slot < 0 || slot >= p.n_slots) {
+    if (threadIdx.x == 0) atomicOr(p.status, JV_STATUS_BAD_ROW);
+    return;
+  }
+  const T* row = (const T*)p.proj + (size_t)t * p.stride;
+  float* S_g = p.state + (size_t)slot * p.slot_stride + c;
+  const float zl = to_f32(row[p.z_off + c]), y = to_f32(row[p.x_off + c]), g = to_f32(row[p.g_off + c]), S0 = *S_g;
+  float a, b;
+  gru_pair<EXACT>(zl + zb, y + xb, a, b);
+  const float S = fmaf(a, S0, b);
+  *S_g = S;
+  ((T*)p.out)[(size_t)t * p.out_stride + c] = from_f32<T>(p.scale * S * silu_of<EXACT>(g));
+}
+}  // namespace
+
+// proj: rows of `stride` elements of `dtype` with the three pre-activations (C columns each) at the given columns;
+// z_bias, x_bias: [C] of `w_dtype`; out: rows of `out_stride` elements of `dtype`; state: row of slot 0, rows
+// `slot_stride` floats apart.  singles != 0: every entry has exactly one token.
+JV_EXPORT int jv_min_gru(const void* proj, int dtype, long long stride, int z_off, int x_off, int g_off, const void* z_bias,
+                         const void* x_bias, int w_dtype, void* out, long long out_stride, float* state,
+                         long long slot_stride, const int* cu_seqlens, const int* slots, int n_slots, int entries,
+                         int channels, float scale, int singles, int* status, cudaStream_t stream) {
+  if (entries == 0 || channels == 0) return JV_OK;
+  GruParams p;
+  p.proj = proj; p.stride = stride; p.z_off = z_off; p.x_off = x_off; p.g_off = g_off; p.z_bias = z_bias; p.x_bias = x_bias;
+  p.out = out; p.out_stride = out_stride; p.state = state; p.slot_stride = slot_stride; p.cu_seqlens = cu_seqlens;
+  p.slots = slots; p.n_slots = n_slots; p.channels = channels; p.scale = scale; p.status = status;
+  JV_DISPATCH_DTYPE(dtype, T, JV_DISPATCH_DTYPE(w_dtype, W, {
+    if (singles)
+      return jv_launch(gru_single_kernel<T, W>, dim3(entries, (channels + 127) / 128), dim3(128), 0, stream, p);
+    // half a warp's worth of channels a block where whole warps would leave multiprocessors without a block
+    if ((long long)entries * ((channels + 31) / 32) < 120)
+      return jv_launch(gru_scan_kernel<T, W, 16>, dim3(entries, (channels + 15) / 16), dim3(THREADS), 0, stream, p);
+    return jv_launch(gru_scan_kernel<T, W, 32>, dim3(entries, (channels + 31) / 32), dim3(THREADS), 0, stream, p);
+  }));
+  return JV_ERR_UNSUPPORTED;
+}

@@ -6,6 +6,9 @@
 // `keep` best groups stay; the `top` largest s among those are chosen, largest first (lowest index on a tie);
 // weight = s (divided by the chosen scores' sum plus `renorm_eps` if `renorm`), times `weight_scale`.
 //
+// jv_moe_route_table: no router: row token_ids[t] of an integer table [vocab, top] names the experts of token t, each with
+// the weight 1/top.
+//
 // jv_moe_align, one block: puts the (token, choice) pairs in the order of their experts, every expert's run
 // padded to a multiple of `tile` rows so that a row tile of the grouped products belongs to one expert:
 //   sorted_token[pos] = token (-1: padding), pos_of[token*top + k] = pos, tile_expert[tile] = expert (-1: unused),
@@ -104,6 +107,23 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(
   }
 }
 
+__global__ void __launch_bounds__(128) moe_route_table_kernel(const int* __restrict__ tokens, const int* __restrict__ table,
+                                                              int vocab, int experts, int top, int pairs,
+                                                              int* __restrict__ ids, float* __restrict__ weights,
+                                                              int* __restrict__ status) {
+  pdl_trigger();
+  pdl_wait();
+  const int i = blockIdx.x * 128 + threadIdx.x;
+  if (i >= pairs) return;
+  const int t = i / top, tok = tokens[t];
+  int e = 0;
+  if (tok < 0 || tok >= vocab) atomicOr(status, JV_STATUS_BAD_TOKEN);
+  else e = table[(size_t)tok * top + (i - t * top)];
+  if (e < 0 || e >= experts) { atomicOr(status, JV_STATUS_BAD_ROW); e = 0; }
+  ids[i] = e;
+  weights[i] = 1.f / (float)top;
+}
+
 __global__ void __launch_bounds__(1024) moe_align_kernel(const int* __restrict__ ids, int pairs, int top, int experts,
                                                          int tile, int max_tiles, int* __restrict__ sorted_token,
                                                          int* __restrict__ pos_of, int* __restrict__ tile_expert,
@@ -186,6 +206,16 @@ JV_EXPORT int jv_moe_route(const float* z, int z_stride, int n, int experts, int
   const int blocks = (n + ROUTE_WARPS - 1) / ROUTE_WARPS;
   return jv_launch(moe_route_kernel, dim3(blocks), dim3(ROUTE_WARPS * 32), smem, stream, z, z_stride, n, experts, top,
                    groups, keep, renorm, scoring, group_mode, renorm_eps, weight_scale, ids, weights);
+}
+
+// tokens: [n] ids; table: [vocab, top]; ids: [n, top] int32; weights: [n, top] float.
+JV_EXPORT int jv_moe_route_table(const int* tokens, const int* table, int vocab, int experts, int top, int n, int* ids,
+                                 float* weights, int* status, cudaStream_t stream) {
+  if (n == 0) return JV_OK;
+  if (experts < 1 || top < 1 || top > experts) return JV_ERR_UNSUPPORTED;
+  const int pairs = n * top;
+  return jv_launch(moe_route_table_kernel, dim3((pairs + 127) / 128), dim3(128), 0, stream, tokens, table, vocab, experts,
+                   top, pairs, ids, weights, status);
 }
 
 // ids: [pairs] experts of the (token, choice) pairs, pairs = n * top; sorted_token: [max_tiles * tile];

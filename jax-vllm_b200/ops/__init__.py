@@ -400,7 +400,7 @@ def attn_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.
               n_work: int, n_q_heads: int, n_kv_heads: int, head_dim: int, window: int, scale: float,
               split_size: int = 0, n_splits: int = 0, v_dim: int = 0, score_cap: float = 0.0, sigmoid: bool = False,
               bias: torch.Tensor | None = None, head_scale: torch.Tensor | None = None,
-              dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None) -> None:
+              dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None, out_scale: float = 1.0) -> None:
     """Paged causal attention on CUDA cores (csrc/attn_simt.cu).  `work` is [n_work, 2] int32
     (entry, first token of the tile); with `n_splits` > 0 the work items are single tokens
     whose keys are split into `n_splits` ranges of `split_size` positions.  `v_dim` > 0: only that many
@@ -408,7 +408,8 @@ def attn_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.
     the leading part of its keys is passed as both caches).
 
     The value cache may have other heads and another row size than the key cache ([pages, page, value heads,
-    value size]): key head g then reads value head g % value heads.  `score_cap` > 0 caps the scaled scores by
+    value size]): group g of query heads (n_kv_heads groups) then reads value head g % value heads, and key head g % key
+    heads of the key cache.  `out_scale` multiplies the heads' outputs.  `score_cap` > 0 caps the scaled scores by
     cap * tanh(score / cap); `sigmoid` replaces the softmax by independent weights sigmoid(score + bias[query
     head]); `out` may be float32 whatever the type of q.  `head_scale` [query heads] multiplies the scaled scores of
     its head; `dist_bias` [query heads, distances] is added to the score of a key that lies so many positions back
@@ -421,7 +422,7 @@ def attn_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.
     if out.dtype not in (q.dtype, torch.float32) or out.stride(1) != 1:
         raise KernelError("attn_simt: out must have the type of q or float32, and unit column stride")
     if k_cache.dim() != 4 or v_cache.dim() != 4 or k_cache.shape[:2] != v_cache.shape[:2] or \
-            k_cache.shape[2:] != (n_kv_heads, head_dim) or n_kv_heads % v_cache.shape[2]:
+            k_cache.shape[3] != head_dim or n_kv_heads % k_cache.shape[2] or n_kv_heads % v_cache.shape[2]:
         raise KernelError(f"attn_simt: caches {tuple(k_cache.shape)} / {tuple(v_cache.shape)} do not fit "
                           f"{n_kv_heads} key heads of {head_dim}")
     n_v_heads, v_row = v_cache.shape[2], v_cache.shape[3]
@@ -442,13 +443,13 @@ def attn_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.
                                              c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                              c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int,
                                              c_int, c_float, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
-                                             c_void_p, c_void_p, c_void_p])
+                                             c_void_p, c_int, c_float, c_void_p, c_void_p])
     _check(f(q.data_ptr(), q_stride, out.data_ptr(), out.stride(0), _code(q, "q"), _ptr(part_o), _ptr(part_ml),
              k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), block_table.shape[1],
              cu_seqlens.data_ptr(), start_pos.data_ptr(), work.data_ptr(), n_work, n_q_heads, n_kv_heads, head_dim,
              k_cache.shape[1], k_cache.shape[0], int(window), float(scale), int(split_size), int(n_splits), v_dim,
              n_v_heads, v_row, float(score_cap), 1 if sigmoid else 0, _ptr(bias), 1 if out.dtype != q.dtype else 0,
-             _ptr(head_scale), _ptr(dist_bias), n_dist, _ptr(sink),
+             _ptr(head_scale), _ptr(dist_bias), n_dist, _ptr(sink), k_cache.shape[2], float(out_scale),
              _status_ptr(q.device), _stream()), "attn_simt", launches=2 if n_splits > 0 else 1)
 
 
@@ -491,9 +492,9 @@ def attn_general_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache:
                      n_work: int, n_q_heads: int, n_kv_heads: int, scale: float, split_size: int = 0, n_splits: int = 0,
                      score_cap: float = 0.0, sigmoid: bool = False, bias: torch.Tensor | None = None,
                      head_scale: torch.Tensor | None = None, dist_bias: torch.Tensor | None = None,
-                     sink: torch.Tensor | None = None, window: int = 0) -> None:
-    """Paged causal attention on the tensor cores with the options of `attn_simt`: the key size is the key
-    cache's row, the value size and the value heads the value cache's; bfloat16 in, bfloat16 or float32 out.
+                     sink: torch.Tensor | None = None, window: int = 0, out_scale: float = 1.0) -> None:
+    """Paged causal attention on the tensor cores with the options of `attn_simt`: the key size and the key heads are the
+    key cache's, the value size and the value heads the value cache's; bfloat16 in, bfloat16 or float32 out.
     `window`: the mask as one number (`mask_code`)."""
     n_dist = _score_extras("attn_general_mma", n_q_heads, head_scale, dist_bias, sink)
     for t, nm in ((q, "q"), (k_cache, "k_cache"), (v_cache, "v_cache")):
@@ -506,7 +507,7 @@ def attn_general_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache:
     if out.dtype not in (torch.bfloat16, torch.float32) or out.stride(1) != 1:
         raise KernelError("attn_general_mma: out must be bfloat16 or float32 with unit column stride")
     if k_cache.dim() != 4 or v_cache.dim() != 4 or k_cache.shape[:2] != v_cache.shape[:2] or \
-            k_cache.shape[2] != n_kv_heads or n_kv_heads % v_cache.shape[2]:
+            n_kv_heads % k_cache.shape[2] or n_kv_heads % v_cache.shape[2]:
         raise KernelError(f"attn_general_mma: caches {tuple(k_cache.shape)} / {tuple(v_cache.shape)} do not fit")
     key_dim, n_v_heads, value_dim = k_cache.shape[3], v_cache.shape[2], v_cache.shape[3]
     if bias is not None:
@@ -521,13 +522,14 @@ def attn_general_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache:
     f = _fn(attn_general_mma_library(key_dim, value_dim), "jv_attn_general_mma",
             [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-             c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p])
+             c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
     _check(f(q.data_ptr(), q_stride, out.data_ptr(), out.stride(0), 1 if out.dtype == torch.float32 else 0, _ptr(part_o),
              _ptr(part_ml), _ptr(counters), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(),
              block_table.shape[1], cu_seqlens.data_ptr(), start_pos.data_ptr(), work.data_ptr(), n_work, n_q_heads,
              n_kv_heads, n_v_heads, key_dim, value_dim, k_cache.shape[1], k_cache.shape[0], int(window), float(scale),
              float(score_cap), 1 if sigmoid else 0, _ptr(bias), _ptr(head_scale), _ptr(dist_bias), n_dist, _ptr(sink),
-             int(split_size), int(n_splits), _status_ptr(q.device), _stream()), "attn_general_mma")
+             int(split_size), int(n_splits), k_cache.shape[2], float(out_scale), _status_ptr(q.device), _stream()),
+           "attn_general_mma")
 
 
 def attn_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.Tensor, positions: torch.Tensor,
@@ -1245,6 +1247,20 @@ def moe_align(ids: torch.Tensor, experts: int, tile: int):
     return sorted_token, pos_of, tile_expert[:max_tiles], tile_expert[max_tiles:]
 
 
+def moe_route_table(tokens: torch.Tensor, table: torch.Tensor, experts: int):
+    """(ids [n, top] int32, weights [n, top] float32 = 1 / top): the experts that row tokens[t] of the integer table
+    [vocab, top] names (csrc/moe_route.cu)."""
+    _cuda(tokens, "tokens", torch.int32); _cuda(table, "table", torch.int32)
+    n, (vocab, top) = tokens.numel(), table.shape
+    ids = torch.empty((n, top), dtype=torch.int32, device=table.device)
+    weights = torch.empty((n, top), dtype=torch.float32, device=table.device)
+    f = _fn("moe_route", "jv_moe_route_table", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
+                                                c_void_p])
+    _check(f(tokens.data_ptr(), table.data_ptr(), vocab, int(experts), top, n, ids.data_ptr(), weights.data_ptr(),
+             _status_ptr(table.device), _stream()), "moe_route_table")
+    return ids, weights
+
+
 MOE_ACTS = {None: 0, "gelu": 1}
 
 
@@ -1651,8 +1667,10 @@ def short_conv(x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor | None
 def head_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.Tensor, positions: torch.Tensor,
                  token_entry: torch.Tensor, block_table: torch.Tensor, freq: torch.Tensor | None, interleaved: bool,
                  q_norm_w, k_norm_w, eps: float, value_norm: bool, value_freq: torch.Tensor | None, k_cache, v_cache,
-                 n_q_heads: int, n_k_heads: int, n_v_heads: int, key_dim: int, value_dim: int) -> None:
-    """Per head: RMSNorm of queries and keys with one weight vector [key_dim] shared by the heads (or none), rotation of
+                 n_q_heads: int, n_k_heads: int, n_v_heads: int, key_dim: int, value_dim: int,
+                 unit_heads: bool = False) -> None:
+    """Per head: RMSNorm of queries and keys with one weight vector [key_dim] shared by the heads (none: no norm, or with
+    `unit_heads` a norm without a weight), rotation of
     the first 2 * len(freq) elements (pairs in halves or `interleaved`); values divided by their root mean square
     (`value_norm`) and rotated by their own position over 2 * len(value_freq) elements; keys and values written to
     their pages (both caches None: queries only).  32-bit arithmetic."""
@@ -1692,14 +1710,14 @@ def head_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: 
         raise KernelError("head_prepare: the projection row is too short")
     f = _fn("head_prepare", "jv_head_prepare",
             [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
-             c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
-             c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+             c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
+             c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
     _check(f(proj.data_ptr(), _code(proj, "proj"), proj.stride(0), q_off, k_off, v_off, q_out.data_ptr(),
              positions.data_ptr(), token_entry.data_ptr(), block_table.data_ptr(), block_table.shape[1], _ptr(freq), rot,
              _ptr(value_freq), v_rot, 1 if interleaved else 0, _ptr(q_norm_w), _ptr(k_norm_w), w_code, float(eps),
-             1 if value_norm else 0, _ptr(k_cache) if writes else 0, _ptr(v_cache) if writes else 0, n, n_q_heads,
-             n_k_heads, n_v_heads, key_dim, value_dim, page_size, num_pages, _status_ptr(proj.device), _stream()),
-           "head_prepare")
+             1 if value_norm else 0, 1 if unit_heads else 0, _ptr(k_cache) if writes else 0, _ptr(v_cache) if writes else 0,
+             n, n_q_heads, n_k_heads, n_v_heads, key_dim, value_dim, page_size, num_pages, _status_ptr(proj.device),
+             _stream()), "head_prepare")
 
 
 def head_rotate(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, interleaved: bool, heads: int, dim: int,
@@ -1733,6 +1751,107 @@ def rms_rows(x: torch.Tensor, weight: torch.Tensor | None, eps: float) -> torch.
                                             c_int, c_int, c_void_p])
     _check(f(x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), _code(x, "x"), _ptr(weight),
              0 if weight is None else _code(weight, "weight"), float(eps), x.shape[0], x.shape[1], _stream()), "rms_rows")
+    return out
+
+
+# ------------------------------------------------ scores mixed across heads (csrc/talk_prepare.cu)
+def talk_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.Tensor, talk: torch.Tensor,
+                 positions: torch.Tensor, token_entry: torch.Tensor, block_table: torch.Tensor, freq: torch.Tensor | None,
+                 unit_eps: float | None, k_cache, v_cache, n_q_heads: int, n_kv_heads: int, key_dim: int,
+                 value_dim: int) -> None:
+    """Queries and keys rotated in halves over their first 2 * len(freq) elements and divided head by head by their root
+    mean square (`unit_eps`, None: not); keys and values written to their pages; and the queries that give scores mixed
+    across heads by `talk` [H, H] float32: `q_out` [n, H * (G * D)], head h holding at key head c the mixture
+    sum over c's query heads g of talk[h, g] * q_g, so that its product with a token's whole key row is the mixed score.
+    Both caches None: queries only.  32-bit arithmetic."""
+    _cuda(proj, "proj", contiguous=False); _cuda(q_out, "q_out", proj.dtype); _cuda(talk, "talk", torch.float32)
+    _cuda(positions, "positions", torch.int32); _cuda(token_entry, "token_entry", torch.int32)
+    _cuda(block_table, "block_table", torch.int32)
+    n = proj.shape[0]
+    if proj.stride(1) != 1 or q_out.shape != (n, n_q_heads * n_kv_heads * key_dim) or talk.shape != (n_q_heads, n_q_heads) or \
+            q_off + n_q_heads * key_dim > proj.shape[1]:
+        raise KernelError("talk_prepare: shapes do not fit")
+    rot = 0
+    if freq is not None:
+        _cuda(freq, "freq", torch.float32)
+        rot = 2 * freq.numel()
+    writes = k_cache is not None
+    page_size = num_pages = 1
+    if writes:
+        _cuda(k_cache, "k_cache", proj.dtype); _cuda(v_cache, "v_cache", proj.dtype)
+        if k_cache.shape[2:] != (n_kv_heads, key_dim) or v_cache.shape[2:] != (n_kv_heads, value_dim) or \
+                k_cache.shape[:2] != v_cache.shape[:2] or \
+                max(k_off + n_kv_heads * key_dim, v_off + n_kv_heads * value_dim) > proj.shape[1]:
+            raise KernelError("talk_prepare: the caches do not fit the heads")
+        num_pages, page_size = k_cache.shape[0], k_cache.shape[1]
+    f = _fn("talk_prepare", "jv_talk_prepare",
+            [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+             c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(f(proj.data_ptr(), _code(proj, "proj"), proj.stride(0), q_off, k_off, v_off, q_out.data_ptr(), talk.data_ptr(),
+             positions.data_ptr(), token_entry.data_ptr(), block_table.data_ptr(), block_table.shape[1], _ptr(freq), rot,
+             0 if unit_eps is None else 1, float(unit_eps or 0.0), _ptr(k_cache) if writes else 0,
+             _ptr(v_cache) if writes else 0, n, n_q_heads, n_kv_heads, key_dim, value_dim, page_size, num_pages,
+             _status_ptr(proj.device), _stream()), "talk_prepare")
+
+
+# ------------------------------------------------ recurrence with gates of the current token (csrc/min_gru.cu)
+def min_gru(proj: torch.Tensor, z_off: int, x_off: int, g_off: int, z_bias: torch.Tensor, x_bias: torch.Tensor,
+            state: torch.Tensor, cu_seqlens: torch.Tensor, slots: torch.Tensor, n_entries: int, channels: int,
+            out: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
+    """S <- (1 - z) S + z * candidate(y) element by element along every entry's tokens, z = sigmoid(. + z_bias), y = . +
+    x_bias, candidate(y) = y + 1/2 where y >= 0 and sigmoid(y) elsewhere; out = scale * S * silu(g).  The three
+    pre-activations are column ranges of the rows of `proj`; `state` [slots, channels] float32 holds S of every sequence
+    and is renewed; `out` [n, channels] may be a column range of wider rows."""
+    _cuda(proj, "proj", contiguous=False); _cuda(out, "out", proj.dtype, contiguous=False)
+    _cuda(z_bias, "z_bias"); _cuda(x_bias, "x_bias", z_bias.dtype); _cuda(state, "state", torch.float32, contiguous=False)
+    _cuda(cu_seqlens, "cu_seqlens", torch.int32); _cuda(slots, "slots", torch.int32)
+    n = proj.shape[0]
+    if proj.stride(1) != 1 or out.stride(1) != 1 or out.shape != (n, channels) or z_bias.numel() != channels or \
+            x_bias.numel() != channels or max(z_off, x_off, g_off) + channels > proj.shape[1] or \
+            state.stride(1) != 1 or state.shape[1] < channels:
+        raise KernelError("min_gru: shapes do not fit")
+    f = _fn("min_gru", "jv_min_gru", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
+                                      c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
+                                      c_int, c_void_p, c_void_p])
+    _check(f(proj.data_ptr(), _code(proj, "proj"), proj.stride(0), z_off, x_off, g_off, z_bias.data_ptr(), x_bias.data_ptr(),
+             _code(z_bias, "z_bias"), out.data_ptr(), out.stride(0), state.data_ptr(), state.stride(0), cu_seqlens.data_ptr(),
+             slots.data_ptr(), state.shape[0], n_entries, channels, float(scale), 1 if n == n_entries else 0,
+             _status_ptr(proj.device), _stream()), "min_gru")
+    return out
+
+
+# ------------------------------------------------ activation of normed powers (csrc/poly_norm.cu)
+def poly_norm(z, coef: torch.Tensor, eps: float, out: torch.Tensor | None = None,
+              out_dtype: torch.dtype | None = None) -> torch.Tensor:
+    """a N(z) + b N(z^2) + c N(z^3) + e for every row of `z` [n, width] (a tensor, possibly a column range, or a
+    PartialSum), powers element by element, N(y) = y / sqrt(mean(y^2) + eps) over the row, `coef` = (a, b, c, e)."""
+    _cuda(coef, "coef")
+    if coef.numel() != 4:
+        raise KernelError("poly_norm: four numbers")
+    parts, part_stride = 1, 0
+    if isinstance(z, PartialSum):
+        z = _cuda(z.parts, "z parts", torch.float32)
+        parts, part_stride = z.shape[0], z.stride(0)
+        n, width = z.shape[1:]
+        row_stride = z.stride(1)
+    else:
+        _cuda(z, "z", contiguous=False)
+        n, width = z.shape
+        row_stride = z.stride(0)
+        if z.stride(1) != 1:
+            raise KernelError("poly_norm: rows have unit column stride")
+        out_dtype = out_dtype or z.dtype
+    if out is None:
+        if out_dtype is None:
+            raise KernelError("poly_norm of a PartialSum needs out_dtype")
+        out = torch.empty((n, width), dtype=out_dtype, device=z.device)
+    _cuda(out, "out", contiguous=False)
+    if out.shape != (n, width) or out.stride(1) != 1:
+        raise KernelError("poly_norm: out has the shape of z")
+    f = _fn("poly_norm", "jv_poly_norm", [c_void_p, c_int, c_longlong, c_int, c_longlong, c_void_p, c_int, c_longlong, c_void_p,
+                                          c_int, c_float, c_int, c_int, c_void_p])
+    _check(f(z.data_ptr(), _code(z, "z"), row_stride, parts, part_stride, out.data_ptr(), _code(out, "out"), out.stride(0),
+             coef.data_ptr(), _code(coef, "coef"), float(eps), n, width, _stream()), "poly_norm")
     return out
 
 

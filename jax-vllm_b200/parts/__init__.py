@@ -1,4 +1,4 @@
-from . import (attention, block, dense_mlp, feed_forward, general_attention, latent_attention, mixer_pair, norm,  # noqa: F401
+from . import (attention, block, dense_mlp, feed_forward, general_attention, latent_attention, min_gru, mixer_pair, norm,  # noqa: F401
                position, recurrent, routed_experts, state_space, token_input)  # noqa: F401  (register the built-in kinds)
 from .base import (BuildContext, FixedStateNeed, PagedKVNeed, PagedLayerCache, Part, StateLayerCache, StepContext,
                    TensorSpec)

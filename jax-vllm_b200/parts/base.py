@@ -31,7 +31,9 @@ class TensorSpec:
     (the part reads it when it binds); random weights give it `FREE_AXIS`."""
     shape: tuple
     kind: str = "matrix"        # "matrix", "vector" (norm weights and the like) or "table" (integers)
-    init: str = "normal"        # random mode: "normal" = N(0, 0.02); "ones_normal" = 1 + N(0, 0.1)
+    init: str = "normal"        # random mode: "normal" = N(0, 0.02); "ones_normal" = 1 + N(0, 0.1); "eye_normal" = a
+                                #   matrix near the identity, 1 on the diagonal + N(0, 0.1) everywhere
+    below: int = 0              # random mode, tables: rows of different integers from 0 .. below - 1 (0: zeros)
 
 
 FREE_AXIS = 16

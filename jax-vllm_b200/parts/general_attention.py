@@ -3,8 +3,10 @@
     row  = x @ [W_q; W_k; W_v; W_g]^T                    one product over the packed matrix
     q, k   whole-projection RMSNorm, query temperature, rotation of a leading part of every head;
            k, v -> cache (v = k as projected where the spec says so)      csrc/attn_prepare.cu, 32-bit
-           or, head by head: RMSNorm with one weight vector shared by the heads, rotation in halves or interleaved
-           pairs, values unit-normed and rotated by their own position      csrc/head_prepare.cu, 32-bit
+           or, head by head: RMSNorm with one weight vector shared by the heads (or none), rotation in halves or
+           interleaved pairs, values unit-normed and rotated by their own position      csrc/head_prepare.cu, 32-bit
+           or, with scores mixed across heads (`talk`, below): rotation in halves, unit norm per head, and the mixture of
+           the query heads                                                    csrc/talk_prepare.cu, 32-bit
     a    = sum_j w_ij v_j over the visible keys, w = softmax(cap(q.k * scale)) or sigmoid(q.k * scale + bias_h)
     o    = a, or a1 - lam * a2 for two score maps, unit-normed; times a sigmoid gate        csrc/attn_finish.cu
            with rotated values every head of a is first turned back by the query's position   csrc/head_prepare.cu
@@ -14,6 +16,12 @@ Keys have `key_dim` elements a head and values `value_dim`; the value cache has 
 maps the rows of W_q and W_k are re-ordered when the weights are bound, from head by head [map 1 | map 2] to all
 heads' map 1 followed by all heads' map 2: the attention kernel then sees 2H query heads on 2G key heads with
 the ordinary grouping (query head i on key head i // (H/G)), and key head g reads value head g % G.
+
+With `talk` the scaled scores of the H heads are mixed by a matrix T before the softmax, s_h = sum_g T[h, g] r_g.  Since
+r_g = q_g . k_c for the key head c that g reads, s_h is the product of the token's WHOLE key row (its key heads side by
+side, G * D elements) with a query that holds at key head c the mixture sum_{g on c} T[h, g] q_g: the preparation forms
+those queries once a token, and the attention kernels run H query heads on one key head of G * D elements under G value
+heads.  The cache holds what it would hold without the mixing.
 
 The part also offers its two products to an arrangement that packs them with another part's
 (`in_weight`, `from_projection`, `out_weight`): both then read the same normed input in one product and add
@@ -77,8 +85,15 @@ class GeneralAttention(Part):
         self.mask = ops.mask_code(spec.window, spec.chunk)
         # heads prepared one by one (csrc/head_prepare.cu) where the layer asks for what only that kernel does
         interleaved = self.position is not None and getattr(self.position, "layout", "halves") == "interleaved"
+        self.unit_heads = spec.head_norm_eps is not None and not spec.head_norm_weight
+        self.talking = bool(spec.talk)
         self.by_head = (spec.head_norm_eps is not None or spec.value_norm_eps is not None or spec.rotate_values
-                        or interleaved)
+                        or interleaved or self.talking)
+        if self.talking and (spec.value_norm_eps is not None or spec.rotate_values or interleaved or spec.head_temperature
+                             or spec.distance_bias is not None or spec.weights != "softmax"
+                             or (spec.head_norm_eps is not None and spec.head_norm_weight)):
+            raise ValueError("scores mixed across heads are built for softmax weights, rotation in halves and heads normed "
+                             "without a weight")
         if self.by_head and (spec.whole_norm_eps is not None or spec.query_temperature is not None
                              or spec.values_from_keys or spec.twin is not None):
             raise ValueError("norms per head, normed or rotated values and interleaved pairs are built without a "
@@ -91,34 +106,42 @@ class GeneralAttention(Part):
             self.value_freq = self.position.frequencies(self.dv).to(ctx.device)
         if self.by_head:            # neither the whole-projection preparation nor (without a gate) the finishing kernel runs
             unused = ("attn_prepare",) + (("attn_finish",) if spec.gate is None else ())
-            self.kernels = tuple(k for k in self.kernels if k not in unused) + ("head_prepare",)
+            self.kernels = tuple(k for k in self.kernels if k not in unused) + \
+                ("talk_prepare" if self.talking else "head_prepare",)
         # Which attention kernel: once queries and keys are prepared, a mixer with one softmax map, no cap and
         # values shaped like its keys IS the plain grouped-query attention, and goes the way of that mixer (the
         # tcgen05 kernels for heads of 128, mma.sync for 16/32/64, in bfloat16).  Every other bfloat16 mixer with
         # sizes in steps of 16 takes the tensor-core kernel compiled for its pair of sizes; the rest, and 32-bit,
         # the CUDA-core kernel.
         # a temperature per head, a bias by distance and a sink are options of both of these
-        self.extras = spec.head_temperature or spec.distance_bias is not None or spec.sink
-        if self.extras and (spec.twin is not None or (spec.sink and spec.weights != "softmax")):
-            raise ValueError("head temperature, distance bias and sink are built for one softmax map")
+        self.has_sink = spec.sink or spec.sink_score is not None
+        self.out_scale = float(spec.output_scale)
+        self.extras = spec.head_temperature or spec.distance_bias is not None or self.has_sink or self.out_scale != 1.0
+        if self.extras and (spec.twin is not None or (self.has_sink and spec.weights != "softmax")):
+            raise ValueError("head temperature, distance bias, sink and output scale are built for one softmax map")
+        if spec.sink and spec.sink_score is not None:
+            raise ValueError("a sink is learned or fixed, not both")
+        # the key row that the attention kernels see: with mixed scores the G key heads side by side, under one key head
+        self.dk, self.nk = (self.hk * self.d, 1) if self.talking else (self.d, self.hk)
         plain = (spec.twin is None and spec.weights == "softmax" and not spec.score_cap and self.hv == self.hk
-                 and self.dv == self.d and not self.extras)
+                 and self.dv == self.d and not self.extras and not self.talking)
         self.plain = self.general = None
         if plain and ops.attn_mma_supports(ctx.dtype, self.d):
             self.plain = Attention(AttentionSpec(spec.hidden_size, self.hq, self.hk, self.d, spec.scale, prefix="",
                                                  window=self.mask or None), self.prefix, ctx)
             self.kernels += tuple(k for k in self.plain.kernels if k not in self.kernels and k != "rope_kv")
-        elif ops.attn_general_mma_supports(ctx.dtype, self.d, self.dv):
-            self.general = ops.attn_general_mma_library(self.d, self.dv)
+        elif ops.attn_general_mma_supports(ctx.dtype, self.dk, self.dv):
+            self.general = ops.attn_general_mma_library(self.dk, self.dv)
             self.kernels += (self.general,)
         # heads of 128 with sigmoid weights, or with a softmax that has a temperature per head, a bias by distance or a
         # sink: prompt portions that fill a 128-row tile go to the tcgen05 kernel
         self.big_tiles = (self.general is not None and not spec.score_cap and self.hv == self.hk and self.dv == self.d == 128
-                          and spec.twin is None and (spec.weights == "sigmoid") != bool(self.extras))
+                          and spec.twin is None and (spec.weights == "sigmoid") != bool(self.extras)
+                          and self.out_scale == 1.0 and not self.talking)
         if self.big_tiles:
             self.kernels += ("attn_tcgen05",)
         self.w_in = self.w_o = self.q_norm = self.k_norm = self.bias = None
-        self.head_scale = self.dist_bias = self.sink = None
+        self.head_scale = self.dist_bias = self.sink = self.talk = None
         self.lam = 0.0
         # columns of the packed projection
         self.k_off = self.hq * self.d
@@ -130,7 +153,7 @@ class GeneralAttention(Part):
 
     # -------------------------------------------------------------------- weights
     def _names(self):
-        keys = ("q", "k", "v", "g", "o", "q_norm", "k_norm", "bias", "temp", "rel", "sink")
+        keys = ("q", "k", "v", "g", "o", "q_norm", "k_norm", "bias", "temp", "rel", "sink", "talk")
         return {k: f"{self.prefix}.{n}" for k, n in zip(keys, self.spec.names)}
 
     def tensor_specs(self):
@@ -145,7 +168,7 @@ class GeneralAttention(Part):
         if s.whole_norm_eps is not None:
             specs[n["q_norm"]] = TensorSpec((self.hq * self.d,), kind="vector", init="ones_normal")
             specs[n["k_norm"]] = TensorSpec((self.hk * self.d,), kind="vector", init="ones_normal")
-        if s.head_norm_eps is not None:
+        if s.head_norm_eps is not None and s.head_norm_weight:
             specs[n["q_norm"]] = TensorSpec((self.d,), kind="vector", init="ones_normal")
             specs[n["k_norm"]] = TensorSpec((self.d,), kind="vector", init="ones_normal")
         if s.score_bias:
@@ -160,6 +183,8 @@ class GeneralAttention(Part):
             specs[n["rel"]] = TensorSpec((-1 if rows is None else int(rows), self.h), kind="vector", init="normal")
         if s.sink:
             specs[n["sink"]] = TensorSpec((self.h,), kind="vector", init="normal")
+        if s.talk:
+            specs[n["talk"]] = TensorSpec((self.h, self.h), init="eye_normal")
         return specs
 
     def _maps_first(self, w: torch.Tensor, heads: int) -> torch.Tensor:
@@ -180,7 +205,7 @@ class GeneralAttention(Part):
             mats = [m.to(torch.float32) for m in mats]
         self.w_in = torch.cat(mats, dim=0).contiguous()
         self.w_o = self.compute_weight(tensors[n["o"]], self.ctx).contiguous()
-        if s.whole_norm_eps is not None or s.head_norm_eps is not None:
+        if s.whole_norm_eps is not None or (s.head_norm_eps is not None and s.head_norm_weight):
             self.q_norm, self.k_norm = tensors[n["q_norm"]].contiguous(), tensors[n["k_norm"]].contiguous()
             if self.q_norm.dtype != self.k_norm.dtype:
                 self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
@@ -195,6 +220,10 @@ class GeneralAttention(Part):
             self.dist_bias = rel[torch.tensor(rows, device=rel.device)].t().contiguous()
         if s.sink:
             self.sink = tensors[n["sink"]].to(torch.float32).contiguous()
+        elif s.sink_score is not None:
+            self.sink = torch.full((self.h,), float(s.sink_score), dtype=torch.float32, device=self.w_in.device)
+        if s.talk:
+            self.talk = tensors[n["talk"]].to(torch.float32).contiguous()
         if s.twin is not None:
             lq1, lk1, lq2, lk2 = (tensors[f"{self.prefix}.{name}"].double() for name in s.twin.names)
             self.lam = math.exp(float((lq1 * lk1).sum())) - math.exp(float((lq2 * lk2).sum())) + float(s.twin.offset)
@@ -244,14 +273,19 @@ class GeneralAttention(Part):
         s, dt, n = self.spec, self.ctx.dtype, step.n_tokens
         table = step.block_tables[cache.group]
         writes = self.writes_cache and cache.writes
-        q = torch.empty((n, self.hq * self.d), dtype=dt, device=row.device)
+        q = torch.empty((n, self.hq * self.dk), dtype=dt, device=row.device)
         coef, every = s.query_temperature if s.query_temperature is not None else (0.0, 0)
         freq = self.position.table() if self.position is not None else None
-        if self.by_head:
+        if self.talking:
+            ops.talk_prepare(row, 0, self.k_off, self.v_off, q, self.talk, step.positions, step.token_entry, table, freq,
+                             s.head_norm_eps, cache.k if writes else None, cache.v if writes else None, self.hq, self.hk,
+                             self.d, self.dv)
+        elif self.by_head:
             ops.head_prepare(row, 0, self.k_off, self.v_off, q, step.positions, step.token_entry, table, freq,
                              self.interleaved, self.q_norm, self.k_norm, s.head_norm_eps or s.value_norm_eps or 0.0,
                              s.value_norm_eps is not None, self.value_freq, cache.k if writes else None,
-                             cache.v if writes else None, self.hq, self.hk, self.hv, self.d, self.dv)
+                             cache.v if writes else None, self.hq, self.hk, self.hv, self.d, self.dv,
+                             unit_heads=self.unit_heads)
         else:
             ops.attn_prepare(row, 0, self.k_off, self.v_off, q, step.positions, step.token_entry, table, freq,
                              self.q_norm, self.k_norm, s.whole_norm_eps or 0.0, coef, every, cache.k if writes else None,
@@ -265,7 +299,8 @@ class GeneralAttention(Part):
             return ops.head_rotate(a, step.positions, self.value_freq, self.interleaved, self.h, self.dv, sign=-1.0, out=out)
         if self.value_freq is not None:
             raise ValueError("rotated values with a gate or two score maps are not built")
-        direct = twin is None and gate is None and out.is_contiguous()
+        # the kernels that these options go to write rows of any stride
+        direct = twin is None and gate is None and (out.is_contiguous() or self.plain is None)
         # two maps are subtracted in 32-bit: the attention kernel leaves them as floats
         a = out if direct else torch.empty((n, self.hq * self.dv), dtype=torch.float32 if twin is not None else dt,
                                            device=row.device)
@@ -280,17 +315,18 @@ class GeneralAttention(Part):
         s = self.spec
         if self.plain is not None:
             return self.plain.attend(q, a, step, cache, table)
-        common = (cache.k, cache.v, table, step.cu_seqlens, step.start_pos)
+        keys = cache.k.view(*cache.k.shape[:2], self.nk, self.dk) if self.talking else cache.k
+        common = (keys, cache.v, table, step.cu_seqlens, step.start_pos)
         extra = dict(score_cap=s.score_cap or 0.0, sigmoid=s.weights == "sigmoid", bias=self.bias)
         if self.extras:
-            extra.update(head_scale=self.head_scale, dist_bias=self.dist_bias, sink=self.sink)
+            extra.update(head_scale=self.head_scale, dist_bias=self.dist_bias, sink=self.sink, out_scale=self.out_scale)
         if self.general is not None:
             def kernel(work, n_work, **split):
                 ops.attn_general_mma(q, q.stride(0), a, *common, work, n_work, self.hq, self.hk, s.scale,
                                      window=self.mask, **split, **extra)
         else:
             def kernel(work, n_work, **split):
-                ops.attn_simt(q, q.stride(0), a, *common, work, n_work, self.hq, self.hk, self.d, self.mask, s.scale,
+                ops.attn_simt(q, q.stride(0), a, *common, work, n_work, self.hq, self.hk, self.dk, self.mask, s.scale,
                               v_dim=self.dv, **split, **extra)
         for cls in self.tile_classes(cache.k.shape[1]):
             work, n_work = step.tile_work[cls]

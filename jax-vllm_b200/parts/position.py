@@ -1,10 +1,14 @@
 """Rotary position encoding: inv_freq[j] = 1 / theta^(2j/dim) / scaling_factor, j < dim/2, in 32-bit
-(jllm/model/common.py:51-55; the factor is linear scaling of positions).  `layout` names the pairs that turn together:
-"halves" (element i with i + dim/2) or "interleaved" (2i with 2i + 1); a mixer's preparation kernel must know it.  The part only owns the table; the rotation itself is
-applied to queries and keys inside the mixer's preparation kernel (csrc/rope_kv.cu), which
+(jllm/model/common.py:51-55; the factor is linear scaling of positions).  With `bands` = (factor, low, high, original) a
+frequency is scaled by its wavelength l = 2 pi / f instead: kept where l < original/high, divided by the factor where
+l > original/low, and between the two (1 - s) f / factor + s f with s = (original/l - low) / (high - low).  `layout` names the pairs that turn together:
+"halves" (element i with i + dim/2) or "interleaved" (2i with 2i + 1); a mixer's preparation kernel must know it.  The part only owns the table; the rotation
+itself is applied to queries and keys inside the mixer's preparation kernel (csrc/rope_kv.cu), which
 forms the angle position * inv_freq[j] and its cos and sin in 32-bit."""
 
 from __future__ import annotations
+
+import math
 
 import torch
 
@@ -21,13 +25,26 @@ class Rope(Part):
         self.factor = float(getattr(spec, "scaling_factor", 1.0))
         if self.layout not in ("halves", "interleaved") or not self.factor > 0:
             raise ValueError(f"rotation: layout {self.layout!r} or scaling factor {self.factor} is not built")
+        self.bands = getattr(spec, "bands", None)
+        if self.bands is not None:
+            self.bands = tuple(float(v) for v in self.bands)
+            factor, low, high, original = self.bands
+            if not (factor > 0 and low > 0 and high >= low and original > 0):
+                raise ValueError(f"rotation: bands {self.bands} (factor, low, high, original) do not fit")
         self.wide = torch.float64 if getattr(spec, "exact_table", False) else torch.float32
         self.inv_freq = self.frequencies(self.dim, self.factor).to(ctx.device)
 
     def frequencies(self, dim: int, factor: float = 1.0) -> torch.Tensor:
-        """theta^(-2j/dim) / factor for j < dim/2, as float32 on the CPU."""
+        """theta^(-2j/dim) / factor (scaled by bands, if there are any) for j < dim/2, as float32 on the CPU."""
         exponents = torch.arange(0, dim, 2, dtype=self.wide) / dim
-        return (1.0 / (self.theta ** exponents) / factor).to(torch.float32)
+        freq = 1.0 / (self.theta ** exponents) / factor
+        if self.bands is not None:
+            div, low, high, original = self.bands
+            wavelength = 2.0 * math.pi / freq
+            s = (original / wavelength - low) / (high - low)
+            mixed = (1.0 - s) * freq / div + s * freq
+            freq = torch.where(wavelength < original / high, freq, torch.where(wavelength > original / low, freq / div, mixed))
+        return freq.to(torch.float32)
 
     def table(self):
         return self.inv_freq

@@ -1,9 +1,11 @@
 """A mixture of small feed-forward experts, each down(act(up(x))), no biases; or, with the activation
 "clamped_glu", experts with a gate matrix: g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit),
-down(g * sigmoid(1.702 g) * (u + 1)) (the two matrices are stacked, the activation is a kernel of its own).
+down(g * sigmoid(1.702 g) * (u + 1)), or with "swiglu" down(silu(W_gate x) * (W_up x)) (the two matrices are stacked, the
+activation is a kernel of its own).
 
     z        = x @ W_router^T           32-bit accumulation and result (ops.linear)
     ids, w   = route(z)                 softmax scores in 32-bit, group-limited choice of the top_k (csrc/moe_route.cu)
+               or, with `scoring` "table", no router: a table names each token id's experts, all weights 1 / top_k
     order    = pairs sorted by expert   every expert's rows padded to a row tile (csrc/moe_route.cu, jv_moe_align)
     a        = act(x[token] @ W_up_e^T) grouped product, rows gathered as they are read, activation in its epilogue
     y        = a @ W_down_e^T           grouped product
@@ -26,13 +28,16 @@ class RoutedExperts(Part):
     kernels = ("moe_route", "moe_gemm_simt", "gemm_simt")
 
     def __init__(self, spec, prefix, ctx):
-        if spec.activation not in ("gelu", "clamped_glu"):
-            raise ValueError(f"routed experts: activation {spec.activation!r} is not built (gelu and clamped_glu are)")
-        if spec.scoring not in ops.ROUTER_SCORINGS or spec.group_score not in ops.GROUP_SCORES:
+        if spec.activation not in ("gelu", "clamped_glu", "swiglu"):
+            raise ValueError(f"routed experts: activation {spec.activation!r} is not built (gelu, clamped_glu and swiglu are)")
+        self.by_table = spec.scoring == "table"
+        if (spec.scoring not in ops.ROUTER_SCORINGS and not self.by_table) or spec.group_score not in ops.GROUP_SCORES:
             raise ValueError(f"routed experts: scoring {spec.scoring!r} with group score {spec.group_score!r} is not "
-                             f"built ({', '.join(ops.ROUTER_SCORINGS)}; {', '.join(ops.GROUP_SCORES)})")
-        self.gated = spec.activation == "clamped_glu"
-        if self.gated and not spec.limit > 0:
+                             f"built ({', '.join(ops.ROUTER_SCORINGS)}, table; {', '.join(ops.GROUP_SCORES)})")
+        if self.by_table and (spec.n_groups != 1 or spec.vocab_size < 1):
+            raise ValueError("routed experts: a table has a row per token id and knows no groups")
+        self.gated = spec.activation in ("clamped_glu", "swiglu")
+        if spec.activation == "clamped_glu" and not spec.limit > 0:
             raise ValueError("routed experts: the clamped activation needs a positive limit")
         if self.gated:
             self.kernels = ("moe_route", "moe_gemm_simt", "gemm_simt", "activation")
@@ -41,11 +46,14 @@ class RoutedExperts(Part):
             raise ValueError(f"routed experts: {E} experts, {n} groups, {keep} kept, top {spec.top_k} do not fit")
         self.spec, self.ctx = spec, ctx
         self.prefix = f"{prefix}.{spec.prefix}" if spec.prefix else prefix
-        self.w_router = self.w_up = self.w_down = None
+        self.w_router = self.table = self.w_up = self.w_down = None
 
     def tensor_specs(self):
         p, s = self.prefix, self.spec
-        out = {f"{p}.router": TensorSpec((s.num_experts, s.hidden_size))}
+        if self.by_table:
+            out = {f"{p}.table": TensorSpec((s.vocab_size, s.top_k), kind="table", below=s.num_experts)}
+        else:
+            out = {f"{p}.router": TensorSpec((s.num_experts, s.hidden_size))}
         for e in range(s.num_experts):
             if self.gated:
                 out[f"{p}.e{e}.gate"] = TensorSpec((s.expert_size, s.hidden_size))
@@ -55,7 +63,10 @@ class RoutedExperts(Part):
 
     def bind(self, tensors):
         p, s = self.prefix, self.spec
-        self.w_router = self.compute_weight(tensors[f"{p}.router"], self.ctx).contiguous()
+        if self.by_table:
+            self.table = tensors[f"{p}.table"].to(torch.int32).contiguous()
+        else:
+            self.w_router = self.compute_weight(tensors[f"{p}.router"], self.ctx).contiguous()
         ups = [self.compute_weight(tensors[f"{p}.e{e}.up"], self.ctx) for e in range(s.num_experts)]
         if self.gated:      # [gate; up] of an expert stacked: one grouped product makes both
             gates = [self.compute_weight(tensors[f"{p}.e{e}.gate"], self.ctx) for e in range(s.num_experts)]
@@ -80,23 +91,34 @@ class RoutedExperts(Part):
         return (ops.moe_gemm_tcgen05_supports(self.ctx.dtype, self.w_up) and ops.moe_gemm_tcgen05_supports(self.ctx.dtype, self.w_down)
                 and min(s.expert_size, s.hidden_size) >= self.TCGEN05_MIN_SIZE)
 
+    def _choose(self, x, step):
+        """(experts, weights) [n, top_k] of every token."""
+        s = self.spec
+        if self.by_table:
+            return ops.moe_route_table(step.token_ids, self.table, s.num_experts)
+        logits = ops.linear(x, self.w_router, torch.float32)       # 32-bit accumulation, 32-bit result
+        return ops.moe_route(logits, s.top_k, s.n_groups, s.keep_groups, s.renormalize, s.scoring, s.group_score,
+                             s.renorm_eps, s.weight_scale)
+
+    def _gate(self, gu):
+        """The activation of experts with a gate matrix, from rows [gate | up]."""
+        return ops.swiglu(gu) if self.spec.activation == "swiglu" else ops.glu_clamped(gu, self.spec.limit)
+
     def forward(self, x, step):
         s, dt = self.spec, self.ctx.dtype
-        logits = ops.linear(x, self.w_router, torch.float32)       # 32-bit accumulation, 32-bit result
-        ids, weights = ops.moe_route(logits, s.top_k, s.n_groups, s.keep_groups, s.renormalize, s.scoring, s.group_score,
-                                     s.renorm_eps, s.weight_scale)
+        ids, weights = self._choose(x, step)
         first = None if self.gated else "gelu"
         if self._tensor_cores():
             _, pos_of, tile_expert, used = ops.moe_align(ids, s.num_experts, ops.MOE_TCGEN05_TILE)
             rows = ops.moe_gather_rows(x, pos_of, tile_expert.numel() * ops.MOE_TCGEN05_TILE)
             act = ops.moe_gemm_tcgen05(rows, self.w_up, tile_expert, act=first, used_tiles=used)
             if self.gated:
-                act = ops.glu_clamped(act, s.limit)
+                act = self._gate(act)
             return ops.PickedRows(ops.moe_gemm_tcgen05(act, self.w_down, tile_expert, used_tiles=used), pos_of, weights)
         sorted_token, pos_of, tile_expert, _ = ops.moe_align(ids, s.num_experts, ops.moe_gemm_simt_tile())
         act = ops.moe_gemm_simt(x, sorted_token, self.w_up, tile_expert, dt, act=first)
         if self.gated:
-            act = ops.glu_clamped(act, s.limit)
+            act = self._gate(act)
         y = ops.moe_gemm_simt(act, None, self.w_down, tile_expert, dt)
         return ops.PickedRows(y, pos_of, weights)
 

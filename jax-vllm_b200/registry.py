@@ -63,6 +63,9 @@ def _register_builtin() -> None:
     from .models.gogivik import ARCHITECTURE as GOGIVIK, GogivikConfig
 
     register_architecture(GOGIVIK, GogivikConfig)
+    from .models.tidarax import ARCHITECTURE as TIDARAX, TidaraxConfig
+
+    register_architecture(TIDARAX, TidaraxConfig)
 
 
 _register_builtin()

@@ -2,7 +2,8 @@
 
 Each tensor is drawn from its own generator, seeded from (seed, name), so the values do
 not depend on the order in which tensors are made or on how parts pack them.  Matrices
-and tables of floats are N(0, 0.02); norm weights are 1 + N(0, 0.1).  `write_model_folder`
+and tables of floats are N(0, 0.02); norm weights are 1 + N(0, 0.1); mixing matrices are the identity + N(0, 0.1);
+rows of integer tables are different integers below the table's bound.  `write_model_folder`
 makes a folder (config.json, model.safetensors) that loads like any other.
 """
 
@@ -30,10 +31,16 @@ def random_tensor(name: str, spec, seed: int, dtype: torch.dtype, device="cpu") 
     gen.manual_seed(tensor_seed(seed, name))
     shape = tuple(FREE_AXIS if d == -1 else d for d in spec.shape)
     if spec.kind == "table":
-        return torch.zeros(shape, dtype=torch.int32, device=device)
+        if not spec.below:
+            return torch.zeros(shape, dtype=torch.int32, device=device)
+        # the places of the smallest of `below` random numbers: different within a row, every choice equally likely
+        keys = torch.rand((shape[0], spec.below), generator=gen, dtype=torch.float32, device=device)
+        return keys.argsort(dim=1)[:, :shape[1]].to(torch.int32).contiguous()
     z = torch.randn(shape, generator=gen, dtype=torch.float32, device=device)
     if spec.init == "ones_normal":
         z = 1.0 + NORM_STD * z
+    elif spec.init == "eye_normal":
+        z = torch.eye(shape[0], shape[1], device=device) + NORM_STD * z
     else:
         z = MATRIX_STD * z
     return z.to(dtype)
