@@ -5,12 +5,14 @@
 //
 // zl, yl and g are column ranges of the packed projection; everything from them on is 32-bit, the state is a row of
 // floats in the request's state slot.  Since the gates do not read the state, a run of tokens is one affine map of it:
-// S -> A S + B with A the product of the (1 - z) and B what the run makes of a zero state.  A block takes CB channels of
-// one entry in tiles of tokens: every thread reads TPT tokens of one channel (the loads of the next tile fly while this
-// one is computed), forms their (a, b) pairs in registers and the pair (A, B) of its run, the runs of a tile are chained
-// through shared memory from the state that the tile before left, and every thread goes through its tokens again from
-// its true start.  One pass over memory, one launch; the order of the sums differs from token by token by 32-bit
-// rounding only.  A step of single tokens is a flat kernel, one thread a channel.
+// S -> (1 - D) S + B with 1 - D the product of the (1 - z) and B what the run makes of a zero state.  Every update is
+// written as S + z (candidate - S), and D is carried rather than 1 - D: a gate close to zero keeps its relative precision
+// over thousands of tokens, which 1 - z rounded to 32-bit does not.  A block takes CB channels of one entry in tiles of
+// tokens: every thread reads TPT tokens of one channel (the loads of the next tile fly while this one is computed), forms
+// their gates and candidates in registers and the pair (D, B) of its run, the runs of a tile are chained through shared
+// memory from the state that the tile before left, and every thread goes through its tokens again from its true start.
+// One pass over memory, one launch; the order of the sums differs from token by token by 32-bit rounding only.  A step of
+// single tokens is a flat kernel, one thread a channel.
 #include "common.cuh"
 #include <math.h>
 
@@ -34,14 +36,14 @@ struct GruParams {
 template <bool EXACT> __device__ __forceinline__ float exp_of(float x) { return EXACT ? expf(x) : __expf(x); }
 template <bool EXACT> __device__ __forceinline__ float recip(float x) { return EXACT ? 1.f / x : __fdividef(1.f, x); }
 
-// (a, b) of one token: S <- a S + b.
+// Gate and candidate of one token.
 template <bool EXACT>
-__device__ __forceinline__ void gru_pair(float zl, float y, float& a, float& b) {
+__device__ __forceinline__ void gru_pair(float zl, float y, float& z, float& c) {
   const float e = exp_of<EXACT>(fminf(zl, 80.f));          // e^zl, kept finite
-  a = recip<EXACT>(1.f + e);                               // 1 - z
-  const float c = y >= 0.f ? y + 0.5f : recip<EXACT>(1.f + exp_of<EXACT>(fminf(-y, 80.f)));
-  b = e * a * c;                                           // z * candidate
+  z = e * recip<EXACT>(1.f + e);
+  c = y >= 0.f ? y + 0.5f : recip<EXACT>(1.f + exp_of<EXACT>(fminf(-y, 80.f)));
 }
+__device__ __forceinline__ float blend(float S, float z, float c) { return fmaf(z, c - S, S); }
 template <bool EXACT>
 __device__ __forceinline__ float silu_of(float g) { return g * recip<EXACT>(1.f + exp_of<EXACT>(fminf(-g, 80.f))); }
 
@@ -50,7 +52,7 @@ template <typename T, typename W, int CB>
 __global__ void __launch_bounds__(THREADS, 1) gru_scan_kernel(const GruParams p) {
   constexpr int RUNS = THREADS / CB, TILE = RUNS * TPT;
   constexpr bool EXACT = sizeof(T) == 4;
-  __shared__ float As[RUNS][CB], Bs[RUNS][CB];
+  __shared__ float Ds[RUNS][CB], Bs[RUNS][CB];
   __shared__ float carry[2][CB];
   pdl_trigger();
   const int cl = threadIdx.x % CB, run = threadIdx.x / CB;
@@ -86,27 +88,27 @@ __global__ void __launch_bounds__(THREADS, 1) gru_scan_kernel(const GruParams p)
   fetch(t0);
   int which = 0;
   for (int tile0 = t0; tile0 < t1; tile0 += TILE, which ^= 1) {
-    float a[TPT], b[TPT], g[TPT];
-    float A = 1.f, B = 0.f;
+    float z[TPT], cand[TPT], g[TPT];
+    float D = 0.f, B = 0.f;
 #pragma unroll
     for (int i = 0; i < TPT; ++i) {
-      gru_pair<EXACT>(to_f32(zr[i]) + zb, to_f32(xr[i]) + xb, a[i], b[i]);
+      gru_pair<EXACT>(to_f32(zr[i]) + zb, to_f32(xr[i]) + xb, z[i], cand[i]);
       g[i] = to_f32(gr[i]);
-      if (tile0 + run * TPT + i >= t1) { a[i] = 1.f; b[i] = 0.f; }      // no token: the state passes
-      A *= a[i];
-      B = fmaf(a[i], B, b[i]);
+      if (tile0 + run * TPT + i >= t1) z[i] = 0.f;         // no token: the state passes
+      D = blend(D, z[i], 1.f);
+      B = blend(B, z[i], cand[i]);
     }
     if (tile0 + TILE < t1) fetch(tile0 + TILE);
-    As[run][cl] = A;
+    Ds[run][cl] = D;
     Bs[run][cl] = B;
     __syncthreads();
     float S = carry[which][cl];
-    for (int r = 0; r < run; ++r) S = fmaf(As[r][cl], S, Bs[r][cl]);
-    if (run == RUNS - 1) carry[which ^ 1][cl] = fmaf(A, S, B);
+    for (int r = 0; r < run; ++r) S = fmaf(-Ds[r][cl], S, S) + Bs[r][cl];
+    if (run == RUNS - 1) carry[which ^ 1][cl] = fmaf(-D, S, S) + B;
 #pragma unroll
     for (int i = 0; i < TPT; ++i) {
       const int t = tile0 + run * TPT + i;
-      S = fmaf(a[i], S, b[i]);
+      S = blend(S, z[i], cand[i]);
       if (live && t < t1) ((T*)p.out)[(size_t)t * p.out_stride + c] = from_f32<T>(p.scale * S * silu_of<EXACT>(g[i]));
     }
     __syncthreads();                                       // the runs' pairs have been read; the carry is there
@@ -131,9 +133,9 @@ __global__ void __launch_bounds__(128) gru_single_kernel(const GruParams p) {
   const T* row = (const T*)p.proj + (size_t)t * p.stride;
   float* S_g = p.state + (size_t)slot * p.slot_stride + c;
   const float zl = to_f32(row[p.z_off + c]), y = to_f32(row[p.x_off + c]), g = to_f32(row[p.g_off + c]), S0 = *S_g;
-  float a, b;
-  gru_pair<EXACT>(zl + zb, y + xb, a, b);
-  const float S = fmaf(a, S0, b);
+  float z, cand;
+  gru_pair<EXACT>(zl + zb, y + xb, z, cand);
+  const float S = blend(S0, z, cand);
   *S_g = S;
   ((T*)p.out)[(size_t)t * p.out_stride + c] = from_f32<T>(p.scale * S * silu_of<EXACT>(g));
 }
