@@ -1,0 +1,366 @@
+// Attention of single tokens whose scores are products with a token's WHOLE cached key row (KD elements, the key heads
+// side by side: scores mixed across heads, see talk_prepare.cu), bfloat16, the value heads as in grouped-query attention
+// (query head h reads value head h / (H / G)).
+//
+// Every query head reads every byte of the keys, so a block takes ALL heads of one request over a range of keys (grid:
+// request x range) and each cached byte is read once from memory.  Tiles of KT keys come in by bulk copies (one a key row,
+// one a value row) into two stages, the next tile's under way while this one is worked on:
+//   scores     S [H, KT] = Q [H, KD] K^T on the tensor cores (mma.sync m16n8k16, 32-bit accumulation): a warp takes 16 heads
+//              x 8 keys, and where that gives fewer than eight pieces of work, a part of KD
+//   softmax    running (max, sum) a head in 32-bit, one warp a head, one lane a key
+//   output     O [H, DV] += P V in 32-bit on the CUDA cores: a thread keeps two columns of a value head for all query heads
+//              that read it (a decoded token's few rows would leave most of a tensor-core tile empty); P stays 32-bit
+// Each range leaves its unnormalised output and (max, sum); a second kernel merges a head's ranges in ascending order and
+// lets the sink join the denominator.  Every wait on a barrier is bounded and reports to the status word.
+#include "common.cuh"
+#include "mbarrier.cuh"
+#include <math.h>
+
+namespace {
+constexpr int THREADS = 256, WARPS = THREADS / 32;
+constexpr int MAX_SPLIT = 256;                  // keys of a range
+constexpr float LOG2E = 1.4426950408889634f;
+
+struct Params {
+  const __nv_bfloat16* q; int q_stride;
+  __nv_bfloat16* out; int out_stride;
+  float* part_o; float* part_ml;
+  const __nv_bfloat16* k_cache; const __nv_bfloat16* v_cache;
+  const int* block_table; int table_width;
+  const int* cu_seqlens; const int* start_pos; const int* work;
+  int H, G, KD, DV, page_size, num_pages;
+  float scale_log2, out_scale;
+  const float* sink;           // [H] or null
+  int KT, k_parts;             // keys of a tile; parts of KD that warps share a score tile in
+  int split_size, n_splits;
+  int* status;
+};
+
+__device__ __forceinline__ void bulk_copy(void* dst, const void* src, int bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n"
+               ::"r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldmatrix_x2(uint32_t (&r)[2], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// Offsets (bytes) of the arrays in dynamic shared memory, for the kernel and its launcher.
+struct Layout {
+  int q_row, k_row, v_row, s_row;              // elements from row to row
+  size_t q, k, v, s, total;                    // s: [k_parts][H16][s_row] floats
+  __host__ __device__ Layout(int H, int G, int KD, int DV, int KT, int k_parts) {
+    const int H16 = (H + 15) / 16 * 16;
+    q_row = k_row = KD + 8; v_row = G * DV; s_row = KT + 4;
+    q = 0;
+    k = q + sizeof(__nv_bfloat16) * (size_t)H16 * q_row;
+    v = k + sizeof(__nv_bfloat16) * (size_t)2 * KT * k_row;
+    s = v + sizeof(__nv_bfloat16) * (size_t)2 * KT * v_row;
+    total = s + sizeof(float) * (size_t)k_parts * H16 * s_row;
+  }
+};
+
+// HT: query heads of a value head, rounded up; IT: column pairs a thread keeps.
+template <int HT, int IT>
+__global__ void __launch_bounds__(THREADS) attn_rows_decode_kernel(const Params p) {
+  extern __shared__ __align__(128) unsigned char smem[];
+  __shared__ long long slots[MAX_SPLIT];        // cache slot of every key of the range (-1: none)
+  __shared__ float row_m[256], row_l[256], row_alpha[256];
+  __shared__ __align__(8) uint64_t bars[2];
+  const int H = p.H, G = p.G, KD = p.KD, DV = p.DV, KT = p.KT, HPT = H / G;
+  const Layout L(H, G, KD, DV, KT, p.k_parts);
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem + L.q);
+  __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(smem + L.k);
+  __nv_bfloat16* vs = reinterpret_cast<__nv_bfloat16*>(smem + L.v);
+  float* ss = reinterpret_cast<float*>(smem + L.s);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  pdl_trigger();
+  if (tid == 0) {
+    mbar_init(&bars[0], THREADS);
+    mbar_init(&bars[1], THREADS);
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+  }
+  pdl_wait();
+  const int entry = p.work[2 * blockIdx.x];
+  const int pos = p.start_pos[entry];
+  const int j_lo = blockIdx.y * p.split_size, j_hi = min(pos + 1, j_lo + p.split_size);
+  if (blockIdx.y == 0 && tid == 0 && pos / p.split_size >= p.n_splits) atomicOr(p.status, JV_STATUS_BAD_ROW);
+  if (j_lo >= j_hi) return;
+  const int token = p.cu_seqlens[entry];
+  for (int i = tid; i < j_hi - j_lo; i += THREADS) {
+    const int j = j_lo + i, pi = j / p.page_size;
+    const int page = pi < p.table_width ? p.block_table[(size_t)entry * p.table_width + pi] : -1;
+    long long s = -1;
+    if (page < 0 || page >= p.num_pages) atomicOr(p.status, JV_STATUS_BAD_PAGE);
+    else s = (long long)page * p.page_size + (j - pi * p.page_size);
+    slots[i] = s;
+  }
+  const int H16 = (H + 15) / 16 * 16, CH = KD / 8;
+  for (int c = tid; c < H16 * CH; c += THREADS) {
+    const int h = c / CH, part = c - h * CH;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (h < H) v = *reinterpret_cast<const uint4*>(p.q + (size_t)token * p.q_stride + (size_t)h * KD + part * 8);
+    *reinterpret_cast<uint4*>(qs + (size_t)h * L.q_row + part * 8) = v;
+  }
+  for (int h = tid; h < H; h += THREADS) { row_m[h] = -INFINITY; row_l[h] = 0.f; }
+  __syncthreads();
+
+  const int n_tiles = (j_hi - j_lo + KT - 1) / KT;
+  // Tile t into stage t & 1: thread n < KT its key row, thread KT + n its value row (KT <= 64); every thread arrives once.
+  auto issue = [&](int t) {
+    uint64_t* bar = &bars[t & 1];
+    const int n = tid < KT ? tid : tid - KT;
+    if (tid < 2 * KT) {
+      const bool is_v = tid >= KT;
+      const int i = t * KT + n;
+      const long long slot = i < j_hi - j_lo ? slots[i] : -1;
+      const int elems = is_v ? G * DV : KD;
+      __nv_bfloat16* dst = is_v ? vs + (size_t)((t & 1) * KT + n) * L.v_row : ks + (size_t)((t & 1) * KT + n) * L.k_row;
+      if (slot >= 0) {
+        mbar_expect_tx(bar, elems * 2);
+        bulk_copy(dst, (is_v ? p.v_cache : p.k_cache) + slot * elems, elems * 2, bar);
+      } else {                                   // no key here: zeros
+        for (int c = 0; c < elems / 8; ++c) *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(0, 0, 0, 0);
+        mbar_arrive(bar);
+      }
+    } else {
+      mbar_arrive(bar);
+    }
+  };
+  issue(0);
+  if (n_tiles > 1) issue(1);
+
+  // ---- this thread's columns of the output
+  const int pairs = G * DV / 2;
+  float acc[IT][HT][2];
+#pragma unroll
+  for (int i = 0; i < IT; ++i)
+#pragma unroll
+    for (int g = 0; g < HT; ++g) acc[i][g][0] = acc[i][g][1] = 0.f;
+
+  const int mt = H16 / 16, nt = KT / 8, kp = p.k_parts, k_steps = KD / 16;
+  for (int t = 0; t < n_tiles; ++t) {
+    const int buf = t & 1;
+    // every thread takes the same way out: all saw the tile, or the block stops (status word set)
+    if (!__syncthreads_and(mbar_wait(&bars[buf], (t >> 1) & 1))) {
+      if (tid == 0) atomicOr(p.status, JV_STATUS_WAIT_EXPIRED);
+      mbar_wait(&bars[buf], (t >> 1) & 1);       // once more, bounded, for copies that may still be landing
+      if (t + 1 < n_tiles) mbar_wait(&bars[buf ^ 1], ((t + 1) >> 1) & 1);
+      return;
+    }
+    // ---- scores
+    for (int u = warp; u < mt * nt * kp; u += WARPS) {
+      const int part = u % kp, n8 = (u / kp) % nt, m16 = u / (kp * nt);
+      const int k0 = k_steps * part / kp, k1 = k_steps * (part + 1) / kp;
+      const __nv_bfloat16* qa = qs + (size_t)(m16 * 16 + (lane & 15)) * L.q_row + (lane >> 4) * 8;
+      const __nv_bfloat16* kb = ks + (size_t)(buf * KT + n8 * 8 + (lane & 7)) * L.k_row + ((lane >> 3) & 3) * 8;
+      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+      int k = k0;
+#pragma unroll 2
+      for (; k + 2 <= k1; k += 2) {              // two independent sums
+        uint32_t a0[4], a1[4], b[4];
+        ldmatrix_x4(a0, qa + k * 16);
+        ldmatrix_x4(a1, qa + k * 16 + 16);
+        ldmatrix_x4(b, kb + k * 16);
+        mma_bf16(c0, a0, b[0], b[1]);
+        mma_bf16(c1, a1, b[2], b[3]);
+      }
+      if (k < k1) {
+        uint32_t a0[4], b[2];
+        ldmatrix_x4(a0, qa + k * 16);
+        ldmatrix_x2(b, ks + (size_t)(buf * KT + n8 * 8 + (lane & 7)) * L.k_row + ((lane >> 3) & 1) * 8 + k * 16);
+        mma_bf16(c0, a0, b[0], b[1]);
+      }
+      float* dst = ss + ((size_t)part * H16 + m16 * 16 + (lane >> 2)) * L.s_row + n8 * 8 + (lane & 3) * 2;
+      *reinterpret_cast<float2*>(dst) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
+      *reinterpret_cast<float2*>(dst + 8 * L.s_row) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
+    }
+    __syncthreads();
+    // ---- softmax: one warp a head; the weights replace the first part's scores
+    const int here = min(KT, j_hi - j_lo - t * KT);
+    for (int h = warp; h < H; h += WARPS) {
+      float* row = ss + (size_t)h * L.s_row;
+      float v[2];
+      float mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int j = lane + 32 * i;
+        v[i] = -INFINITY;
+        if (j < here) {
+          float s = row[j];
+          for (int q = 1; q < kp; ++q) s += row[(size_t)q * H16 * L.s_row + j];
+          v[i] = s * p.scale_log2;
+        }
+        mx = fmaxf(mx, v[i]);
+      }
+      mx = warp_max(mx);
+      const float m_old = row_m[h], m_new = fmaxf(m_old, mx);          // finite: a tile has at least one key
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int j = lane + 32 * i;
+        if (j < KT) {
+          const float e = j < here ? exp2f(v[i] - m_new) : 0.f;
+          row[j] = e;
+          sum += e;
+        }
+      }
+      sum = warp_sum(sum);
+      __syncwarp();
+      if (lane == 0) {
+        const float alpha = m_old == -INFINITY ? 0.f : exp2f(m_old - m_new);
+        row_alpha[h] = alpha;
+        row_m[h] = m_new;
+        row_l[h] = row_l[h] * alpha + sum;
+      }
+    }
+    __syncthreads();
+    // ---- output
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+      const int pr = tid + i * THREADS;
+      if (pr < pairs) {
+        const int c = pr / (DV / 2);
+        const __nv_bfloat16* vcol = vs + (size_t)buf * KT * L.v_row + pr * 2;
+        const float* prow = ss + (size_t)c * HPT * L.s_row;
+#pragma unroll
+        for (int g = 0; g < HT; ++g)
+          if (g < HPT) { const float al = row_alpha[c * HPT + g]; acc[i][g][0] *= al; acc[i][g][1] *= al; }
+        for (int j = 0; j < KT; j += 4) {
+          float2 v[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[e] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vcol + (size_t)(j + e) * L.v_row));
+#pragma unroll
+          for (int g = 0; g < HT; ++g)
+            if (g < HPT) {
+              const float4 w = *reinterpret_cast<const float4*>(prow + (size_t)g * L.s_row + j);
+              acc[i][g][0] = fmaf(w.x, v[0].x, acc[i][g][0]); acc[i][g][1] = fmaf(w.x, v[0].y, acc[i][g][1]);
+              acc[i][g][0] = fmaf(w.y, v[1].x, acc[i][g][0]); acc[i][g][1] = fmaf(w.y, v[1].y, acc[i][g][1]);
+              acc[i][g][0] = fmaf(w.z, v[2].x, acc[i][g][0]); acc[i][g][1] = fmaf(w.z, v[2].y, acc[i][g][1]);
+              acc[i][g][0] = fmaf(w.w, v[3].x, acc[i][g][0]); acc[i][g][1] = fmaf(w.w, v[3].y, acc[i][g][1]);
+            }
+        }
+      }
+    }
+    __syncthreads();                             // the stage and the weights have been read
+    if (t + 2 < n_tiles) {
+      asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+      issue(t + 2);
+    }
+  }
+  // ---- what the range leaves
+#pragma unroll
+  for (int i = 0; i < IT; ++i) {
+    const int pr = tid + i * THREADS;
+    if (pr < pairs) {
+      const int c = pr / (DV / 2), d = pr * 2 - c * DV;
+#pragma unroll
+      for (int g = 0; g < HT; ++g)
+        if (g < HPT) {
+          const size_t at = ((size_t)blockIdx.x * H + c * HPT + g) * p.n_splits + blockIdx.y;
+          *reinterpret_cast<float2*>(p.part_o + at * DV + d) = make_float2(acc[i][g][0], acc[i][g][1]);
+        }
+    }
+  }
+  for (int h = tid; h < H; h += THREADS) {
+    const size_t at = ((size_t)blockIdx.x * H + h) * p.n_splits + blockIdx.y;
+    p.part_ml[2 * at] = row_m[h];
+    p.part_ml[2 * at + 1] = row_l[h];
+  }
+}
+
+// One block a (request, head): the ranges in ascending order; maxima are exponents of two.
+__global__ void __launch_bounds__(128) attn_rows_merge_kernel(const Params p) {
+  pdl_trigger();
+  pdl_wait();
+  const int entry = p.work[2 * blockIdx.x], h = blockIdx.y;
+  const int last = min(p.start_pos[entry] / p.split_size, p.n_splits - 1);
+  const size_t base = ((size_t)blockIdx.x * p.H + h) * p.n_splits;
+  // the sink is one more part, with no value: maximum sink, sum 1
+  const float sk = p.sink != nullptr ? p.sink[h] * LOG2E : -INFINITY;
+  float m = sk;
+  for (int s = 0; s <= last; ++s) m = fmaxf(m, p.part_ml[2 * (base + s)]);
+  float l = p.sink != nullptr ? exp2f(sk - m) : 0.f;
+  for (int s = 0; s <= last; ++s) l += exp2f(p.part_ml[2 * (base + s)] - m) * p.part_ml[2 * (base + s) + 1];
+  const float inv = p.out_scale / l;
+  for (int d = threadIdx.x; d < p.DV; d += blockDim.x) {
+    float o = 0.f;
+#pragma unroll 4
+    for (int s = 0; s <= last; ++s) o = fmaf(exp2f(p.part_ml[2 * (base + s)] - m), p.part_o[(base + s) * p.DV + d], o);
+    p.out[(size_t)p.cu_seqlens[entry] * p.out_stride + (size_t)h * p.DV + d] = __float2bfloat16_rn(o * inv);
+  }
+}
+
+// Keys of a tile: as many as let two stages fit beside the queries, 64 at most.
+int tile_keys(int H, int G, int KD, int DV, int* k_parts) {
+  const int H16 = (H + 15) / 16 * 16;
+  for (int kt = 64; kt >= 16; kt /= 2) {
+    int kp = 1;
+    while (kp < 8 && (H16 / 16) * (kt / 8) * kp < WARPS && KD / 16 >= 2 * kp) kp *= 2;
+    if (2 * kt * 2 * (size_t)(KD + G * DV) <= 132 * 1024 && Layout(H, G, KD, DV, kt, kp).total <= 220 * 1024) {
+      *k_parts = kp;
+      return kt;
+    }
+  }
+  return 0;
+}
+
+template <int HT, int IT>
+int launch(const Params& p, int n_work, size_t smem, cudaStream_t stream) {
+  auto kern = attn_rows_decode_kernel<HT, IT>;
+  static bool ready[JV_MAX_DEVICES];
+  if (!jv_once_per_device(ready, [&] {
+        return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) == cudaSuccess;
+      }))
+    return JV_ERR_UNSUPPORTED;
+  const int rc = jv_launch(kern, dim3(n_work, p.n_splits), dim3(THREADS), smem, stream, p);
+  if (rc != JV_OK) return rc;
+  return jv_launch(attn_rows_merge_kernel, dim3(n_work, p.H), dim3(128), 0, stream, p);
+}
+}  // namespace
+
+// 1 if the kernel takes these sizes: KD a multiple of 16, DV of 8, up to 16 query heads a value head and 256 in all.
+JV_EXPORT int jv_attn_rows_decode_supports(int H, int G, int KD, int DV) {
+  if (G < 1 || H < 1 || H % G || H > 256 || KD % 16 || KD < 16 || DV % 8 || DV < 8) return 0;
+  const int hpt = H / G, ht = hpt <= 4 ? 4 : hpt <= 8 ? 8 : 16;
+  const int it = (G * DV / 2 + THREADS - 1) / THREADS;
+  int kp;
+  return hpt <= 16 && it <= 4 && ht * it <= 32 && tile_keys(H, G, KD, DV, &kp) > 0;
+}
+
+// q: rows of q_stride elements, head h of a token at column h*KD; out: rows of out_stride, head h at h*DV; k_cache:
+// [num_pages, page_size, KD], v_cache: [num_pages, page_size, G*DV]; work: [n_work, 2] entries of one token; part_o:
+// [n_work * H * n_splits * DV] and part_ml: [n_work * H * n_splits * 2] floats of scratch; split_size: keys of a range, up to
+// 256; sink: [H] floats or null.
+JV_EXPORT int jv_attn_rows_decode(const void* q, int q_stride, void* out, int out_stride, float* part_o, float* part_ml,
+                                  const void* k_cache, const void* v_cache, const int* block_table, int table_width,
+                                  const int* cu_seqlens, const int* start_pos, const int* work, int n_work, int H, int G,
+                                  int KD, int DV, int page_size, int num_pages, float scale, float out_scale,
+                                  const float* sink, int split_size, int n_splits, int* status, cudaStream_t stream) {
+  if (n_work == 0) return JV_OK;
+  if (!jv_attn_rows_decode_supports(H, G, KD, DV) || split_size < 1 || split_size > MAX_SPLIT || n_splits < 1 ||
+      n_splits > 65535 || (q_stride % 8) || ((uintptr_t)q % 16) || ((uintptr_t)k_cache % 16) || ((uintptr_t)v_cache % 16))
+    return JV_ERR_UNSUPPORTED;
+  Params p;
+  p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride; p.out = (__nv_bfloat16*)out; p.out_stride = out_stride;
+  p.part_o = part_o; p.part_ml = part_ml; p.k_cache = (const __nv_bfloat16*)k_cache; p.v_cache = (const __nv_bfloat16*)v_cache;
+  p.block_table = block_table; p.table_width = table_width; p.cu_seqlens = cu_seqlens; p.start_pos = start_pos; p.work = work;
+  p.H = H; p.G = G; p.KD = KD; p.DV = DV; p.page_size = page_size; p.num_pages = num_pages; p.scale_log2 = scale * LOG2E;
+  p.out_scale = out_scale; p.sink = sink; p.split_size = split_size; p.n_splits = n_splits; p.status = status;
+  p.KT = tile_keys(H, G, KD, DV, &p.k_parts);
+  const size_t smem = Layout(H, G, KD, DV, p.KT, p.k_parts).total;
+  const int hpt = H / G, it = (G * DV / 2 + THREADS - 1) / THREADS;
+  if (hpt <= 4) return it <= 1 ? launch<4, 1>(p, n_work, smem, stream) : it <= 2 ? launch<4, 2>(p, n_work, smem, stream)
+                                                                                 : launch<4, 4>(p, n_work, smem, stream);
+  if (hpt <= 8) return it <= 1 ? launch<8, 1>(p, n_work, smem, stream) : it <= 2 ? launch<8, 2>(p, n_work, smem, stream)
+                                                                                 : launch<8, 4>(p, n_work, smem, stream);
+  return it <= 1 ? launch<16, 1>(p, n_work, smem, stream) : launch<16, 2>(p, n_work, smem, stream);
+}

@@ -138,8 +138,15 @@ class GeneralAttention(Part):
         self.big_tiles = (self.general is not None and not spec.score_cap and self.hv == self.hk and self.dv == self.d == 128
                           and spec.twin is None and (spec.weights == "sigmoid") != bool(self.extras)
                           and self.out_scale == 1.0 and not self.talking)
-        if self.big_tiles:
+        # scores mixed across heads: heads of 128 go to the same kernel in its form for whole key rows, portions of any
+        # length where no kernel with smaller tiles takes rows that long; single tokens to the kernel that reads each row once
+        self.whole_rows = (self.talking and not spec.score_cap and self.hv == self.hk and self.dv == self.d == 128)
+        self.rows_decode = (self.talking and not spec.score_cap and not self.mask and self.general is None
+                            and ops.attn_rows_decode_supports(ctx.dtype, self.hq, self.hv, self.dk, self.dv))
+        if self.big_tiles or (self.whole_rows and ctx.dtype == torch.bfloat16):
             self.kernels += ("attn_tcgen05",)
+        if self.rows_decode:
+            self.kernels += ("attn_rows_decode",)
         self.w_in = self.w_o = self.q_norm = self.k_norm = self.bias = None
         self.head_scale = self.dist_bias = self.sink = self.talk = None
         self.lam = 0.0
@@ -238,14 +245,22 @@ class GeneralAttention(Part):
     def tile_classes(self, page_size: int):
         if self.plain is not None:
             return self.plain.tile_classes(page_size)
+        return [cls for cls, _ in self._tile_kernels(page_size)]
+
+    def _tile_kernels(self, page_size: int):
+        """The work lists of entries of several tokens, each with whether the tcgen05 prompt kernel takes it."""
+        big = 0
+        if (self.big_tiles or self.whole_rows) and ops.attn_tcgen05_supports(self.ctx.dtype, self.d, self.hq, self.hk,
+                                                                             page_size, 0):
+            big = ops.attn_tcgen05_tokens_per_tile(self.hq, self.hk)
         if self.general is not None:
             small = ops.attn_general_mma_tokens_per_tile(self.hq, self.hk)
-            if self.big_tiles and ops.attn_tcgen05_supports(self.ctx.dtype, self.d, self.hq, self.hk, page_size, 0):
-                big = ops.attn_tcgen05_tokens_per_tile(self.hq, self.hk)
-                if big > small:
-                    return [(small, 2, big), (big, big, self.FOREVER)]
-            return [(small, 2, self.FOREVER)]
-        return [(ops.attn_simt_tokens_per_tile(self.hq, self.hk), 2, self.FOREVER)]
+            if big > small:
+                return [((small, 2, big), False), ((big, big, self.FOREVER), True)]
+            return [((small, 2, self.FOREVER), False)]
+        if self.whole_rows and big:
+            return [((big, 2, self.FOREVER), True)]
+        return [((ops.attn_simt_tokens_per_tile(self.hq, self.hk), 2, self.FOREVER), False)]
 
     # ----------------------------------------------------------------------- step
     def in_weight(self) -> torch.Tensor:
@@ -328,16 +343,20 @@ class GeneralAttention(Part):
             def kernel(work, n_work, **split):
                 ops.attn_simt(q, q.stride(0), a, *common, work, n_work, self.hq, self.hk, self.dk, self.mask, s.scale,
                               v_dim=self.dv, **split, **extra)
-        for cls in self.tile_classes(cache.k.shape[1]):
+        for cls, big in self._tile_kernels(cache.k.shape[1]):
             work, n_work = step.tile_work[cls]
-            if n_work and cls[1] > 2:                      # the class of whole 128-row tiles
-                ops.attn_tcgen05(q, q.stride(0), a, *common, work, n_work, self.hq, self.hk, self.d, s.scale,
-                                 sigmoid=s.weights == "sigmoid", bias=self.bias, head_scale=self.head_scale,
-                                 dist_bias=self.dist_bias, sink=self.sink, window=self.mask)
+            if n_work and big:                             # 128-row tiles
+                ops.attn_tcgen05(q, q.stride(0), a, cache.k, cache.v, *common[2:], work, n_work, self.hq, self.hk, self.d,
+                                 s.scale, sigmoid=s.weights == "sigmoid", bias=self.bias, head_scale=self.head_scale,
+                                 dist_bias=self.dist_bias, sink=self.sink, window=self.mask, whole_rows=self.talking,
+                                 out_scale=self.out_scale)
             elif n_work:
                 kernel(work, n_work)
         dwork, n_dec = step.decode_work
-        if n_dec:
+        if n_dec and self.rows_decode:
+            ops.attn_rows_decode(q, q.stride(0), a, *common, dwork, n_dec, self.hq, s.scale, step.max_seq_len,
+                                 sink=self.sink, out_scale=self.out_scale)
+        elif n_dec:
             split = self.ctx.decode_split_size
             kernel(dwork, n_dec, split_size=split, n_splits=max(1, -(-step.max_seq_len // split)))
 
