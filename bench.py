@@ -694,6 +694,8 @@ def design(name: str, layers, sizes, steps, warmup) -> int:
         return design_nufapel(layers or 3, sizes, steps, warmup)
     if name == "gogivik":
         return design_gogivik(layers or 3, sizes, steps, warmup)
+    if name == "tidarax":
+        return design_tidarax(layers or 2, sizes, steps, warmup)
     if name != "guronex":
         print(f"bench.py: no design {name!r}")
         return 2
@@ -1106,6 +1108,154 @@ def design_gogivik(layers, sizes, steps, warmup) -> int:
     return 0
 
 
+# ------------------------------------------------------------------ the Tidarax design beside Nufapel and Loselix
+# Layer sizes for `--design tidarax`: layers of attention with scores mixed across heads beside a minimal gated recurrence,
+# over a dense feed-forward with the activation of normed powers and over experts that a table names, in turn; beside
+# Nufapel's layers of the same arrangement (attention with a distance bias beside a matrix memory, over dense and routed
+# feed-forwards) and Loselix softmax-attention layers, both of equal width, heads and feed-forward work per token.  "w2k":
+# the width of a 1B-class model; "w4k" and "w4k8": an 8B-class width with 4 and with 8 key heads; "small": heads of 64.
+TIDARAX_SIZES = {
+    "w2k": dict(width=2048, heads=16, kv=4, dim=128, vdim=128, gru=2048, ff=8192, experts=32, top=4, eff=1024,
+                mem=(8, 128, 256)),
+    "w4k": dict(width=4096, heads=32, kv=4, dim=128, vdim=128, gru=4096, ff=16384, experts=32, top=4, eff=2048,
+                mem=(8, 256, 512)),
+    "w4k8": dict(width=4096, heads=32, kv=8, dim=128, vdim=128, gru=4096, ff=16384, experts=32, top=4, eff=2048,
+                 mem=(8, 256, 512)),
+    "small": dict(width=1024, heads=16, kv=4, dim=64, vdim=64, gru=1024, ff=4096, experts=16, top=2, eff=1024,
+                  mem=(4, 64, 128)),
+}
+TIDARAX_KINDS = ("dense", "moe")
+
+
+def tidarax_configs(z, layers, vocab=32000):
+    H, G = z["heads"], z["kv"]
+    rot = {"base": 5e5, "dims": z["dim"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}
+    mixer = {"left": {"heads": H, "kv_heads": G, "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5, "rot": rot},
+             "right": {"width": z["gru"]}, "left_scale": 0.9, "right_scale": 1.1}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    copy = lambda x: json.loads(json.dumps(x))
+    tidarax = {"architecture": "Tidarax", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-5},
+               "layers": [copy({"type": "parallel", "mixer": mixer, "mlp": (dense, moe)[i % 2]}) for i in range(layers)]}
+    nz = dict(z, delta=(1, 8), rank=8, buckets=32, bias_max=1024, groups=(4, 2))
+    nufapel, loselix = nufapel_configs(nz, 3, vocab)
+    pairs = (nufapel["layers"][0], nufapel["layers"][2])
+    nufapel = dict(nufapel, layers=[copy(pairs[i % 2]) for i in range(layers)])
+    loselix = dict(loselix, layers=[copy(loselix["layers"][0]) for _ in range(layers)])
+    return tidarax, nufapel, loselix
+
+
+def tidarax_parts(model, z, layer_index, batch, tokens, reps, pk):
+    """Layer `layer_index` of a Tidarax model in parts, each alone: the attention kernel, the preparation of its queries
+    (rotation, unit norm, mixture, cache write), the recurrence (from the projected row to the gated state), the whole
+    mixer, the feed-forward and its activation.  One prompt of `tokens` tokens, then one decode step of `batch` requests at
+    CONTEXT tokens.  Rooflines: the slower of FLOPs at the measured bf16 peak and bytes at the measured copy bandwidth;
+    attention counts what the mixing needs at least, per pair of tokens and head the products with one key head, one row
+    of the mixing matrix and one value head (the kernels run the product with the whole key row instead)."""
+    import torch
+    from jax_vllm_b200 import make_driver, ops
+    from jax_vllm_b200.engine import StepEntry
+    W = z["width"]
+    flush = torch.zeros(160 << 20, dtype=torch.int16, device="cuda")
+    layer = model.layers[layer_index]
+    mixer, ff = layer.mixer, layer.feed_forward
+    att, gru = mixer.sides
+    out = {}
+    for phase in ("prefill", "decode"):
+        if phase == "prefill":
+            driver = make_driver(model, max_num_seqs=1, max_model_len=tokens + 16, block_size=PAGE, prefix_cache=False,
+                                 max_tokens_per_step=tokens, cuda_graphs=False)
+            rc = driver.cache.admit("p")
+            driver.cache.grow(rc, tokens)
+            entries = [StepEntry(rc, [(i * 7919 + 13) % 1000 for i in range(tokens)], (tokens - 1,))]
+            n, pairs, keys, seqs = tokens, tokens * (tokens + 1) // 2, tokens, 1
+        else:
+            driver = make_driver(model, max_num_seqs=batch, max_model_len=CONTEXT + 64, block_size=PAGE, prefix_cache=False,
+                                 cuda_graphs=False)
+            rcs = fake_context(driver, batch, CONTEXT)
+            for rc in rcs:
+                driver.cache.grow(rc, rc.num_tokens + 1)
+            entries = [StepEntry(rc, [b], (0,)) for b, rc in enumerate(rcs)]
+            n, pairs, keys, seqs = batch, batch * (CONTEXT + 1), batch * (CONTEXT + 1), batch
+        step = driver.runner.builder.build(entries)
+        cache = driver.runner.layer_caches[layer_index]
+        table = step.block_tables[cache[0].group]
+        x = (torch.randn((n, W), device="cuda") * 0.5).to(torch.bfloat16)
+        row = (torch.randn((n, mixer.in_rows), device="cuda") * 0.5).to(torch.bfloat16)
+        q = torch.empty((n, att.hq * att.dk), dtype=torch.bfloat16, device="cuda")
+        a = torch.empty((n, att.hq * att.dv), dtype=torch.bfloat16, device="cuda")
+        s = torch.empty((n, gru.c), dtype=torch.bfloat16, device="cuda")
+        bw, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+        prep = lambda: ops.talk_prepare(row, 0, att.k_off, att.v_off, q, att.talk, step.positions, step.token_entry, table,
+                                        att.position.table(), 1e-5, cache[0].k, cache[0].v, att.hq, att.hk, att.d, att.dv)
+        prep()
+        flops = 2 * att.hq * (att.d + att.hq + att.dv) * pairs
+        nbytes = keys * (att.hk * att.d + att.hv * att.dv) * 2 + n * att.hq * (att.dk + att.dv) * 2
+        jobs = [("attention kernel", lambda: att.attend(q, a, step, cache[0], table), (flops / tf * 1e6, nbytes / bw * 1e6)),
+                ("query preparation", prep, (0.0, n * (2 * att.in_rows - att.hq * att.d + att.hq * att.dk) * 2 / bw * 1e6)),
+                ("recurrence", lambda: gru.from_projection(row[:, att.in_rows:], step, cache[1], s),
+                 (0.0, (n * gru.c * 4 * 2 + seqs * gru.c * 8) / bw * 1e6)),
+                ("mixer", lambda: mixer.forward(x, step, cache), None)]
+        if layer_index % 2 == 0:
+            z_up = (torch.randn((n, z["ff"]), device="cuda")).to(torch.bfloat16)
+            jobs.append(("activation", lambda: ff.from_projection(z_up, step), (0.0, n * z["ff"] * 4 / bw * 1e6)))
+            ff_flops, ff_bytes = 2 * n * 2 * z["ff"] * W, 2 * z["ff"] * W * 2
+        else:
+            hit = z["experts"] * (1 - (1 - z["top"] / z["experts"]) ** n)
+            ff_flops, ff_bytes = 2 * n * z["top"] * 3 * z["eff"] * W, hit * 3 * z["eff"] * W * 2
+        jobs.append(("feed-forward", lambda: ff.forward(x, step), (ff_flops / tf * 1e6, ff_bytes / bw * 1e6)))
+        res = {}
+        for name, fn, roof in jobs:
+            us = time_part(fn, reps, flush)
+            res[name] = {"us": round(us, 1)}
+            if roof is not None:
+                ideal = max(roof)
+                res[name].update(roofline_us=round(ideal, 1), bound="flops" if roof[0] >= roof[1] else "bytes",
+                                 of_roofline=round(ideal / us, 3))
+        driver.runner.check_kernels()
+        out[phase] = res
+        del driver
+        torch.cuda.empty_cache()
+    return out
+
+
+def design_tidarax(layers, sizes, steps, warmup) -> int:
+    import torch
+    from jax_vllm_b200 import random_model, registry
+    pk, pk_src = peaks()
+    sizes = [t for t in sizes if t in TIDARAX_SIZES] or ["w2k", "w4k", "w4k8"]
+    out = {"design": "tidarax", "layers": layers, "prefill_tokens": PREFILL_TOKENS, "decode_batch": 8, "context": CONTEXT,
+           "dtype": "bf16", "data": "synthetic (random weights, seed 5)", "peaks": pk, "peak_source": pk_src, "sizes": {}}
+    for tag in sizes:
+        z = TIDARAX_SIZES[tag]
+        row = {}
+        for kind, cfg in zip(("tidarax", "nufapel", "loselix"), tidarax_configs(z, layers)):
+            model = random_model(registry.config_from_dict(cfg), seed=5, dtype="bf16", device="cuda:0")
+            with ClockSampler() as clocks:
+                pms = time_prefill(model, PREFILL_TOKENS, warmup=2, reps=5)
+                dms, launches, _, _ = time_decode(model, 8, steps, warmup)
+            row[kind] = dict(prefill_tok_s=round(PREFILL_TOKENS / (pms / 1e3), 1), prefill_ms=round(pms, 3),
+                             decode_tok_s=round(8 / (dms / 1e3), 1), decode_ms_per_step=round(dms, 4),
+                             decode_launches_per_step=launches, clocks=clocks.summary)
+            mhz = float(clocks.summary.get("sm_max_mhz") or 1965.0)
+            if kind == "loselix":
+                row[kind]["parts"] = design_parts(model, kind, dict(z, soft=(z["dim"], z["vdim"], z["dim"] // 2)), 0, 8,
+                                                  PREFILL_TOKENS, 7, pk)
+            elif kind == "nufapel":
+                # the parts' code tells dense from routed feed-forwards by the layer's number (0: dense, else routed)
+                row[kind]["parts"] = {TIDARAX_KINDS[i]: nufapel_parts(model, z, i, 8, PREFILL_TOKENS, 7, pk, mhz)
+                                      for i in range(min(2, layers))}
+            else:
+                row[kind]["config"] = dict(z)
+                row[kind]["parts"] = {TIDARAX_KINDS[i]: tidarax_parts(model, z, i, 8, PREFILL_TOKENS, 7, pk)
+                                      for i in range(min(2, layers))}
+            del model
+            torch.cuda.empty_cache()
+        out["sizes"][tag] = row
+    print(json.dumps(out))
+    return 0
+
+
 def reference_arm():
     why = ("the reference (jllm) needs jax, jaxlib and equinox and the hatchling build backend; none is installed "
            "and none is in the offline wheelhouse, so it can neither be installed nor run here")
@@ -1132,12 +1282,13 @@ def main():
     ap.add_argument("--with-workloads", action="store_true",
                     help="after the headline run, also run the two serving workloads and add their lines under `workloads`")
     ap.add_argument("--design", default=None, metavar="NAME",
-                    help="guronex, loselix, nufapel or gogivik: that design's prefill and decode throughput at a few layer sizes "
-                         "beside its closest neighbour of equal size (Qwen3; for nufapel, Loselix), with the rooflines of "
+                    help="guronex, loselix, nufapel, gogivik or tidarax: that design's prefill and decode throughput at a few layer sizes "
+                         "beside its closest neighbours of equal size (Qwen3; later designs beside earlier ones), with the rooflines of "
                          "its kernels (see design())")
     ap.add_argument("--sizes", default="lite,mid,row576",
                     help="with --design: which of its layer sizes, comma-separated (guronex: lite,mid,row576; loselix: "
-                         "w2k,w4k,mix, all by default; nufapel and gogivik: w2k,w4k,small, the first two by default)")
+                         "w2k,w4k,mix, all by default; nufapel and gogivik: w2k,w4k,small, the first two by default; tidarax: w2k,w4k,w4k8,small, the "
+                         "first three by default)")
     ap.add_argument("--micro-eager", action="store_true",
                     help="with --micro: plain launches instead of replays of a CUDA graph (for a profiler)")
     args = ap.parse_args()
