@@ -4,10 +4,12 @@
 //
 // Every query head reads every byte of the keys, so a block takes ALL heads of one request over a range of keys (grid:
 // request x range) and each cached byte is read once from memory.  Tiles of KT keys come in by bulk copies (one a key row,
-// one a value row) into two stages, the next tile's under way while this one is worked on:
+// one a value row) into two stages, the next tile's under way while this one is worked on; two blocks share a
+// multiprocessor where their stages allow it:
 //   scores     S [H, KT] = Q [H, KD] K^T on the tensor cores (mma.sync m16n8k16, 32-bit accumulation): a warp takes 16 heads
-//              x 8 keys, and where that gives fewer than eight pieces of work, a part of KD
-//   softmax    running (max, sum) a head in 32-bit, one warp a head, one lane a key
+//              and a part of KD, keeps its piece of the queries in registers for the whole range, and goes over the keys of
+//              the tile; the parts of a score are added up by its reader
+//   softmax    running (max, sum) a head in 32-bit, eight lanes a head
 //   output     O [H, DV] += P V in 32-bit on the CUDA cores: a thread keeps two columns of a value head for all query heads
 //              that read it (a decoded token's few rows would leave most of a tensor-core tile empty); P stays 32-bit
 // Each range leaves its unnormalised output and (max, sum); a second kernel merges a head's ranges in ascending order and
@@ -19,6 +21,7 @@
 namespace {
 constexpr int THREADS = 256, WARPS = THREADS / 32;
 constexpr int MAX_SPLIT = 256;                  // keys of a range
+constexpr int MAX_HEADS = 128;
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct Params {
@@ -31,7 +34,7 @@ struct Params {
   int H, G, KD, DV, page_size, num_pages;
   float scale_log2, out_scale;
   const float* sink;           // [H] or null
-  int KT, k_parts;             // keys of a tile; parts of KD that warps share a score tile in
+  int KT, k_parts;             // keys of a tile; parts of KD that warps share the scores of 16 heads in
   int split_size, n_splits;
   int* status;
 };
@@ -55,29 +58,28 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
 
 // Offsets (bytes) of the arrays in dynamic shared memory, for the kernel and its launcher.
 struct Layout {
-  int q_row, k_row, v_row, s_row;              // elements from row to row
-  size_t q, k, v, s, total;                    // s: [k_parts][H16][s_row] floats
+  int k_row, v_row, s_row;                     // elements from row to row
+  size_t k, v, s, total;                       // s: [k_parts][H16][s_row] floats
   __host__ __device__ Layout(int H, int G, int KD, int DV, int KT, int k_parts) {
     const int H16 = (H + 15) / 16 * 16;
-    q_row = k_row = KD + 8; v_row = G * DV; s_row = KT + 4;
-    q = 0;
-    k = q + sizeof(__nv_bfloat16) * (size_t)H16 * q_row;
+    k_row = KD + 8; v_row = G * DV; s_row = KT + 4;
+    k = 0;
     v = k + sizeof(__nv_bfloat16) * (size_t)2 * KT * k_row;
     s = v + sizeof(__nv_bfloat16) * (size_t)2 * KT * v_row;
     total = s + sizeof(float) * (size_t)k_parts * H16 * s_row;
   }
 };
 
-// HT: query heads of a value head, rounded up; IT: column pairs a thread keeps.
-template <int HT, int IT>
-__global__ void __launch_bounds__(THREADS) attn_rows_decode_kernel(const Params p) {
+// HT: query heads of a value head, rounded up; IT: column pairs a thread keeps; KS: steps of 16 elements of KD a warp keeps
+// of the queries.
+template <int HT, int IT, int KS>
+__global__ void __launch_bounds__(THREADS, HT * IT <= 16 ? 2 : 1) attn_rows_decode_kernel(const Params p) {
   extern __shared__ __align__(128) unsigned char smem[];
   __shared__ long long slots[MAX_SPLIT];        // cache slot of every key of the range (-1: none)
-  __shared__ float row_m[256], row_l[256], row_alpha[256];
+  __shared__ float row_m[MAX_HEADS], row_l[MAX_HEADS], row_alpha[MAX_HEADS];
   __shared__ __align__(8) uint64_t bars[2];
   const int H = p.H, G = p.G, KD = p.KD, DV = p.DV, KT = p.KT, HPT = H / G;
   const Layout L(H, G, KD, DV, KT, p.k_parts);
-  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem + L.q);
   __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(smem + L.k);
   __nv_bfloat16* vs = reinterpret_cast<__nv_bfloat16*>(smem + L.v);
   float* ss = reinterpret_cast<float*>(smem + L.s);
@@ -103,14 +105,7 @@ __global__ void __launch_bounds__(THREADS) attn_rows_decode_kernel(const Params 
     else s = (long long)page * p.page_size + (j - pi * p.page_size);
     slots[i] = s;
   }
-  const int H16 = (H + 15) / 16 * 16, CH = KD / 8;
-  for (int c = tid; c < H16 * CH; c += THREADS) {
-    const int h = c / CH, part = c - h * CH;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (h < H) v = *reinterpret_cast<const uint4*>(p.q + (size_t)token * p.q_stride + (size_t)h * KD + part * 8);
-    *reinterpret_cast<uint4*>(qs + (size_t)h * L.q_row + part * 8) = v;
-  }
-  for (int h = tid; h < H; h += THREADS) { row_m[h] = -INFINITY; row_l[h] = 0.f; }
+  for (int h = tid; h < MAX_HEADS; h += THREADS) { row_m[h] = -INFINITY; row_l[h] = 0.f; }
   __syncthreads();
 
   const int n_tiles = (j_hi - j_lo + KT - 1) / KT;
@@ -138,6 +133,26 @@ __global__ void __launch_bounds__(THREADS) attn_rows_decode_kernel(const Params 
   issue(0);
   if (n_tiles > 1) issue(1);
 
+  // ---- this warp's queries: 16 heads, k steps [k0, k1) of 16 elements, as operand fragments
+  const int H16 = (H + 15) / 16 * 16, mt = H16 / 16, kp = p.k_parts, k_steps = KD / 16;
+  const int m16 = warp % mt, part = warp / mt;
+  const bool scores_here = part < kp;
+  const int k0 = k_steps * part / kp, k1 = scores_here ? k_steps * (part + 1) / kp : k0;
+  uint32_t qa[KS][4];
+  {
+    const int h0 = m16 * 16 + (lane >> 2), h1 = h0 + 8;
+    const __nv_bfloat16* q0 = p.q + (size_t)token * p.q_stride + (lane & 3) * 2;
+#pragma unroll
+    for (int i = 0; i < KS; ++i) {
+      const int k = (k0 + i) * 16;
+      const bool in = k0 + i < k1;
+      qa[i][0] = in && h0 < H ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)h0 * KD + k) : 0u;
+      qa[i][1] = in && h1 < H ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)h1 * KD + k) : 0u;
+      qa[i][2] = in && h0 < H ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)h0 * KD + k + 8) : 0u;
+      qa[i][3] = in && h1 < H ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)h1 * KD + k + 8) : 0u;
+    }
+  }
+
   // ---- this thread's columns of the output
   const int pairs = G * DV / 2;
   float acc[IT][HT][2];
@@ -146,7 +161,6 @@ __global__ void __launch_bounds__(THREADS) attn_rows_decode_kernel(const Params 
 #pragma unroll
     for (int g = 0; g < HT; ++g) acc[i][g][0] = acc[i][g][1] = 0.f;
 
-  const int mt = H16 / 16, nt = KT / 8, kp = p.k_parts, k_steps = KD / 16;
   for (int t = 0; t < n_tiles; ++t) {
     const int buf = t & 1;
     // every thread takes the same way out: all saw the tile, or the block stops (status word set)
@@ -156,66 +170,65 @@ __global__ void __launch_bounds__(THREADS) attn_rows_decode_kernel(const Params 
       if (t + 1 < n_tiles) mbar_wait(&bars[buf ^ 1], ((t + 1) >> 1) & 1);
       return;
     }
-    // ---- scores
-    for (int u = warp; u < mt * nt * kp; u += WARPS) {
-      const int part = u % kp, n8 = (u / kp) % nt, m16 = u / (kp * nt);
-      const int k0 = k_steps * part / kp, k1 = k_steps * (part + 1) / kp;
-      const __nv_bfloat16* qa = qs + (size_t)(m16 * 16 + (lane & 15)) * L.q_row + (lane >> 4) * 8;
-      const __nv_bfloat16* kb = ks + (size_t)(buf * KT + n8 * 8 + (lane & 7)) * L.k_row + ((lane >> 3) & 3) * 8;
-      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
-      int k = k0;
-#pragma unroll 2
-      for (; k + 2 <= k1; k += 2) {              // two independent sums
-        uint32_t a0[4], a1[4], b[4];
-        ldmatrix_x4(a0, qa + k * 16);
-        ldmatrix_x4(a1, qa + k * 16 + 16);
-        ldmatrix_x4(b, kb + k * 16);
-        mma_bf16(c0, a0, b[0], b[1]);
-        mma_bf16(c1, a1, b[2], b[3]);
+    // ---- scores: 8 keys at a time
+    if (scores_here) {
+      const __nv_bfloat16* kb = ks + (size_t)(buf * KT + (lane & 7)) * L.k_row + k0 * 16 + (lane >> 3) * 8;
+      float* dst = ss + ((size_t)part * H16 + m16 * 16 + (lane >> 2)) * L.s_row + (lane & 3) * 2;
+      const int n_here = k1 - k0;
+      for (int n8 = 0; n8 < KT / 8; ++n8, kb += 8 * L.k_row, dst += 8) {
+        float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < KS; i += 2) {          // two independent sums
+          if (i + 1 < n_here) {
+            uint32_t b[4];
+            ldmatrix_x4(b, kb + i * 16);
+            mma_bf16(c0, qa[i], b[0], b[1]);
+            mma_bf16(c1, qa[i + 1], b[2], b[3]);
+          } else if (i < n_here) {                 // one step is left: the upper lanes' addresses are not used
+            uint32_t b[2];
+            ldmatrix_x2(b, kb + i * 16 - ((lane & 16) ? 16 : 0));
+            mma_bf16(c0, qa[i], b[0], b[1]);
+          }
+        }
+        *reinterpret_cast<float2*>(dst) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
+        *reinterpret_cast<float2*>(dst + 8 * L.s_row) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
       }
-      if (k < k1) {
-        uint32_t a0[4], b[2];
-        ldmatrix_x4(a0, qa + k * 16);
-        ldmatrix_x2(b, ks + (size_t)(buf * KT + n8 * 8 + (lane & 7)) * L.k_row + ((lane >> 3) & 1) * 8 + k * 16);
-        mma_bf16(c0, a0, b[0], b[1]);
-      }
-      float* dst = ss + ((size_t)part * H16 + m16 * 16 + (lane >> 2)) * L.s_row + n8 * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(dst) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
-      *reinterpret_cast<float2*>(dst + 8 * L.s_row) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
     __syncthreads();
-    // ---- softmax: one warp a head; the weights replace the first part's scores
+    // ---- softmax: eight lanes a head; the weights replace the first part's scores
     const int here = min(KT, j_hi - j_lo - t * KT);
-    for (int h = warp; h < H; h += WARPS) {
+    for (int h = tid >> 3; h < H16; h += THREADS / 8) {        // whole warps stay together: H16 is a multiple of 4
       float* row = ss + (size_t)h * L.s_row;
-      float v[2];
+      float v[8];
       float mx = -INFINITY;
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int j = lane + 32 * i;
+      for (int i = 0; i < 8; ++i) {
+        const int j = (lane & 7) + 8 * i;
         v[i] = -INFINITY;
         if (j < here) {
-          float s = row[j];
-          for (int q = 1; q < kp; ++q) s += row[(size_t)q * H16 * L.s_row + j];
-          v[i] = s * p.scale_log2;
+          float x = row[j];
+          for (int q = 1; q < kp; ++q) x += row[(size_t)q * H16 * L.s_row + j];
+          v[i] = x * p.scale_log2;
         }
         mx = fmaxf(mx, v[i]);
       }
-      mx = warp_max(mx);
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       const float m_old = row_m[h], m_new = fmaxf(m_old, mx);          // finite: a tile has at least one key
       float sum = 0.f;
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int j = lane + 32 * i;
+      for (int i = 0; i < 8; ++i) {
+        const int j = (lane & 7) + 8 * i;
         if (j < KT) {
           const float e = j < here ? exp2f(v[i] - m_new) : 0.f;
           row[j] = e;
           sum += e;
         }
       }
-      sum = warp_sum(sum);
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
       __syncwarp();
-      if (lane == 0) {
+      if ((lane & 7) == 0) {
         const float alpha = m_old == -INFINITY ? 0.f : exp2f(m_old - m_new);
         row_alpha[h] = alpha;
         row_m[h] = m_new;
@@ -279,61 +292,79 @@ __global__ void __launch_bounds__(THREADS) attn_rows_decode_kernel(const Params 
 
 // One block a (request, head): the ranges in ascending order; maxima are exponents of two.
 __global__ void __launch_bounds__(128) attn_rows_merge_kernel(const Params p) {
+  __shared__ float weight[128];
   pdl_trigger();
   pdl_wait();
-  const int entry = p.work[2 * blockIdx.x], h = blockIdx.y;
-  const int last = min(p.start_pos[entry] / p.split_size, p.n_splits - 1);
+  const int entry = p.work[2 * blockIdx.x], h = blockIdx.y, lane = threadIdx.x & 31;
+  const int n = min(p.start_pos[entry] / p.split_size, p.n_splits - 1) + 1;
   const size_t base = ((size_t)blockIdx.x * p.H + h) * p.n_splits;
-  // the sink is one more part, with no value: maximum sink, sum 1
+  const float2* ml = reinterpret_cast<const float2*>(p.part_ml) + base;
+  // the sink is one more part, with no value: maximum sink, sum 1; every warp forms the maximum and the sum for itself
   const float sk = p.sink != nullptr ? p.sink[h] * LOG2E : -INFINITY;
   float m = sk;
-  for (int s = 0; s <= last; ++s) m = fmaxf(m, p.part_ml[2 * (base + s)]);
-  float l = p.sink != nullptr ? exp2f(sk - m) : 0.f;
-  for (int s = 0; s <= last; ++s) l += exp2f(p.part_ml[2 * (base + s)] - m) * p.part_ml[2 * (base + s) + 1];
+  for (int s = lane; s < n; s += 32) m = fmaxf(m, ml[s].x);
+  m = warp_max(m);
+  float l = 0.f;
+  for (int s = lane; s < n; s += 32) l += exp2f(ml[s].x - m) * ml[s].y;
+  l = warp_sum(l) + (p.sink != nullptr ? exp2f(sk - m) : 0.f);
   const float inv = p.out_scale / l;
-  for (int d = threadIdx.x; d < p.DV; d += blockDim.x) {
+  const size_t out_at = (size_t)p.cu_seqlens[entry] * p.out_stride + (size_t)h * p.DV;
+  for (int d0 = 0; d0 < p.DV; d0 += 128) {
+    const int d = d0 + threadIdx.x;
     float o = 0.f;
-#pragma unroll 4
-    for (int s = 0; s <= last; ++s) o = fmaf(exp2f(p.part_ml[2 * (base + s)] - m), p.part_o[(base + s) * p.DV + d], o);
-    p.out[(size_t)p.cu_seqlens[entry] * p.out_stride + (size_t)h * p.DV + d] = __float2bfloat16_rn(o * inv);
+    for (int s0 = 0; s0 < n; s0 += 128) {
+      __syncthreads();
+      if (s0 + (int)threadIdx.x < n) weight[threadIdx.x] = exp2f(ml[s0 + threadIdx.x].x - m);
+      __syncthreads();
+      const int upto = min(128, n - s0);
+      if (d < p.DV) {
+        const float* src = p.part_o + (base + s0) * p.DV + d;
+#pragma unroll 8
+        for (int s = 0; s < upto; ++s) o = fmaf(weight[s], src[(size_t)s * p.DV], o);
+      }
+    }
+    if (d < p.DV) p.out[out_at + d] = __float2bfloat16_rn(o * inv);
   }
 }
 
-// Keys of a tile: as many as let two stages fit beside the queries, 64 at most.
-int tile_keys(int H, int G, int KD, int DV, int* k_parts) {
-  const int H16 = (H + 15) / 16 * 16;
-  for (int kt = 64; kt >= 16; kt /= 2) {
-    int kp = 1;
-    while (kp < 8 && (H16 / 16) * (kt / 8) * kp < WARPS && KD / 16 >= 2 * kp) kp *= 2;
-    if (2 * kt * 2 * (size_t)(KD + G * DV) <= 132 * 1024 && Layout(H, G, KD, DV, kt, kp).total <= 220 * 1024) {
-      *k_parts = kp;
-      return kt;
-    }
-  }
+// Parts of KD that the warps of 16 heads share.
+int parts_of(int H) { return WARPS / ((H + 15) / 16); }
+
+// Keys of a tile: as many as let two blocks share a multiprocessor, 64 at most and 8 at least (then one block may need
+// most of the shared memory).
+int tile_keys(int H, int G, int KD, int DV) {
+  for (int kt = 64; kt >= 8; kt /= 2)
+    if (Layout(H, G, KD, DV, kt, parts_of(H)).total <= (kt > 8 ? 104 : 200) * 1024) return kt;
   return 0;
 }
 
-template <int HT, int IT>
+template <int HT, int IT, int KS>
 int launch(const Params& p, int n_work, size_t smem, cudaStream_t stream) {
-  auto kern = attn_rows_decode_kernel<HT, IT>;
+  auto kern = attn_rows_decode_kernel<HT, IT, KS>;
   static bool ready[JV_MAX_DEVICES];
   if (!jv_once_per_device(ready, [&] {
-        return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) == cudaSuccess;
+        return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) == cudaSuccess;
       }))
     return JV_ERR_UNSUPPORTED;
   const int rc = jv_launch(kern, dim3(n_work, p.n_splits), dim3(THREADS), smem, stream, p);
   if (rc != JV_OK) return rc;
   return jv_launch(attn_rows_merge_kernel, dim3(n_work, p.H), dim3(128), 0, stream, p);
 }
+
+template <int HT, int IT>
+int launch_steps(const Params& p, int n_work, size_t smem, cudaStream_t stream) {
+  return (p.KD / 16 + p.k_parts - 1) / p.k_parts <= 8 ? launch<HT, IT, 8>(p, n_work, smem, stream)
+                                                      : launch<HT, IT, 16>(p, n_work, smem, stream);
+}
 }  // namespace
 
-// 1 if the kernel takes these sizes: KD a multiple of 16, DV of 8, up to 16 query heads a value head and 256 in all.
+// 1 if the kernel takes these sizes: KD a multiple of 16, DV of 8, up to 16 query heads a value head and 128 in all, and
+// what a thread keeps in registers: 16 steps of the queries, 32 pairs of outputs.
 JV_EXPORT int jv_attn_rows_decode_supports(int H, int G, int KD, int DV) {
-  if (G < 1 || H < 1 || H % G || H > 256 || KD % 16 || KD < 16 || DV % 8 || DV < 8) return 0;
+  if (G < 1 || H < 1 || H % G || H > MAX_HEADS || KD % 16 || KD < 16 || DV % 8 || DV < 8) return 0;
   const int hpt = H / G, ht = hpt <= 4 ? 4 : hpt <= 8 ? 8 : 16;
   const int it = (G * DV / 2 + THREADS - 1) / THREADS;
-  int kp;
-  return hpt <= 16 && it <= 4 && ht * it <= 32 && tile_keys(H, G, KD, DV, &kp) > 0;
+  return hpt <= 16 && it <= 4 && ht * it <= 32 && (KD / 16 + parts_of(H) - 1) / parts_of(H) <= 16 && tile_keys(H, G, KD, DV) > 0;
 }
 
 // q: rows of q_stride elements, head h of a token at column h*KD; out: rows of out_stride, head h at h*DV; k_cache:
@@ -355,12 +386,12 @@ JV_EXPORT int jv_attn_rows_decode(const void* q, int q_stride, void* out, int ou
   p.block_table = block_table; p.table_width = table_width; p.cu_seqlens = cu_seqlens; p.start_pos = start_pos; p.work = work;
   p.H = H; p.G = G; p.KD = KD; p.DV = DV; p.page_size = page_size; p.num_pages = num_pages; p.scale_log2 = scale * LOG2E;
   p.out_scale = out_scale; p.sink = sink; p.split_size = split_size; p.n_splits = n_splits; p.status = status;
-  p.KT = tile_keys(H, G, KD, DV, &p.k_parts);
+  p.KT = tile_keys(H, G, KD, DV); p.k_parts = parts_of(H);
   const size_t smem = Layout(H, G, KD, DV, p.KT, p.k_parts).total;
   const int hpt = H / G, it = (G * DV / 2 + THREADS - 1) / THREADS;
-  if (hpt <= 4) return it <= 1 ? launch<4, 1>(p, n_work, smem, stream) : it <= 2 ? launch<4, 2>(p, n_work, smem, stream)
-                                                                                 : launch<4, 4>(p, n_work, smem, stream);
-  if (hpt <= 8) return it <= 1 ? launch<8, 1>(p, n_work, smem, stream) : it <= 2 ? launch<8, 2>(p, n_work, smem, stream)
-                                                                                 : launch<8, 4>(p, n_work, smem, stream);
-  return it <= 1 ? launch<16, 1>(p, n_work, smem, stream) : launch<16, 2>(p, n_work, smem, stream);
+  if (hpt <= 4) return it <= 1 ? launch_steps<4, 1>(p, n_work, smem, stream) : it <= 2 ? launch_steps<4, 2>(p, n_work, smem, stream)
+                                                                                       : launch_steps<4, 4>(p, n_work, smem, stream);
+  if (hpt <= 8) return it <= 1 ? launch_steps<8, 1>(p, n_work, smem, stream) : it <= 2 ? launch_steps<8, 2>(p, n_work, smem, stream)
+                                                                                       : launch_steps<8, 4>(p, n_work, smem, stream);
+  return it <= 1 ? launch_steps<16, 1>(p, n_work, smem, stream) : launch_steps<16, 2>(p, n_work, smem, stream);
 }

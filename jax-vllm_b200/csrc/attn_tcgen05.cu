@@ -20,24 +20,14 @@
 //            exp2, write P; when a row's maximum has moved, rescale O in TMEM first.  At an item's end O / sum
 //            leaves through the item's query buffer and a TMA store.
 // The score buffer of the next tile (of this item or the next) is filled while the softmax of a tile runs.
-//
-// Key rows of several pieces (`chunks` NC > 1): the scores of every query head are the product of the token's WHOLE key row,
-// NC pieces of 128 (its key heads side by side), with a query of the same size, under one value head per group of query
-// heads as before (scores mixed across heads: talk_prepare.cu forms such queries).  S = sum_c Q_c K_c^T then accumulates
-// over the pieces; a stage of keys is one piece of a tile.  Up to four pieces the queries of an item stay in shared memory
-// (two items of two pieces, or one item of three or four); more pieces stream with the keys, a stage being the pair
-// (Q_c, K_c).
 // Shared memory moves 128 bytes a clock, which a 128x128x16 product with both operands there needs all by
 // itself: P therefore never goes through shared memory.  Every mbarrier wait is bounded by a clock deadline and
 // reports to the status word instead of spinning.
 //
 // Restrictions (the caller falls back to the mma.sync kernel otherwise): bfloat16, head size 128, no
 // window, HPT up to 16, page size a power of two from 8 to 128.
-#include "common.cuh"
-#include "mbarrier.cuh"
+#include "tcgen05.cuh"
 
-#include <cuda.h>
-#include <cudaTypedefs.h>
 #include <math.h>
 
 namespace {
@@ -45,16 +35,7 @@ namespace {
 constexpr int D = 128, ROWS = 128, BN = 128;
 constexpr int TILE_BYTES = 128 * 128 * 2;       // a 128 x 128 bfloat16 tile: two halves of [128 rows][128 bytes]
 constexpr int HALF_BYTES = 128 * 128;            // one half: 128 rows of 128 bytes
-constexpr int MAX_STAGES = 3;
-constexpr int SMEM_TILES = 7;                    // 7 tiles of 32 KB
-// How the tiles are used, by the number of pieces of a key row NC (0: any number, streamed with their queries): queries of
-// QB items, KS stages of keys, VS stages of values.
-template <int NC> struct Plan;
-template <> struct Plan<1> { static constexpr int QB = 2, KS = 2, VS = 3; static constexpr bool STREAM = false; };
-template <> struct Plan<2> { static constexpr int QB = 2, KS = 2, VS = 1; static constexpr bool STREAM = false; };
-template <> struct Plan<3> { static constexpr int QB = 1, KS = 3, VS = 1; static constexpr bool STREAM = false; };
-template <> struct Plan<4> { static constexpr int QB = 1, KS = 2, VS = 1; static constexpr bool STREAM = false; };
-template <> struct Plan<0> { static constexpr int QB = 1, KS = 2, VS = 2; static constexpr bool STREAM = true; };   // and one tile for the output
+constexpr int K_STAGES = 2, V_STAGES = 3, Q_BUFFERS = 2;   // 7 tiles of 32 KB
 constexpr int THREADS = 352;                     // key producer warp, mma warp, 8 softmax warps, value producer warp
 constexpr int SOFTMAX_THREADS = 256;
 constexpr int TMEM_COLS = 512;                   // S0: [0,128)  S1: [128,256)  O: [256,384)  P0: [384,448)  P1: [448,512)
@@ -73,163 +54,18 @@ struct Params {
   // added to the score of key j (untouched by the scales); exp(sink[h]) counts once in the denominator.  Each may be null.
   const float* head_scale; const float* dist_bias; int n_dist; const float* sink;
   int window;                  // the mask as one number (common.cuh, first_visible): 0, a window (> 0) or chunks (< 0)
-  int chunks;                  // pieces of 128 of a key row that all heads share (1: key heads of their own, one a group)
   float out_scale;             // multiplies the output
   int* status;
 };
 
-__device__ __forceinline__ void tma_load_3d(void* dst, const CUtensorMap* map, int x, int y, int z, uint64_t* bar) {
-  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];\n"
-               ::"r"(smem_u32(dst)), "l"(map), "r"(x), "r"(y), "r"(z), "r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void tma_load_4d(void* dst, const CUtensorMap* map, int x, int y, int z, int w, uint64_t* bar) {
-  asm volatile("cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5}], [%6];\n"
-               ::"r"(smem_u32(dst)), "l"(map), "r"(x), "r"(y), "r"(z), "r"(w), "r"(smem_u32(bar)) : "memory");
-}
-
-__device__ __forceinline__ void tma_store_3d(const CUtensorMap* map, const void* src, int x, int y, int z) {
-  asm volatile("cp.async.bulk.tensor.3d.global.shared::cta.bulk_group [%0, {%1, %2, %3}], [%4];\n"
-               ::"l"(map), "r"(x), "r"(y), "r"(z), "r"(smem_u32(src)) : "memory");
-}
-
-// Descriptor of a K-major operand tile (rows of 128 bytes along k, 8-row groups 1024 bytes apart, 128-byte swizzle).
-__device__ __forceinline__ uint64_t desc_k_major(uint32_t addr) {
-  return (uint64_t)((addr & 0x3FFFF) >> 4) | ((uint64_t)1 << 16) | ((uint64_t)(1024 >> 4) << 32) | ((uint64_t)1 << 46) |
-         ((uint64_t)2 << 61);
-}
-// Descriptor of an MN-major operand tile: rows of 128 bytes run along n (64 elements), consecutive rows are
-// consecutive k, 8 rows = 1024 bytes (stride byte offset); the next 64 n are HALF_BYTES further (leading byte offset).
-__device__ __forceinline__ uint64_t desc_mn_major(uint32_t addr) {
-  return (uint64_t)((addr & 0x3FFFF) >> 4) | ((uint64_t)(HALF_BYTES >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) |
-         ((uint64_t)1 << 46) | ((uint64_t)2 << 61);
-}
-// bfloat16 x bfloat16 -> float, M = 128, N = 128; B K-major (S = Q K^T) or MN-major (O = P V).
-constexpr uint32_t IDESC_QK = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(128 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-constexpr uint32_t IDESC_PV = IDESC_QK | (1u << 16);
-
-__device__ __forceinline__ void umma(uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile("{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-               "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}\n"
-               ::"r"(tmem_d), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
-}
-// The same with the A operand in tensor memory (rows = lanes, two 16-bit elements of k per column).
-__device__ __forceinline__ void umma_a_tmem(uint32_t tmem_d, uint32_t tmem_a, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile("{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-               "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}\n"
-               ::"r"(tmem_d), "r"(tmem_a), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
-}
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, float (&v)[32]) {
-  uint32_t r[32];
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-      "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];\n"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
-        "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
-        "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr));
-  asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
-#pragma unroll
-  for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-}
-// The same without waiting: several loads can be in flight; tmem_ld_wait() before the values are used.
-__device__ __forceinline__ void tmem_ld32_issue(uint32_t taddr, uint32_t (&r)[32]) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-      "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];\n"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
-        "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
-        "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory"); }
-
-__device__ __forceinline__ void tmem_st32(uint32_t taddr, const float (&v)[32]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};\n"
-      ::"r"(taddr), "r"(__float_as_uint(v[0])), "r"(__float_as_uint(v[1])), "r"(__float_as_uint(v[2])), "r"(__float_as_uint(v[3])),
-        "r"(__float_as_uint(v[4])), "r"(__float_as_uint(v[5])), "r"(__float_as_uint(v[6])), "r"(__float_as_uint(v[7])),
-        "r"(__float_as_uint(v[8])), "r"(__float_as_uint(v[9])), "r"(__float_as_uint(v[10])), "r"(__float_as_uint(v[11])),
-        "r"(__float_as_uint(v[12])), "r"(__float_as_uint(v[13])), "r"(__float_as_uint(v[14])), "r"(__float_as_uint(v[15])),
-        "r"(__float_as_uint(v[16])), "r"(__float_as_uint(v[17])), "r"(__float_as_uint(v[18])), "r"(__float_as_uint(v[19])),
-        "r"(__float_as_uint(v[20])), "r"(__float_as_uint(v[21])), "r"(__float_as_uint(v[22])), "r"(__float_as_uint(v[23])),
-        "r"(__float_as_uint(v[24])), "r"(__float_as_uint(v[25])), "r"(__float_as_uint(v[26])), "r"(__float_as_uint(v[27])),
-        "r"(__float_as_uint(v[28])), "r"(__float_as_uint(v[29])), "r"(__float_as_uint(v[30])), "r"(__float_as_uint(v[31]))
-      : "memory");
-  asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
-}
-// 1 / x to about 2^-23 relative (1 / inf = 0): the weights it makes are rounded to bfloat16 right away
-__device__ __forceinline__ float fast_rcp(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ float fast_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ void tmem_st32_bits(uint32_t taddr, const uint32_t (&v)[32]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};\n"
-      ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]),
-        "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]), "r"(v[16]), "r"(v[17]), "r"(v[18]), "r"(v[19]),
-        "r"(v[20]), "r"(v[21]), "r"(v[22]), "r"(v[23]), "r"(v[24]), "r"(v[25]), "r"(v[26]), "r"(v[27]), "r"(v[28]), "r"(v[29]),
-        "r"(v[30]), "r"(v[31])
-      : "memory");
-  asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
-}
-__device__ __forceinline__ float max3(float a, float b, float c) {
-  float d;
-  asm("max.f32 %0, %1, %2, %3;\n" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-  return d;
-}
-// Two 32-bit floats in one 64-bit register pair, for the packed fma and add of sm_100.
-__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %2};\n" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ void unpack2(uint64_t v, float& lo, float& hi) {
-  asm("mov.b64 {%0, %1}, %2;\n" : "=f"(lo), "=f"(hi) : "l"(v));
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
-  uint64_t d;
-  asm("add.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-#define TC_FENCE_BEFORE() asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory")
-#define TC_FENCE_AFTER() asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory")
-#define PROXY_FENCE() asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory")
-
-// Barrier of the two softmax warps that share 32 rows (64 threads; barriers 1..4, one for each pair) that also
-// tells every one of them whether any had `flag` set.
-__device__ __forceinline__ bool pair_barrier_or(int quad, bool flag) {
-  uint32_t any;
-  asm volatile("{\n.reg .pred p, q;\nsetp.ne.b32 q, %2, 0;\nbar.red.or.pred p, %1, 64, q;\nselp.u32 %0, 1, 0, p;\n}\n"
-               : "=r"(any) : "r"(quad + 1), "r"((uint32_t)flag) : "memory");
-  return any != 0;
-}
-__device__ __forceinline__ void pair_barrier(int quad) { asm volatile("bar.sync %0, 64;\n" ::"r"(quad + 1) : "memory"); }
-
 struct Shared {
-  // queries: one pair of barriers an item's buffer; with one buffer (QB = 1) pair 0 is for the item's first piece, through
-  // whose place the output leaves, and pair 1 for the others, which are free as soon as the item's last scores are formed
-  uint64_t q_full[2], q_free[2], k_full[MAX_STAGES], k_empty[MAX_STAGES], v_full[MAX_STAGES], v_empty[MAX_STAGES];
+  uint64_t q_full[Q_BUFFERS], q_free[Q_BUFFERS], k_full[K_STAGES], k_empty[K_STAGES], v_full[V_STAGES], v_empty[V_STAGES];
   uint64_t s_full[2], p_full[2], o_done[2];
   uint64_t o_free;              // the softmax threads have read an item's output: the next item's may be written
   uint64_t drain;               // used only after a wait ran out (see the tear-down)
   uint32_t tmem_base;
   int failed;                   // a role gave up on a wait
-  int armed_q[2], armed_k[MAX_STAGES], armed_v[MAX_STAGES];   // parity of the phase a producer armed last; -1: never
+  int armed_q[Q_BUFFERS], armed_k[K_STAGES], armed_v[V_STAGES];   // parity of the phase a producer armed last; -1: never
   float xch[2][128];            // a row's two softmax threads exchange their maxima (and at the end their sums)
 };
 
@@ -241,25 +77,18 @@ struct Item {
   int tile0, n_tiles;               // the first key tile (keys tile0 * BN ..) and the number of key tiles
 };
 
-template <int NCT>
 __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map,
                                                                   const __grid_constant__ CUtensorMap k_map,
                                                                   const __grid_constant__ CUtensorMap v_map,
                                                                   const __grid_constant__ CUtensorMap out_map,
                                                                   const Params p) {
-  using PL = Plan<NCT>;
-  constexpr int QB = PL::QB, K_STAGES = PL::KS, V_STAGES = PL::VS;
-  constexpr bool STREAM = PL::STREAM;
-  constexpr bool ONE_BUFFER = !STREAM && QB == 1;
-  const int NC = NCT > 0 ? NCT : p.chunks;
   pdl_trigger();      // a kernel launched behind this one (decode attention of the same step) may take the multiprocessors that the first blocks to end leave free
   extern __shared__ unsigned char smem_raw[];
   unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
-  unsigned char* q_s = base;                                   // [buffers][pieces][2 halves of d][128 rows][128 B]; streamed: the output's tile
-  unsigned char* k_s = q_s + (STREAM ? 1 : QB * NCT) * TILE_BYTES;             // [stages] tiles [2 halves of d][128 keys][128 B]; streamed:
-  unsigned char* v_s = k_s + (STREAM ? 2 : 1) * K_STAGES * TILE_BYTES;         //   the piece's queries, then its keys
-  Shared* sh = reinterpret_cast<Shared*>(base + SMEM_TILES * TILE_BYTES);      // [stages][2 halves of d][128 keys][128 B] values before it
-  constexpr int K_STRIDE = (STREAM ? 2 : 1) * TILE_BYTES, K_OFF = STREAM ? TILE_BYTES : 0;
+  unsigned char* q_s = base;                                   // [buffers][2 halves of d][128 rows][128 B]
+  unsigned char* k_s = q_s + Q_BUFFERS * TILE_BYTES;           // [stages][2 halves of d][128 keys][128 B]
+  unsigned char* v_s = k_s + K_STAGES * TILE_BYTES;            // [stages][2 halves of d][128 keys][128 B]
+  Shared* sh = reinterpret_cast<Shared*>(v_s + V_STAGES * TILE_BYTES);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int G = p.n_q_heads / p.n_kv_heads, HPT = p.hpt;
   const int n_items = p.n_work * p.n_kv_heads, n_blocks = gridDim.x;
@@ -291,7 +120,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
   };
 
   if (threadIdx.x == 0) {
-    for (int b = 0; b < 2; ++b) { mbar_init(&sh->q_full[b], 1); mbar_init(&sh->q_free[b], 1); sh->armed_q[b] = -1; }
+    for (int b = 0; b < Q_BUFFERS; ++b) { mbar_init(&sh->q_full[b], 1); mbar_init(&sh->q_free[b], 1); sh->armed_q[b] = -1; }
     for (int s = 0; s < K_STAGES; ++s) { mbar_init(&sh->k_full[s], 1); mbar_init(&sh->k_empty[s], 1); sh->armed_k[s] = -1; }
     for (int s = 0; s < V_STAGES; ++s) { mbar_init(&sh->v_full[s], 1); mbar_init(&sh->v_empty[s], 1); sh->armed_v[s] = -1; }
     mbar_init(&sh->s_full[0], 1); mbar_init(&sh->s_full[1], 1);
@@ -322,36 +151,28 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
     // --------------------------------------------------------------- producers
     const int which = warp == 0 ? 0 : 1;                        // keys (and queries) or values
     const int stages = which ? V_STAGES : K_STAGES;
-    const int pieces = which ? 1 : NC;                          // stages of a tile
     pdl_wait();                         // queries, keys and values are the work of the kernels before this one
     const int P = p.page_size, pages_per_tile = BN / P;
     uint64_t* full_bars = which ? sh->v_full : sh->k_full;
     uint64_t* empty_bars = which ? sh->v_empty : sh->k_empty;
     int* armed = which ? sh->armed_v : sh->armed_k;
-    unsigned char* tiles = which ? v_s : k_s + K_OFF;
-    const int tile_stride = which ? TILE_BYTES : K_STRIDE;
-    const int q_bytes = 2 * 128 * G * p.tokens_per_tile;        // of one piece: two boxes of 64 d x G heads x tokens
+    unsigned char* tiles = which ? v_s : k_s;
     const CUtensorMap* map = which ? &v_map : &k_map;
     bool ok = true;
-    int gt = 0, n = 0;                  // stages of tiles and items of this block so far
-    auto load_q = [&](const Item& it, int tile, int c, uint64_t* bar) {
-      tma_load_3d(q_s + tile * TILE_BYTES, &q_map, c * D, it.kv_head * G, it.q_first, bar);
-      tma_load_3d(q_s + tile * TILE_BYTES + HALF_BYTES, &q_map, c * D + 64, it.kv_head * G, it.q_first, bar);
-    };
+    int gt = 0, n = 0;                  // tiles and items of this block so far
     for (int r = 0; r < n_rounds && ok; ++r) {
       const int L = item_of_round(r);
       if (L < 0) continue;
       const Item it = load_item(L);
       if (it.n_tiles == 0) continue;
-      if (!STREAM && which == 0 && lane == 0) {
-        // two buffers: all pieces, once the item two before this one has left through this buffer; one buffer: all but the
-        // first piece, once the item before has formed its last scores
-        const int qb = ONE_BUFFER ? 1 : n % QB, ph = (n / QB) & 1, first = ONE_BUFFER ? 1 : 0;
-        ok = mbar_wait(&sh->q_free[qb], ph ^ 1);
+      if (which == 0 && lane == 0) {
+        const int qb = n % Q_BUFFERS, ph = (n / Q_BUFFERS) & 1;
+        ok = mbar_wait(&sh->q_free[qb], ph ^ 1);                 // the item two before this one has left through this buffer
         if (ok) {
           sh->armed_q[qb] = ph;
-          mbar_expect_tx(&sh->q_full[qb], (NC - first) * q_bytes);
-          for (int c = first; c < NC; ++c) load_q(it, ONE_BUFFER ? c : qb * NC + c, c, &sh->q_full[qb]);
+          mbar_expect_tx(&sh->q_full[qb], 2 * 128 * G * p.tokens_per_tile);      // two boxes of 64 d x G heads x tokens
+          tma_load_3d(q_s + qb * TILE_BYTES, &q_map, 0, it.kv_head * G, it.q_first, &sh->q_full[qb]);
+          tma_load_3d(q_s + qb * TILE_BYTES + HALF_BYTES, &q_map, 64, it.kv_head * G, it.q_first, &sh->q_full[qb]);
         }
       }
       ok = __shfl_sync(0xffffffffu, ok, 0);
@@ -368,33 +189,20 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
       };
       // the block-table entries of a tile are read while the tile before it is loaded
       int pages = tile_pages(0);
-      for (int j = 0; j < it.n_tiles && ok; ++j) {
+      for (int j = 0; j < it.n_tiles && ok; ++j, ++gt) {
         const int pages_next = tile_pages(j + 1);
+        const int s = gt % stages, ph = (gt / stages) & 1;
+        unsigned char* dst = tiles + s * TILE_BYTES;
         const int n_pages = __popc(__ballot_sync(0xffffffffu, pages >= 0));
-        for (int cc = 0; cc < pieces && ok; ++cc, ++gt) {
-          const int c = cc + 1 == pieces ? 0 : cc + 1;           // the first piece last
-          const int s = gt % stages, ph = (gt / stages) & 1;
-          unsigned char* dst = tiles + s * tile_stride;
-          if (lane == 0) {
-            if (ONE_BUFFER && which == 0 && j == 0 && c == 0) {  // the output of the item before has left through this place
-              ok = mbar_wait(&sh->q_free[0], (n & 1) ^ 1);
-              if (ok) { sh->armed_q[0] = n & 1; mbar_expect_tx(&sh->q_full[0], q_bytes); load_q(it, 0, 0, &sh->q_full[0]); }
-            }
-            ok = ok && mbar_wait(&empty_bars[s], ph ^ 1);
-            if (ok) {
-              armed[s] = ph;
-              const bool with_q = STREAM && which == 0;
-              mbar_expect_tx(&full_bars[s], n_pages * P * 128 * 2 + (with_q ? q_bytes : 0));
-              if (with_q) load_q(it, 1 + 2 * s, c, &full_bars[s]);       // the tile before the stage's keys
-            }
-          }
-          ok = __shfl_sync(0xffffffffu, ok, 0);      // also orders the announcement before the copies
-          // lane i issues the two boxes of page i
-          if (ok && pages >= 0) {
-            const int head = (which || NC == 1) ? it.kv_head : c;
-            tma_load_4d(dst + lane * P * 128, map, 0, head, 0, pages, &full_bars[s]);
-            tma_load_4d(dst + HALF_BYTES + lane * P * 128, map, 64, head, 0, pages, &full_bars[s]);
-          }
+        if (lane == 0) {
+          ok = mbar_wait(&empty_bars[s], ph ^ 1);
+          if (ok) { armed[s] = ph; mbar_expect_tx(&full_bars[s], n_pages * P * 128 * 2); }
+        }
+        ok = __shfl_sync(0xffffffffu, ok, 0);      // also orders the announcement before the copies
+        // lane i issues the two boxes of page i
+        if (ok && pages >= 0) {
+          tma_load_4d(dst + lane * P * 128, map, 0, it.kv_head, 0, pages, &full_bars[s]);
+          tma_load_4d(dst + HALF_BYTES + lane * P * 128, map, 64, it.kv_head, 0, pages, &full_bars[s]);
         }
         pages = pages_next;
       }
@@ -404,9 +212,19 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
   } else if (warp == 1) {
     // -------------------------------------------------------------- mma issuer
     if (lane == 0) {
-      // descriptors of the first query, key and value tile; a tile further is TILE_BYTES / 16 more
-      const uint64_t q_desc = desc_k_major(smem_u32(STREAM ? k_s : q_s));
-      const uint64_t k_desc = desc_k_major(smem_u32(k_s + K_OFF)), v_desc = desc_mn_major(smem_u32(v_s));
+      uint64_t q_desc[Q_BUFFERS][2], k_desc[K_STAGES][2], v_desc[V_STAGES];
+#pragma unroll
+      for (int b = 0; b < Q_BUFFERS; ++b) {
+        q_desc[b][0] = desc_k_major(smem_u32(q_s + b * TILE_BYTES));
+        q_desc[b][1] = desc_k_major(smem_u32(q_s + b * TILE_BYTES + HALF_BYTES));
+      }
+#pragma unroll
+      for (int st = 0; st < K_STAGES; ++st) {
+        k_desc[st][0] = desc_k_major(smem_u32(k_s + st * TILE_BYTES));
+        k_desc[st][1] = desc_k_major(smem_u32(k_s + st * TILE_BYTES + HALF_BYTES));
+      }
+#pragma unroll
+      for (int st = 0; st < V_STAGES; ++st) v_desc[st] = desc_mn_major(smem_u32(v_s + st * TILE_BYTES), HALF_BYTES);
       // Where this thread stands in the block's sequence of tiles: round, item number, tile of the item, its tiles.
       // The item after the current one is looked up when the current one begins, so that the loads for it have
       // long arrived when its first scores are due (while the current item's last softmax runs).
@@ -431,25 +249,17 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
         return b;
       };
       auto issue_qk = [&](const At& a, int gt) -> bool {          // S[gt % 2] = Q K^T for tile gt of the sequence
-        const int qb = a.n % QB;
-        if (!STREAM && a.j == 0 && !mbar_wait(&sh->q_full[ONE_BUFFER ? 1 : qb], (a.n / QB) & 1)) return false;
+        const int qb = a.n % Q_BUFFERS, s = gt % K_STAGES;
+        if (a.j == 0 && !mbar_wait(&sh->q_full[qb], (a.n / Q_BUFFERS) & 1)) return false;
+        if (!mbar_wait(&sh->k_full[s], (gt / K_STAGES) & 1)) return false;
+        TC_FENCE_AFTER();
+        const uint64_t q0 = q_desc[qb][0], q1 = q_desc[qb][1], k0 = k_desc[s][0], k1 = k_desc[s][1];
         const uint32_t tmem_s = tmem + (gt & 1) * 128;
-        for (int cc = 0; cc < NC; ++cc) {
-          const int c = cc + 1 == NC ? 0 : cc + 1;                 // the first piece last
-          const int at = gt * NC + cc, s = at % K_STAGES;
-          if (ONE_BUFFER && a.j == 0 && c == 0 && !mbar_wait(&sh->q_full[0], a.n & 1)) return false;
-          if (!mbar_wait(&sh->k_full[s], (at / K_STAGES) & 1)) return false;
-          TC_FENCE_AFTER();
-          const uint64_t q0 = q_desc + (uint64_t)((STREAM ? s * K_STRIDE : (ONE_BUFFER ? c : qb * NC + c) * TILE_BYTES) >> 4);
-          const uint64_t k0 = k_desc + (uint64_t)((s * K_STRIDE) >> 4);
-          const uint64_t q1 = q0 + (HALF_BYTES >> 4), k1 = k0 + (HALF_BYTES >> 4);
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk) umma(tmem_s, q0 + 2 * kk, k0 + 2 * kk, IDESC_QK, (cc | kk) != 0);
+        for (int kk = 0; kk < 4; ++kk) umma(tmem_s, q0 + 2 * kk, k0 + 2 * kk, IDESC_QK, kk != 0);
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk) umma(tmem_s, q1 + 2 * kk, k1 + 2 * kk, IDESC_QK, 1);
-          umma_commit(&sh->k_empty[s]);
-        }
-        if (ONE_BUFFER && a.j == a.nt - 1) umma_commit(&sh->q_free[1]);    // the item's other pieces have been used for the last time
+        for (int kk = 0; kk < 4; ++kk) umma(tmem_s, q1 + 2 * kk, k1 + 2 * kk, IDESC_QK, 1);
+        umma_commit(&sh->k_empty[s]);
         umma_commit(&sh->s_full[gt & 1]);
         return true;
       };
@@ -457,10 +267,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
       if (cur.r < n_rounds) ok = issue_qk(cur, 0);
       for (int gt = 0; cur.r < n_rounds && ok; ++gt) {
         const At nxt = after(cur);
-        // the next scores while this tile's softmax runs; with one query buffer the next item's have to wait until this
-        // item's output has left
-        const bool later = ONE_BUFFER && nxt.n != cur.n;
-        if (nxt.r < n_rounds && !later) ok = issue_qk(nxt, gt + 1);
+        if (nxt.r < n_rounds) ok = issue_qk(nxt, gt + 1);          // the next scores while this tile's softmax runs
         if (!ok) break;
         const int s = gt % V_STAGES;
         if (!mbar_wait(&sh->p_full[gt & 1], (gt >> 1) & 1) || !mbar_wait(&sh->v_full[s], (gt / V_STAGES) & 1)) { ok = false; break; }
@@ -471,10 +278,9 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
         const uint32_t tmem_p = tmem + TMEM_P + (gt & 1) * 64;
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk)   // 16 keys further: 8 columns of P, 16 rows (2048 bytes) down V
-          umma_a_tmem(tmem_o, tmem_p + kk * 8, v_desc + (uint64_t)((s * TILE_BYTES) >> 4) + kk * (16 * 128 / 16), IDESC_PV, (cur.j | kk) != 0);
+          umma_a_tmem(tmem_o, tmem_p + kk * 8, v_desc[s] + kk * (16 * 128 / 16), IDESC_PV, (cur.j | kk) != 0);
         umma_commit(&sh->v_empty[s]);
         umma_commit(&sh->o_done[gt & 1]);
-        if (nxt.r < n_rounds && later) ok = issue_qk(nxt, gt + 1);
         cur = nxt;
       }
       if (!ok) { atomicOr(p.status, JV_STATUS_WAIT_EXPIRED); sh->failed = 1; }
@@ -678,7 +484,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
         }
       }
       // ---- the item's output: O / sum, each thread its 64 columns; the row's sum is the two threads' together
-      const int g_last = gt - 1, qb = n % QB;
+      const int g_last = gt - 1, qb = n % Q_BUFFERS;
       sh->xch[half][row] = l_run;
       pair_barrier(quad);
       const float l_row = sh->xch[0][row] + sh->xch[1][row];
@@ -696,8 +502,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
       // A whole tile leaves through shared memory (where the item's queries were: every product with them has
       // completed) and one TMA store per half of the head; threads that write their 128 bytes to rows 8 KB apart in
       // memory take five times as long.
-      unsigned char* out_s = q_s + qb * (STREAM ? 1 : NCT) * TILE_BYTES;    // the item's first piece (streamed: a tile of its own)
-      unsigned char* row_base = out_s + half * HALF_BYTES + row * 128;
+      unsigned char* row_base = q_s + qb * TILE_BYTES + half * HALF_BYTES + row * 128;
       __nv_bfloat16* dst = p.out + (size_t)(it.q_first + t) * p.out_stride + (size_t)(it.kv_head * G + hh) * D + half * 64;
       if (got) {
         TC_FENCE_AFTER();
@@ -725,15 +530,10 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
         if (threadIdx.x == 64) {
           if (got) {
             // started here, waited for after the next item's first tile (or at the end): this thread's warp is not held up
-            tma_store_3d(&out_map, out_s, 0, it.kv_head * G, it.q_first);
-            tma_store_3d(&out_map, out_s + HALF_BYTES, 64, it.kv_head * G, it.q_first);
+            tma_store_3d(&out_map, q_s + qb * TILE_BYTES, 0, it.kv_head * G, it.q_first);
+            tma_store_3d(&out_map, q_s + qb * TILE_BYTES + HALF_BYTES, 64, it.kv_head * G, it.q_first);
             asm volatile("cp.async.bulk.commit_group;\n" ::: "memory");
-            if (QB > 1) {
-              stored = qb;
-            } else {                                             // the next item needs the place before it can begin
-              asm volatile("cp.async.bulk.wait_group.read 0;\n" ::: "memory");
-              mbar_arrive(&sh->q_free[0]);
-            }
+            stored = qb;
           } else {
             mbar_arrive(&sh->q_free[qb]);
           }
@@ -758,7 +558,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
     // in this block's shared memory; both get a bounded time to finish before tensor memory is freed and the block ends
     if (warp == 1 && lane == 0) drain_products_after_failure(&sh->drain);
     if (warp == 0 && lane == 0) {
-      for (int b = 0; b < 2; ++b)
+      for (int b = 0; b < Q_BUFFERS; ++b)
         if (sh->armed_q[b] >= 0) drain_copies_after_failure(&sh->q_full[b], sh->armed_q[b]);
       for (int s = 0; s < K_STAGES; ++s)
         if (sh->armed_k[s] >= 0) drain_copies_after_failure(&sh->k_full[s], sh->armed_k[s]);
@@ -774,30 +574,6 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
   }
 }
 
-PFN_cuTensorMapEncodeTiled_v12000 encode_fn() {
-  static PFN_cuTensorMapEncodeTiled_v12000 fn = nullptr;
-  if (fn == nullptr) {
-    void* ptr = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) == cudaSuccess &&
-        q == cudaDriverEntryPointSuccess)
-      fn = reinterpret_cast<PFN_cuTensorMapEncodeTiled_v12000>(ptr);
-  }
-  return fn;
-}
-
-template <int NCT>
-int launch(int blocks, cudaStream_t stream, const CUtensorMap& q_map, const CUtensorMap& k_map, const CUtensorMap& v_map,
-           const CUtensorMap& out_map, const Params& p) {
-  constexpr size_t smem = TILE_BYTES * SMEM_TILES + sizeof(Shared) + 1024;
-  static_assert(Plan<NCT>::STREAM || Plan<NCT>::QB * NCT + Plan<NCT>::KS + Plan<NCT>::VS <= SMEM_TILES, "tiles");
-  static bool ready[JV_MAX_DEVICES];
-  if (!jv_once_per_device(ready, [&] {
-        return cudaFuncSetAttribute(attn_tcgen05_kernel<NCT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess;
-      }))
-    return JV_ERR_UNSUPPORTED;
-  return jv_launch(attn_tcgen05_kernel<NCT>, dim3(blocks), dim3(THREADS), smem, stream, q_map, k_map, v_map, out_map, p);
-}
 }  // namespace
 
 // 1 if this kernel takes the case (else the caller uses the mma.sync kernel).
@@ -818,17 +594,14 @@ JV_EXPORT int jv_attn_tcgen05_tokens_per_tile(int n_q_heads, int n_kv_heads) { r
 // sigmoid != 0: the weights are sigmoid(q.k * scale + bias[query head]) instead of a softmax (bias: [n_q_heads] floats or null).
 // head_scale [n_q_heads], dist_bias [n_q_heads][n_dist], sink [n_q_heads] (floats, each may be null; softmax only): see Params.
 // window: the mask as one number (0: every earlier key; > 0: a window; < 0: chunks of -window positions).
-// chunks > 1 (then n_kv_heads): every query head has chunks * 128 elements (head h of a token at column h*chunks*128) and
-// its scores are products with a token's whole key row, the n_kv_heads key heads side by side.
 // out_scale multiplies the output.
 JV_EXPORT int jv_attn_tcgen05_ex(const void* q, int q_stride, int n_tokens, void* out, int out_stride, const void* k_cache,
                                  const void* v_cache, const int* block_table, int table_width, const int* cu_seqlens,
                                  const int* start_pos, const int* work, int n_work, int n_q_heads, int n_kv_heads,
                                  int head_dim, int page_size, int num_pages, float scale, int sigmoid, const float* bias,
                                  const float* head_scale, const float* dist_bias, int n_dist, const float* sink,
-                                 int window, int chunks, float out_scale, int* status, cudaStream_t stream) {
+                                 int window, float out_scale, int* status, cudaStream_t stream) {
   if (n_work == 0) return JV_OK;
-  if (chunks < 1 || (chunks > 1 && chunks != n_kv_heads)) return JV_ERR_UNSUPPORTED;
   if ((dist_bias != nullptr && n_dist < 1) || (sigmoid && (head_scale != nullptr || dist_bias != nullptr || sink != nullptr)))
     return JV_ERR_UNSUPPORTED;
   if (!jv_attn_tcgen05_supports(head_dim, n_q_heads, n_kv_heads, page_size, 0)) return JV_ERR_UNSUPPORTED;
@@ -841,9 +614,8 @@ JV_EXPORT int jv_attn_tcgen05_ex(const void* q, int q_stride, int n_tokens, void
   CUtensorMap q_map, k_map, v_map, out_map;
   for (int which = 0; which < 2; ++which) {
     // queries and output: (d, head, token); a box is 64 d x G heads x (128 / G) tokens = 128 rows, head fastest
-    const int d = which ? D : D * chunks;
-    const cuuint64_t dims[3] = {(cuuint64_t)d, (cuuint64_t)n_q_heads, (cuuint64_t)n_tokens};
-    const cuuint64_t strides[2] = {(cuuint64_t)d * 2, (cuuint64_t)(which ? out_stride : q_stride) * 2};
+    const cuuint64_t dims[3] = {(cuuint64_t)D, (cuuint64_t)n_q_heads, (cuuint64_t)n_tokens};
+    const cuuint64_t strides[2] = {(cuuint64_t)D * 2, (cuuint64_t)(which ? out_stride : q_stride) * 2};
     const cuuint32_t box[3] = {64, (cuuint32_t)G, (cuuint32_t)(ROWS / G)};
     const cuuint32_t es[3] = {1, 1, 1};
     if (fn(which ? &out_map : &q_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, which ? out : const_cast<void*>(q), dims, strides, box, es,
@@ -868,7 +640,13 @@ JV_EXPORT int jv_attn_tcgen05_ex(const void* q, int q_stride, int n_tokens, void
   p.page_size = page_size; p.num_pages = num_pages; p.hpt = G; p.tokens_per_tile = ROWS / G;
   p.scale_log2 = scale * LOG2E; p.status = status; p.sigmoid = sigmoid ? 1 : 0; p.bias = bias;
   p.head_scale = head_scale; p.dist_bias = dist_bias; p.n_dist = n_dist; p.sink = sink; p.window = window;
-  p.chunks = chunks; p.out_scale = out_scale;
+  p.out_scale = out_scale;
+  constexpr size_t smem = TILE_BYTES * (Q_BUFFERS + K_STAGES + V_STAGES) + sizeof(Shared) + 1024;
+  static bool ready[JV_MAX_DEVICES];
+  if (!jv_once_per_device(ready, [&] {
+        return cudaFuncSetAttribute(attn_tcgen05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess;
+      }))
+    return JV_ERR_UNSUPPORTED;
   // persistent blocks: one per multiprocessor (or per item, if there are fewer)
   static int sm_count[JV_MAX_DEVICES];
   int dev = 0;
@@ -878,13 +656,7 @@ JV_EXPORT int jv_attn_tcgen05_ex(const void* q, int q_stride, int n_tokens, void
     sm_count[dev] = 148;
   const long long items = (long long)n_work * n_kv_heads;
   const int blocks = items < sm_count[dev] ? (int)items : sm_count[dev];
-  switch (chunks) {
-    case 1: return launch<1>(blocks, stream, q_map, k_map, v_map, out_map, p);
-    case 2: return launch<2>(blocks, stream, q_map, k_map, v_map, out_map, p);
-    case 3: return launch<3>(blocks, stream, q_map, k_map, v_map, out_map, p);
-    case 4: return launch<4>(blocks, stream, q_map, k_map, v_map, out_map, p);
-    default: return launch<0>(blocks, stream, q_map, k_map, v_map, out_map, p);
-  }
+  return jv_launch(attn_tcgen05_kernel, dim3(blocks), dim3(THREADS), smem, stream, q_map, k_map, v_map, out_map, p);
 }
 
 JV_EXPORT int jv_attn_tcgen05(const void* q, int q_stride, int n_tokens, void* out, int out_stride, const void* k_cache,
@@ -893,5 +665,5 @@ JV_EXPORT int jv_attn_tcgen05(const void* q, int q_stride, int n_tokens, void* o
                               int head_dim, int page_size, int num_pages, float scale, int* status, cudaStream_t stream) {
   return jv_attn_tcgen05_ex(q, q_stride, n_tokens, out, out_stride, k_cache, v_cache, block_table, table_width, cu_seqlens,
                             start_pos, work, n_work, n_q_heads, n_kv_heads, head_dim, page_size, num_pages, scale, 0, nullptr,
-                            nullptr, nullptr, 0, nullptr, 0, 1, 1.f, status, stream);
+                            nullptr, nullptr, 0, nullptr, 0, 1.f, status, stream);
 }

@@ -751,13 +751,12 @@ def attn_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: tor
                  n_work: int, n_q_heads: int, n_kv_heads: int, head_dim: int, scale: float, sigmoid: bool = False,
                  bias: torch.Tensor | None = None, head_scale: torch.Tensor | None = None,
                  dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None, window: int = 0,
-                 whole_rows: bool = False, out_scale: float = 1.0) -> None:
+                 out_scale: float = 1.0) -> None:
     """Paged causal attention of prompt portions on tcgen05 tensor cores with scores and output in tensor
     memory (csrc/attn_tcgen05.cu); `work` lists 128-row tiles of `attn_tcgen05_tokens_per_tile` tokens.  With
     `sigmoid` the weight of a visible key is sigmoid(score * scale + bias[query head]) instead of a softmax;
     `head_scale`, `dist_bias` and `sink` as for `attn_simt` (softmax only); `window`: the mask as one number
-    (`mask_code`).  `whole_rows`: every query head has the size of a token's whole key row (the key heads side by side) and
-    its scores are products with that (scores mixed across heads).  `out_scale` multiplies the output."""
+    (`mask_code`).  `out_scale` multiplies the output."""
     n_dist = _score_extras("attn_tcgen05", n_q_heads, head_scale, dist_bias, sink)
     for t, nm in ((q, "q"), (out, "out"), (k_cache, "k_cache"), (v_cache, "v_cache")):
         _cuda(t, nm, torch.bfloat16, contiguous=(nm not in ("q", "out")))     # q and out may be some heads of wider rows
@@ -774,12 +773,38 @@ def attn_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: tor
     f = _fn("attn_tcgen05", "jv_attn_tcgen05_ex", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                    c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                    c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
-                                                   c_int, c_int, c_float, c_void_p, c_void_p])
+                                                   c_int, c_float, c_void_p, c_void_p])
     _check(f(q.data_ptr(), q_stride, q.shape[0], out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
              block_table.data_ptr(), block_table.shape[1], cu_seqlens.data_ptr(), start_pos.data_ptr(), work.data_ptr(),
              n_work, n_q_heads, n_kv_heads, head_dim, k_cache.shape[1], k_cache.shape[0], float(scale),
              1 if sigmoid else 0, _ptr(bias), _ptr(head_scale), _ptr(dist_bias), n_dist, _ptr(sink), int(window),
-             n_kv_heads if whole_rows else 1, float(out_scale), _status_ptr(q.device), _stream()), "attn_tcgen05")
+             float(out_scale), _status_ptr(q.device), _stream()), "attn_tcgen05")
+
+
+def attn_rows_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                      block_table: torch.Tensor, cu_seqlens: torch.Tensor, start_pos: torch.Tensor, work: torch.Tensor,
+                      n_work: int, n_q_heads: int, n_kv_heads: int, scale: float, sink: torch.Tensor | None = None,
+                      out_scale: float = 1.0) -> None:
+    """Attention of prompt portions whose queries have the size of a token's whole key row, `n_kv_heads` (two or more) pieces
+    of 128 (csrc/attn_rows_tcgen05.cu): caches [pages, page, n_kv_heads, 128]; `work` as for `attn_tcgen05`, whose
+    `attn_tcgen05_supports` says which sizes are taken.  No window."""
+    _score_extras("attn_rows_tcgen05", n_q_heads, None, None, sink)
+    for t, nm in ((q, "q"), (out, "out"), (k_cache, "k_cache"), (v_cache, "v_cache")):
+        _cuda(t, nm, torch.bfloat16, contiguous=(nm not in ("q", "out")))
+    for t, nm in ((block_table, "block_table"), (cu_seqlens, "cu_seqlens"), (start_pos, "start_pos"), (work, "work")):
+        _cuda(t, nm, torch.int32)
+    if n_work == 0:
+        return
+    if k_cache.shape[2:] != (n_kv_heads, 128) or v_cache.shape != k_cache.shape or out.stride(1) != 1 or q.stride(1) != 1 or \
+            q.shape[1] < n_q_heads * n_kv_heads * 128 or out.shape[1] < n_q_heads * 128:
+        raise KernelError("attn_rows_tcgen05: the caches, queries or output do not fit the heads")
+    f = _fn("attn_rows_tcgen05", "jv_attn_rows_tcgen05",
+            [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
+             c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p])
+    _check(f(q.data_ptr(), q_stride, q.shape[0], out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
+             block_table.data_ptr(), block_table.shape[1], cu_seqlens.data_ptr(), start_pos.data_ptr(), work.data_ptr(),
+             n_work, n_q_heads, n_kv_heads, k_cache.shape[1], k_cache.shape[0], float(scale), float(out_scale), _ptr(sink),
+             _status_ptr(q.device), _stream()), "attn_rows_tcgen05")
 
 
 DECODE_TCGEN05_MAX_REQUESTS = 512
@@ -863,15 +888,16 @@ def attn_decode_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cac
 
 def attn_rows_decode_supports(dtype: torch.dtype, n_q_heads: int, n_v_heads: int, row: int, value_dim: int) -> bool:
     """Whether the decode kernel for whole key rows takes these sizes (csrc/attn_rows_decode.cu): bfloat16, rows in steps
-    of 16, values in steps of 8, what a thread keeps of the output in registers, two stages of 16 keys in shared memory."""
-    if dtype != torch.bfloat16 or row % 16 or row < 16 or value_dim % 8 or value_dim < 8 or n_q_heads % n_v_heads or n_q_heads > 256:
+    of 16, values in steps of 8, what a thread keeps of queries and output in registers, two stages of 8 keys in shared
+    memory."""
+    if dtype != torch.bfloat16 or row % 16 or row < 16 or value_dim % 8 or value_dim < 8 or n_q_heads % n_v_heads or n_q_heads > 128:
         return False
-    group = n_q_heads // n_v_heads
+    group, heads16 = n_q_heads // n_v_heads, -(-n_q_heads // 16) * 16
     pairs = -(-n_v_heads * value_dim // 512)                 # column pairs a thread
-    heads16 = -(-n_q_heads // 16) * 16
-    smem = 2 * (heads16 * (row + 8) + 32 * (row + 8 + n_v_heads * value_dim)) + 4 * 8 * heads16 * 20
+    parts = 8 // (heads16 // 16)                             # parts of a row that warps share
+    smem = 32 * (row + 8 + n_v_heads * value_dim) + 4 * parts * heads16 * 12
     return group <= 16 and pairs <= 4 and (4 if group <= 4 else 8 if group <= 8 else 16) * pairs <= 32 and \
-        64 * (row + n_v_heads * value_dim) <= 132 * 1024 and smem <= 220 * 1024
+        -(-row // 16 // parts) <= 16 and smem <= 200 * 1024
 
 
 def attn_rows_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
@@ -891,7 +917,7 @@ def attn_rows_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache:
     if k_cache.dim() != 4 or k_cache.shape[2] != 1 or k_cache.shape[:2] != v_cache.shape[:2] or out.stride(1) != 1:
         raise KernelError("attn_rows_decode: one key row a token, and out with unit column stride")
     row, groups, dv = k_cache.shape[3], v_cache.shape[2], v_cache.shape[3]
-    split = 64 if n_work <= 4 else 128 if n_work <= 10 else 256
+    split = 64 if n_work <= 12 else 128 if n_work <= 24 else 256
     n_splits = max(1, -(-max_seq_len // split))
     part_o = torch.empty(n_work * n_q_heads * n_splits * dv, dtype=torch.float32, device=q.device)
     part_ml = torch.empty(n_work * n_q_heads * n_splits * 2, dtype=torch.float32, device=q.device)

@@ -138,13 +138,15 @@ class GeneralAttention(Part):
         self.big_tiles = (self.general is not None and not spec.score_cap and self.hv == self.hk and self.dv == self.d == 128
                           and spec.twin is None and (spec.weights == "sigmoid") != bool(self.extras)
                           and self.out_scale == 1.0 and not self.talking)
-        # scores mixed across heads: heads of 128 go to the same kernel in its form for whole key rows, portions of any
-        # length where no kernel with smaller tiles takes rows that long; single tokens to the kernel that reads each row once
-        self.whole_rows = (self.talking and not spec.score_cap and self.hv == self.hk and self.dv == self.d == 128)
+        # scores mixed across heads: prompt portions on heads of 128 go to the tcgen05 kernel for whole key rows (of one key
+        # head: to the ordinary one), portions of any length where no kernel with smaller tiles takes rows that long; single
+        # tokens to the kernel that reads each row once
+        self.whole_rows = (self.talking and not spec.score_cap and not self.mask and self.hv == self.hk
+                           and self.dv == self.d == 128)
         self.rows_decode = (self.talking and not spec.score_cap and not self.mask and self.general is None
                             and ops.attn_rows_decode_supports(ctx.dtype, self.hq, self.hv, self.dk, self.dv))
         if self.big_tiles or (self.whole_rows and ctx.dtype == torch.bfloat16):
-            self.kernels += ("attn_tcgen05",)
+            self.kernels += ("attn_rows_tcgen05" if self.talking and self.hk > 1 else "attn_tcgen05",)
         if self.rows_decode:
             self.kernels += ("attn_rows_decode",)
         self.w_in = self.w_o = self.q_norm = self.k_norm = self.bias = None
@@ -345,11 +347,13 @@ class GeneralAttention(Part):
                               v_dim=self.dv, **split, **extra)
         for cls, big in self._tile_kernels(cache.k.shape[1]):
             work, n_work = step.tile_work[cls]
-            if n_work and big:                             # 128-row tiles
+            if n_work and big and self.talking and self.hk > 1:
+                ops.attn_rows_tcgen05(q, q.stride(0), a, cache.k, cache.v, *common[2:], work, n_work, self.hq, self.hk, s.scale,
+                                      sink=self.sink, out_scale=self.out_scale)
+            elif n_work and big:                           # 128-row tiles
                 ops.attn_tcgen05(q, q.stride(0), a, cache.k, cache.v, *common[2:], work, n_work, self.hq, self.hk, self.d,
                                  s.scale, sigmoid=s.weights == "sigmoid", bias=self.bias, head_scale=self.head_scale,
-                                 dist_bias=self.dist_bias, sink=self.sink, window=self.mask, whole_rows=self.talking,
-                                 out_scale=self.out_scale)
+                                 dist_bias=self.dist_bias, sink=self.sink, window=self.mask, out_scale=self.out_scale)
             elif n_work:
                 kernel(work, n_work)
         dwork, n_dec = step.decode_work
