@@ -10,8 +10,8 @@
 //              and a part of KD, keeps its piece of the queries in registers for the whole range, and goes over the keys of
 //              the tile; the parts of a score are added up by its reader
 //   softmax    running (max, sum) a head in 32-bit, eight lanes a head
-//   output     O [H, DV] += P V in 32-bit on the CUDA cores: a thread keeps two columns of a value head for all query heads
-//              that read it (a decoded token's few rows would leave most of a tensor-core tile empty); P stays 32-bit
+//   output     O [H, DV] += P V on the tensor cores, a warp 16 columns of a value head at a time for all query heads that
+//              read it (rows of the tile without a head are zero); P is rounded to bfloat16 as in the prompt kernels
 // Each range leaves its unnormalised output and (max, sum); a second kernel merges a head's ranges in ascending order and
 // lets the sink join the denominator.  Every wait on a barrier is bounded and reports to the status word.
 #include "common.cuh"
@@ -34,7 +34,7 @@ struct Params {
   int H, G, KD, DV, page_size, num_pages;
   float scale_log2, out_scale;
   const float* sink;           // [H] or null
-  int KT, k_parts;             // keys of a tile; parts of KD that warps share the scores of 16 heads in
+  int KT;                      // keys of a tile
   int split_size, n_splits;
   int* status;
 };
@@ -56,38 +56,52 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ float fast_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int N> struct Int { static constexpr int value = N; };
+
 // Offsets (bytes) of the arrays in dynamic shared memory, for the kernel and its launcher.
 struct Layout {
-  int k_row, v_row, s_row;                     // elements from row to row
-  size_t k, v, s, total;                       // s: [k_parts][H16][s_row] floats
+  int k_row, v_row, s_row, p_row;              // elements from row to row
+  size_t k, v, s, w, total;                    // s: [k_parts][H16][s_row] floats; w: [H16][p_row] bfloat16
   __host__ __device__ Layout(int H, int G, int KD, int DV, int KT, int k_parts) {
     const int H16 = (H + 15) / 16 * 16;
-    k_row = KD + 8; v_row = G * DV; s_row = KT + 4;
+    k_row = KD + 8; v_row = G * DV + 8; s_row = KT + 4; p_row = KT + 8;
     k = 0;
     v = k + sizeof(__nv_bfloat16) * (size_t)2 * KT * k_row;
     s = v + sizeof(__nv_bfloat16) * (size_t)2 * KT * v_row;
-    total = s + sizeof(float) * (size_t)k_parts * H16 * s_row;
+    w = s + sizeof(float) * (size_t)k_parts * H16 * s_row;
+    total = w + sizeof(__nv_bfloat16) * (size_t)H16 * p_row;
   }
 };
 
-// HT: query heads of a value head, rounded up; IT: column pairs a thread keeps; KS: steps of 16 elements of KD a warp keeps
-// of the queries.
-template <int HT, int IT, int KS>
-__global__ void __launch_bounds__(THREADS, HT * IT <= 16 ? 2 : 1) attn_rows_decode_kernel(const Params p) {
+// NP: pieces of 16 output columns a warp keeps; KP: parts of KD that warps share the scores of 16 heads in; KS: steps of 16
+// elements of KD a warp keeps of the queries.
+template <int NP, int KP, int KS>
+__global__ void __launch_bounds__(THREADS, NP * 8 + KS * 4 <= 64 ? 2 : 1) attn_rows_decode_kernel(const Params p) {
   extern __shared__ __align__(128) unsigned char smem[];
   __shared__ long long slots[MAX_SPLIT];        // cache slot of every key of the range (-1: none)
   __shared__ float row_m[MAX_HEADS], row_l[MAX_HEADS], row_alpha[MAX_HEADS];
   __shared__ __align__(8) uint64_t bars[2];
   const int H = p.H, G = p.G, KD = p.KD, DV = p.DV, KT = p.KT, HPT = H / G;
-  const Layout L(H, G, KD, DV, KT, p.k_parts);
+  const Layout L(H, G, KD, DV, KT, KP);
   __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(smem + L.k);
   __nv_bfloat16* vs = reinterpret_cast<__nv_bfloat16*>(smem + L.v);
   float* ss = reinterpret_cast<float*>(smem + L.s);
+  __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(smem + L.w);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   pdl_trigger();
   if (tid == 0) {
-    mbar_init(&bars[0], THREADS);
-    mbar_init(&bars[1], THREADS);
+    mbar_init(&bars[0], WARPS);
+    mbar_init(&bars[1], WARPS);
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
   }
   pdl_wait();
@@ -109,35 +123,33 @@ __global__ void __launch_bounds__(THREADS, HT * IT <= 16 ? 2 : 1) attn_rows_deco
   __syncthreads();
 
   const int n_tiles = (j_hi - j_lo + KT - 1) / KT;
-  // Tile t into stage t & 1: thread n < KT its key row, thread KT + n its value row (KT <= 64); every thread arrives once.
+  // Tile t into stage t & 1: a key row and a value row a copy, every warp its share of the rows (issuing a copy takes some
+  // sixty clocks).  Rows past the last key are not copied: their scores are masked, and their value rows become zero (they
+  // may hold anything, and their weights are zero).
   auto issue = [&](int t) {
     uint64_t* bar = &bars[t & 1];
-    const int n = tid < KT ? tid : tid - KT;
-    if (tid < 2 * KT) {
-      const bool is_v = tid >= KT;
-      const int i = t * KT + n;
-      const long long slot = i < j_hi - j_lo ? slots[i] : -1;
-      const int elems = is_v ? G * DV : KD;
-      __nv_bfloat16* dst = is_v ? vs + (size_t)((t & 1) * KT + n) * L.v_row : ks + (size_t)((t & 1) * KT + n) * L.k_row;
-      if (slot >= 0) {
-        mbar_expect_tx(bar, elems * 2);
-        bulk_copy(dst, (is_v ? p.v_cache : p.k_cache) + slot * elems, elems * 2, bar);
-      } else {                                   // no key here: zeros
-        for (int c = 0; c < elems / 8; ++c) *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(0, 0, 0, 0);
-        mbar_arrive(bar);
-      }
-    } else {
-      mbar_arrive(bar);
+    const int here = min(KT, j_hi - j_lo - t * KT), k_bytes = KD * 2, v_bytes = G * DV * 2;
+    const int n = warp + WARPS * (lane >> 1), at = (t & 1) * KT + n;       // two lanes a row: keys, values
+    const bool is_v = lane & 1;
+    const long long slot = n < here ? slots[t * KT + n] : -1;
+    const int n_k = __popc(__ballot_sync(0xffffffffu, slot >= 0 && !is_v));
+    if (lane == 0) mbar_expect_tx(bar, n_k * (k_bytes + v_bytes));
+    __syncwarp();                                // the announcement before the copies
+    if (slot >= 0) {
+      if (is_v) bulk_copy(vs + (size_t)at * L.v_row, p.v_cache + slot * (G * DV), v_bytes, bar);
+      else bulk_copy(ks + (size_t)at * L.k_row, p.k_cache + slot * KD, k_bytes, bar);
+    } else if (is_v && n < KT) {
+      for (int c = 0; c < G * DV / 8; ++c) *reinterpret_cast<uint4*>(vs + (size_t)at * L.v_row + c * 8) = make_uint4(0, 0, 0, 0);
     }
   };
   issue(0);
   if (n_tiles > 1) issue(1);
 
   // ---- this warp's queries: 16 heads, k steps [k0, k1) of 16 elements, as operand fragments
-  const int H16 = (H + 15) / 16 * 16, mt = H16 / 16, kp = p.k_parts, k_steps = KD / 16;
+  const int H16 = (H + 15) / 16 * 16, mt = H16 / 16, k_steps = KD / 16;
   const int m16 = warp % mt, part = warp / mt;
-  const bool scores_here = part < kp;
-  const int k0 = k_steps * part / kp, k1 = scores_here ? k_steps * (part + 1) / kp : k0;
+  const bool scores_here = part < KP;
+  const int k0 = k_steps * part / KP, k1 = scores_here ? k_steps * (part + 1) / KP : k0;
   uint32_t qa[KS][4];
   {
     const int h0 = m16 * 16 + (lane >> 2), h1 = h0 + 8;
@@ -153,13 +165,18 @@ __global__ void __launch_bounds__(THREADS, HT * IT <= 16 ? 2 : 1) attn_rows_deco
     }
   }
 
-  // ---- this thread's columns of the output
-  const int pairs = G * DV / 2;
-  float acc[IT][HT][2];
+  // ---- this warp's columns of the output: pieces warp * NP .. of 16 columns, for up to 16 query heads of a value head
+  const int pieces = G * DV / 16, first_piece = warp * NP;
+  float acc[NP][2][4];
 #pragma unroll
-  for (int i = 0; i < IT; ++i)
+  for (int i = 0; i < NP; ++i)
 #pragma unroll
-    for (int g = 0; g < HT; ++g) acc[i][g][0] = acc[i][g][1] = 0.f;
+    for (int e = 0; e < 4; ++e) acc[i][0][e] = acc[i][1][e] = 0.f;
+  const int g0 = lane >> 2, g1 = g0 + 8;         // this lane's two rows: query heads of the value head
+  const bool in0 = g0 < HPT, in1 = g1 < HPT;
+  int head0[NP];                                 // the first query head of a piece's value head (-1: no such piece)
+#pragma unroll
+  for (int i = 0; i < NP; ++i) head0[i] = first_piece + i < pieces ? (first_piece + i) * 16 / DV * HPT : -1;
 
   for (int t = 0; t < n_tiles; ++t) {
     const int buf = t & 1;
@@ -195,71 +212,73 @@ __global__ void __launch_bounds__(THREADS, HT * IT <= 16 ? 2 : 1) attn_rows_deco
       }
     }
     __syncthreads();
-    // ---- softmax: eight lanes a head; the weights replace the first part's scores
+    // ---- softmax: eight lanes a head
     const int here = min(KT, j_hi - j_lo - t * KT);
     for (int h = tid >> 3; h < H16; h += THREADS / 8) {        // whole warps stay together: H16 is a multiple of 4
-      float* row = ss + (size_t)h * L.s_row;
-      float v[8];
-      float mx = -INFINITY;
+      const float* row = ss + (size_t)h * L.s_row + (lane & 7);
+      __nv_bfloat16* wrow = ps + (size_t)h * L.p_row + (lane & 7);
+      auto softmax = [&](auto columns) {
+        constexpr int C = decltype(columns)::value;            // keys of a lane
+        float v[C];
+        float mx = -INFINITY;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int j = (lane & 7) + 8 * i;
-        v[i] = -INFINITY;
-        if (j < here) {
-          float x = row[j];
-          for (int q = 1; q < kp; ++q) x += row[(size_t)q * H16 * L.s_row + j];
-          v[i] = x * p.scale_log2;
+        for (int i = 0; i < C; ++i) {
+          float x[KP];
+#pragma unroll
+          for (int q = 0; q < KP; ++q) x[q] = row[(size_t)q * H16 * L.s_row + 8 * i];
+#pragma unroll
+          for (int q = 1; q < KP; ++q) x[0] += x[q];
+          v[i] = (lane & 7) + 8 * i < here ? x[0] * p.scale_log2 : -INFINITY;
+          mx = fmaxf(mx, v[i]);
         }
-        mx = fmaxf(mx, v[i]);
-      }
 #pragma unroll
-      for (int o = 4; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float m_old = row_m[h], m_new = fmaxf(m_old, mx);          // finite: a tile has at least one key
-      float sum = 0.f;
+        for (int o = 4; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float m_old = row_m[h], m_new = fmaxf(m_old, mx);        // finite: a tile has at least one key
+        float sum = 0.f;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int j = (lane & 7) + 8 * i;
-        if (j < KT) {
-          const float e = j < here ? exp2f(v[i] - m_new) : 0.f;
-          row[j] = e;
+        for (int i = 0; i < C; ++i) {
+          const float e = fast_exp2(v[i] - m_new);
+          wrow[8 * i] = __float2bfloat16_rn(e);
           sum += e;
         }
-      }
 #pragma unroll
-      for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-      __syncwarp();
-      if ((lane & 7) == 0) {
-        const float alpha = m_old == -INFINITY ? 0.f : exp2f(m_old - m_new);
-        row_alpha[h] = alpha;
-        row_m[h] = m_new;
-        row_l[h] = row_l[h] * alpha + sum;
-      }
+        for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        if ((lane & 7) == 0) {
+          const float alpha = fast_exp2(m_old - m_new);                // of -inf: 0
+          row_alpha[h] = alpha;
+          row_m[h] = m_new;
+          row_l[h] = row_l[h] * alpha + sum;
+        }
+        __syncwarp();
+      };
+      if (KT == 16) softmax(Int<2>{});
+      else if (KT == 32) softmax(Int<4>{});
+      else softmax(Int<8>{});
     }
     __syncthreads();
     // ---- output
 #pragma unroll
-    for (int i = 0; i < IT; ++i) {
-      const int pr = tid + i * THREADS;
-      if (pr < pairs) {
-        const int c = pr / (DV / 2);
-        const __nv_bfloat16* vcol = vs + (size_t)buf * KT * L.v_row + pr * 2;
-        const float* prow = ss + (size_t)c * HPT * L.s_row;
+    for (int i = 0; i < NP; ++i) {
+      if (head0[i] >= 0) {
+        const int h0 = head0[i] + g0, h1 = head0[i] + g1;
+        const float al0 = in0 ? row_alpha[h0] : 1.f, al1 = in1 ? row_alpha[h1] : 1.f;
 #pragma unroll
-        for (int g = 0; g < HT; ++g)
-          if (g < HPT) { const float al = row_alpha[c * HPT + g]; acc[i][g][0] *= al; acc[i][g][1] *= al; }
-        for (int j = 0; j < KT; j += 4) {
-          float2 v[4];
-#pragma unroll
-          for (int e = 0; e < 4; ++e) v[e] = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vcol + (size_t)(j + e) * L.v_row));
-#pragma unroll
-          for (int g = 0; g < HT; ++g)
-            if (g < HPT) {
-              const float4 w = *reinterpret_cast<const float4*>(prow + (size_t)g * L.s_row + j);
-              acc[i][g][0] = fmaf(w.x, v[0].x, acc[i][g][0]); acc[i][g][1] = fmaf(w.x, v[0].y, acc[i][g][1]);
-              acc[i][g][0] = fmaf(w.y, v[1].x, acc[i][g][0]); acc[i][g][1] = fmaf(w.y, v[1].y, acc[i][g][1]);
-              acc[i][g][0] = fmaf(w.z, v[2].x, acc[i][g][0]); acc[i][g][1] = fmaf(w.z, v[2].y, acc[i][g][1]);
-              acc[i][g][0] = fmaf(w.w, v[3].x, acc[i][g][0]); acc[i][g][1] = fmaf(w.w, v[3].y, acc[i][g][1]);
-            }
+        for (int e = 0; e < 2; ++e) {
+          acc[i][e][0] *= al0; acc[i][e][1] *= al0;
+          acc[i][e][2] *= al1; acc[i][e][3] *= al1;
+        }
+        const __nv_bfloat16* w0 = ps + h0 * L.p_row + (lane & 3) * 2;
+        const __nv_bfloat16* w1 = ps + h1 * L.p_row + (lane & 3) * 2;
+        const __nv_bfloat16* vb = vs + (buf * KT + ((lane >> 3) & 1) * 8 + (lane & 7)) * L.v_row + (first_piece + i) * 16 + (lane >> 4) * 8;
+        for (int k = 0; k < KT; k += 16, vb += 16 * L.v_row) {
+          uint32_t a[4], b[4];
+          a[0] = in0 ? *reinterpret_cast<const uint32_t*>(w0 + k) : 0u;
+          a[1] = in1 ? *reinterpret_cast<const uint32_t*>(w1 + k) : 0u;
+          a[2] = in0 ? *reinterpret_cast<const uint32_t*>(w0 + k + 8) : 0u;
+          a[3] = in1 ? *reinterpret_cast<const uint32_t*>(w1 + k + 8) : 0u;
+          ldmatrix_x4_trans(b, vb);
+          mma_bf16(acc[i][0], a, b[0], b[1]);
+          mma_bf16(acc[i][1], a, b[2], b[3]);
         }
       }
     }
@@ -271,16 +290,19 @@ __global__ void __launch_bounds__(THREADS, HT * IT <= 16 ? 2 : 1) attn_rows_deco
   }
   // ---- what the range leaves
 #pragma unroll
-  for (int i = 0; i < IT; ++i) {
-    const int pr = tid + i * THREADS;
-    if (pr < pairs) {
-      const int c = pr / (DV / 2), d = pr * 2 - c * DV;
+  for (int i = 0; i < NP; ++i) {
+    const int piece = first_piece + i;
+    if (piece < pieces) {
+      const int c = piece * 16 / DV, d = piece * 16 - c * DV + (lane & 3) * 2;
 #pragma unroll
-      for (int g = 0; g < HT; ++g)
+      for (int half = 0; half < 2; ++half) {
+        const int g = half ? g1 : g0;
         if (g < HPT) {
-          const size_t at = ((size_t)blockIdx.x * H + c * HPT + g) * p.n_splits + blockIdx.y;
-          *reinterpret_cast<float2*>(p.part_o + at * DV + d) = make_float2(acc[i][g][0], acc[i][g][1]);
+          float* o = p.part_o + (((size_t)blockIdx.x * H + c * HPT + g) * p.n_splits + blockIdx.y) * DV + d;
+          *reinterpret_cast<float2*>(o) = make_float2(acc[i][0][2 * half], acc[i][0][2 * half + 1]);
+          *reinterpret_cast<float2*>(o + 8) = make_float2(acc[i][1][2 * half], acc[i][1][2 * half + 1]);
         }
+      }
     }
   }
   for (int h = tid; h < H; h += THREADS) {
@@ -328,19 +350,22 @@ __global__ void __launch_bounds__(128) attn_rows_merge_kernel(const Params p) {
 }
 
 // Parts of KD that the warps of 16 heads share.
-int parts_of(int H) { return WARPS / ((H + 15) / 16); }
+int parts_of(int H) {
+  const int mt = (H + 15) / 16;
+  return mt <= 1 ? 8 : mt <= 2 ? 4 : mt <= 4 ? 2 : 1;
+}
 
-// Keys of a tile: as many as let two blocks share a multiprocessor, 64 at most and 8 at least (then one block may need
+// Keys of a tile: as many as let two blocks share a multiprocessor, 64 at most and 16 at least (then one block may need
 // most of the shared memory).
 int tile_keys(int H, int G, int KD, int DV) {
-  for (int kt = 64; kt >= 8; kt /= 2)
-    if (Layout(H, G, KD, DV, kt, parts_of(H)).total <= (kt > 8 ? 104 : 200) * 1024) return kt;
+  for (int kt = 64; kt >= 16; kt /= 2)
+    if (Layout(H, G, KD, DV, kt, parts_of(H)).total <= (kt > 16 ? 104 : 200) * 1024) return kt;
   return 0;
 }
 
-template <int HT, int IT, int KS>
+template <int NP, int KP, int KS>
 int launch(const Params& p, int n_work, size_t smem, cudaStream_t stream) {
-  auto kern = attn_rows_decode_kernel<HT, IT, KS>;
+  auto kern = attn_rows_decode_kernel<NP, KP, KS>;
   static bool ready[JV_MAX_DEVICES];
   if (!jv_once_per_device(ready, [&] {
         return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) == cudaSuccess;
@@ -351,20 +376,22 @@ int launch(const Params& p, int n_work, size_t smem, cudaStream_t stream) {
   return jv_launch(attn_rows_merge_kernel, dim3(n_work, p.H), dim3(128), 0, stream, p);
 }
 
-template <int HT, int IT>
-int launch_steps(const Params& p, int n_work, size_t smem, cudaStream_t stream) {
-  return (p.KD / 16 + p.k_parts - 1) / p.k_parts <= 8 ? launch<HT, IT, 8>(p, n_work, smem, stream)
-                                                      : launch<HT, IT, 16>(p, n_work, smem, stream);
+template <int NP>
+int launch_parts(const Params& p, int n_work, size_t smem, cudaStream_t stream) {
+  const int kp = parts_of(p.H), steps = (p.KD / 16 + kp - 1) / kp;
+  if (kp == 8) return launch<NP, 8, 8>(p, n_work, smem, stream);
+  if (kp == 4) return steps <= 8 ? launch<NP, 4, 8>(p, n_work, smem, stream) : launch<NP, 4, 16>(p, n_work, smem, stream);
+  if (kp == 2) return launch<NP, 2, 16>(p, n_work, smem, stream);
+  return launch<NP, 1, 16>(p, n_work, smem, stream);
 }
 }  // namespace
 
-// 1 if the kernel takes these sizes: KD a multiple of 16, DV of 8, up to 16 query heads a value head and 128 in all, and
-// what a thread keeps in registers: 16 steps of the queries, 32 pairs of outputs.
+// 1 if the kernel takes these sizes: KD and DV multiples of 16, up to 16 query heads a value head and 128 in all, and what a
+// warp keeps in registers: 16 steps of the queries, 8 pieces of 16 columns of the output.
 JV_EXPORT int jv_attn_rows_decode_supports(int H, int G, int KD, int DV) {
-  if (G < 1 || H < 1 || H % G || H > MAX_HEADS || KD % 16 || KD < 16 || DV % 8 || DV < 8) return 0;
-  const int hpt = H / G, ht = hpt <= 4 ? 4 : hpt <= 8 ? 8 : 16;
-  const int it = (G * DV / 2 + THREADS - 1) / THREADS;
-  return hpt <= 16 && it <= 4 && ht * it <= 32 && (KD / 16 + parts_of(H) - 1) / parts_of(H) <= 16 && tile_keys(H, G, KD, DV) > 0;
+  if (G < 1 || H < 1 || H % G || H > MAX_HEADS || KD % 16 || KD < 16 || DV % 16 || DV < 16) return 0;
+  const int kp = parts_of(H), steps = (KD / 16 + kp - 1) / kp;
+  return H / G <= 16 && G * DV <= 1024 && steps <= (kp == 8 ? 8 : 16) && tile_keys(H, G, KD, DV) > 0;
 }
 
 // q: rows of q_stride elements, head h of a token at column h*KD; out: rows of out_stride, head h at h*DV; k_cache:
@@ -386,12 +413,9 @@ JV_EXPORT int jv_attn_rows_decode(const void* q, int q_stride, void* out, int ou
   p.block_table = block_table; p.table_width = table_width; p.cu_seqlens = cu_seqlens; p.start_pos = start_pos; p.work = work;
   p.H = H; p.G = G; p.KD = KD; p.DV = DV; p.page_size = page_size; p.num_pages = num_pages; p.scale_log2 = scale * LOG2E;
   p.out_scale = out_scale; p.sink = sink; p.split_size = split_size; p.n_splits = n_splits; p.status = status;
-  p.KT = tile_keys(H, G, KD, DV); p.k_parts = parts_of(H);
-  const size_t smem = Layout(H, G, KD, DV, p.KT, p.k_parts).total;
-  const int hpt = H / G, it = (G * DV / 2 + THREADS - 1) / THREADS;
-  if (hpt <= 4) return it <= 1 ? launch_steps<4, 1>(p, n_work, smem, stream) : it <= 2 ? launch_steps<4, 2>(p, n_work, smem, stream)
-                                                                                       : launch_steps<4, 4>(p, n_work, smem, stream);
-  if (hpt <= 8) return it <= 1 ? launch_steps<8, 1>(p, n_work, smem, stream) : it <= 2 ? launch_steps<8, 2>(p, n_work, smem, stream)
-                                                                                       : launch_steps<8, 4>(p, n_work, smem, stream);
-  return it <= 1 ? launch_steps<16, 1>(p, n_work, smem, stream) : launch_steps<16, 2>(p, n_work, smem, stream);
+  p.KT = tile_keys(H, G, KD, DV);
+  const size_t smem = Layout(H, G, KD, DV, p.KT, parts_of(H)).total;
+  const int np = (G * DV / 16 + WARPS - 1) / WARPS;
+  return np <= 2 ? launch_parts<2>(p, n_work, smem, stream) : np <= 4 ? launch_parts<4>(p, n_work, smem, stream)
+                                                                      : launch_parts<8>(p, n_work, smem, stream);
 }

@@ -887,17 +887,14 @@ def attn_decode_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cac
 
 
 def attn_rows_decode_supports(dtype: torch.dtype, n_q_heads: int, n_v_heads: int, row: int, value_dim: int) -> bool:
-    """Whether the decode kernel for whole key rows takes these sizes (csrc/attn_rows_decode.cu): bfloat16, rows in steps
-    of 16, values in steps of 8, what a thread keeps of queries and output in registers, two stages of 8 keys in shared
-    memory."""
-    if dtype != torch.bfloat16 or row % 16 or row < 16 or value_dim % 8 or value_dim < 8 or n_q_heads % n_v_heads or n_q_heads > 128:
+    """Whether the decode kernel for whole key rows takes these sizes (csrc/attn_rows_decode.cu): bfloat16, rows and values
+    in steps of 16, what a warp keeps of queries and output in registers, two stages of 16 keys in shared memory."""
+    if dtype != torch.bfloat16 or row % 16 or row < 16 or value_dim % 16 or value_dim < 16 or n_q_heads % n_v_heads or n_q_heads > 128:
         return False
-    group, heads16 = n_q_heads // n_v_heads, -(-n_q_heads // 16) * 16
-    pairs = -(-n_v_heads * value_dim // 512)                 # column pairs a thread
-    parts = 8 // (heads16 // 16)                             # parts of a row that warps share
-    smem = 32 * (row + 8 + n_v_heads * value_dim) + 4 * parts * heads16 * 12
-    return group <= 16 and pairs <= 4 and (4 if group <= 4 else 8 if group <= 8 else 16) * pairs <= 32 and \
-        -(-row // 16 // parts) <= 16 and smem <= 200 * 1024
+    heads16 = -(-n_q_heads // 16) * 16
+    parts = 8 if heads16 <= 16 else 4 if heads16 <= 32 else 2 if heads16 <= 64 else 1       # parts of a row that warps share
+    smem = 64 * (row + n_v_heads * value_dim + 16) + 4 * parts * heads16 * 20 + 2 * heads16 * 24
+    return n_q_heads // n_v_heads <= 16 and n_v_heads * value_dim <= 1024 and -(-row // 16 // parts) <= (8 if parts == 8 else 16) and smem <= 200 * 1024
 
 
 def attn_rows_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
