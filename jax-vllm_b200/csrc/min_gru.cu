@@ -103,6 +103,7 @@ __global__ void __launch_bounds__(THREADS, 1) gru_scan_kernel(const GruParams p)
     Bs[run][cl] = B;
     __syncthreads();
     float S = carry[which][cl];
+#pragma unroll 8
     for (int r = 0; r < run; ++r) S = fmaf(-Ds[r][cl], S, S) + Bs[r][cl];
     if (run == RUNS - 1) carry[which ^ 1][cl] = fmaf(-D, S, S) + B;
 #pragma unroll

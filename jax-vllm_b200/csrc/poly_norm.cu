@@ -140,9 +140,12 @@ int launch(const void* in, long long in_stride, void* out, long long out_stride,
   const bool vec = width % VEC == 0 && in_stride % VEC == 0 && out_stride % VEC == 0 && part_stride % VEC == 0 &&
                    (uintptr_t)in % ai == 0 && (uintptr_t)out % ao == 0;
   const int per = width / VEC;
-  // a few long rows: as many threads as the row has vectors, up to 1,024; many rows: 256 threads with more vectors each
-  int threads = n <= 148 ? 1024 : 256;
+  // a few rows: as many threads as a row has vectors, up to 1,024; many rows: four vectors a thread where that leaves 128
+  // threads at least
+  int threads = 1024;
   while (threads > 64 && threads / 2 >= per) threads /= 2;
+  if (n > 148)
+    while (threads > 128 && (per + threads / 2 - 1) / (threads / 2) <= 4) threads /= 2;
   const int iters = (per + threads - 1) / threads;
 #define JV_POLY(I)                                                                                                          \
   if (vec && iters <= I)                                                                                                    \

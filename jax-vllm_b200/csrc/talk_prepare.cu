@@ -17,8 +17,9 @@
 // they are to v_cache[page, slot, G, DV].
 //
 // One block a token (or, for a few tokens, several blocks a token that share its mixed heads; only the first writes the
-// cache).  The queries of the token lie in shared memory as floats; a thread keeps 4 elements of the query heads of one
-// key head in registers and forms its elements of every mixed head from them.
+// cache).  All of the token's queries and keys come into shared memory as floats in one go, are normed and rotated there, one
+// warp a head, and the keys leave for their page; a thread keeps 4 elements of the query heads of one key head in registers
+// and forms its elements of every mixed head from them.
 #include "common.cuh"
 
 namespace {
@@ -35,18 +36,31 @@ struct TalkParams {
   void* k_cache; void* v_cache;
   int n, n_q_heads, n_kv_heads, key_dim, value_dim, page_size, num_pages;
   int parts;                         // blocks per token
+  int vec_in;                        // the projection's rows and offsets allow 4 elements an access
   int* status;
 };
 
 template <typename T, int V> struct Pack;
-template <> struct Pack<float, 1> { static __device__ __forceinline__ void store(float* p, const float (&v)[1]) { *p = v[0]; } };
+template <> struct Pack<float, 1> {
+  static __device__ __forceinline__ void store(float* p, const float (&v)[1]) { *p = v[0]; }
+};
 template <> struct Pack<float, 4> {
   static __device__ __forceinline__ void store(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+  static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  }
 };
 template <> struct Pack<__nv_bfloat16, 1> {
   static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[1]) { *p = __float2bfloat16_rn(v[0]); }
 };
 template <> struct Pack<__nv_bfloat16, 4> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[4]) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&a);
+    const float2 f0 = __bfloat1622float2(h[0]), f1 = __bfloat1622float2(h[1]);
+    v[0] = f0.x; v[1] = f0.y; v[2] = f1.x; v[3] = f1.y;
+  }
   static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[4]) {
     uint2 u;
     __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
@@ -62,8 +76,8 @@ __global__ void __launch_bounds__(THREADS) talk_prepare_kernel(const TalkParams 
   extern __shared__ __align__(16) float smem[];
   pdl_trigger();
   const int H = p.n_q_heads, G = p.n_kv_heads, D = p.key_dim, HPT = H / G, half = p.rot_dim >> 1;
-  float* qs = smem;                                    // [H][D], 16-byte aligned rows where VEC = 4
-  float* cs = qs + (((size_t)H * D + 3) & ~(size_t)3);  // [half] cosines, then [half] sines
+  float* qs = smem;                                    // [H + G][D]: query heads, then key heads
+  float* cs = qs + (((size_t)(H + G) * D + 3) & ~(size_t)3);  // [half] cosines, then [half] sines
   float* sn = cs + half;
   float* ts = sn + half;                               // [mixed heads of this block][H]
   const int t = blockIdx.x / p.parts, part = blockIdx.x - t * p.parts;
@@ -72,50 +86,58 @@ __global__ void __launch_bounds__(THREADS) talk_prepare_kernel(const TalkParams 
   for (int i = tid; i < (h_hi - h_lo) * H; i += THREADS) ts[i] = p.talk[(size_t)h_lo * H + i];   // a weight: before the wait
   pdl_wait();
   const int posi = p.positions[t];
-  for (int j = tid; j < half; j += THREADS) sincosf((float)posi * p.freq[j], &sn[j], &cs[j]);
-  __syncthreads();
   const T* row = (const T*)p.proj + (size_t)t * p.row_stride;
-
-  // ---- query heads into shared memory; the block that writes the cache takes the key and value heads as well
   const bool writes = p.k_cache != nullptr && part == 0;
+
+  // ---- queries (and, for the block that writes the cache, keys) into shared memory
+  const int n_heads = H + (writes ? G : 0);
+  if (VEC == 4 && p.vec_in) {
+    for (int i = tid; i < n_heads * D / 4; i += THREADS) {
+      const int e = i * 4;
+      float v[4];
+      Pack<T, 4>::load(row + (e < H * D ? p.q_off + e : p.k_off + e - H * D), v);
+      *reinterpret_cast<float4*>(qs + e) = make_float4(v[0], v[1], v[2], v[3]);
+    }
+  } else {
+    for (int e = tid; e < n_heads * D; e += THREADS) qs[e] = to_f32(row[e < H * D ? p.q_off + e : p.k_off + e - H * D]);
+  }
+  for (int j = tid; j < half; j += THREADS) sincosf((float)posi * p.freq[j], &sn[j], &cs[j]);
   size_t slot = 0;
-  bool page_ok = true;
+  bool page_ok = false;
   if (writes) {
     const int pi = posi / p.page_size;
     const int page = (posi >= 0 && pi < p.table_width) ? p.block_table[(size_t)p.token_entry[t] * p.table_width + pi] : -1;
     page_ok = page >= 0 && page < p.num_pages;
-    if (page_ok) slot = (size_t)page * p.page_size + (posi - pi * p.page_size);
-    else if (tid == 0) atomicOr(p.status, JV_STATUS_BAD_PAGE);
-  }
-  const int n_heads = H + ((writes && page_ok) ? 2 * G : 0);
-  for (int h = warp; h < n_heads; h += THREADS / 32) {
-    if (h >= H + G) {                                   // a value head: copied
-      const int g = h - H - G;
-      const T* src = row + p.v_off + (size_t)g * p.value_dim;
-      T* dst = (T*)p.v_cache + (slot * G + g) * p.value_dim;
-      for (int d = lane; d < p.value_dim; d += 32) dst[d] = src[d];
-      continue;
+    if (page_ok) {
+      slot = (size_t)page * p.page_size + (posi - pi * p.page_size);
+      T* dst = (T*)p.v_cache + slot * G * p.value_dim;           // the values of all heads, as they are
+      for (int e = tid; e < G * p.value_dim; e += THREADS) dst[e] = row[p.v_off + e];
+    } else if (tid == 0) {
+      atomicOr(p.status, JV_STATUS_BAD_PAGE);
     }
-    const bool is_q = h < H;
-    const T* src = row + (is_q ? p.q_off + (size_t)h * D : p.k_off + (size_t)(h - H) * D);
+  }
+  __syncthreads();
+
+  // ---- norm and rotation, one warp a head
+  for (int h = warp; h < n_heads; h += THREADS / 32) {
+    float* x = qs + (size_t)h * D;
     float inv = 1.f;
     if (p.normed) {
       float ss = 0.f;
-      for (int d = lane; d < D; d += 32) { const float v = to_f32(src[d]); ss += v * v; }
+      for (int d = lane; d < D; d += 32) ss = fmaf(x[d], x[d], ss);
       inv = rsqrtf(warp_sum(ss) / (float)D + p.eps);
     }
-    float* qd = qs + (size_t)h * D;
-    T* kd = (T*)p.k_cache + (slot * G + (h - H)) * D;
+    T* kd = (h >= H && page_ok) ? (T*)p.k_cache + (slot * G + (h - H)) * D : nullptr;
     for (int j = lane; j < half; j += 32) {
-      const float u = to_f32(src[j]) * inv, v = to_f32(src[j + half]) * inv;
+      const float u = x[j] * inv, v = x[j + half] * inv;
       const float a = u * cs[j] - v * sn[j], b = v * cs[j] + u * sn[j];
-      if (is_q) { qd[j] = a; qd[j + half] = b; }
-      else { kd[j] = from_f32<T>(a); kd[j + half] = from_f32<T>(b); }
+      x[j] = a; x[j + half] = b;
+      if (kd != nullptr) { kd[j] = from_f32<T>(a); kd[j + half] = from_f32<T>(b); }
     }
     for (int d = p.rot_dim + lane; d < D; d += 32) {
-      const float u = to_f32(src[d]) * inv;
-      if (is_q) qd[d] = u;
-      else kd[d] = from_f32<T>(u);
+      const float u = x[d] * inv;
+      x[d] = u;
+      if (kd != nullptr) kd[d] = from_f32<T>(u);
     }
   }
   __syncthreads();
@@ -190,8 +212,10 @@ JV_EXPORT int jv_talk_prepare(const void* proj, int dtype, long long row_stride,
   p.parts = 1;
   while (p.parts < 8 && n * p.parts * 2 <= 148 && n_q_heads / (p.parts * 2) >= 2) p.parts *= 2;
   const size_t head_rows = (n_q_heads + p.parts - 1) / p.parts;
-  const size_t smem = sizeof(float) * ((((size_t)n_q_heads * key_dim + 3) & ~(size_t)3) + rot_dim + head_rows * n_q_heads);
+  const size_t smem = sizeof(float) * ((((size_t)(n_q_heads + n_kv_heads) * key_dim + 3) & ~(size_t)3) + rot_dim + head_rows * n_q_heads);
   if (smem > 200 * 1024) return JV_ERR_UNSUPPORTED;
+  const size_t unit = dtype == 0 ? 16 : 8;
+  p.vec_in = row_stride % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && (uintptr_t)proj % unit == 0;
   const bool vec = key_dim % 4 == 0 && (uintptr_t)q_out % 16 == 0;
   JV_DISPATCH_DTYPE(dtype, T, {
     if (vec) return launch<T, 4>(p, smem, stream);
