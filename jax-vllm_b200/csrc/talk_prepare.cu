@@ -17,9 +17,8 @@
 // they are to v_cache[page, slot, G, DV].
 //
 // One block a token (or, for a few tokens, several blocks a token that share its mixed heads; only the first writes the
-// cache).  All of the token's queries and keys come into shared memory as floats in one go, are normed and rotated there, one
-// warp a head, and the keys leave for their page; a thread keeps 4 elements of the query heads of one key head in registers
-// and forms its elements of every mixed head from them.
+// cache).  One warp norms and rotates a head; the queries lie in shared memory as floats, and a thread keeps 4 elements of
+// the query heads of one key head in registers and forms its elements of every mixed head from them.
 #include "common.cuh"
 
 namespace {
@@ -36,7 +35,6 @@ struct TalkParams {
   void* k_cache; void* v_cache;
   int n, n_q_heads, n_kv_heads, key_dim, value_dim, page_size, num_pages;
   int parts;                         // blocks per token
-  int vec_in;                        // the projection's rows and offsets allow 4 elements an access
   int* status;
 };
 
@@ -46,21 +44,11 @@ template <> struct Pack<float, 1> {
 };
 template <> struct Pack<float, 4> {
   static __device__ __forceinline__ void store(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
-  static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
-    const float4 a = *reinterpret_cast<const float4*>(p);
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-  }
 };
 template <> struct Pack<__nv_bfloat16, 1> {
   static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[1]) { *p = __float2bfloat16_rn(v[0]); }
 };
 template <> struct Pack<__nv_bfloat16, 4> {
-  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[4]) {
-    const uint2 a = *reinterpret_cast<const uint2*>(p);
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&a);
-    const float2 f0 = __bfloat1622float2(h[0]), f1 = __bfloat1622float2(h[1]);
-    v[0] = f0.x; v[1] = f0.y; v[2] = f1.x; v[3] = f1.y;
-  }
   static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[4]) {
     uint2 u;
     __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
@@ -70,75 +58,116 @@ template <> struct Pack<__nv_bfloat16, 4> {
   }
 };
 
-// VEC: elements of a mixed head that a thread forms together (4 where the key size allows it).
-template <typename T, int VEC>
+// VEC: elements of a mixed head that a thread forms together (4 where the key size allows it).  HPTC: query heads of a key
+// head, 4 or 8 (0: any number).  ND: the key size in 32s where a rotation by whole 32s lets a lane hold both elements of its
+// pairs in registers, 2 or 4 (0: any size, pairs through shared memory).
+template <typename T, int VEC, int HPTC, int ND>
 __global__ void __launch_bounds__(THREADS) talk_prepare_kernel(const TalkParams p) {
   extern __shared__ __align__(16) float smem[];
   pdl_trigger();
-  const int H = p.n_q_heads, G = p.n_kv_heads, D = p.key_dim, HPT = H / G, half = p.rot_dim >> 1;
-  float* qs = smem;                                    // [H + G][D]: query heads, then key heads
-  float* cs = qs + (((size_t)(H + G) * D + 3) & ~(size_t)3);  // [half] cosines, then [half] sines
-  float* sn = cs + half;
-  float* ts = sn + half;                               // [mixed heads of this block][H]
+  const int H = p.n_q_heads, G = p.n_kv_heads, D = p.key_dim, HPT = HPTC > 0 ? HPTC : H / G, half = p.rot_dim >> 1;
+  float* ts = smem;                                    // [mixed heads of this block][H]
   const int t = blockIdx.x / p.parts, part = blockIdx.x - t * p.parts;
   const int h_lo = (int)((long long)H * part / p.parts), h_hi = (int)((long long)H * (part + 1) / p.parts);
+  float* qs = ts + (((h_hi - h_lo) * H + 3) & ~3);     // [H][D]
+  float* ks = qs + (((size_t)H * D + 3) & ~(size_t)3);  // ND == 0: [G][D], then the angles' [half] cosines and sines
+  float* cs = ks + (size_t)G * D;
+  float* sn = cs + half;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   for (int i = tid; i < (h_hi - h_lo) * H; i += THREADS) ts[i] = p.talk[(size_t)h_lo * H + i];   // a weight: before the wait
   pdl_wait();
   const int posi = p.positions[t];
   const T* row = (const T*)p.proj + (size_t)t * p.row_stride;
   const bool writes = p.k_cache != nullptr && part == 0;
-
-  // ---- queries (and, for the block that writes the cache, keys) into shared memory
   const int n_heads = H + (writes ? G : 0);
-  if (VEC == 4 && p.vec_in) {
-    for (int i = tid; i < n_heads * D / 4; i += THREADS) {
-      const int e = i * 4;
-      float v[4];
-      Pack<T, 4>::load(row + (e < H * D ? p.q_off + e : p.k_off + e - H * D), v);
-      *reinterpret_cast<float4*>(qs + e) = make_float4(v[0], v[1], v[2], v[3]);
-    }
-  } else {
-    for (int e = tid; e < n_heads * D; e += THREADS) qs[e] = to_f32(row[e < H * D ? p.q_off + e : p.k_off + e - H * D]);
+  constexpr int WARPS = THREADS / 32;
+  // element e of the token's query and key heads, in the order [query heads][key heads]
+  auto source = [&](int h) { return row + (h < H ? p.q_off + h * D : p.k_off + (h - H) * D); };
+  T raw[ND > 0 ? ND : 1];
+  if (ND > 0 && warp < n_heads) {
+#pragma unroll
+    for (int i = 0; i < ND; ++i) raw[i] = source(warp)[lane + 32 * i];
   }
-  for (int j = tid; j < half; j += THREADS) sincosf((float)posi * p.freq[j], &sn[j], &cs[j]);
   size_t slot = 0;
   bool page_ok = false;
   if (writes) {
     const int pi = posi / p.page_size;
     const int page = (posi >= 0 && pi < p.table_width) ? p.block_table[(size_t)p.token_entry[t] * p.table_width + pi] : -1;
     page_ok = page >= 0 && page < p.num_pages;
-    if (page_ok) {
-      slot = (size_t)page * p.page_size + (posi - pi * p.page_size);
-      T* dst = (T*)p.v_cache + slot * G * p.value_dim;           // the values of all heads, as they are
-      for (int e = tid; e < G * p.value_dim; e += THREADS) dst[e] = row[p.v_off + e];
-    } else if (tid == 0) {
-      atomicOr(p.status, JV_STATUS_BAD_PAGE);
+    if (page_ok) slot = (size_t)page * p.page_size + (posi - pi * p.page_size);
+    else if (tid == 0) atomicOr(p.status, JV_STATUS_BAD_PAGE);
+  }
+  if (ND > 0) {
+    // ---- one warp a head, pairs within a lane: element lane + 32 i turns with lane + 32 (i + half / 32)
+    const int hi = half >> 5;
+    float c[ND > 0 ? ND : 1], s[ND > 0 ? ND : 1];
+#pragma unroll
+    for (int i = 0; i < ND / 2; ++i)
+      if (i < hi) sincosf((float)posi * p.freq[lane + 32 * i], &s[i], &c[i]);
+    for (int h = warp; h < n_heads; h += WARPS) {
+      float x[ND > 0 ? ND : 1];
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < ND; ++i) { x[i] = to_f32(raw[i]); ss = fmaf(x[i], x[i], ss); }
+      if (h + WARPS < n_heads) {                       // the next head's loads fly while this one is worked on
+#pragma unroll
+        for (int i = 0; i < ND; ++i) raw[i] = source(h + WARPS)[lane + 32 * i];
+      }
+      if (p.normed) {
+        const float inv = rsqrtf(warp_sum(ss) / (float)D + p.eps);
+#pragma unroll
+        for (int i = 0; i < ND; ++i) x[i] *= inv;
+      }
+#pragma unroll
+      for (int i = 0; i < ND / 2; ++i)
+#pragma unroll
+        for (int o = 1; o <= ND / 2; ++o)              // the partner's place, i + hi, as a constant
+          if (o == hi && i < hi) {
+            const float u = x[i], v = x[i + o];
+            x[i] = u * c[i] - v * s[i];
+            x[i + o] = v * c[i] + u * s[i];
+          }
+      if (h < H) {
+#pragma unroll
+        for (int i = 0; i < ND; ++i) qs[(size_t)h * D + lane + 32 * i] = x[i];
+      } else if (page_ok) {
+        T* kd = (T*)p.k_cache + (slot * G + (h - H)) * D + lane;
+#pragma unroll
+        for (int i = 0; i < ND; ++i) kd[32 * i] = from_f32<T>(x[i]);
+      }
+    }
+  } else {
+    for (int e = tid; e < n_heads * D; e += THREADS) {
+      const int h = e / D;
+      (h < H ? qs[e] : ks[e - H * D]) = to_f32(source(h)[e - h * D]);
+    }
+    for (int j = tid; j < half; j += THREADS) sincosf((float)posi * p.freq[j], &sn[j], &cs[j]);
+    __syncthreads();
+    for (int h = warp; h < n_heads; h += WARPS) {
+      float* x = h < H ? qs + (size_t)h * D : ks + (size_t)(h - H) * D;
+      float inv = 1.f;
+      if (p.normed) {
+        float ss = 0.f;
+        for (int d = lane; d < D; d += 32) ss = fmaf(x[d], x[d], ss);
+        inv = rsqrtf(warp_sum(ss) / (float)D + p.eps);
+      }
+      T* kd = (h >= H && page_ok) ? (T*)p.k_cache + (slot * G + (h - H)) * D : nullptr;
+      for (int j = lane; j < half; j += 32) {
+        const float u = x[j] * inv, v = x[j + half] * inv;
+        const float a = u * cs[j] - v * sn[j], b = v * cs[j] + u * sn[j];
+        x[j] = a; x[j + half] = b;
+        if (kd != nullptr) { kd[j] = from_f32<T>(a); kd[j + half] = from_f32<T>(b); }
+      }
+      for (int d = p.rot_dim + lane; d < D; d += 32) {
+        const float u = x[d] * inv;
+        x[d] = u;
+        if (kd != nullptr) kd[d] = from_f32<T>(u);
+      }
     }
   }
-  __syncthreads();
-
-  // ---- norm and rotation, one warp a head
-  for (int h = warp; h < n_heads; h += THREADS / 32) {
-    float* x = qs + (size_t)h * D;
-    float inv = 1.f;
-    if (p.normed) {
-      float ss = 0.f;
-      for (int d = lane; d < D; d += 32) ss = fmaf(x[d], x[d], ss);
-      inv = rsqrtf(warp_sum(ss) / (float)D + p.eps);
-    }
-    T* kd = (h >= H && page_ok) ? (T*)p.k_cache + (slot * G + (h - H)) * D : nullptr;
-    for (int j = lane; j < half; j += 32) {
-      const float u = x[j] * inv, v = x[j + half] * inv;
-      const float a = u * cs[j] - v * sn[j], b = v * cs[j] + u * sn[j];
-      x[j] = a; x[j + half] = b;
-      if (kd != nullptr) { kd[j] = from_f32<T>(a); kd[j + half] = from_f32<T>(b); }
-    }
-    for (int d = p.rot_dim + lane; d < D; d += 32) {
-      const float u = x[d] * inv;
-      x[d] = u;
-      if (kd != nullptr) kd[d] = from_f32<T>(u);
-    }
+  if (page_ok) {                                       // the values of all heads, as they are
+    T* dst = (T*)p.v_cache + slot * G * p.value_dim;
+    for (int e = tid; e < G * p.value_dim; e += THREADS) dst[e] = row[p.v_off + e];
   }
   __syncthreads();
 
@@ -149,37 +178,59 @@ __global__ void __launch_bounds__(THREADS) talk_prepare_kernel(const TalkParams 
     const int sub = i / places, at = (i - sub * places) * VEC;
     const int c = at / D, d = at - c * D;
     const float* q0 = qs + (size_t)c * HPT * D + d;      // query heads of key head c, D apart
-    float q[GROUP_REGS][VEC];
+    constexpr int REGS = HPTC > 0 ? HPTC : GROUP_REGS;
+    float q[REGS][VEC];
 #pragma unroll
-    for (int g = 0; g < GROUP_REGS; ++g)
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) q[g][e] = g < HPT ? q0[(size_t)g * D + e] : 0.f;
+    for (int g = 0; g < REGS; ++g) {
+      if (VEC == 4) {
+        const float4 f = g < HPT ? *reinterpret_cast<const float4*>(q0 + (size_t)g * D) : make_float4(0.f, 0.f, 0.f, 0.f);
+        q[g][0] = f.x; q[g][VEC > 1 ? 1 : 0] = f.y; q[g][VEC > 2 ? 2 : 0] = f.z; q[g][VEC > 3 ? 3 : 0] = f.w;
+      } else {
+        q[g][0] = g < HPT ? q0[(size_t)g * D] : 0.f;
+      }
+    }
     const int n_here = h_hi - h_lo, lo = n_here * sub / subs, hi = n_here * (sub + 1) / subs;
+    T* dst = (T*)p.q_out + ((size_t)t * H + h_lo) * GD + at;
+#pragma unroll 2
     for (int h = lo; h < hi; ++h) {
-      const float* w = ts + (size_t)h * H + c * HPT;
+      const float* w = ts + h * H + c * HPT;
       float acc[VEC];
 #pragma unroll
       for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+      if (HPTC > 0) {
 #pragma unroll
-      for (int g = 0; g < GROUP_REGS; ++g)
-        if (g < HPT) {
+        for (int g = 0; g < HPTC; g += 4) {
+          const float4 wg = *reinterpret_cast<const float4*>(w + g);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            acc[e] = fmaf(wg.x, q[g][e], acc[e]);
+            acc[e] = fmaf(wg.y, q[g + 1][e], acc[e]);
+            acc[e] = fmaf(wg.z, q[g + 2][e], acc[e]);
+            acc[e] = fmaf(wg.w, q[g + 3][e], acc[e]);
+          }
+        }
+      } else {
+#pragma unroll
+        for (int g = 0; g < REGS; ++g)
+          if (g < HPT) {
+            const float wg = w[g];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc[e] = fmaf(wg, q[g][e], acc[e]);
+          }
+        for (int g = REGS; g < HPT; ++g) {
           const float wg = w[g];
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) acc[e] = fmaf(wg, q[g][e], acc[e]);
+          for (int e = 0; e < VEC; ++e) acc[e] = fmaf(wg, q0[(size_t)g * D + e], acc[e]);
         }
-      for (int g = GROUP_REGS; g < HPT; ++g) {
-        const float wg = w[g];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) acc[e] = fmaf(wg, q0[(size_t)g * D + e], acc[e]);
       }
-      Pack<T, VEC>::store((T*)p.q_out + ((size_t)t * H + h_lo + h) * GD + at, acc);
+      Pack<T, VEC>::store(dst + (size_t)h * GD, acc);
     }
   }
 }
 
-template <typename T, int VEC>
+template <typename T, int VEC, int HPTC, int ND>
 int launch(const TalkParams& p, size_t smem, cudaStream_t stream) {
-  auto kern = talk_prepare_kernel<T, VEC>;
+  auto kern = talk_prepare_kernel<T, VEC, HPTC, ND>;
   static bool ready[JV_MAX_DEVICES];
   if (!jv_once_per_device(ready, [&] {
         return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) == cudaSuccess;
@@ -212,14 +263,20 @@ JV_EXPORT int jv_talk_prepare(const void* proj, int dtype, long long row_stride,
   p.parts = 1;
   while (p.parts < 8 && n * p.parts * 2 <= 148 && n_q_heads / (p.parts * 2) >= 2) p.parts *= 2;
   const size_t head_rows = (n_q_heads + p.parts - 1) / p.parts;
-  const size_t smem = sizeof(float) * ((((size_t)(n_q_heads + n_kv_heads) * key_dim + 3) & ~(size_t)3) + rot_dim + head_rows * n_q_heads);
+  const size_t up4 = ~(size_t)3;
+  const size_t smem = sizeof(float) * (((head_rows * n_q_heads + 3) & up4) + (((size_t)n_q_heads * key_dim + 3) & up4) +
+                                       (size_t)n_kv_heads * key_dim + rot_dim);
   if (smem > 200 * 1024) return JV_ERR_UNSUPPORTED;
-  const size_t unit = dtype == 0 ? 16 : 8;
-  p.vec_in = row_stride % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && (uintptr_t)proj % unit == 0;
   const bool vec = key_dim % 4 == 0 && (uintptr_t)q_out % 16 == 0;
+  const int hpt = n_q_heads / n_kv_heads;
+  const int nd = (vec && rot_dim % 64 == 0) ? (key_dim == 128 ? 4 : key_dim == 64 ? 2 : 0) : 0;
   JV_DISPATCH_DTYPE(dtype, T, {
-    if (vec) return launch<T, 4>(p, smem, stream);
-    return launch<T, 1>(p, smem, stream);
+    if (!vec) return launch<T, 1, 0, 0>(p, smem, stream);
+    if (nd == 4) return hpt == 4 ? launch<T, 4, 4, 4>(p, smem, stream) : hpt == 8 ? launch<T, 4, 8, 4>(p, smem, stream)
+                                                                                  : launch<T, 4, 0, 4>(p, smem, stream);
+    if (nd == 2) return hpt == 4 ? launch<T, 4, 4, 2>(p, smem, stream) : hpt == 8 ? launch<T, 4, 8, 2>(p, smem, stream)
+                                                                                  : launch<T, 4, 0, 2>(p, smem, stream);
+    return launch<T, 4, 0, 0>(p, smem, stream);
   });
   return JV_ERR_UNSUPPORTED;
 }
