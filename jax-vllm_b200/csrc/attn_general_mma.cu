@@ -30,13 +30,13 @@
 
 namespace {
 constexpr int KD = JV_KEY_DIM, VD = JV_VALUE_DIM;
-static_assert(KD % 16 == 0 && VD % 16 == 0 && KD >= 16 && VD >= 16 && KD <= 256 && VD <= 256, "sizes in steps of 16");
+static_assert(KD % 16 == 0 && VD % 16 == 0 && KD >= 16 && VD >= 16 && KD <= 512 && VD <= 256, "sizes in steps of 16");
 
 constexpr int BN = 64;         // keys per tile
 constexpr int NWARPS = 4;
 constexpr int THREADS = NWARPS * 32;
 constexpr int ROWS_PREFILL = 16 * NWARPS;
-constexpr int DECODE_STAGES = 3;
+constexpr int DECODE_STAGES = KD > 256 ? 2 : 3;
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct Params {
@@ -699,7 +699,7 @@ JV_EXPORT int jv_attn_general_mma(const void* q, int q_stride, void* out, int ou
   if ((q_stride % 8) || (out_stride % 2) || ((uintptr_t)q % 16) || ((uintptr_t)out % 8) || ((uintptr_t)k_cache % 16) ||
       ((uintptr_t)v_cache % 16))
     return JV_ERR_UNSUPPORTED;   // 16-byte copies need aligned rows
-  if (prefill_smem() > 227 * 1024 || decode_smem() > 227 * 1024) return JV_ERR_UNSUPPORTED;
+  if ((n_splits > 0 ? decode_smem() : prefill_smem()) > 227 * 1024) return JV_ERR_UNSUPPORTED;
   Params p;
   p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride; p.out = out; p.out_stride = out_stride; p.out_f32 = out_f32 ? 1 : 0;
   p.part_o = part_o; p.part_ml = part_ml; p.counters = counters;

@@ -468,14 +468,14 @@ def _score_extras(who: str, n_q_heads: int, head_scale, dist_bias, sink) -> int:
     return dist_bias.shape[1]
 
 
-GENERAL_MMA_MAX_KEY, GENERAL_MMA_MAX_VALUE = 256, 128
+GENERAL_MMA_MAX_KEY, GENERAL_MMA_MAX_VALUE = 512, 128
 
 
 def attn_general_mma_supports(dtype: torch.dtype, key_dim: int, value_dim: int) -> bool:
     """Whether the tensor-core kernel for keys and values of different sizes takes these (csrc/attn_general_mma.cu):
-    bfloat16, sizes in steps of 16."""
+    bfloat16, sizes in steps of 16, two stages of 64 keys and values beside 64 queries in shared memory."""
     return (dtype == torch.bfloat16 and key_dim % 16 == 0 and value_dim % 16 == 0
-            and 16 <= key_dim <= GENERAL_MMA_MAX_KEY and 16 <= value_dim <= GENERAL_MMA_MAX_VALUE)
+            and 2 * (192 * (key_dim + 8) + 128 * (value_dim + 8)) <= 227 * 1024 and 16 <= key_dim <= GENERAL_MMA_MAX_KEY and 16 <= value_dim <= GENERAL_MMA_MAX_VALUE)
 
 
 def attn_general_mma_library(key_dim: int, value_dim: int) -> str:

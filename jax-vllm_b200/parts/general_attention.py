@@ -143,7 +143,7 @@ class GeneralAttention(Part):
         # tokens to the kernel that reads each row once
         self.whole_rows = (self.talking and not spec.score_cap and not self.mask and self.hv == self.hk
                            and self.dv == self.d == 128)
-        self.rows_decode = (self.talking and not spec.score_cap and not self.mask and self.general is None
+        self.rows_decode = (self.talking and self.hk > 1 and not spec.score_cap and not self.mask
                             and ops.attn_rows_decode_supports(ctx.dtype, self.hq, self.hv, self.dk, self.dv))
         if self.big_tiles or (self.whole_rows and ctx.dtype == torch.bfloat16):
             self.kernels += ("attn_rows_tcgen05" if self.talking and self.hk > 1 else "attn_tcgen05",)

@@ -172,6 +172,7 @@ def test_mixed_queries_alone(H, G, D, E, rot, tokens, dtype):
 
 # name: (query heads, key heads, key size, value size, what serves it in bfloat16)
 TALK_CASES = {"general_96x48": (4, 2, 48, 48), "general_256x32": (8, 8, 32, 32), "general_16x64": (1, 1, 16, 64),
+              "general_512x64": (16, 8, 64, 64), "general_384x128": (6, 6, 64, 128), "many_heads": (96, 6, 32, 32),
               "odd_sizes": (3, 3, 21, 7), "wide_rows": (4, 4, 96, 40), "very_wide_rows": (12, 12, 130, 20),
               "one_key_head": (16, 1, 64, 32), "heads_of_128_on_2": (4, 2, 128, 128), "heads_of_128_on_4": (8, 4, 128, 128),
               "heads_of_128_on_8": (8, 8, 128, 128), "heads_of_128_on_1": (3, 1, 128, 128),
