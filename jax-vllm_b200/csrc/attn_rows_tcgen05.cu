@@ -37,6 +37,7 @@ constexpr int SOFTMAX_THREADS = 256;
 constexpr int TMEM_COLS = 512;                  // S0: [0,128)  S1: [128,256)  O: [256,384)  P0: [384,448)  P1: [448,512)
 constexpr int TMEM_O = 256, TMEM_P = 384;
 constexpr int MAX_STAGES = 4;
+constexpr int MAX_LISTED = 32;                  // rounds whose item a block looks up once, for all roles
 constexpr float LOG2E = 1.4426950408889634f;
 
 // By the number of pieces NC (0: five or more): items whose queries have a place, pieces that stay there, ring stages.
@@ -65,6 +66,7 @@ struct Shared {
   uint32_t tmem_base;
   int failed;                   // a role gave up on a wait
   int armed_q[2], armed[MAX_STAGES];   // parity of the phase the producer armed last; -1: never
+  int4 items[MAX_LISTED];       // the block's first items: entry, first row, first position, (group << 16 | tokens)
   float xch[2][128];            // a row's two softmax threads exchange their maxima (and at the end their sums)
 };
 
@@ -108,17 +110,23 @@ __global__ void __launch_bounds__(THREADS, 1) attn_rows_tcgen05_kernel(const __g
     return L < n_items ? L : -1;
   };
   const int n_rounds = (n_items + n_blocks - 1) / n_blocks;
-  auto load_item = [&](int L) -> Item {
+  auto look_up = [&](int r) -> int4 {
+    const int L = item_of_round(r);
+    if (L < 0) return make_int4(0, 0, 0, 0);
+    const int w = p.n_work - 1 - L / p.n_kv_heads, kv_head = L % p.n_kv_heads;
+    const int entry = p.work[2 * w], q_off = p.work[2 * w + 1];
+    const int q_begin = p.cu_seqlens[entry];
+    const int tokens = max(0, min(p.tokens_per_tile, p.cu_seqlens[entry + 1] - q_begin - q_off));
+    return make_int4(entry, q_begin + q_off, p.start_pos[entry] + q_off, kv_head << 16 | tokens);
+  };
+  auto load_item = [&](int r) -> Item {
+    const int4 v = r < MAX_LISTED ? sh->items[r] : look_up(r);
     Item it;
-    const int w = p.n_work - 1 - L / p.n_kv_heads;
-    it.kv_head = L % p.n_kv_heads;
-    it.entry = p.work[2 * w];
-    const int q_off = p.work[2 * w + 1];
-    const int q_begin = p.cu_seqlens[it.entry];
-    const int q_len = p.cu_seqlens[it.entry + 1] - q_begin;
-    it.q_first = q_begin + q_off;
-    it.tokens_here = min(p.tokens_per_tile, q_len - q_off);
-    it.pos_first = p.start_pos[it.entry] + q_off;
+    it.entry = v.x;
+    it.q_first = v.y;
+    it.pos_first = v.z;
+    it.kv_head = v.w >> 16;
+    it.tokens_here = v.w & 0xffff;
     it.j_hi = it.pos_first + it.tokens_here;
     it.n_tiles = it.tokens_here > 0 ? (it.j_hi + BN - 1) / BN : 0;
     it.turn = it.n_tiles > 0 ? blockIdx.x % it.n_tiles : 0;
@@ -127,9 +135,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_rows_tcgen05_kernel(const __g
   // the first item with tiles from round r on; r becomes its round
   auto next_item = [&](int& r, Item& out) -> bool {
     for (; r < n_rounds; ++r) {
-      const int L = item_of_round(r);
-      if (L < 0) continue;
-      out = load_item(L);
+      out = load_item(r);
       if (out.n_tiles > 0) return true;
     }
     return false;
@@ -146,6 +152,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_rows_tcgen05_kernel(const __g
     sh->failed = 0;
     mbar_fence_init();
   }
+  for (int r = threadIdx.x; r < min(n_rounds, MAX_LISTED); r += THREADS) sh->items[r] = look_up(r);
   __syncthreads();
   // the producer starts at once; the others wait until the second warp has its tensor memory
   if (warp >= 1) {
@@ -166,32 +173,28 @@ __global__ void __launch_bounds__(THREADS, 1) attn_rows_tcgen05_kernel(const __g
     const int P = p.page_size, pages_per_tile = BN / P;
     const int q_bytes = 2 * 128 * HPT * p.tokens_per_tile;      // of one piece: two boxes of 64 d x heads x tokens
     bool ok = true;
-    int rc = 0;                         // stages filled so far
-    // page ids of a tile: lane i reads the i-th (a tile has at most 16 pages); -1 = no page needed or none there
+    // page ids of a tile: lane i reads the i-th (a tile has at most 16 pages); NOT_NEEDED, or what the table says (-1: none)
+    constexpr int NOT_NEEDED = -2;
     auto tile_pages = [&](const Item& it, int j) -> int {
       const int pi = it.tile(j) * pages_per_tile + lane;
-      int page = -1;
-      if (lane < pages_per_tile && pi * P < it.j_hi && pi < p.table_width) {
-        page = p.block_table[(size_t)it.entry * p.table_width + pi];
-        if (page < 0 || page >= p.num_pages) { atomicOr(p.status, JV_STATUS_BAD_PAGE); page = -1; }
-      }
-      return page;
+      if (lane >= pages_per_tile || pi * P >= it.j_hi) return NOT_NEEDED;
+      return pi < p.table_width ? p.block_table[(size_t)it.entry * p.table_width + pi] : -1;
     };
     auto load_q = [&](const Item& it, int c, unsigned char* dst, uint64_t* bar) {
       tma_load_3d(dst, &q_map, c * D, it.kv_head * HPT, it.q_first, bar);
       tma_load_3d(dst + HALF_BYTES, &q_map, c * D + 64, it.kv_head * HPT, it.q_first, bar);
     };
-    // a stage with the rows that the lanes' pages hold of piece (or value head) c
-    auto put_rows = [&](const CUtensorMap* map, int c, int pages) {
-      const int s = rc % STAGES, ph = (rc / STAGES) & 1;
-      const int n_pages = __popc(__ballot_sync(0xffffffffu, pages >= 0));
-      if (lane == 0 && ok) {
-        ok = mbar_wait(&sh->empty[s], ph ^ 1);
-        if (ok) { sh->armed[s] = ph; mbar_expect_tx(&sh->full[s], n_pages * P * 256); }
+    // a stage with the rows that the lanes' pages hold of piece (or value head) c.  The announcement need not come before the
+    // copies: the phase cannot complete before lane 0 has arrived.
+    int s_at = 0, s_ph = 0;             // the next stage and the parity of its phase
+    auto put_rows = [&](const CUtensorMap* map, int c, int pages, int n_pages) {
+      ok = __all_sync(0xffffffffu, mbar_wait(&sh->empty[s_at], s_ph ^ 1)) && ok;
+      if (ok) {
+        uint64_t* bar = &sh->full[s_at];
+        if (lane == 0) { sh->armed[s_at] = s_ph; mbar_expect_tx(bar, n_pages * P * 256); }
+        if (pages >= 0) tma_load_5d(r_s + s_at * TILE_BYTES + lane * P * 256, map, 0, 0, 2 * c, 0, pages, bar);
       }
-      ok = __shfl_sync(0xffffffffu, ok, 0);                     // also orders the announcement before the copies
-      if (ok && pages >= 0) tma_load_5d(r_s + s * TILE_BYTES + lane * P * 256, map, 0, 0, 2 * c, 0, pages, &sh->full[s]);
-      ++rc;
+      if (++s_at == STAGES) { s_at = 0; s_ph ^= 1; }
     };
     auto put_queries = [&](const Item& it, int n) {             // the pieces that stay (with one place: all but piece 0)
       if (lane == 0 && ok) {
@@ -205,106 +208,121 @@ __global__ void __launch_bounds__(THREADS, 1) attn_rows_tcgen05_kernel(const __g
       }
       ok = __shfl_sync(0xffffffffu, ok, 0);
     };
-    auto put_keys = [&](const Item& it, int n, bool first_tile, int pages) {
-      for (int cc = 0; cc < NC && ok; ++cc) {
+    auto put_keys = [&](const Item& it, int n, bool first_tile, int pages, int n_pages) {
+      for (int cc = 0; cc < NC; ++cc) {
         const int c = cc + 1 == NC ? 0 : cc + 1;                // piece 0 last
-        if (ONE && first_tile && c == 0 && lane == 0) {         // the output of the item before has left through this place
-          ok = mbar_wait(&sh->q_free[0], (n & 1) ^ 1);
-          if (ok) { sh->armed_q[0] = n & 1; mbar_expect_tx(&sh->q_full[0], q_bytes); load_q(it, 0, q_s, &sh->q_full[0]); }
+        if (ONE && first_tile && c == 0) {                      // the output of the item before has left through this place
+          ok = __all_sync(0xffffffffu, mbar_wait(&sh->q_free[0], (n & 1) ^ 1)) && ok;
+          if (ok && lane == 0) { sh->armed_q[0] = n & 1; mbar_expect_tx(&sh->q_full[0], q_bytes); load_q(it, 0, q_s, &sh->q_full[0]); }
         }
         if (NCT == 0 && c >= KEPT) {                            // a streamed piece: its queries first
-          const int s = rc % STAGES, ph = (rc / STAGES) & 1;
-          if (lane == 0) {
-            ok = mbar_wait(&sh->empty[s], ph ^ 1);
-            if (ok) { sh->armed[s] = ph; mbar_expect_tx(&sh->full[s], q_bytes); load_q(it, c, r_s + s * TILE_BYTES, &sh->full[s]); }
+          ok = __all_sync(0xffffffffu, mbar_wait(&sh->empty[s_at], s_ph ^ 1)) && ok;
+          if (ok && lane == 0) {
+            sh->armed[s_at] = s_ph;
+            mbar_expect_tx(&sh->full[s_at], q_bytes);
+            load_q(it, c, r_s + s_at * TILE_BYTES, &sh->full[s_at]);
           }
-          ++rc;
+          if (++s_at == STAGES) { s_at = 0; s_ph ^= 1; }
         }
-        ok = __shfl_sync(0xffffffffu, ok, 0);
-        put_rows(&k_map, c, pages);
+        put_rows(&k_map, c, pages, n_pages);
       }
     };
-    int r = 0, n = 0;
-    Item it, nx;
-    bool have = next_item(r, it);
-    int pages = -1;
-    if (have) {
-      pages = tile_pages(it, 0);
-      put_queries(it, 0);
-      put_keys(it, 0, true, pages);
+    // what the table says -> pages to copy from (-1: none), with a report of those that should be there
+    auto usable = [&](int said, int& n_pages) -> int {
+      const bool there = said >= 0 && said < p.num_pages;
+      if (said != NOT_NEEDED && !there) atomicOr(p.status, JV_STATUS_BAD_PAGE);
+      n_pages = __popc(__ballot_sync(0xffffffffu, there));
+      return there ? said : -1;
+    };
+    // the tiles of all items as one sequence; a tile's page ids are asked for two tiles before they are used
+    struct At { Item it; int r, n, j; bool valid; };
+    auto after = [&](const At& x) -> At {
+      At y = x;
+      if (!x.valid) return y;
+      if (++y.j < x.it.n_tiles) return y;
+      y.j = 0;
+      ++y.n;
+      ++y.r;
+      y.valid = next_item(y.r, y.it);
+      return y;
+    };
+    At cur;
+    cur.r = cur.n = cur.j = 0;
+    cur.valid = next_item(cur.r, cur.it);
+    At nxt = after(cur);
+    int n_pages = 0, n_pages_next = 0;
+    int pages = usable(cur.valid ? tile_pages(cur.it, 0) : NOT_NEEDED, n_pages);
+    int said_next = nxt.valid ? tile_pages(nxt.it, nxt.j) : NOT_NEEDED;
+    if (cur.valid) {
+      put_queries(cur.it, 0);
+      put_keys(cur.it, 0, true, pages, n_pages);
     }
-    while (have && ok) {
-      int rn = r + 1;
-      const bool more = next_item(rn, nx);
-      for (int j = 0; j < it.n_tiles && ok; ++j) {
-        int pages_next = -1;
-        if (j + 1 < it.n_tiles) {
-          pages_next = tile_pages(it, j + 1);
-          put_keys(it, n, false, pages_next);
-          put_rows(&v_map, it.kv_head, pages);
-        } else {
-          if (ONE) put_rows(&v_map, it.kv_head, pages);
-          if (more) {
-            pages_next = tile_pages(nx, 0);
-            put_queries(nx, n + 1);
-            put_keys(nx, n + 1, true, pages_next);
-          }
-          if (!ONE) put_rows(&v_map, it.kv_head, pages);
-        }
-        pages = pages_next;
+    while (cur.valid && ok) {
+      const At next2 = after(nxt);
+      const int said_next2 = next2.valid ? tile_pages(next2.it, next2.j) : NOT_NEEDED;
+      const bool values_first = ONE && (!nxt.valid || nxt.n != cur.n);
+      const int pages_next = usable(said_next, n_pages_next);
+      if (values_first) put_rows(&v_map, cur.it.kv_head, pages, n_pages);
+      if (nxt.valid) {
+        if (nxt.n != cur.n) put_queries(nxt.it, nxt.n);
+        put_keys(nxt.it, nxt.n, nxt.n != cur.n, pages_next, n_pages_next);
       }
-      it = nx;
-      r = rn;
-      have = more;
-      ++n;
+      if (!values_first) put_rows(&v_map, cur.it.kv_head, pages, n_pages);
+      cur = nxt;
+      nxt = next2;
+      pages = pages_next;
+      n_pages = n_pages_next;
+      said_next = said_next2;
     }
     if (!ok && lane == 0) { atomicOr(p.status, JV_STATUS_WAIT_EXPIRED); sh->failed = 1; }
   } else if (warp == 1) {
     // -------------------------------------------------------------- mma issuer
-    // The whole warp walks through the stages; lane 0 issues the products.
+    // The whole warp walks through the tiles; lane 0 takes a tile's stages of keys and issues the products.
     const uint64_t q_desc = desc_k_major(smem_u32(q_s)), rq_desc = desc_k_major(smem_u32(r_s));
     const uint64_t k_desc = desc_k_major(smem_u32(r_s), GROUP_BYTES);
     const uint64_t v_desc = desc_mn_major(smem_u32(r_s), GROUP_BYTES / 2, GROUP_BYTES);
-    int rc = 0;                         // stages taken so far
+    int s_at = 0, s_ph = 0;             // the next stage and the parity of its phase
+    auto next_stage = [&]() { if (++s_at == STAGES) { s_at = 0; s_ph ^= 1; } };
     auto wait = [&](uint64_t* bar, int parity) -> bool { return __all_sync(0xffffffffu, mbar_wait(bar, parity)); };
-    auto issue_qk = [&](int n, int j, int n_tiles, int gt) -> bool {        // S[gt % 2] = sum_c Q_c K_c^T
-      if (j == 0 && !wait(&sh->q_full[ONE ? 1 : n % QB], (n / QB) & 1)) return false;
+    auto issue_qk_lane = [&](int n, int j, int n_tiles, int gt) -> bool {   // S[gt % 2] = sum_c Q_c K_c^T
+      if (j == 0 && !mbar_wait(&sh->q_full[ONE ? 1 : n % QB], (n / QB) & 1)) return false;
       const uint32_t tmem_s = tmem + (gt & 1) * 128;
+      const uint64_t q_item = q_desc + (uint64_t)(((n % QB) * KEPT * TILE_BYTES) >> 4);
+#pragma unroll (NCT > 0 ? NCT : 1)
       for (int cc = 0; cc < NC; ++cc) {
         const int c = cc + 1 == NC ? 0 : cc + 1;
-        if (ONE && j == 0 && c == 0 && !wait(&sh->q_full[0], n & 1)) return false;
-        uint64_t q0;
+        if (ONE && j == 0 && c == 0 && !mbar_wait(&sh->q_full[0], n & 1)) return false;
+        uint64_t q0 = q_item + (uint64_t)((c * TILE_BYTES) >> 4);
         int sq = -1;
         if (NCT == 0 && c >= KEPT) {
-          sq = rc % STAGES;
-          if (!wait(&sh->full[sq], (rc / STAGES) & 1)) return false;
-          ++rc;
+          sq = s_at;
+          if (!mbar_wait(&sh->full[sq], s_ph)) return false;
+          next_stage();
           q0 = rq_desc + (uint64_t)((sq * TILE_BYTES) >> 4);
-        } else {
-          q0 = q_desc + (uint64_t)((((n % QB) * KEPT + c) * TILE_BYTES) >> 4);
         }
-        const int s = rc % STAGES;
-        if (!wait(&sh->full[s], (rc / STAGES) & 1)) return false;
-        ++rc;
-        if (lane == 0) {
-          TC_FENCE_AFTER();
-          const uint64_t k0 = k_desc + (uint64_t)((s * TILE_BYTES) >> 4);
-          const uint64_t q1 = q0 + (HALF_BYTES >> 4), k1 = k0 + (GROUP_BYTES / 2 >> 4);
+        const int s = s_at;
+        if (!mbar_wait(&sh->full[s], s_ph)) return false;
+        next_stage();
+        TC_FENCE_AFTER();
+        const uint64_t k0 = k_desc + (uint64_t)((s * TILE_BYTES) >> 4);
+        const uint64_t q1 = q0 + (HALF_BYTES >> 4), k1 = k0 + (GROUP_BYTES / 2 >> 4);
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk) umma(tmem_s, q0 + 2 * kk, k0 + 2 * kk, IDESC_QK, (cc | kk) != 0);
+        for (int kk = 0; kk < 4; ++kk) umma(tmem_s, q0 + 2 * kk, k0 + 2 * kk, IDESC_QK, (cc | kk) != 0);
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk) umma(tmem_s, q1 + 2 * kk, k1 + 2 * kk, IDESC_QK, 1);
-          if (sq >= 0) umma_commit(&sh->empty[sq]);
-          umma_commit(&sh->empty[s]);
-        }
-        __syncwarp();
+        for (int kk = 0; kk < 4; ++kk) umma(tmem_s, q1 + 2 * kk, k1 + 2 * kk, IDESC_QK, 1);
+        if (sq >= 0) umma_commit(&sh->empty[sq]);
+        umma_commit(&sh->empty[s]);
       }
-      if (lane == 0) {
-        if (ONE && j == n_tiles - 1) umma_commit(&sh->q_free[1]);   // the other pieces have been used for the last time
-        umma_commit(&sh->s_full[gt & 1]);
-      }
-      __syncwarp();
+      if (ONE && j == n_tiles - 1) umma_commit(&sh->q_free[1]);     // the other pieces have been used for the last time
+      umma_commit(&sh->s_full[gt & 1]);
       return true;
+    };
+    auto issue_qk = [&](int n, int j, int n_tiles, int gt) -> bool {
+      bool fine = true;
+      if (lane == 0) fine = issue_qk_lane(n, j, n_tiles, gt);
+      s_at = __shfl_sync(0xffffffffu, s_at, 0);
+      s_ph = __shfl_sync(0xffffffffu, s_ph, 0);
+      return __all_sync(0xffffffffu, fine);
     };
     bool ok = true;
     int r = 0, n = 0, gt = 0;
@@ -324,9 +342,9 @@ __global__ void __launch_bounds__(THREADS, 1) attn_rows_tcgen05_kernel(const __g
         const bool later = ONE && last;
         if (has_next && !later) ok = next_scores();
         if (!ok) break;
-        const int s = rc % STAGES;
-        if (!wait(&sh->full[s], (rc / STAGES) & 1)) { ok = false; break; }
-        ++rc;
+        const int s = s_at;
+        if (!wait(&sh->full[s], s_ph)) { ok = false; break; }
+        next_stage();
         const int first = it.j_hi - it.tile(j) * BN;
         if (first < BN) {
           // the keys end within the tile: the value rows past the end become zero (they may hold anything, and their weights
@@ -559,6 +577,7 @@ template <int NCT>
 int launch(int blocks, cudaStream_t stream, const CUtensorMap& q_map, const CUtensorMap& k_map, const CUtensorMap& v_map,
            const CUtensorMap& out_map, const Params& p) {
   constexpr size_t smem = TILE_BYTES * SMEM_TILES + sizeof(Shared) + 1024;
+  static_assert(smem <= 227 * 1024, "shared memory");
   static bool ready[JV_MAX_DEVICES];
   if (!jv_once_per_device(ready, [&] {
         return cudaFuncSetAttribute(attn_rows_tcgen05_kernel<NCT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess;
