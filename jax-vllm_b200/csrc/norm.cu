@@ -200,6 +200,107 @@ JV_EXPORT int jv_rmsnorm(float* h, const void* delta, int delta_dtype, const int
   return JV_ERR_UNSUPPORTED;
 }
 
+// The norm behind a routed feed-forward: what is added to row r is sum_s coef[r, s] * y[pick[r, s], :] (s ascending, 32-bit),
+// the weighted rows of its experts, picked up as they are added.  Rows of 8 elements a thread and pass where sizes and
+// addresses allow (VEC), else one.
+template <typename TD, typename TW, typename TY, bool VEC>
+__global__ void __launch_bounds__(1024) rmsnorm_pick_kernel(float* __restrict__ h, const TD* __restrict__ picked,
+                                                            const int* __restrict__ pick, const float* __restrict__ coef,
+                                                            int parts, int picked_rows, const int* __restrict__ rows,
+                                                            const TW* __restrict__ weight, TY* __restrict__ y, int hidden,
+                                                            float eps, int n_rows_total, int* __restrict__ status) {
+  constexpr int V = VEC ? 8 : 1, TOGETHER = 4;
+  extern __shared__ float kept[];                 // [hidden]: the row after the sum
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const int i = blockIdx.x;
+  int r = i;
+  if (rows != nullptr) {
+    r = rows[i];
+    if (r < 0 || r >= n_rows_total) {
+      if (threadIdx.x == 0) atomicOr(status, JV_STATUS_BAD_ROW);
+      for (int c = threadIdx.x; c < hidden; c += blockDim.x) y[(size_t)i * hidden + c] = from_f32<TY>(0.f);
+      return;
+    }
+  }
+  float* hr = h + (size_t)r * hidden;
+  const int* pk = pick + (size_t)r * parts;
+  const float* cf = coef + (size_t)r * parts;
+  if (threadIdx.x < parts && (pk[threadIdx.x] < 0 || pk[threadIdx.x] >= picked_rows)) atomicOr(status, JV_STATUS_BAD_ROW);
+  float ss = 0.f;
+  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
+    float v[8], d[8];
+    if (VEC) load8<float>(hr + c, v);
+    else v[0] = hr[c];
+#pragma unroll
+    for (int k = 0; k < V; ++k) d[k] = 0.f;
+    for (int s0 = 0; s0 < parts; s0 += TOGETHER) {      // four rows ask for their loads together, then add in their order
+      float e[TOGETHER][8], w[TOGETHER];
+#pragma unroll
+      for (int s = 0; s < TOGETHER; ++s) {
+        const int src = s0 + s < parts ? pk[s0 + s] : -1;
+        const bool ok = src >= 0 && src < picked_rows;
+        w[s] = ok ? cf[s0 + s] : 0.f;
+        const TD* row = picked + (size_t)(ok ? src : 0) * hidden + c;
+        if (ok) {
+          if (VEC) load8<TD>(row, e[s]);
+          else e[s][0] = to_f32(*row);
+        }
+      }
+#pragma unroll
+      for (int s = 0; s < TOGETHER; ++s)
+        if (w[s] != 0.f) {
+#pragma unroll
+          for (int k = 0; k < V; ++k) d[k] = fmaf(w[s], e[s][k], d[k]);
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      v[k] += d[k];
+      ss += v[k] * v[k];
+      kept[c + k] = v[k];
+    }
+    if (rows == nullptr) {
+      if (VEC) store8<float>(hr + c, v);
+      else hr[c] = v[0];
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float inv = rsqrtf(ss / (float)hidden + eps);
+  TY* yr = y + (size_t)i * hidden;
+  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {     // a thread's own elements
+    float w[8];
+    if (VEC) load8<TW>(weight + c, w);
+    else w[0] = to_f32(weight[c]);
+#pragma unroll
+    for (int k = 0; k < V; ++k) w[k] *= kept[c + k] * inv;
+    if (VEC) store8<TY>(yr + c, w);
+    else yr[c] = from_f32<TY>(w[0]);
+  }
+}
+
+// As jv_rmsnorm, with the sum of picked rows as delta: picked [picked_rows, hidden] of dtype `delta_dtype`, pick and coef
+// [n_total, parts].
+JV_EXPORT int jv_rmsnorm_pick(float* h, const void* picked, int delta_dtype, const int* pick, const float* coef, int parts,
+                              int picked_rows, const int* rows, const void* weight, int weight_dtype, void* y, int out_dtype,
+                              int n_out, int n_total, int hidden, float eps, int* status, cudaStream_t stream) {
+  if (n_out == 0) return JV_OK;
+  const size_t smem = sizeof(float) * (size_t)hidden;
+  if (parts < 1 || parts > 64 || smem > 48 * 1024 - 256) return JV_ERR_UNSUPPORTED;
+  const bool vec = hidden % 8 == 0 && ((uintptr_t)h % 16) == 0 && ((uintptr_t)picked % 16) == 0 && ((uintptr_t)weight % 16) == 0 &&
+                   ((uintptr_t)y % 16) == 0;
+  const int units = vec ? hidden / 8 : hidden;
+  int threads = 64;                               // `parts` threads at least
+  while (threads < 512 && threads < units) threads *= 2;
+  JV_DISPATCH_DTYPE(out_dtype, TY, JV_DISPATCH_DTYPE(weight_dtype, TW, JV_DISPATCH_DTYPE(delta_dtype, TD, {
+      return jv_launch(vec ? rmsnorm_pick_kernel<TD, TW, TY, true> : rmsnorm_pick_kernel<TD, TW, TY, false>, dim3(n_out),
+                       dim3(threads), smem, stream, h, (const TD*)picked, pick, coef, parts, picked_rows, rows,
+                       (const TW*)weight, (TY*)y, hidden, eps, n_total, status);
+  })));
+  return JV_ERR_UNSUPPORTED;
+}
+
 // Adds delta into the 32-bit stream without a norm: h[r, :] += delta[r, :].
 template <typename TD>
 __global__ void residual_add_kernel(float* __restrict__ h, const TD* __restrict__ delta, size_t n, int parts,

@@ -257,7 +257,7 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor | Non
 # ----------------------------------------------------------------------------- norm
 def rmsnorm(h: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
             delta: torch.Tensor | None = None, rows: torch.Tensor | None = None) -> torch.Tensor:
-    """RMSNorm of rows of the float32 stream `h`, after adding `delta` (if given).
+    """RMSNorm of rows of the float32 stream `h`, after adding `delta` (a tensor, a PartialSum or PickedRows, if given).
 
     Without `rows` every row is normalised and, when `delta` is given, `h` is updated
     in place with the sum.  With `rows` (int32) only those rows are produced and `h`
@@ -267,11 +267,22 @@ def rmsnorm(h: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.
     n_total, hidden = h.shape
     if weight.shape != (hidden,):
         raise KernelError(f"norm weight has shape {tuple(weight.shape)}, rows have {hidden} elements")
-    delta, n_parts, part_stride = _delta_parts(delta, h)
     if rows is not None:
         _cuda(rows, "rows", torch.int32)
     n_out = n_total if rows is None else rows.numel()
     y = torch.empty((n_out, hidden), dtype=out_dtype, device=h.device)
+    if isinstance(delta, PickedRows) and delta.pick.shape[1] <= 64 and hidden <= 12000:
+        picked, pick, coef = _cuda(delta.rows, "rows to pick"), _cuda(delta.pick, "pick", torch.int32), \
+            _cuda(delta.coef, "coef", torch.float32)
+        if delta.shape != h.shape or coef.shape != pick.shape:
+            raise KernelError("the picked rows do not fit the stream")
+        f = _fn("norm", "jv_rmsnorm_pick", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                                            c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+        _check(f(h.data_ptr(), picked.data_ptr(), _code(picked, "rows to pick"), pick.data_ptr(), coef.data_ptr(),
+                 pick.shape[1], picked.shape[0], _ptr(rows), weight.data_ptr(), _code(weight, "weight"), y.data_ptr(),
+                 _code(y, "out"), n_out, n_total, hidden, float(eps), _status_ptr(h.device), _stream()), "rmsnorm_pick")
+        return y
+    delta, n_parts, part_stride = _delta_parts(delta, h)
     f = _fn("norm", "jv_rmsnorm", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int,
                                    c_int, c_int, c_int, c_float, c_int, c_longlong, c_void_p, c_void_p])
     _check(f(h.data_ptr(), _ptr(delta), 0 if delta is None else _code(delta, "delta"), _ptr(rows),

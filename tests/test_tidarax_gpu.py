@@ -341,6 +341,33 @@ def test_experts_named_by_a_table_alone(E, top, F, W, n, dtype):
     assert (got - want).abs().max() < tol * max(1.0, want.abs().max().item())
 
 
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("n,hidden,top", [(5, 40, 1), (7, 33, 3), (200, 2048, 4), (3, 8192, 9)])
+def test_a_norm_that_picks_up_the_experts_rows(n, hidden, top, dtype):
+    """The sum of weighted rows added and normed in one pass, for all rows (the stream is updated) and for chosen rows (it
+    is not), against the two steps apart."""
+    from jax_vllm_b200 import ops
+    g = torch.Generator().manual_seed(n + hidden)
+    h = torch.randn((n, hidden), generator=g)
+    rows = torch.randn((2 * n + 3, hidden), generator=g).to(dtype)
+    pick = torch.randint(0, 2 * n + 3, (n, top), generator=g, dtype=torch.int32)
+    coef = torch.randn((n, top), generator=g)
+    w = (1.0 + 0.1 * torch.randn(hidden, generator=g)).to(dtype)
+    full = h.double() + torch.einsum("ns,nsc->nc", coef.double(), rows.double()[pick.long()])
+    want = tp.unit(full, 1e-5) * w.double()
+    hc = h.cuda()
+    delta = ops.PickedRows(rows.cuda(), pick.cuda(), coef.cuda())
+    some = torch.tensor([n - 1, 0, n // 2], dtype=torch.int32)
+    y = ops.rmsnorm(hc, w.cuda(), 1e-5, dtype, delta=delta, rows=some.cuda())
+    assert torch.equal(hc.cpu(), h)
+    tol = 2e-5 if dtype == torch.float32 else 2e-2
+    assert (y.double().cpu() - want[some.long()]).abs().max() < tol * want.abs().max()
+    y = ops.rmsnorm(hc, w.cuda(), 1e-5, dtype, delta=delta)
+    ops.check_status()
+    assert (y.double().cpu() - want).abs().max() < tol * want.abs().max()
+    assert (hc.double().cpu() - full).abs().max() < 1e-5 * full.abs().max()
+
+
 def test_a_table_that_names_no_expert_is_reported():
     from jax_vllm_b200 import ops
     table = torch.tensor([[0, 1], [2, 5]], dtype=torch.int32).cuda()
