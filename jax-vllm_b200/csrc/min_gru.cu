@@ -31,21 +31,27 @@ struct GruParams {
   int* status;
 };
 
-// EXACT (32-bit projections): library exponentials and divisions; else the short forms, whose error is far below the
-// 16-bit rounding of what they are given.
-template <bool EXACT> __device__ __forceinline__ float exp_of(float x) { return EXACT ? expf(x) : __expf(x); }
-template <bool EXACT> __device__ __forceinline__ float recip(float x) { return EXACT ? 1.f / x : __fdividef(1.f, x); }
+// sigmoid(x) = 1 / (1 + e^-x): of a large negative x the sum is infinite and the result 0, and a small result keeps its
+// relative precision.  EXACT (32-bit projections): library exponential and division; else one instruction each for the
+// power of two and the reciprocal, whose error is far below the 16-bit rounding of what they are given.
+template <bool EXACT> __device__ __forceinline__ float sigmoid_of(float x) {
+  if (EXACT) return 1.f / (1.f + expf(-x));
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(x * -1.4426950408889634f));
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(r) : "f"(1.f + e));
+  return r;
+}
 
 // Gate and candidate of one token.
 template <bool EXACT>
 __device__ __forceinline__ void gru_pair(float zl, float y, float& z, float& c) {
-  const float e = exp_of<EXACT>(fminf(zl, 80.f));          // e^zl, kept finite
-  z = e * recip<EXACT>(1.f + e);
-  c = y >= 0.f ? y + 0.5f : recip<EXACT>(1.f + exp_of<EXACT>(fminf(-y, 80.f)));
+  z = sigmoid_of<EXACT>(zl);
+  const float low = sigmoid_of<EXACT>(y);
+  c = y >= 0.f ? y + 0.5f : low;
 }
 __device__ __forceinline__ float blend(float S, float z, float c) { return fmaf(z, c - S, S); }
 template <bool EXACT>
-__device__ __forceinline__ float silu_of(float g) { return g * recip<EXACT>(1.f + exp_of<EXACT>(fminf(-g, 80.f))); }
+__device__ __forceinline__ float silu_of(float g) { return g * sigmoid_of<EXACT>(g); }
 
 // CB channels a block, THREADS / CB runs of TPT tokens a tile.
 template <typename T, typename W, int CB>
@@ -69,32 +75,33 @@ __global__ void __launch_bounds__(THREADS, 1) gru_scan_kernel(const GruParams p)
   }
   float* S_g = p.state + (size_t)slot * p.slot_stride + c;
   if (run == 0) carry[0][cl] = live ? *S_g : 0.f;
-  const T* zp = (const T*)p.proj + p.z_off + c;
-  const T* xp = (const T*)p.proj + p.x_off + c;
-  const T* gp = (const T*)p.proj + p.g_off + c;
+  const T* row = (const T*)p.proj + c;
   T zr[TPT], xr[TPT], gr[TPT];
   auto fetch = [&](int tile0) {
+    const int first = tile0 + run * TPT, n_here = live ? t1 - first : 0;
+    const T* at = row + (size_t)first * p.stride;
+    if (n_here >= TPT) {
 #pragma unroll
-    for (int i = 0; i < TPT; ++i) {
-      const int t = tile0 + run * TPT + i;
-      if (live && t < t1) {
-        const size_t at = (size_t)t * p.stride;
-        zr[i] = zp[at]; xr[i] = xp[at]; gr[i] = gp[at];
-      } else {
+      for (int i = 0; i < TPT; ++i, at += p.stride) { zr[i] = at[p.z_off]; xr[i] = at[p.x_off]; gr[i] = at[p.g_off]; }
+    } else {
+#pragma unroll
+      for (int i = 0; i < TPT; ++i, at += p.stride) {
         zr[i] = xr[i] = gr[i] = from_f32<T>(0.f);
+        if (i < n_here) { zr[i] = at[p.z_off]; xr[i] = at[p.x_off]; gr[i] = at[p.g_off]; }
       }
     }
   };
   fetch(t0);
   int which = 0;
   for (int tile0 = t0; tile0 < t1; tile0 += TILE, which ^= 1) {
+    const int first = tile0 + run * TPT, n_here = live ? t1 - first : 0;
     float z[TPT], cand[TPT], g[TPT];
     float D = 0.f, B = 0.f;
 #pragma unroll
     for (int i = 0; i < TPT; ++i) {
       gru_pair<EXACT>(to_f32(zr[i]) + zb, to_f32(xr[i]) + xb, z[i], cand[i]);
-      g[i] = to_f32(gr[i]);
-      if (tile0 + run * TPT + i >= t1) z[i] = 0.f;         // no token: the state passes
+      g[i] = p.scale * silu_of<EXACT>(to_f32(gr[i]));
+      if (i >= n_here) z[i] = 0.f;                         // no token: the state passes
       D = blend(D, z[i], 1.f);
       B = blend(B, z[i], cand[i]);
     }
@@ -106,11 +113,19 @@ __global__ void __launch_bounds__(THREADS, 1) gru_scan_kernel(const GruParams p)
 #pragma unroll 8
     for (int r = 0; r < run; ++r) S = fmaf(-Ds[r][cl], S, S) + Bs[r][cl];
     if (run == RUNS - 1) carry[which ^ 1][cl] = fmaf(-D, S, S) + B;
+    T* out = (T*)p.out + (size_t)first * p.out_stride + c;
+    if (n_here >= TPT) {
 #pragma unroll
-    for (int i = 0; i < TPT; ++i) {
-      const int t = tile0 + run * TPT + i;
-      S = blend(S, z[i], cand[i]);
-      if (live && t < t1) ((T*)p.out)[(size_t)t * p.out_stride + c] = from_f32<T>(p.scale * S * silu_of<EXACT>(g[i]));
+      for (int i = 0; i < TPT; ++i, out += p.out_stride) {
+        S = blend(S, z[i], cand[i]);
+        *out = from_f32<T>(S * g[i]);
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < TPT; ++i, out += p.out_stride) {
+        S = blend(S, z[i], cand[i]);
+        if (i < n_here) *out = from_f32<T>(S * g[i]);
+      }
     }
     __syncthreads();                                       // the runs' pairs have been read; the carry is there
   }

@@ -252,7 +252,7 @@ def test_recurrence_alone(C, dtype):
     unused slot stays as it was.  Gates far on both sides of zero; input and output are column ranges."""
     from jax_vllm_b200 import ops
     g = torch.Generator().manual_seed(C)
-    first, second, third, slots, n_slots = [1300, 1, 512, 9], [1, 3, 260, 1], [1, 1, 1, 1], [3, 0, 4, 1], 6
+    first, second, third, slots, n_slots = [1300, 1, 1537, 9], [1, 3, 260, 1], [1, 1, 1, 1], [3, 0, 4, 1], 6
     zb, xb = (torch.randn(C, generator=g).to(dtype) for _ in range(2))
     total = [a + b + c for a, b, c in zip(first, second, third)]
     full = [(3.0 * torch.randn((t, 3 * C), generator=g)).to(dtype) for t in total]
