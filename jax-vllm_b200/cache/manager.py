@@ -5,14 +5,15 @@ Layers are put into groups by what they need: all layers with the same `PagedKVN
 table per request; a page id of a group addresses the same page in every layer of the
 group.  Layers with a `FixedStateNeed` get a row per state slot instead.  Pages are given
 back when a request ends, when it is preempted, and - in a group with a window or with
-chunks - as soon as every position of a page lies before what the next query can see.
+chunks - as soon as every position of a page lies before what the next query can see (under a
+window that keeps the first tokens of a sequence, their pages stay).
 
 Prefix reuse (jllm/engine/cache.py:20-57): full pages are hashed in a chain over the
 tokens; a new request takes the longest run of pages whose hashes are known, in every
 group, but always leaves at least its last token to compute.  A group with a window needs
 only the pages that the window of the next query still reaches: the hit is the longest
 prefix whose pages are known from the start in every group without a window and over the
-last `window` positions in every group with one; the pages before that are entered as
+last `window` positions (and the kept first ones) in every group with one; the others are entered as
 given back, as they would be had the request computed the prefix itself.  Reuse is
 switched off for models with fixed-size state, which a page hit does not restore.
 """
@@ -188,15 +189,15 @@ class CacheManager:
             n = len(hashes)                               # pages known from the start where there is no window
             windowed = [g for g, grp in enumerate(self.groups) if grp.need.window is not None or grp.need.chunk is not None]
             while n > 0 and not all(found[i][g] is not None for g in windowed
-                                    for i in range(self._first_page_needed(g, n * P), n)):
+                                    for i in range(n) if self._page_needed(g, i, n * P)):
                 n -= 1
             for g, grp in enumerate(self.groups):
-                first = self._first_page_needed(g, n * P)
                 for i in range(n):
-                    if i >= first:
+                    needed = self._page_needed(g, i, n * P)
+                    if needed:
                         grp.pool.touch(found[i][g])
-                    rc.tables[g].append(found[i][g] if i >= first else -1)
-                rc.freed_upto[g] = first
+                    rc.tables[g].append(found[i][g] if needed else -1)
+                rc.freed_upto[g] = self._first_page_needed(g, n * P)
             rc.hashes = hashes[:n]
             rc.num_tokens = n * P
             rc.tokens = list(prompt[:rc.num_tokens])
@@ -215,6 +216,15 @@ class CacheManager:
         if need.chunk is not None:
             first = max(first, num_tokens - num_tokens % need.chunk)
         return first // self.page_size
+
+    def _kept_pages(self, g: int) -> int:
+        """How many pages at the start of a request in group g hold tokens that stay visible under the window."""
+        need = self.groups[g].need
+        return -(-need.keep_first // self.page_size) if need.window is not None else 0
+
+    def _page_needed(self, g: int, i: int, num_tokens: int) -> bool:
+        """Whether a query at position >= num_tokens can still see a key of logical page i in group g."""
+        return i < self._kept_pages(g) or i >= self._first_page_needed(g, num_tokens)
 
     def pages_needed(self, rc: RequestCache, new_len: int) -> list:
         """Pages each group must still allocate so that positions < new_len have a page."""
@@ -259,7 +269,7 @@ class CacheManager:
             if grp.need.window is None and grp.need.chunk is None:
                 continue
             upto = self._first_page_needed(g, rc.num_tokens)
-            for i in range(rc.freed_upto[g], min(upto, len(rc.tables[g]))):
+            for i in range(max(rc.freed_upto[g], self._kept_pages(g)), min(upto, len(rc.tables[g]))):
                 if rc.tables[g][i] >= 0:
                     grp.pool.release([rc.tables[g][i]])
                     rc.tables[g][i] = -1

@@ -35,6 +35,10 @@ class RopeSpec:
     # scaling by wavelength, (factor, low, high, original): a frequency whose wavelength is below original/high stays, one
     # above original/low is divided by the factor, those between are a straight mixture of both
     bands: Optional[tuple] = None
+    # YaRN, (factor, original, fast, slow): a pair that turns more than `fast` times over `original` positions keeps its
+    # frequency, one that turns fewer than `slow` times has it divided by the factor, those between are mixed by the pair's
+    # number; the cosines and sines of queries and keys are multiplied by 0.1 ln(factor) + 1
+    yarn: Optional[tuple] = None
 
 
 @dataclass(frozen=True)
@@ -57,6 +61,7 @@ class GatedMLPSpec:
     intermediate_size: int
     activation: str = "silu"
     prefix: str = "mlp"
+    names: tuple = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
     kind: str = "gated_mlp"
 
 
@@ -110,6 +115,7 @@ class GeneralAttentionSpec:
     # position encoding's theta and layout), cached so; every head's output turned back by the query's position
     rotate_values: bool = False
     window: Optional[int] = None            # a query sees its own position and the window - 1 before it
+    keep_first: int = 0                     # under a window: the first so many tokens of a sequence stay visible
     chunk: Optional[int] = None             # a query sees the earlier positions of its chunk, chunks counted from 0
     prefix: str = "mix"
     # tensor names below the prefix: queries, keys, values, gate, output, whole-projection norms, score bias,
@@ -153,6 +159,24 @@ class DeltaRuleSpec:
     # output norm weight, output projection
     names: tuple = ("r", "k", "v", "g", "a", "a.b", "w1", "w2", "w0", "norm", "o")
     kind: str = "delta_rule"
+
+
+@dataclass(frozen=True)
+class GatedLinearAttentionSpec:
+    """A matrix state per head with a decay per key channel: S <- diag(a) S + k v^T, o = S^T q * q_scale, a =
+    sigmoid(W_a2 W_a1 x + b)^(1/tau).  Each head's o is RMS-normed with one weight vector that the heads share, times
+    silu(W_g x).  The rank of the decay's pair of matrices is the first one's row count."""
+    hidden_size: int
+    num_heads: int
+    key_dim: int
+    value_dim: int
+    tau: float
+    q_scale: float
+    norm_eps: float
+    prefix: str = "mix"
+    # query, key, value, output gate, decay down- and up-projection and its bias, output norm weight, output projection
+    names: tuple = ("q", "k", "v", "g", "a1", "a2", "a2.b", "norm", "o")
+    kind: str = "gated_linear_attention"
 
 
 @dataclass(frozen=True)
@@ -267,6 +291,10 @@ class RoutedExpertsSpec:
     weight_scale: float = 1.0      # multiplies the weights at the end
     limit: float = 0.0             # of the clamped activation
     vocab_size: int = 0            # rows of the table (scoring "table")
+    # experts are chosen by score plus a learned number per expert (tensor name below the prefix), weighted without it
+    correction: Optional[str] = None
+    identity: int = 0              # this many further experts, the last of the router's, give their input itself
+    shared_size: int = 0           # a gated silu expert of this size that every token uses, added (tensors "shared.*")
     prefix: str = "mlp"
     kind: str = "routed_experts"
 
@@ -292,7 +320,7 @@ class LayerSpec:
     mixer: Any
     feed_forward: Any              # None: the layer has no feed-forward (arrangements that allow it)
     mixer_norm: NormSpec
-    ffn_norm: Optional[NormSpec]
+    ffn_norm: Optional[NormSpec]   # "parallel": None where both branches read the mixer's norm
     cache_from: Optional[int] = None
     kind: str = "pre_norm"
     residual_scale: float = 1.0    # multiplies every branch before it is added to the stream
@@ -325,6 +353,7 @@ class ModelSpec:
     # learned vectors added to every token's stream right before places of the run order: (tensor name [rows, hidden],
     # ((place, row), ...)), or None
     pass_vectors: Optional[tuple] = None
+    embedding_scale: float = 1.0            # multiplies the embedding's rows as they enter the stream
     logit_softcap: Optional[float] = None   # logits <- cap * tanh(logits / cap)
     logit_scale: Optional[float] = None     # logits <- logits * scale
     unused_tensors: tuple = ()    # names that a folder may hold without the model reading them

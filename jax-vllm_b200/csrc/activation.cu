@@ -2,11 +2,11 @@
 // evaluated in 32-bit.  `gu` is what the packed gate|up projection writes: blocks of `block` gate
 // columns followed by the `block` up columns of the same indices (block == inter: all gate columns,
 // then all up columns), so gate_i = gu[n, (i / block) * 2 * block + i % block] and up_i is `block`
-// columns further.
+// columns further.  Rows of `act` lie `act_stride` elements apart (a column range of wider rows).
 #include "common.cuh"
 
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ act, int inter, int block, size_t total) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ act, size_t act_stride, int inter, int block, size_t total) {
   pdl_trigger();
   pdl_wait();
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -18,13 +18,13 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ act, int
     const float g = to_f32(gu[n * 2 * inter + col]);
     const float u = to_f32(gu[n * 2 * inter + col + block]);
     const float s = g / (1.f + expf(-g));
-    act[idx] = from_f32<T>(s * u);
+    act[n * act_stride + i] = from_f32<T>(s * u);
   }
 }
 
 // Same, 16 bytes per access (block a multiple of the vector length, rows 16-byte aligned).
 template <typename T>
-__global__ void swiglu_vec_kernel(const T* __restrict__ gu, T* __restrict__ act, int inter, int block, size_t total_vec) {
+__global__ void swiglu_vec_kernel(const T* __restrict__ gu, T* __restrict__ act, size_t act_stride, int inter, int block, size_t total_vec) {
   pdl_trigger();
   pdl_wait();
   constexpr int V = 16 / sizeof(T);
@@ -46,14 +46,14 @@ __global__ void swiglu_vec_kernel(const T* __restrict__ gu, T* __restrict__ act,
       const float gv = to_f32(g[k]);
       o[k] = from_f32<T>(gv / (1.f + expf(-gv)) * to_f32(u[k]));
     }
-    *reinterpret_cast<uint4*>(act + n * inter + i) = o4;
+    *reinterpret_cast<uint4*>(act + n * act_stride + i) = o4;
   }
 }
 
 // The same for a gate|up given as `parts` 32-bit tensors [n, 2*inter] `part_stride` elements apart, whose sum it is
 // (the sums over the parts of k that a split product leaves), four columns per thread and pass.
 template <typename T>
-__global__ void swiglu_parts_kernel(const float* __restrict__ gu, T* __restrict__ act, int inter, int block, size_t total_vec,
+__global__ void swiglu_parts_kernel(const float* __restrict__ gu, T* __restrict__ act, size_t act_stride, int inter, int block, size_t total_vec,
                                     int parts, size_t part_stride) {
   pdl_trigger();
   pdl_wait();
@@ -86,7 +86,7 @@ __global__ void swiglu_parts_kernel(const float* __restrict__ gu, T* __restrict_
       g.x += g2.x; g.y += g2.y; g.z += g2.z; g.w += g2.w;
       u.x += u2.x; u.y += u2.y; u.z += u2.z; u.w += u2.w;
     }
-    T* dst = act + n * inter + i;
+    T* dst = act + n * act_stride + i;
     dst[0] = from_f32<T>(g.x / (1.f + expf(-g.x)) * u.x);
     dst[1] = from_f32<T>(g.y / (1.f + expf(-g.y)) * u.y);
     dst[2] = from_f32<T>(g.z / (1.f + expf(-g.z)) * u.z);
@@ -94,10 +94,10 @@ __global__ void swiglu_parts_kernel(const float* __restrict__ gu, T* __restrict_
   }
 }
 
-// gu: [n, 2*inter]; act: [n, inter]; both of dtype `dtype`; block: see above (a divisor of inter).
+// gu: [n, 2*inter]; act: n rows of inter elements, act_stride apart; both of dtype `dtype`; block: see above (a divisor of inter).
 // parts > 1: gu is `parts` float tensors [n, 2*inter], part_stride elements apart, and act is of dtype `dtype`
 // (block and part_stride multiples of 4, gu 16-byte aligned).
-JV_EXPORT int jv_swiglu(const void* gu, void* act, int dtype, int n, int inter, int block, int parts, long long part_stride,
+JV_EXPORT int jv_swiglu(const void* gu, void* act, long long act_stride, int dtype, int n, int inter, int block, int parts, long long part_stride,
                         cudaStream_t stream) {
   const size_t total = (size_t)n * inter;
   if (total == 0) return JV_OK;
@@ -108,22 +108,22 @@ JV_EXPORT int jv_swiglu(const void* gu, void* act, int dtype, int n, int inter, 
     size_t blocks = (total_vec + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     JV_DISPATCH_DTYPE(dtype, T, return jv_launch(swiglu_parts_kernel<T>, dim3((int)blocks), dim3(256), 0, stream,
-                                                  (const float*)gu, (T*)act, inter, block, total_vec, parts, (size_t)part_stride));
+                                                  (const float*)gu, (T*)act, (size_t)act_stride, inter, block, total_vec, parts, (size_t)part_stride));
     return JV_ERR_UNSUPPORTED;
   }
   const int vec = dtype == 0 ? 4 : 8;
-  if (block % vec == 0 && ((uintptr_t)gu % 16) == 0 && ((uintptr_t)act % 16) == 0) {
+  if (block % vec == 0 && act_stride % vec == 0 && ((uintptr_t)gu % 16) == 0 && ((uintptr_t)act % 16) == 0) {
     const size_t total_vec = total / vec;
     size_t blocks = (total_vec + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     JV_DISPATCH_DTYPE(dtype, T, return jv_launch(swiglu_vec_kernel<T>, dim3((int)blocks), dim3(256), 0, stream,
-                                                  (const T*)gu, (T*)act, inter, block, total_vec));
+                                                  (const T*)gu, (T*)act, (size_t)act_stride, inter, block, total_vec));
     return JV_ERR_UNSUPPORTED;
   }
   size_t blocks = (total + 255) / 256;
   if (blocks > 148 * 32) blocks = 148 * 32;
   JV_DISPATCH_DTYPE(dtype, T, return jv_launch(swiglu_kernel<T>, dim3((int)blocks), dim3(256), 0, stream,
-                                                (const T*)gu, (T*)act, inter, block, total));
+                                                (const T*)gu, (T*)act, (size_t)act_stride, inter, block, total));
   return JV_ERR_UNSUPPORTED;
 }
 

@@ -13,6 +13,8 @@
 //   head scale     the scaled score of query head h is multiplied by head_scale[h] (a temperature per head)
 //   distance bias  dist_bias[h][min(pos - j, n_dist - 1)] is added to the score of key j; no scale touches it
 //   sink           exp(sink[h]) counts once in the softmax's denominator; it has no key and no value
+//   kept tokens    under a window the first `keep` positions of a sequence stay visible.  A tile's keys are counted as
+//                  places in one run (common.cuh, KeyRun): the kept positions first, then those of the window
 //
 // Scores are scaled and masked in 32-bit, the running softmax keeps (max, sum) in 32-bit, weights are rounded to
 // bfloat16 for the second product.  Tiles, the split of a decoded token's keys and the merge by the block that ends
@@ -48,6 +50,7 @@ struct Params {
   const int* cu_seqlens; const int* start_pos;
   const int* work;
   int n_q_heads, n_kv_heads, page_size, num_pages, window;
+  int keep;                    // positions below this one stay visible under a window
   float scale;                 // multiplies q.k
   float score_cap;             // > 0: s <- cap * tanh(s / cap)
   int sigmoid;                 // independent weights sigmoid(s + bias[query head])
@@ -94,14 +97,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // is then 4 modulo 8, so the eight 16-byte rows that one ldmatrix phase reads fall into distinct banks.
 template <int D> struct Tile { static constexpr int STRIDE = D + 8; };
 
-// Cache slots (page * page_size + place in the page) of keys [j0, j0 + BN) (-1: beyond j_end, or no
-// page), one per thread n < BN: the block table is read once per key, ahead of the copies.
-__device__ __forceinline__ void tile_rows(long long* rows, const Params& p, int entry, int kv_head, int j0, int j_end,
+// Cache slots (page * page_size + place in the page) of the keys at places [n0, n0 + BN) of the run (-1: beyond n_end, or
+// no page), one per thread n < BN: the block table is read once per key, ahead of the copies.
+__device__ __forceinline__ void tile_rows(long long* rows, const Params& p, int entry, const KeyRun& run, int n0, int n_end,
                                           int tid) {
   if (tid < BN) {
-    const int j = j0 + tid;
     long long off = -1;
-    if (j < j_end) {
+    if (n0 + tid < n_end) {
+      const int j = run.position(n0 + tid);
       const int pi = j / p.page_size;
       const int page = pi < p.table_width ? p.block_table[(size_t)entry * p.table_width + pi] : -1;
       if (page < 0 || page >= p.num_pages) atomicOr(p.status, JV_STATUS_BAD_PAGE);
@@ -205,21 +208,27 @@ __device__ __forceinline__ float fast_exp2(float x) {
 // Turns one warp's raw products of a tile into weights.  The products are scaled (and capped) first.  Softmax:
 // exponentials against the running maximum of the thread's two rows, (max, sum) updated, output accumulators
 // rescaled.  Sigmoid: every weight stands alone, nothing is kept.  With MASK the visibility test is applied
-// (key0 + nb*8 + (lane%4)*2 + (i&1) is the key of s[nb][i]; pos0/pos1 are the positions of rows lane/4 and
-// lane/4 + 8, -1 for an unused row); tiles that lie wholly inside every row's visible range go without it.
+// (n0 + nb*8 + (lane%4)*2 + (i&1) is the place in the run of s[nb][i]'s key; pos0/pos1 are the positions of rows lane/4
+// and lane/4 + 8, -1 for an unused row); tiles that lie wholly inside every row's visible range go without it.
 template <int NB, bool MASK>
 __device__ __forceinline__ void weights_tile(float (&s)[NB][4], float (&o)[VD / 8][4], float (&m)[2], float (&l)[2],
-                                             int pos0, int pos1, int key0, int j_end, int window, float scale0,
+                                             int pos0, int pos1, const KeyRun& run, int n0, int n_end, int window, int keep,
+                                             float scale0,
                                              float scale1, const float* dist0, const float* dist1, int n_dist,
                                              float cap, bool sigmoid, float bias0, float bias1, int lane) {
   const float cap_exp = cap > 0.f ? 2.f * LOG2E / cap : 0.f;
+  const int first0 = MASK ? first_visible(pos0, window) : 0, first1 = MASK ? first_visible(pos1, window) : 0;
+  auto visible = [&](int nb, int i) {
+    const int n = n0 + nb * 8 + (lane & 3) * 2 + (i & 1), key = run.position(n);
+    return n < n_end && key <= ((i < 2) ? pos0 : pos1) && (key >= ((i < 2) ? first0 : first1) || key < keep);
+  };
 #pragma unroll
   for (int nb = 0; nb < NB; ++nb)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       float v = s[nb][i] * ((i < 2) ? scale0 : scale1);
       if (dist0 != nullptr) {     // by how far back the key lies; rows without a position and hidden keys read column 0
-        const int back = ((i < 2) ? pos0 : pos1) - (key0 + nb * 8 + (lane & 3) * 2 + (i & 1));
+        const int back = ((i < 2) ? pos0 : pos1) - run.position(n0 + nb * 8 + (lane & 3) * 2 + (i & 1));
         v += __ldg(((i < 2) ? dist0 : dist1) + min(max(back, 0), n_dist - 1));
       }
       // tanh(x) = 1 - 2 / (1 + e^(2x)): one ex2 and one reciprocal; its absolute error (about 1e-7) times the cap is
@@ -232,12 +241,7 @@ __device__ __forceinline__ void weights_tile(float (&s)[NB][4], float (&o)[VD / 
     for (int nb = 0; nb < NB; ++nb)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        bool vis = true;
-        if (MASK) {
-          const int key = key0 + nb * 8 + (lane & 3) * 2 + (i & 1);
-          const int pos = (i < 2) ? pos0 : pos1;
-          vis = key < j_end && key <= pos && key >= first_visible(pos, window);
-        }
+        const bool vis = !MASK || visible(nb, i);
         const float x = s[nb][i] + ((i < 2) ? bias0 : bias1);
         s[nb][i] = vis ? fast_rcp(1.f + fast_exp2(-x * LOG2E)) : 0.f;
       }
@@ -248,12 +252,7 @@ __device__ __forceinline__ void weights_tile(float (&s)[NB][4], float (&o)[VD / 
   for (int nb = 0; nb < NB; ++nb)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      if (MASK) {
-        const int key = key0 + nb * 8 + (lane & 3) * 2 + (i & 1);
-        const int pos = (i < 2) ? pos0 : pos1;
-        const bool vis = key < j_end && key <= pos && key >= first_visible(pos, window);
-        if (!vis) s[nb][i] = -INFINITY;
-      }
+      if (MASK && !visible(nb, i)) s[nb][i] = -INFINITY;
       mx[i >> 1] = fmaxf(mx[i >> 1], s[nb][i]);
     }
   float alpha[2], m_scaled[2];
@@ -318,7 +317,8 @@ __global__ void __launch_bounds__(THREADS) attn_prefill_general_kernel(const Par
   if (tokens_here <= 0) return;
   const int pos_first = ctx + q_off;
   const int j_lo = first_visible(pos_first, p.window);
-  const int j_hi = pos_first + tokens_here;   // exclusive
+  const KeyRun run(j_lo, p.keep);
+  const int n_keys = run.places(pos_first + tokens_here);
 
   // ---- queries of the tile (unused rows zero)
   constexpr int CH = KD / 8;
@@ -329,9 +329,9 @@ __global__ void __launch_bounds__(THREADS) attn_prefill_general_kernel(const Par
     const size_t off = valid ? (size_t)(q_begin + q_off + t) * p.q_stride + (size_t)(kv_head * G + hh) * KD + part * 8 : 0;
     cp_async16(qs + r * SK + part * 8, p.q + off, valid);
   }
-  const int n_tiles = (j_hi - j_lo + BN - 1) / BN;
-  tile_rows(rows[0], p, entry, kv_head, j_lo, j_hi, tid);
-  tile_rows(rows[1], p, entry, kv_head, j_lo + BN, j_hi, tid);
+  const int n_tiles = (n_keys + BN - 1) / BN;
+  tile_rows(rows[0], p, entry, run, 0, n_keys, tid);
+  tile_rows(rows[1], p, entry, run, BN, n_keys, tid);
   cp_async_commit();                      // the queries
   __syncthreads();
   issue_tile(ks, vs, rows[0], p, kv_head, &bars[0], tid);
@@ -368,6 +368,7 @@ __global__ void __launch_bounds__(THREADS) attn_prefill_general_kernel(const Par
     warp_last = max(warp_last, __shfl_xor_sync(0xffffffffu, warp_last, o));
     warp_first = min(warp_first, __shfl_xor_sync(0xffffffffu, warp_first, o));
   }
+  const int warp_vis = first_visible(warp_last, p.window);     // keys before it are hidden from the warp's last row
 
   float o_acc[VD / 8][4];
 #pragma unroll
@@ -381,14 +382,14 @@ __global__ void __launch_bounds__(THREADS) attn_prefill_general_kernel(const Par
     if (t + 1 < n_tiles)
       issue_tile(ks + (buf ^ 1) * BN * SK, vs + (buf ^ 1) * BN * SV, rows[buf ^ 1], p, kv_head, &bars[buf ^ 1], tid);
     // rows of tile t+2 go where those of tile t were (read when tile t was issued, an iteration ago)
-    if (t + 2 < n_tiles) tile_rows(rows[buf], p, entry, kv_head, j_lo + (t + 2) * BN, j_hi, tid);
+    if (t + 2 < n_tiles) tile_rows(rows[buf], p, entry, run, (t + 2) * BN, n_keys, tid);
     if (t == 0) cp_async_wait<0>();
     // every thread takes the same way out: all saw the tile, or the block stops (status word set)
     if (!__syncthreads_and(wait_tile(&bars[buf], (t >> 1) & 1, p))) {
       wait_tile(&bars[buf], (t >> 1) & 1, p);   // once more, bounded, for copies that may still be landing
       return;
     }
-    const int key0 = j_lo + t * BN;
+    const int n0 = t * BN, key0 = run.position(n0);
     if (key0 <= warp_last) {
       float s[BN / 8][4];
 #pragma unroll
@@ -397,12 +398,12 @@ __global__ void __launch_bounds__(THREADS) attn_prefill_general_kernel(const Par
         for (int i = 0; i < 4; ++i) s[nb][i] = 0.f;
       qk_tile<KD, BN / 8>(s, qs + warp * 16 * SK, ks + buf * BN * SK, lane);
       // the test is needed only where the tile reaches past the first row's position, past the end,
-      // or a window cuts into it
-      if (key0 + BN - 1 > warp_first || key0 + BN > j_hi || p.window != 0)
-        weights_tile<BN / 8, true>(s, o_acc, m, l, pos[0], pos[1], key0, j_hi, p.window, scale[0], scale[1], dist[0], dist[1], p.n_dist, p.score_cap, sigmoid,
+      // or starts before what the last row's window (chunk) shows
+      if (run.position(n0 + BN - 1) > warp_first || n0 + BN > n_keys || key0 < warp_vis)
+        weights_tile<BN / 8, true>(s, o_acc, m, l, pos[0], pos[1], run, n0, n_keys, p.window, p.keep, scale[0], scale[1], dist[0], dist[1], p.n_dist, p.score_cap, sigmoid,
                                    bias[0], bias[1], lane);
       else
-        weights_tile<BN / 8, false>(s, o_acc, m, l, pos[0], pos[1], key0, j_hi, p.window, scale[0], scale[1], dist[0], dist[1], p.n_dist, p.score_cap, sigmoid,
+        weights_tile<BN / 8, false>(s, o_acc, m, l, pos[0], pos[1], run, n0, n_keys, p.window, p.keep, scale[0], scale[1], dist[0], dist[1], p.n_dist, p.score_cap, sigmoid,
                                     bias[0], bias[1], lane);
       pv_tile<VD, BN / 8>(o_acc, s, vs + buf * BN * SV, lane);
     }
@@ -463,10 +464,11 @@ __global__ void __launch_bounds__(THREADS) attn_decode_general_kernel(const Para
   const int G = p.n_q_heads / p.n_kv_heads;
   const int HPT = p.heads_per_tile;
   const int pos_q = p.start_pos[entry];
-  const int vis_lo = first_visible(pos_q, p.window);   // visible keys: [vis_lo, pos_q]
-  const int j_lo = max(vis_lo, (int)blockIdx.z * p.split_size);
-  const int j_hi = min(pos_q + 1, ((int)blockIdx.z + 1) * p.split_size);
-  if (j_lo >= j_hi) return;
+  const KeyRun run(first_visible(pos_q, p.window), p.keep);
+  const int n_vis = run.places(pos_q + 1);             // all of them visible; the splits share the places of the run
+  const int n_lo = blockIdx.z * p.split_size;
+  const int n_hi = min(n_vis, n_lo + p.split_size);
+  if (n_lo >= n_hi) return;
   const int token = p.cu_seqlens[entry];
 
   constexpr int CH = KD / 8;
@@ -477,9 +479,9 @@ __global__ void __launch_bounds__(THREADS) attn_decode_general_kernel(const Para
     const size_t off = valid ? (size_t)token * p.q_stride + (size_t)(kv_head * G + hh) * KD + part * 8 : 0;
     cp_async16(qs + r * SK + part * 8, p.q + off, valid);
   }
-  const int n_tiles = (j_hi - j_lo + BN - 1) / BN;
+  const int n_tiles = (n_hi - n_lo + BN - 1) / BN;
 #pragma unroll
-  for (int st = 0; st < DECODE_STAGES; ++st) tile_rows(rows[st], p, entry, kv_head, j_lo + st * BN, j_hi, tid);
+  for (int st = 0; st < DECODE_STAGES; ++st) tile_rows(rows[st], p, entry, run, n_lo + st * BN, n_hi, tid);
   cp_async_commit();                      // the queries
   __syncthreads();
 #pragma unroll
@@ -525,26 +527,26 @@ __global__ void __launch_bounds__(THREADS) attn_decode_general_kernel(const Para
     }
     // rows of tile t+STAGES go where those of tile t were (read when tile t was issued)
     if (t + DECODE_STAGES < n_tiles)
-      tile_rows(rows[t % DECODE_STAGES], p, entry, kv_head, j_lo + (t + DECODE_STAGES) * BN, j_hi, tid);
+      tile_rows(rows[t % DECODE_STAGES], p, entry, run, n_lo + (t + DECODE_STAGES) * BN, n_hi, tid);
     if (t == 0) cp_async_wait<0>();
     if (!__syncthreads_and(wait_tile(&bars[t % DECODE_STAGES], (t / DECODE_STAGES) & 1, p))) {
       wait_tile(&bars[t % DECODE_STAGES], (t / DECODE_STAGES) & 1, p);
       return;
     }
     const int buf = t % DECODE_STAGES;
-    const int key0 = j_lo + t * BN + warp * 16;      // this warp's 16 keys of the tile
-    if (key0 < j_hi) {
+    const int n0 = n_lo + t * BN + warp * 16;        // this warp's 16 keys of the tile
+    if (n0 < n_hi) {
       float s[2][4];
 #pragma unroll
       for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
         for (int i = 0; i < 4; ++i) s[nb][i] = 0.f;
       qk_tile<KD, 2>(s, qs, ks + (buf * BN + warp * 16) * SK, lane);
-      // keys before j_lo are never loaded, so only the tile that reaches past j_hi needs the test
-      if (key0 + 16 > j_hi)
-        weights_tile<2, true>(s, o_acc, m, l, pos[0], pos[1], key0, j_hi, 0, scale[0], scale[1], dist[0], dist[1], p.n_dist, p.score_cap, sigmoid, bias[0], bias[1], lane);
+      // hidden keys are not in the run, so only the tile that reaches past n_hi needs the test
+      if (n0 + 16 > n_hi)
+        weights_tile<2, true>(s, o_acc, m, l, pos[0], pos[1], run, n0, n_hi, 0, 0, scale[0], scale[1], dist[0], dist[1], p.n_dist, p.score_cap, sigmoid, bias[0], bias[1], lane);
       else
-        weights_tile<2, false>(s, o_acc, m, l, pos[0], pos[1], key0, j_hi, 0, scale[0], scale[1], dist[0], dist[1], p.n_dist, p.score_cap, sigmoid, bias[0], bias[1], lane);
+        weights_tile<2, false>(s, o_acc, m, l, pos[0], pos[1], run, n0, n_hi, 0, 0, scale[0], scale[1], dist[0], dist[1], p.n_dist, p.score_cap, sigmoid, bias[0], bias[1], lane);
       pv_tile<VD, 2>(o_acc, s, vs + (buf * BN + warp * 16) * SV, lane);
     }
     __syncthreads();
@@ -597,8 +599,8 @@ __global__ void __launch_bounds__(THREADS) attn_decode_general_kernel(const Para
   // ---- the block that finishes last among the splits of this (token, kv head, head group) merges them,
   //      in ascending order of the splits whichever block that is.  Nobody waits: a block adds one to the
   //      counter when its partial result is written and leaves unless it brought the count to the total.
-  const int s_first = vis_lo / p.split_size;
-  int s_last = pos_q / p.split_size;
+  constexpr int s_first = 0;
+  int s_last = (n_vis - 1) / p.split_size;
   if (s_last >= p.n_splits) {           // the launch has too few splits for this length
     if (tid == 0) atomicOr(p.status, JV_STATUS_BAD_ROW);
     s_last = p.n_splits - 1;
@@ -690,7 +692,7 @@ JV_EXPORT int jv_attn_general_mma(const void* q, int q_stride, void* out, int ou
                                   int value_dim, int page_size, int num_pages, int window, float scale, float score_cap,
                                   int sigmoid, const float* bias, const float* head_scale, const float* dist_bias,
                                   int n_dist, const float* sink, int split_size, int n_splits, int n_k_heads,
-                                  float out_scale, int* status, cudaStream_t stream) {
+                                  float out_scale, int keep, int* status, cudaStream_t stream) {
   if (n_work == 0) return JV_OK;
   if ((dist_bias != nullptr && n_dist < 1) || (sink != nullptr && sigmoid)) return JV_ERR_UNSUPPORTED;
   if (key_dim != KD || value_dim != VD || n_kv_heads < 1 || n_v_heads < 1 || n_k_heads < 1 ||
@@ -709,7 +711,7 @@ JV_EXPORT int jv_attn_general_mma(const void* q, int q_stride, void* out, int ou
   p.num_pages = num_pages; p.window = window; p.scale = scale; p.score_cap = score_cap; p.sigmoid = sigmoid ? 1 : 0;
   p.bias = bias; p.status = status;
   p.head_scale = head_scale; p.dist_bias = dist_bias; p.n_dist = n_dist; p.sink = sink;
-  p.n_k_heads = n_k_heads; p.out_scale = out_scale;
+  p.n_k_heads = n_k_heads; p.out_scale = out_scale; p.keep = window > 0 ? keep : 0;
   const int G = n_q_heads / n_kv_heads;
   p.heads_per_tile = G < 16 ? G : 16;
   p.n_head_groups = (G + p.heads_per_tile - 1) / p.heads_per_tile;

@@ -8,12 +8,13 @@
 // pairs of ONE kv head, so keys and values are read once for all query heads of the
 // group: row m -> token q_off + m / heads_per_tile, head kv*G + hg*heads_per_tile +
 // m % heads_per_tile.  Keys run over the entry's block table; key j is visible to a
-// query at position p iff j <= p and (window == 0 or j > p - window).  Softmax is the
+// query at position p iff j <= p and (window == 0 or j > p - window or j < keep: the first `keep` tokens of a sequence may stay
+// visible under a window; keys are counted as places in a run, common.cuh, KeyRun).  Softmax is the
 // running (max, sum) form; scores, probabilities and the output sum are float.  Key rows (and queries) longer than
 // `d_chunk` elements come through shared memory in pieces.
 //
-// SPLIT: split s covers key positions [s*split_size, (s+1)*split_size) of the visible
-// range; it writes its unnormalised output sum and (max, sum) to `part_o`/`part_ml`;
+// SPLIT: split s covers the places [s*split_size, (s+1)*split_size) of the run of visible
+// keys; it writes its unnormalised output sum and (max, sum) to `part_o`/`part_ml`;
 // `attn_combine_kernel` merges the splits of a row in ascending order, so the result
 // does not depend on what else is in the batch.
 #include "common.cuh"
@@ -39,6 +40,7 @@ struct AttnParams {
   int n_k_heads;             // key heads (group kv reads key head kv % n_k_heads)
   int d_chunk;               // elements of the key rows that are in shared memory at a time
   float out_scale;           // multiplies the heads' outputs
+  int keep;                  // positions below this one stay visible under a window
   float score_cap;           // > 0: score <- cap * tanh(score / cap), after the scale
   int sigmoid;               // 1: the weight of a visible key is sigmoid(score + bias[query head]), not normalised over keys
   const float* bias;         // [n_q_heads] or null
@@ -76,12 +78,12 @@ __global__ void __launch_bounds__(THREADS) attn_simt_kernel(const AttnParams p) 
 
   // visible key range of the tile
   const int pos_first = ctx + q_off, pos_last = ctx + q_off + tokens_here - 1;
-  int j_lo = first_visible(pos_first, p.window);
-  int j_hi = pos_last + 1;  // exclusive
+  const KeyRun run(first_visible(pos_first, p.window), p.keep);
+  int n_lo = 0, n_hi = run.places(pos_last + 1);  // places of the run, the second exclusive
   if (SPLIT) {
-    j_lo = max(j_lo, blockIdx.z * p.split_size);
-    j_hi = min(j_hi, (blockIdx.z + 1) * p.split_size);
-    if (j_lo >= j_hi) return;
+    n_lo = blockIdx.z * p.split_size;
+    n_hi = min(n_hi, n_lo + p.split_size);
+    if (n_lo >= n_hi) return;
   }
 
   const T* q = (const T*)p.q;
@@ -116,7 +118,7 @@ __global__ void __launch_bounds__(THREADS) attn_simt_kernel(const AttnParams p) 
     for (int c = 0; c < DC; ++c) acc[m][c] = 0.f;
   __syncthreads();
 
-  for (int j0 = j_lo; j0 < j_hi; j0 += BLOCK_N) {
+  for (int n0 = n_lo; n0 < n_hi; n0 += BLOCK_N) {
     float s[4] = {0.f, 0.f, 0.f, 0.f};               // scores: thread (n = lane, rows warp*4 .. warp*4+3)
     for (int d0 = 0; d0 < D; d0 += DCH) {
       const int dn = min(DCH, D - d0);
@@ -124,10 +126,10 @@ __global__ void __launch_bounds__(THREADS) attn_simt_kernel(const AttnParams p) 
       if (D > DCH) load_q(d0, dn);
       // ---- keys and values of this chunk into shared memory (one warp per key row)
       for (int n = warp; n < BLOCK_N; n += THREADS / 32) {
-        const int j = j0 + n;
         const T* krow = nullptr;
         const T* vrow = nullptr;
-        if (j < j_hi) {
+        if (n0 + n < n_hi) {
+          const int j = run.position(n0 + n);
           const int pi = j / p.page_size;
           const int page = pi < p.table_width ? p.block_table[(size_t)entry * p.table_width + pi] : -1;
           if (page < 0 || page >= p.num_pages) {
@@ -153,12 +155,12 @@ __global__ void __launch_bounds__(THREADS) attn_simt_kernel(const AttnParams p) 
     }
 
     {
-      const int j = j0 + lane;
+      const int j = run.position(n0 + lane);
 #pragma unroll
       for (int r = 0; r < 4; ++r) {
         const int m = warp * 4 + r;
         const int pos = row_pos[m];
-        const bool vis = pos >= 0 && j < j_hi && j <= pos && j >= first_visible(pos, p.window);
+        const bool vis = pos >= 0 && n0 + lane < n_hi && j <= pos && (j >= first_visible(pos, p.window) || j < p.keep);
         float sc = s[r] * p.scale;
         if (p.head_scale != nullptr || p.dist_bias != nullptr) {
           const int hq = min(hg * p.heads_per_tile + m % p.heads_per_tile, G - 1) + kv_head * G;
@@ -252,10 +254,9 @@ __global__ void attn_combine_kernel(const AttnParams p) {
   const int entry = p.work[2 * x];
   const int D = p.v_dim;
   const int pos = p.start_pos[entry];
-  const int j_lo = first_visible(pos, p.window);
-  const int j_hi = pos + 1;
-  const int s_first = j_lo / p.split_size;
-  int s_last = (j_hi - 1) / p.split_size;  // inclusive
+  const KeyRun run(first_visible(pos, p.window), p.keep);
+  constexpr int s_first = 0;
+  int s_last = (run.places(pos + 1) - 1) / p.split_size;  // inclusive
   if (s_last >= p.n_splits) {  // the launch has too few splits for this length
     if (threadIdx.x == 0) atomicOr(p.status, JV_STATUS_BAD_ROW);
     s_last = p.n_splits - 1;
@@ -322,7 +323,7 @@ JV_EXPORT int jv_attn_simt_ex(const void* q, int q_stride, void* out, int out_st
                               float scale, int split_size, int n_splits, int v_dim, int n_v_heads, int v_row,
                               float score_cap, int sigmoid, const float* bias, int out_f32, const float* head_scale,
                               const float* dist_bias, int n_dist, const float* sink, int n_k_heads, float out_scale,
-                              int* status, cudaStream_t stream) {
+                              int keep, int* status, cudaStream_t stream) {
   if (n_work == 0) return JV_OK;
   if ((dist_bias != nullptr && n_dist < 1) || (sink != nullptr && sigmoid)) return JV_ERR_UNSUPPORTED;
   if (v_row <= 0) v_row = head_dim;
@@ -337,6 +338,7 @@ JV_EXPORT int jv_attn_simt_ex(const void* q, int q_stride, void* out, int out_st
   AttnParams p;
   p.n_v_heads = n_v_heads; p.v_row = v_row; p.score_cap = score_cap; p.sigmoid = sigmoid ? 1 : 0; p.bias = bias;
   p.out_f32 = out_f32 ? 1 : 0; p.n_k_heads = n_k_heads; p.d_chunk = d_chunk; p.out_scale = out_scale;
+  p.keep = window > 0 ? keep : 0;
   p.head_scale = head_scale; p.dist_bias = dist_bias; p.n_dist = n_dist; p.sink = sink;
   p.q = q; p.q_stride = q_stride; p.out = out; p.out_stride = out_stride;
   p.part_o = part_o; p.part_ml = part_ml; p.k_cache = k_cache; p.v_cache = v_cache;
@@ -394,5 +396,5 @@ JV_EXPORT int jv_attn_simt(const void* q, int q_stride, void* out, int out_strid
   return jv_attn_simt_ex(q, q_stride, out, out_stride, dtype, part_o, part_ml, k_cache, v_cache, block_table,
                          table_width, cu_seqlens, start_pos, work, n_work, n_q_heads, n_kv_heads, head_dim, page_size,
                          num_pages, window, scale, split_size, n_splits, v_dim, n_kv_heads, head_dim, 0.f, 0, nullptr,
-                         0, nullptr, nullptr, 0, nullptr, n_kv_heads, 1.f, status, stream);
+                         0, nullptr, nullptr, 0, nullptr, n_kv_heads, 1.f, 0, status, stream);
 }

@@ -24,8 +24,10 @@
 // itself: P therefore never goes through shared memory.  Every mbarrier wait is bounded by a clock deadline and
 // reports to the status word instead of spinning.
 //
-// Restrictions (the caller falls back to the mma.sync kernel otherwise): bfloat16, head size 128, no
-// window, HPT up to 16, page size a power of two from 8 to 128.
+// Masks: causal, a window, chunks; under a window the first `keep` positions of a sequence may stay visible: an item's
+// tiles are then those of the kept positions (as far as they lie before the window's) followed by the window's.
+//
+// Restrictions (the caller falls back to the mma.sync kernel otherwise): bfloat16, head size 128, HPT up to 16, page size a power of two from 8 to 128.
 #include "tcgen05.cuh"
 
 #include <math.h>
@@ -54,6 +56,8 @@ struct Params {
   // added to the score of key j (untouched by the scales); exp(sink[h]) counts once in the denominator.  Each may be null.
   const float* head_scale; const float* dist_bias; int n_dist; const float* sink;
   int window;                  // the mask as one number (common.cuh, first_visible): 0, a window (> 0) or chunks (< 0)
+  int keep;                    // positions below this one stay visible under a window
+  float score_cap_log2;        // > 0: the scaled score s (bias and head scale included) becomes cap * tanh(s / cap); times log2 e
   float out_scale;             // multiplies the output
   int* status;
 };
@@ -75,6 +79,8 @@ struct Item {
   int tokens_here, pos_first;       // tokens in the tile, position of the first
   int j_lo, j_hi;                   // keys [j_lo, j_hi) are visible to some row: j_lo is the first row's first visible key
   int tile0, n_tiles;               // the first key tile (keys tile0 * BN ..) and the number of key tiles
+  int kept;                         // tiles of kept positions, which come first: tile j < kept holds keys j * BN ..
+  __device__ __forceinline__ int tile(int j) const { return j < kept ? j : j - kept + tile0; }    // among all key tiles of the request
 };
 
 __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map,
@@ -115,7 +121,8 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
     it.j_hi = it.pos_first + it.tokens_here;
     it.j_lo = first_visible(it.pos_first, p.window);
     it.tile0 = it.j_lo / BN;
-    it.n_tiles = it.tokens_here > 0 ? (it.j_hi + BN - 1) / BN - it.tile0 : 0;
+    it.kept = min((p.keep + BN - 1) / BN, it.tile0);
+    it.n_tiles = it.tokens_here > 0 ? (it.j_hi + BN - 1) / BN - it.tile0 + it.kept : 0;
     return it;
   };
 
@@ -179,9 +186,9 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
       // page ids of a tile: lane i reads the i-th (a tile has at most 16 pages); -1 = no page needed or none there
       // (a page whose keys all lie before the first visible one is not needed, and may have been given back)
       auto tile_pages = [&](int j) -> int {
-        const int pi = (j + it.tile0) * pages_per_tile + lane;
+        const int pi = it.tile(j) * pages_per_tile + lane;
         int page = -1;
-        if (j < it.n_tiles && lane < pages_per_tile && pi * P < it.j_hi && (pi + 1) * P > it.j_lo && pi < p.table_width) {
+        if (j < it.n_tiles && lane < pages_per_tile && pi * P < it.j_hi && ((pi + 1) * P > it.j_lo || pi * P < p.keep) && pi < p.table_width) {
           page = p.block_table[(size_t)it.entry * p.table_width + pi];
           if (page < 0 || page >= p.num_pages) { atomicOr(p.status, JV_STATUS_BAD_PAGE); page = -1; }
         }
@@ -315,7 +322,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
       const Item it = upcoming;
       ++r_next;
       more = next_item(r_next, upcoming);
-      const int n_tiles = it.n_tiles, j_hi = it.j_hi, pos_first = it.pos_first, tile0 = it.tile0;
+      const int n_tiles = it.n_tiles, j_hi = it.j_hi, pos_first = it.pos_first;
       const bool row_ok = t < it.tokens_here && hh < G;
       const int pos = row_ok ? pos_first + t : -1;
       const int vis_first = first_visible(pos, p.window);                    // this row's first visible key
@@ -325,7 +332,10 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
       // With a head's own scale or a bias by distance the scores are first brought to the exponent's unit, s * scale *
       // head_scale * log2(e) + bias * log2(e), and the maximum, the reference and the exponentials work on that (`sc`,
       // what still multiplies a score in the exponent, is then 1).  The same for every thread of the block.
-      const bool shaped = p.head_scale != nullptr || p.dist_bias != nullptr;
+      // So they are with a cap: cap * tanh(x / cap) * log2(e) = c - 2 c / (1 + 2^(2 y / cap)), c = cap * log2(e), y = x * log2(e).
+      const bool capped = p.score_cap_log2 > 0.f;
+      const bool shaped = p.head_scale != nullptr || p.dist_bias != nullptr || capped;
+      const float cap_exp = capped ? 2.f * LOG2E / p.score_cap_log2 : 0.f, cap2 = -2.f * p.score_cap_log2;
       const int head = it.kv_head * G + min(hh, G - 1);
       const float sc = shaped ? 1.f : p.scale_log2;
       const float row_scale = p.scale_log2 * (p.head_scale != nullptr ? p.head_scale[head] : 1.f);
@@ -340,7 +350,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
         if (ok) ok = mbar_wait(&sh->s_full[gt & 1], (gt >> 1) & 1);
         ok = __all_sync(0xffffffffu, ok);
         const uint32_t s_addr = tmem + lane_addr + (gt & 1) * 128 + half * 64;
-        const int jt = j + tile0;                                // the tile among all key tiles of the request
+        const int jt = it.tile(j);                               // the tile among all key tiles of the request
         const int key0 = jt * BN + half * 64;                    // first key of this thread's 64
         const bool need_mask = jt * BN + BN > j_hi || jt * BN + BN - 1 > pos_first || jt * BN < vis_first_last;   // block-uniform
         uint32_t sr[2][32];
@@ -359,6 +369,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
               for (int i = 0; i < 32; ++i) {
                 float v = __uint_as_float(sr[c][i]) * row_scale;
                 if (dist_row != nullptr) v = fmaf(__ldg(dist_row + min(max(back0 - (c * 32 + i), 0), last_col)), LOG2E, v);
+                if (capped) v = fmaf(cap2, fast_rcp(1.f + fast_exp2(v * cap_exp)), p.score_cap_log2);
                 sr[c][i] = __float_as_uint(v);
               }
           }
@@ -367,11 +378,12 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
           if (need_mask) {
             const int last = min(pos, j_hi - 1) - key0;          // the last of this thread's 64 keys that counts
             const int first = vis_first - key0;                  // and the first (a window, a chunk)
+            const int kept = p.keep - key0;                      // those before this one count all the same
 #pragma unroll
             for (int c = 0; c < 2; ++c)
 #pragma unroll
               for (int i = 0; i < 32; ++i)
-                if (c * 32 + i > last || c * 32 + i < first) sr[c][i] = __float_as_uint(-INFINITY);
+                if (c * 32 + i > last || (c * 32 + i < first && c * 32 + i >= kept)) sr[c][i] = __float_as_uint(-INFINITY);
           }
           float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -454,9 +466,10 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
           tmem_st32_bits(tmem + lane_addr + TMEM_P + (gt & 1) * 64 + half * 32, pw);
         }
         l_run = l_run * alpha + ((sum[0] + sum[1]) + (sum[2] + sum[3]));
-        // ---- in an item's last tile the value rows past the end become zero (they may hold anything), and in its first
-        // tile those before the first visible key (their pages may not have been loaded)
-        const int rows_before = j == 0 ? it.j_lo - jt * BN : 0;
+        // ---- in an item's last tile the value rows past the end become zero (they may hold anything), and so do those
+        // before the first visible key, kept ones excepted (their pages may not have been loaded)
+        const int zero_from = min(max(p.keep - jt * BN, 0), BN);
+        const int rows_before = max(min(it.j_lo - jt * BN, BN) - zero_from, 0);
         const int rows_upto = (j == n_tiles - 1 && j_hi < jt * BN + BN) ? j_hi - jt * BN : BN;
         if (rows_before > 0 || rows_upto < BN) {
           const int s = gt % V_STAGES;
@@ -465,7 +478,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
             const int n_zero = rows_before + (BN - rows_upto);
             for (int i = (threadIdx.x - 64); i < n_zero * 16; i += SOFTMAX_THREADS) {
               const int z = i / 16, part = i % 16;                // 16 chunks of 16 bytes per row (both halves)
-              const int key_row = z < rows_before ? z : rows_upto + (z - rows_before);
+              const int key_row = z < rows_before ? zero_from + z : rows_upto + (z - rows_before);
               *reinterpret_cast<uint4*>(v_s + s * TILE_BYTES + (part >> 3) * HALF_BYTES + key_row * 128 + (part & 7) * 16) =
                   make_uint4(0, 0, 0, 0);
             }
@@ -594,15 +607,17 @@ JV_EXPORT int jv_attn_tcgen05_tokens_per_tile(int n_q_heads, int n_kv_heads) { r
 // sigmoid != 0: the weights are sigmoid(q.k * scale + bias[query head]) instead of a softmax (bias: [n_q_heads] floats or null).
 // head_scale [n_q_heads], dist_bias [n_q_heads][n_dist], sink [n_q_heads] (floats, each may be null; softmax only): see Params.
 // window: the mask as one number (0: every earlier key; > 0: a window; < 0: chunks of -window positions).
+// keep: under a window the first `keep` positions stay visible.  score_cap > 0 (softmax only): scores become cap * tanh(score / cap).
 // out_scale multiplies the output.
 JV_EXPORT int jv_attn_tcgen05_ex(const void* q, int q_stride, int n_tokens, void* out, int out_stride, const void* k_cache,
                                  const void* v_cache, const int* block_table, int table_width, const int* cu_seqlens,
                                  const int* start_pos, const int* work, int n_work, int n_q_heads, int n_kv_heads,
                                  int head_dim, int page_size, int num_pages, float scale, int sigmoid, const float* bias,
                                  const float* head_scale, const float* dist_bias, int n_dist, const float* sink,
-                                 int window, float out_scale, int* status, cudaStream_t stream) {
+                                 int window, int keep, float score_cap, float out_scale, int* status,
+                                 cudaStream_t stream) {
   if (n_work == 0) return JV_OK;
-  if ((dist_bias != nullptr && n_dist < 1) || (sigmoid && (head_scale != nullptr || dist_bias != nullptr || sink != nullptr)))
+  if ((dist_bias != nullptr && n_dist < 1) || (sigmoid && (score_cap > 0.f || head_scale != nullptr || dist_bias != nullptr || sink != nullptr)))
     return JV_ERR_UNSUPPORTED;
   if (!jv_attn_tcgen05_supports(head_dim, n_q_heads, n_kv_heads, page_size, 0)) return JV_ERR_UNSUPPORTED;
   if ((q_stride % 8) || (out_stride % 8) || ((uintptr_t)q % 16) || ((uintptr_t)out % 16) || ((uintptr_t)k_cache % 16) ||
@@ -640,7 +655,7 @@ JV_EXPORT int jv_attn_tcgen05_ex(const void* q, int q_stride, int n_tokens, void
   p.page_size = page_size; p.num_pages = num_pages; p.hpt = G; p.tokens_per_tile = ROWS / G;
   p.scale_log2 = scale * LOG2E; p.status = status; p.sigmoid = sigmoid ? 1 : 0; p.bias = bias;
   p.head_scale = head_scale; p.dist_bias = dist_bias; p.n_dist = n_dist; p.sink = sink; p.window = window;
-  p.out_scale = out_scale;
+  p.out_scale = out_scale; p.keep = window > 0 ? keep : 0; p.score_cap_log2 = score_cap > 0.f ? score_cap * LOG2E : 0.f;
   constexpr size_t smem = TILE_BYTES * (Q_BUFFERS + K_STAGES + V_STAGES) + sizeof(Shared) + 1024;
   static bool ready[JV_MAX_DEVICES];
   if (!jv_once_per_device(ready, [&] {
@@ -665,5 +680,5 @@ JV_EXPORT int jv_attn_tcgen05(const void* q, int q_stride, int n_tokens, void* o
                               int head_dim, int page_size, int num_pages, float scale, int* status, cudaStream_t stream) {
   return jv_attn_tcgen05_ex(q, q_stride, n_tokens, out, out_stride, k_cache, v_cache, block_table, table_width, cu_seqlens,
                             start_pos, work, n_work, n_q_heads, n_kv_heads, head_dim, page_size, num_pages, scale, 0, nullptr,
-                            nullptr, nullptr, 0, nullptr, 0, 1.f, status, stream);
+                            nullptr, nullptr, 0, nullptr, 0, 0, 0.f, 1.f, status, stream);
 }

@@ -150,7 +150,8 @@ __global__ void branch_norm_add_vec_kernel(float* __restrict__ h, const TD* __re
 
 template <typename TD>
 __global__ void pick_rows_sum_kernel(const TD* __restrict__ y, const int* __restrict__ pick, const float* __restrict__ coef,
-                                     int parts, int y_rows, float* __restrict__ out, int hidden, int* __restrict__ status) {
+                                     int parts, int y_rows, const TD* __restrict__ own, const float* __restrict__ own_coef,
+                                     float* __restrict__ out, int hidden, int* __restrict__ status) {
   pdl_trigger();
   pdl_wait();
   const int r = blockIdx.x;
@@ -159,11 +160,12 @@ __global__ void pick_rows_sum_kernel(const TD* __restrict__ y, const int* __rest
     for (int s = 0; s < parts; ++s) {
       const int src = pick[(size_t)r * parts + s];
       if (src < 0 || src >= y_rows) {
-        if (c == 0) atomicOr(status, JV_STATUS_BAD_ROW);
+        if (c == 0 && (src != -1 || own == nullptr)) atomicOr(status, JV_STATUS_BAD_ROW);
         continue;
       }
       v = fmaf(coef[(size_t)r * parts + s], to_f32(y[(size_t)src * hidden + c]), v);
     }
+    if (own != nullptr) v = fmaf(own_coef[r], to_f32(own[(size_t)r * hidden + c]), v);
     out[(size_t)r * hidden + c] = v;
   }
 }
@@ -214,12 +216,14 @@ JV_EXPORT int jv_branch_norm_add(float* h, const void* y, int y_dtype, long long
 }
 
 // out[r, :] = sum_s coef[r, s] * y[pick[r, s], :] in 32-bit, s ascending: the weighted rows added up for a reader
-// that does not add them itself.
+// that does not add them itself.  own [n, hidden] of the same type with own_coef [n], or null: out[r, :] += own_coef[r] *
+// own[r, :], and a pick of -1 is then no row (without it, it is reported).
 JV_EXPORT int jv_pick_rows_sum(const void* y, int y_dtype, const int* pick, const float* coef, int parts, int y_rows,
-                               float* out, int n, int hidden, int* status, cudaStream_t stream) {
+                               const void* own, const float* own_coef, float* out, int n, int hidden, int* status,
+                               cudaStream_t stream) {
   if (n == 0) return JV_OK;
   JV_DISPATCH_DTYPE(y_dtype, TD, return jv_launch(pick_rows_sum_kernel<TD>, dim3(n), dim3(256), 0, stream, (const TD*)y,
-                                                  pick, coef, parts, y_rows, out, hidden, status));
+                                                  pick, coef, parts, y_rows, (const TD*)own, own_coef, out, hidden, status));
   return JV_ERR_UNSUPPORTED;
 }
 

@@ -76,6 +76,18 @@ __device__ __forceinline__ int first_visible(int pos, int mask) {
   return mask > 0 ? max(0, pos - mask + 1) : mask < 0 ? pos - pos % (-mask) : 0;
 }
 
+// The keys that the queries of one tile may see, as one run of places n = 0, 1, ...: with a window that keeps the first
+// `keep` tokens of a sequence these are positions 0 .. kept - 1 and then the positions from `first` on (`first`: the
+// first position inside the tile's first query's window).  Without kept tokens, or where the window still reaches them,
+// it is one run of positions.
+struct KeyRun {
+  int kept, gap;
+  __device__ __forceinline__ KeyRun(int first, int keep) : kept(min(keep, first)), gap(first - min(keep, first)) {}
+  __device__ __forceinline__ int position(int n) const { return n < kept ? n : n + gap; }
+  // places up to (not including) position `end` >= first
+  __device__ __forceinline__ int places(int end) const { return end - gap; }
+};
+
 // Programmatic dependent launch.  A kernel launched through jv_launch may be made resident while the
 // kernel before it in the stream is still finishing; whatever it does before `pdl_wait()` (index
 // arithmetic, prefetching weights that no kernel writes) overlaps that kernel's tail, and everything

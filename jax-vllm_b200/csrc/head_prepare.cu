@@ -10,7 +10,7 @@
 //                   position, so that the summed output can be turned back by the query's position (jv_head_rotate)
 //
 // The pairs of a rotation are (j, j + dims/2) ("halves") or (2j, 2j + 1) (`interleaved`); the pair (u, v) becomes
-// (u cos a - v sin a, v cos a + u sin a).  Queries go to q_out [n, Hq*D]; keys to k_cache[page, slot, key head, :D];
+// (u cos a - v sin a, v cos a + u sin a), for queries and keys with both cos and sin times `rot_gain`.  Queries go to q_out [n, Hq*D]; keys to k_cache[page, slot, key head, :D];
 // values to v_cache[page, slot, value head, :DV].
 //
 // jv_head_rotate turns every head of rows [n, heads*dim] by sign * position * freq[j] (in place or into `out`).
@@ -26,7 +26,7 @@ struct HeadPrepareParams {
   const void* proj; long long row_stride; int q_off, k_off, v_off;
   void* q_out;
   const int* positions; const int* token_entry; const int* block_table; int table_width;
-  const float* freq; int rot_dim;
+  const float* freq; int rot_dim; float rot_gain;
   const float* v_freq; int v_rot_dim;
   int interleaved;
   const void* q_norm_w; const void* k_norm_w; float eps;
@@ -41,7 +41,7 @@ struct HeadPrepareParams {
 template <typename T, typename TW>
 __device__ __forceinline__ void prepare_head(const T* __restrict__ src, T* __restrict__ dst, int dim, bool normed,
                                              const TW* __restrict__ w, float eps, const float* __restrict__ freq, int rot,
-                                             int interleaved, float pos, int lane) {
+                                             int interleaved, float pos, float gain, int lane) {
   float inv = 1.f;
   if (normed) {
     float ss = 0.f;
@@ -55,6 +55,7 @@ __device__ __forceinline__ void prepare_head(const T* __restrict__ src, T* __res
     if (w != nullptr) { u *= to_f32(w[i0]); v *= to_f32(w[i1]); }
     float sn, cs;
     sincosf(pos * freq[j], &sn, &cs);
+    sn *= gain; cs *= gain;
     dst[i0] = from_f32<T>(u * cs - v * sn);
     dst[i1] = from_f32<T>(v * cs + u * sn);
   }
@@ -82,7 +83,7 @@ __global__ void __launch_bounds__(32 * WARPS) head_prepare_kernel(const HeadPrep
   if (h < p.n_q_heads) {
     prepare_head<T, TW>(row + p.q_off + (size_t)h * p.key_dim, (T*)p.q_out + ((size_t)t * p.n_q_heads + h) * p.key_dim,
                         p.key_dim, p.q_norm_w != nullptr || p.qk_unit != 0, (const TW*)p.q_norm_w, p.eps, p.freq, p.rot_dim,
-                        p.interleaved, pos, lane);
+                        p.interleaved, pos, p.rot_gain, lane);
     return;
   }
   h -= p.n_q_heads;
@@ -97,12 +98,12 @@ __global__ void __launch_bounds__(32 * WARPS) head_prepare_kernel(const HeadPrep
   if (h < p.n_k_heads) {
     prepare_head<T, TW>(row + p.k_off + (size_t)h * p.key_dim, (T*)p.k_cache + (slot * p.n_k_heads + h) * p.key_dim,
                         p.key_dim, p.k_norm_w != nullptr || p.qk_unit != 0, (const TW*)p.k_norm_w, p.eps, p.freq, p.rot_dim,
-                        p.interleaved, pos, lane);
+                        p.interleaved, pos, p.rot_gain, lane);
     return;
   }
   h -= p.n_k_heads;
   prepare_head<T, TW>(row + p.v_off + (size_t)h * p.value_dim, (T*)p.v_cache + (slot * p.n_v_heads + h) * p.value_dim,
-                      p.value_dim, p.v_norm != 0, (const TW*)nullptr, p.eps, p.v_freq, p.v_rot_dim, p.interleaved, pos, lane);
+                      p.value_dim, p.v_norm != 0, (const TW*)nullptr, p.eps, p.v_freq, p.v_rot_dim, p.interleaved, pos, 1.f, lane);
 }
 
 template <typename TI, typename TO>
@@ -157,7 +158,7 @@ __global__ void __launch_bounds__(128) rms_rows_kernel(const T* __restrict__ in,
 // jv_attn_prepare, both null: queries only.
 JV_EXPORT int jv_head_prepare(const void* proj, int dtype, long long row_stride, int q_off, int k_off, int v_off,
                               void* q_out, const int* positions, const int* token_entry, const int* block_table,
-                              int table_width, const float* freq, int rot_dim, const float* v_freq, int v_rot_dim,
+                              int table_width, const float* freq, int rot_dim, float rot_gain, const float* v_freq, int v_rot_dim,
                               int interleaved, const void* q_norm_w, const void* k_norm_w, int w_dtype, float eps,
                               int v_norm, int qk_unit, void* k_cache, void* v_cache, int n, int n_q_heads, int n_k_heads,
                               int n_v_heads, int key_dim, int value_dim, int page_size, int num_pages, int* status,
@@ -170,7 +171,7 @@ JV_EXPORT int jv_head_prepare(const void* proj, int dtype, long long row_stride,
   HeadPrepareParams p;
   p.proj = proj; p.row_stride = row_stride; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.q_out = q_out;
   p.positions = positions; p.token_entry = token_entry; p.block_table = block_table; p.table_width = table_width;
-  p.freq = freq; p.rot_dim = rot_dim; p.v_freq = v_freq; p.v_rot_dim = v_rot_dim; p.interleaved = interleaved ? 1 : 0;
+  p.freq = freq; p.rot_dim = rot_dim; p.rot_gain = rot_gain; p.v_freq = v_freq; p.v_rot_dim = v_rot_dim; p.interleaved = interleaved ? 1 : 0;
   p.q_norm_w = q_norm_w; p.k_norm_w = k_norm_w; p.eps = eps; p.v_norm = v_norm ? 1 : 0; p.qk_unit = qk_unit ? 1 : 0;
   p.k_cache = k_cache; p.v_cache = v_cache; p.n = n; p.n_q_heads = n_q_heads; p.n_k_heads = n_k_heads; p.n_v_heads = n_v_heads;
   p.key_dim = key_dim; p.value_dim = value_dim; p.page_size = page_size; p.num_pages = num_pages; p.status = status;

@@ -9,14 +9,15 @@
 // with r = rows[i] if `rows` is given, else r = i.  When `rows` is given the sum is
 // not written back to h (the gathered rows are the last use of the stream).  Squares,
 // mean, rsqrt and the scaling are 32-bit; the result is rounded once, to the output
-// type.
+// type.  With a second weight the same normed row times that weight is written too, to y2 (two branches that read the
+// stream through a norm each).
 #include "common.cuh"
 
 template <typename TD, typename TW, typename TY>
 __global__ void rmsnorm_kernel(float* __restrict__ h, const TD* __restrict__ delta,
                                const int* __restrict__ rows, const TW* __restrict__ weight,
-                               TY* __restrict__ y, int hidden, float eps, int n_rows_total,
-                               int* __restrict__ status, int parts, size_t part_stride) {
+                               TY* __restrict__ y, const TW* __restrict__ weight2, TY* __restrict__ y2, int hidden, float eps,
+                               int n_rows_total, int* __restrict__ status, int parts, size_t part_stride) {
   __shared__ float scratch[33];
   pdl_trigger();
   pdl_wait();
@@ -52,6 +53,7 @@ __global__ void rmsnorm_kernel(float* __restrict__ h, const TD* __restrict__ del
     float v = hr[c];                          // this thread's own write, if any
     if (dr && !write_back) v += delta_at(c);
     yr[c] = from_f32<TY>(v * inv * to_f32(weight[c]));
+    if (y2 != nullptr) y2[(size_t)i * hidden + c] = from_f32<TY>(v * inv * to_f32(weight2[c]));
   }
 }
 
@@ -90,8 +92,8 @@ template <> __device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16*
 template <typename TD, typename TW, typename TY, int ITERS, int TOGETHER>
 __global__ void __launch_bounds__(ITERS == 1 ? 640 : 1024) rmsnorm_vec_kernel(float* __restrict__ h, const TD* __restrict__ delta,
                                    const int* __restrict__ rows, const TW* __restrict__ weight,
-                                   TY* __restrict__ y, int hidden, float eps, int n_rows_total,
-                                   int* __restrict__ status, int parts, size_t part_stride) {
+                                   TY* __restrict__ y, const TW* __restrict__ weight2, TY* __restrict__ y2, int hidden, float eps,
+                                   int n_rows_total, int* __restrict__ status, int parts, size_t part_stride) {
   __shared__ float scratch[33];
   pdl_trigger();
   pdl_wait();
@@ -155,6 +157,12 @@ __global__ void __launch_bounds__(ITERS == 1 ? 640 : 1024) rmsnorm_vec_kernel(fl
 #pragma unroll
       for (int k = 0; k < 8; ++k) w[k] = v[it][k] * inv * w[k];
       store8<TY>(yr + c, w);
+      if (y2 != nullptr) {
+        load8<TW>(weight2 + c, w);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) w[k] = v[it][k] * inv * w[k];
+        store8<TY>(y2 + (size_t)i * hidden + c, w);
+      }
     }
   }
 }
@@ -162,18 +170,20 @@ __global__ void __launch_bounds__(ITERS == 1 ? 640 : 1024) rmsnorm_vec_kernel(fl
 // h: [n_total, hidden] float (updated in place when delta is given and rows is null);
 // delta: [n_total, hidden] of dtype `delta_dtype` or null, or `delta_parts` such tensors `delta_part_stride`
 // elements apart whose sum it is; rows: [n_out] int32 or null;
-// weight: [hidden] of dtype `weight_dtype`; y: [n_out, hidden] of dtype `out_dtype`.
+// weight: [hidden] of dtype `weight_dtype`; y: [n_out, hidden] of dtype `out_dtype`; weight2, y2: a second weight and
+// output of the same types, or both null (`rows` null).
 JV_EXPORT int jv_rmsnorm(float* h, const void* delta, int delta_dtype, const int* rows,
-                         const void* weight, int weight_dtype, void* y, int out_dtype, int n_out,
-                         int n_total, int hidden, float eps, int delta_parts, long long delta_part_stride, int* status,
+                         const void* weight, int weight_dtype, void* y, int out_dtype, const void* weight2, void* y2,
+                         int n_out, int n_total, int hidden, float eps, int delta_parts, long long delta_part_stride, int* status,
                          cudaStream_t stream) {
   if (n_out == 0) return JV_OK;
-  if (delta_parts < 1 || (delta_part_stride % 8)) return JV_ERR_UNSUPPORTED;
+  if (delta_parts < 1 || (weight2 == nullptr) != (y2 == nullptr) || (y2 != nullptr && rows != nullptr))
+    return JV_ERR_UNSUPPORTED;
   const int parts = delta_parts;
   const size_t part_stride = (size_t)delta_part_stride;
   const bool aligned = ((uintptr_t)h % 16) == 0 && ((uintptr_t)delta % 16) == 0 && ((uintptr_t)weight % 16) == 0 &&
-                       ((uintptr_t)y % 16) == 0;
-  if (hidden % 8 == 0 && hidden <= 1024 * 8 * RM_ITERS && aligned) {
+                       ((uintptr_t)y % 16) == 0 && ((uintptr_t)weight2 % 16) == 0 && ((uintptr_t)y2 % 16) == 0;
+  if (hidden % 8 == 0 && hidden <= 1024 * 8 * RM_ITERS && aligned && delta_part_stride % 8 == 0) {
     const int vecs = hidden / 8;
     int iters = vecs <= 640 ? 1 : (vecs + 511) / 512;     // up to 640 threads, then more passes per thread
     if (iters > RM_ITERS) iters = RM_ITERS;
@@ -182,52 +192,71 @@ JV_EXPORT int jv_rmsnorm(float* h, const void* delta, int delta_dtype, const int
     if (iters == 1 && parts > 1 && n_out <= 256)
       JV_DISPATCH_DTYPE(out_dtype, TY, JV_DISPATCH_DTYPE(weight_dtype, TW, JV_DISPATCH_DTYPE(delta_dtype, TD,
           return jv_launch(rmsnorm_vec_kernel<TD, TW, TY, 1, 8>, dim3(n_out), dim3(vthreads), 0, stream,
-                           h, (const TD*)delta, rows, (const TW*)weight, (TY*)y, hidden, eps, n_total, status, parts, part_stride))));
+                           h, (const TD*)delta, rows, (const TW*)weight, (TY*)y, (const TW*)weight2, (TY*)y2, hidden, eps, n_total, status, parts, part_stride))));
     if (iters == 1)
       JV_DISPATCH_DTYPE(out_dtype, TY, JV_DISPATCH_DTYPE(weight_dtype, TW, JV_DISPATCH_DTYPE(delta_dtype, TD,
           return jv_launch(rmsnorm_vec_kernel<TD, TW, TY, 1, 1>, dim3(n_out), dim3(vthreads), 0, stream,
-                           h, (const TD*)delta, rows, (const TW*)weight, (TY*)y, hidden, eps, n_total, status, parts, part_stride))));
+                           h, (const TD*)delta, rows, (const TW*)weight, (TY*)y, (const TW*)weight2, (TY*)y2, hidden, eps, n_total, status, parts, part_stride))));
     JV_DISPATCH_DTYPE(out_dtype, TY, JV_DISPATCH_DTYPE(weight_dtype, TW, JV_DISPATCH_DTYPE(delta_dtype, TD,
         return jv_launch(rmsnorm_vec_kernel<TD, TW, TY, RM_ITERS, 1>, dim3(n_out), dim3(vthreads), 0, stream,
-                         h, (const TD*)delta, rows, (const TW*)weight, (TY*)y, hidden, eps, n_total, status, parts, part_stride))));
+                         h, (const TD*)delta, rows, (const TW*)weight, (TY*)y, (const TW*)weight2, (TY*)y2, hidden, eps, n_total, status, parts, part_stride))));
     return JV_ERR_UNSUPPORTED;
   }
   int threads = 32;
   while (threads < 512 && threads * 4 < hidden) threads *= 2;
   JV_DISPATCH_DTYPE(out_dtype, TY, JV_DISPATCH_DTYPE(weight_dtype, TW, JV_DISPATCH_DTYPE(delta_dtype, TD,
       return jv_launch(rmsnorm_kernel<TD, TW, TY>, dim3(n_out), dim3(threads), 0, stream,
-                       h, (const TD*)delta, rows, (const TW*)weight, (TY*)y, hidden, eps, n_total, status, parts, part_stride))));
+                       h, (const TD*)delta, rows, (const TW*)weight, (TY*)y, (const TW*)weight2, (TY*)y2, hidden, eps, n_total, status, parts, part_stride))));
   return JV_ERR_UNSUPPORTED;
 }
 
-// The norm behind a routed feed-forward: what is added to row r is sum_s coef[r, s] * y[pick[r, s], :] (s ascending, 32-bit),
-// the weighted rows of its experts, picked up as they are added.  Rows of 8 elements a thread and pass where sizes and
-// addresses allow (VEC), else one.
-template <typename TD, typename TW, typename TY, bool VEC>
-__global__ void __launch_bounds__(1024) rmsnorm_pick_kernel(float* __restrict__ h, const TD* __restrict__ picked,
-                                                            const int* __restrict__ pick, const float* __restrict__ coef,
-                                                            int parts, int picked_rows, const int* __restrict__ rows,
-                                                            const TW* __restrict__ weight, TY* __restrict__ y, int hidden,
-                                                            float eps, int n_rows_total, int* __restrict__ status) {
+// The norm behind a routed feed-forward.  What is added to row r is, in this order and in 32-bit,
+//
+//   delta[r, :]                                    (optional: float or 16-bit, as `parts` tensors like above)
+//   sum_s coef[r, s] * picked[pick[r, s], :]       (s ascending: the weighted rows of its experts)
+//   own_coef[r] * own[r, :]                        (optional: what identity experts give; a pick of -1 is then no row)
+//
+// and the sums are formed as they are added.  Rows of 8 elements a thread and pass where sizes and addresses allow (VEC),
+// else one.
+struct SumParams {
+  float* h;
+  const void* delta; int delta_f32, parts; size_t part_stride;
+  const void* picked; const int* pick; const float* coef; int picks, picked_rows;
+  const void* own; const float* own_coef;
+  const int* rows;
+  const void* weight; void* y;
+  const void* weight2; void* y2;
+  int hidden, n_rows_total;
+  float eps;
+  int* status;
+};
+
+template <typename TP, typename TW, typename TY, bool VEC>
+__global__ void __launch_bounds__(1024) rmsnorm_sum_kernel(const SumParams p) {
   constexpr int V = VEC ? 8 : 1, TOGETHER = 4;
   extern __shared__ float kept[];                 // [hidden]: the row after the sum
   __shared__ float scratch[33];
   pdl_trigger();
   pdl_wait();
-  const int i = blockIdx.x;
+  const int i = blockIdx.x, hidden = p.hidden;
+  TY* yr = (TY*)p.y + (size_t)i * hidden;
   int r = i;
-  if (rows != nullptr) {
-    r = rows[i];
-    if (r < 0 || r >= n_rows_total) {
-      if (threadIdx.x == 0) atomicOr(status, JV_STATUS_BAD_ROW);
-      for (int c = threadIdx.x; c < hidden; c += blockDim.x) y[(size_t)i * hidden + c] = from_f32<TY>(0.f);
+  if (p.rows != nullptr) {
+    r = p.rows[i];
+    if (r < 0 || r >= p.n_rows_total) {
+      if (threadIdx.x == 0) atomicOr(p.status, JV_STATUS_BAD_ROW);
+      for (int c = threadIdx.x; c < hidden; c += blockDim.x) yr[c] = from_f32<TY>(0.f);
       return;
     }
   }
-  float* hr = h + (size_t)r * hidden;
-  const int* pk = pick + (size_t)r * parts;
-  const float* cf = coef + (size_t)r * parts;
-  if (threadIdx.x < parts && (pk[threadIdx.x] < 0 || pk[threadIdx.x] >= picked_rows)) atomicOr(status, JV_STATUS_BAD_ROW);
+  float* hr = p.h + (size_t)r * hidden;
+  const int* pk = p.pick + (size_t)r * p.picks;
+  const float* cf = p.coef + (size_t)r * p.picks;
+  if (threadIdx.x < p.picks) {
+    const int src = pk[threadIdx.x];
+    if ((src < 0 || src >= p.picked_rows) && !(src == -1 && p.own != nullptr)) atomicOr(p.status, JV_STATUS_BAD_ROW);
+  }
+  const float oc = p.own != nullptr ? p.own_coef[r] : 0.f;
   float ss = 0.f;
   for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
     float v[8], d[8];
@@ -235,16 +264,33 @@ __global__ void __launch_bounds__(1024) rmsnorm_pick_kernel(float* __restrict__ 
     else v[0] = hr[c];
 #pragma unroll
     for (int k = 0; k < V; ++k) d[k] = 0.f;
-    for (int s0 = 0; s0 < parts; s0 += TOGETHER) {      // four rows ask for their loads together, then add in their order
+    if (p.delta != nullptr) {
+      const size_t at = (size_t)r * hidden + c;
+      for (int s = 0; s < p.parts; ++s) {
+        float e[8];
+        if (p.delta_f32) {
+          const float* src = (const float*)p.delta + s * p.part_stride + at;
+          if (VEC) load8<float>(src, e);
+          else e[0] = *src;
+        } else {
+          const __nv_bfloat16* src = (const __nv_bfloat16*)p.delta + s * p.part_stride + at;
+          if (VEC) load8<__nv_bfloat16>(src, e);
+          else e[0] = to_f32(*src);
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) d[k] += e[k];
+      }
+    }
+    for (int s0 = 0; s0 < p.picks; s0 += TOGETHER) {    // four rows ask for their loads together, then add in their order
       float e[TOGETHER][8], w[TOGETHER];
 #pragma unroll
       for (int s = 0; s < TOGETHER; ++s) {
-        const int src = s0 + s < parts ? pk[s0 + s] : -1;
-        const bool ok = src >= 0 && src < picked_rows;
+        const int src = s0 + s < p.picks ? pk[s0 + s] : -1;
+        const bool ok = src >= 0 && src < p.picked_rows;
         w[s] = ok ? cf[s0 + s] : 0.f;
-        const TD* row = picked + (size_t)(ok ? src : 0) * hidden + c;
+        const TP* row = (const TP*)p.picked + (size_t)(ok ? src : 0) * hidden + c;
         if (ok) {
-          if (VEC) load8<TD>(row, e[s]);
+          if (VEC) load8<TP>(row, e[s]);
           else e[s][0] = to_f32(*row);
         }
       }
@@ -255,48 +301,68 @@ __global__ void __launch_bounds__(1024) rmsnorm_pick_kernel(float* __restrict__ 
           for (int k = 0; k < V; ++k) d[k] = fmaf(w[s], e[s][k], d[k]);
         }
     }
+    if (oc != 0.f) {
+      float e[8];
+      const TP* row = (const TP*)p.own + (size_t)r * hidden + c;
+      if (VEC) load8<TP>(row, e);
+      else e[0] = to_f32(*row);
+#pragma unroll
+      for (int k = 0; k < V; ++k) d[k] = fmaf(oc, e[k], d[k]);
+    }
 #pragma unroll
     for (int k = 0; k < V; ++k) {
       v[k] += d[k];
       ss += v[k] * v[k];
       kept[c + k] = v[k];
     }
-    if (rows == nullptr) {
+    if (p.rows == nullptr) {
       if (VEC) store8<float>(hr + c, v);
       else hr[c] = v[0];
     }
   }
   ss = block_sum(ss, scratch);
-  const float inv = rsqrtf(ss / (float)hidden + eps);
-  TY* yr = y + (size_t)i * hidden;
-  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {     // a thread's own elements
-    float w[8];
-    if (VEC) load8<TW>(weight + c, w);
-    else w[0] = to_f32(weight[c]);
+  const float inv = rsqrtf(ss / (float)hidden + p.eps);
+  auto write = [&](const TW* weight, TY* out) {
+    for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {   // a thread's own elements
+      float w[8];
+      if (VEC) load8<TW>(weight + c, w);
+      else w[0] = to_f32(weight[c]);
 #pragma unroll
-    for (int k = 0; k < V; ++k) w[k] *= kept[c + k] * inv;
-    if (VEC) store8<TY>(yr + c, w);
-    else yr[c] = from_f32<TY>(w[0]);
-  }
+      for (int k = 0; k < V; ++k) w[k] *= kept[c + k] * inv;
+      if (VEC) store8<TY>(out + c, w);
+      else out[c] = from_f32<TY>(w[0]);
+    }
+  };
+  write((const TW*)p.weight, yr);
+  if (p.y2 != nullptr) write((const TW*)p.weight2, (TY*)p.y2 + (size_t)i * hidden);
 }
 
-// As jv_rmsnorm, with the sum of picked rows as delta: picked [picked_rows, hidden] of dtype `delta_dtype`, pick and coef
-// [n_total, parts].
-JV_EXPORT int jv_rmsnorm_pick(float* h, const void* picked, int delta_dtype, const int* pick, const float* coef, int parts,
-                              int picked_rows, const int* rows, const void* weight, int weight_dtype, void* y, int out_dtype,
-                              int n_out, int n_total, int hidden, float eps, int* status, cudaStream_t stream) {
+// As jv_rmsnorm, with a sum of picked rows in what is added: picked [picked_rows, hidden] and own [n_total, hidden] (or null)
+// of dtype `picked_dtype`, pick and coef [n_total, picks], own_coef [n_total]; delta as for jv_rmsnorm, or null.
+JV_EXPORT int jv_rmsnorm_sum(float* h, const void* delta, int delta_dtype, int delta_parts, long long delta_part_stride,
+                             const void* picked, int picked_dtype, const int* pick, const float* coef, int picks,
+                             int picked_rows, const void* own, const float* own_coef, const int* rows, const void* weight,
+                             int weight_dtype, void* y, int out_dtype, const void* weight2, void* y2, int n_out, int n_total,
+                             int hidden, float eps, int* status, cudaStream_t stream) {
   if (n_out == 0) return JV_OK;
   const size_t smem = sizeof(float) * (size_t)hidden;
-  if (parts < 1 || parts > 64 || smem > 48 * 1024 - 256) return JV_ERR_UNSUPPORTED;
-  const bool vec = hidden % 8 == 0 && ((uintptr_t)h % 16) == 0 && ((uintptr_t)picked % 16) == 0 && ((uintptr_t)weight % 16) == 0 &&
-                   ((uintptr_t)y % 16) == 0;
+  if (picks < 1 || picks > 64 || smem > 48 * 1024 - 256 || delta_parts < 1 || (own != nullptr && own_coef == nullptr) ||
+      (weight2 == nullptr) != (y2 == nullptr) || (y2 != nullptr && rows != nullptr))
+    return JV_ERR_UNSUPPORTED;
+  SumParams p;
+  p.h = h; p.delta = delta; p.delta_f32 = delta_dtype == 0; p.parts = delta_parts; p.part_stride = (size_t)delta_part_stride;
+  p.picked = picked; p.pick = pick; p.coef = coef; p.picks = picks; p.picked_rows = picked_rows; p.own = own;
+  p.own_coef = own_coef; p.rows = rows; p.weight = weight; p.y = y; p.weight2 = weight2; p.y2 = y2; p.hidden = hidden;
+  p.n_rows_total = n_total; p.eps = eps; p.status = status;
+  const bool vec = hidden % 8 == 0 && delta_part_stride % 8 == 0 && ((uintptr_t)h % 16) == 0 && ((uintptr_t)delta % 16) == 0 &&
+                   ((uintptr_t)picked % 16) == 0 && ((uintptr_t)own % 16) == 0 && ((uintptr_t)weight % 16) == 0 &&
+                   ((uintptr_t)y % 16) == 0 && ((uintptr_t)weight2 % 16) == 0 && ((uintptr_t)y2 % 16) == 0;
   const int units = vec ? hidden / 8 : hidden;
-  int threads = 64;                               // `parts` threads at least
+  int threads = 64;                               // `picks` threads at least
   while (threads < 512 && threads < units) threads *= 2;
-  JV_DISPATCH_DTYPE(out_dtype, TY, JV_DISPATCH_DTYPE(weight_dtype, TW, JV_DISPATCH_DTYPE(delta_dtype, TD, {
-      return jv_launch(vec ? rmsnorm_pick_kernel<TD, TW, TY, true> : rmsnorm_pick_kernel<TD, TW, TY, false>, dim3(n_out),
-                       dim3(threads), smem, stream, h, (const TD*)picked, pick, coef, parts, picked_rows, rows,
-                       (const TW*)weight, (TY*)y, hidden, eps, n_total, status);
+  JV_DISPATCH_DTYPE(out_dtype, TY, JV_DISPATCH_DTYPE(weight_dtype, TW, JV_DISPATCH_DTYPE(picked_dtype, TP, {
+      return jv_launch(vec ? rmsnorm_sum_kernel<TP, TW, TY, true> : rmsnorm_sum_kernel<TP, TW, TY, false>, dim3(n_out),
+                       dim3(threads), smem, stream, p);
   })));
   return JV_ERR_UNSUPPORTED;
 }

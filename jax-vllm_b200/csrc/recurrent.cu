@@ -11,6 +11,8 @@
 //
 //   generalized delta rule   w = exp(-e^(-1/2) sigmoid(z_w + w0)), a = sigmoid(z_a + a0), u = k / sqrt(|k|^2 + 1e-6),
 //                            b = a * u                                              (jv_delta_prepare, per token)
+//   gated linear attention   w = sigmoid(z)^(1/tau) per key channel, z = W low + bias with low a few numbers a token (the
+//                            low-rank half of the projection), r = q * q_scale, no removal term    (jv_gla_prepare)
 //   matrix memory with exponential gates and a running maximum m (m starts at 0):
 //                            i = cap tanh((z_i + i0) / cap), f = logsigmoid(cap tanh((z_f + f0) / cap)),
 //                            m' = max(f + m, i), keep = exp(f + m - m'), take = exp(i - m'),
@@ -28,8 +30,8 @@
 // the two dot products of a token are two shuffles each.  A step of single tokens is the same kernel with one token
 // an entry: it then reads and writes the state once, which is all its traffic.
 //
-// jv_head_norm_gate finishes both: each head's output divided by its root mean square, times a weight per element,
-// times sigmoid(gate), rounded for the output product.
+// jv_head_norm_gate finishes all: each head's output divided by its root mean square, times a weight per element (of all
+// heads, or one vector that the heads share), times sigmoid(gate) or silu(gate), rounded for the output product.
 #include "common.cuh"
 #include <math.h>
 
@@ -73,6 +75,46 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const T* __restrict_
 }
 
 __device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+
+// packed [n, heads, 3, D] = (q * q_scale, k, exp(logsigmoid(z) / tau)), z = w_up[e, :] . low + bias[e] in 32-bit.  A block
+// takes TOK tokens, so that a row of w_up is read once for all of them; `low` [n, rank] are columns of the projection.
+template <int TOK, typename T, typename W>
+__global__ void __launch_bounds__(128) gla_prepare_kernel(const T* __restrict__ proj, long long stride, int q_off, int k_off,
+                                                          int low_off, int rank, const W* __restrict__ w_up,
+                                                          const W* __restrict__ bias, float inv_tau, float q_scale,
+                                                          float* __restrict__ packed, int n, int heads, int D) {
+  extern __shared__ float low[];                        // [rank][TOK]
+  pdl_trigger();
+  pdl_wait();
+  const int t0 = blockIdx.x * TOK, tokens = min(TOK, n - t0);
+  for (int i = threadIdx.x; i < rank * TOK; i += blockDim.x) {
+    const int t = i % TOK;
+    low[i] = t < tokens ? to_f32(proj[(size_t)(t0 + t) * stride + low_off + i / TOK]) : 0.f;
+  }
+  __syncthreads();
+  const int e = blockIdx.y * blockDim.x + threadIdx.x;
+  if (e >= heads * D) return;
+  const int h = e / D, d = e - h * D;
+  const float b = to_f32(bias[e]);
+  float z[TOK];
+#pragma unroll
+  for (int t = 0; t < TOK; ++t) z[t] = 0.f;
+  const W* wrow = w_up + (size_t)e * rank;
+  for (int r = 0; r < rank; ++r) {
+    const float w = to_f32(wrow[r]);
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) z[t] = fmaf(w, low[r * TOK + t], z[t]);
+  }
+#pragma unroll
+  for (int t = 0; t < TOK; ++t) {
+    if (t >= tokens) break;
+    const T* row = proj + (size_t)(t0 + t) * stride;
+    float* out = packed + ((size_t)(t0 + t) * heads + h) * 3 * D + d;
+    out[0] = to_f32(row[q_off + e]) * q_scale;
+    out[D] = to_f32(row[k_off + e]);
+    out[2 * D] = expf(log_sigmoid(z[t] + b) * inv_tau);
+  }
+}
 
 // The gates of the matrix memory in two kernels.  (1) One warp per (entry, head) scans the running maximum: the two
 // log gates of 32 tokens are formed side by side, one per lane, then the chain m' = max(f + m, i), which is all that
@@ -526,7 +568,8 @@ template <typename T, typename W>
 __global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* __restrict__ o, const W* __restrict__ weight,
                                                              const T* __restrict__ gate, long long gate_stride,
                                                              T* __restrict__ out, long long out_stride, int heads, int V,
-                                                             float eps, const float* __restrict__ gates) {
+                                                             float eps, const float* __restrict__ gates, int shared_weight,
+                                                             int silu) {
   __shared__ float scratch[33];
   pdl_trigger();
   pdl_wait();
@@ -543,8 +586,11 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* __rest
   ss = block_sum(ss, scratch);
   const float inv = 1.f / sqrtf(ss / (float)V + eps);
   for (int j = threadIdx.x; j < V; j += blockDim.x) {
-    float y = src[j] * den * inv * to_f32(weight[h * V + j]);
-    if (gate != nullptr) y *= 1.f / (1.f + expf(-to_f32(gate[(size_t)n * gate_stride + h * V + j])));
+    float y = src[j] * den * inv * to_f32(weight[(shared_weight ? 0 : h * V) + j]);
+    if (gate != nullptr) {
+      const float g = to_f32(gate[(size_t)n * gate_stride + h * V + j]);
+      y *= (silu ? g : 1.f) / (1.f + expf(-g));
+    }
     out[(size_t)n * out_stride + h * V + j] = from_f32<T>(y);
   }
 }
@@ -561,6 +607,23 @@ JV_EXPORT int jv_delta_prepare(const void* proj, int dtype, long long stride, in
   JV_DISPATCH_DTYPE(dtype, T, JV_DISPATCH_DTYPE(w_dtype, W, return jv_launch(
       delta_prepare_kernel<T, W>, dim3(n, heads), dim3(D > 64 ? 128 : 64), 0, stream, (const T*)proj, stride, r_off, k_off,
       a_off, (const T*)zw, zw_stride, (const W*)a_bias, (const W*)w_bias, packed, heads, D)));
+  return JV_ERR_UNSUPPORTED;
+}
+
+// proj as above with q, k (heads * D each) and `rank` low-rank numbers at the given columns; w_up: [heads * D, rank], bias:
+// [heads * D], both of dtype `w_dtype`; packed: [n, heads, 3, D] float.
+JV_EXPORT int jv_gla_prepare(const void* proj, int dtype, long long stride, int q_off, int k_off, int low_off, int rank,
+                             const void* w_up, const void* bias, int w_dtype, float inv_tau, float q_scale, float* packed,
+                             int n, int heads, int D, cudaStream_t stream) {
+  if (n == 0) return JV_OK;
+  constexpr int MANY = 8;
+  if (rank < 1 || (size_t)rank * MANY * sizeof(float) > 48 * 1024) return JV_ERR_UNSUPPORTED;
+  const int tok = n >= 64 ? MANY : 1;
+  const dim3 grid((n + tok - 1) / tok, (heads * D + 127) / 128);
+  const size_t smem = sizeof(float) * rank * tok;
+  JV_DISPATCH_DTYPE(dtype, T, JV_DISPATCH_DTYPE(w_dtype, W, return jv_launch(
+      tok == MANY ? gla_prepare_kernel<MANY, T, W> : gla_prepare_kernel<1, T, W>, grid, dim3(128), smem, stream, (const T*)proj,
+      stride, q_off, k_off, low_off, rank, (const W*)w_up, (const W*)bias, inv_tau, q_scale, packed, n, heads, D)));
   return JV_ERR_UNSUPPORTED;
 }
 
@@ -613,14 +676,15 @@ JV_EXPORT int jv_state_scan(const float* packed, int removal, const void* v, int
   return JV_ERR_UNSUPPORTED;
 }
 
-// o: [n, heads * V] float; weight: [heads * V] of dtype `w_dtype`; gate: rows of `gate_stride` elements (or null);
+// o: [n, heads * V] float; weight: [heads * V], or [V] shared by the heads (`shared_weight`), of dtype `w_dtype`; the gate
+// multiplies by its sigmoid, or by its silu (`silu`); gate: rows of `gate_stride` elements (or null);
 // out: rows of `out_stride` elements, both of dtype `dtype`.
 JV_EXPORT int jv_head_norm_gate(const float* o, const void* weight, int w_dtype, const void* gate, long long gate_stride,
                                 void* out, int dtype, long long out_stride, int n, int heads, int V, float eps,
-                                const float* gates, cudaStream_t stream) {
+                                const float* gates, int shared_weight, int silu, cudaStream_t stream) {
   if (n == 0) return JV_OK;
   JV_DISPATCH_DTYPE(dtype, T, JV_DISPATCH_DTYPE(w_dtype, W, return jv_launch(
       head_norm_gate_kernel<T, W>, dim3(n, heads), dim3(V > 64 ? 128 : 64), 0, stream, o, (const W*)weight, (const T*)gate,
-      gate_stride, (T*)out, out_stride, heads, V, eps, gates)));
+      gate_stride, (T*)out, out_stride, heads, V, eps, gates, shared_weight, silu)));
   return JV_ERR_UNSUPPORTED;
 }

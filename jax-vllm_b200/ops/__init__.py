@@ -56,10 +56,22 @@ class PickedRows:
     """A result [n, width] given as rows of `rows` [m, width] to be picked and weighted: row r of the result is
     sum_s coef[r, s] * rows[pick[r, s]] (32-bit, s ascending): what a routed feed-forward leaves (its experts'
     outputs in the order of the experts, and for every token where its chosen experts' rows are and what they
-    weigh).  `branch_norm_add` adds the rows up as it reads them; `tensor()` does it for any other reader."""
+    weigh).  `branch_norm_add` and `rmsnorm` add the rows up as they read them; `tensor()` does it for any other reader.
+    With `own` [n, width] and `own_coef` [n], own_coef[r] * own[r] is added (what identity experts give), and a pick of -1
+    is no row."""
 
-    def __init__(self, rows: torch.Tensor, pick: torch.Tensor, coef: torch.Tensor):
-        self.rows, self.pick, self.coef = rows, pick, coef
+    def __init__(self, rows: torch.Tensor, pick: torch.Tensor, coef: torch.Tensor, own: torch.Tensor | None = None,
+                 own_coef: torch.Tensor | None = None):
+        self.rows, self.pick, self.coef, self.own, self.own_coef = rows, pick, coef, own, own_coef
+
+    def check(self):
+        _cuda(self.rows, "rows to pick"); _cuda(self.pick, "pick", torch.int32); _cuda(self.coef, "coef", torch.float32)
+        if self.coef.shape != self.pick.shape:
+            raise KernelError("picked rows: a coefficient per pick")
+        if self.own is not None:
+            _cuda(self.own, "own rows", self.rows.dtype); _cuda(self.own_coef, "own_coef", torch.float32)
+            if tuple(self.own.shape) != tuple(self.shape) or self.own_coef.numel() != self.pick.shape[0]:
+                raise KernelError("picked rows: own rows have the result's shape, with a coefficient each")
 
     @property
     def shape(self):
@@ -70,14 +82,34 @@ class PickedRows:
         return self.rows.device
 
     def tensor(self, dtype: torch.dtype = torch.float32) -> torch.Tensor:
-        _cuda(self.rows, "rows"); _cuda(self.pick, "pick", torch.int32); _cuda(self.coef, "coef", torch.float32)
+        self.check()
         n, width = self.shape
         out = torch.empty((n, width), dtype=torch.float32, device=self.device)
-        f = _fn("branch_norm", "jv_pick_rows_sum", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int,
-                                                    c_int, c_void_p, c_void_p])
+        f = _fn("branch_norm", "jv_pick_rows_sum", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                                                    c_void_p, c_int, c_int, c_void_p, c_void_p])
         _check(f(self.rows.data_ptr(), _code(self.rows, "rows"), self.pick.data_ptr(), self.coef.data_ptr(),
-                 self.pick.shape[1], self.rows.shape[0], out.data_ptr(), n, width, _status_ptr(self.device), _stream()),
-               "pick_rows_sum")
+                 self.pick.shape[1], self.rows.shape[0], _ptr(self.own), _ptr(self.own_coef), out.data_ptr(), n, width,
+                 _status_ptr(self.device), _stream()), "pick_rows_sum")
+        return out if dtype == torch.float32 else out.to(dtype)
+
+
+class BranchSum:
+    """A result that is the sum of `delta` (a tensor or a PartialSum) and `picked` (a PickedRows): a layer whose two
+    branches leave together, one of them routed.  `rmsnorm` adds both as it reads them; `tensor()` serves any other reader."""
+
+    def __init__(self, delta, picked: PickedRows):
+        self.delta, self.picked = delta, picked
+
+    @property
+    def shape(self):
+        return self.picked.shape
+
+    @property
+    def device(self):
+        return self.picked.device
+
+    def tensor(self, dtype: torch.dtype = torch.float32) -> torch.Tensor:
+        out = residual_add(self.picked.tensor(), self.delta)
         return out if dtype == torch.float32 else out.to(dtype)
 
 
@@ -238,8 +270,8 @@ def wait_probe(cycles: int, arrive: bool, device=None) -> tuple:
 
 # ------------------------------------------------------------------------ embedding
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor | None = None,
-                 accumulate: bool = False) -> torch.Tensor:
-    """out[n, :] = table[ids[n], :] as float32; with `accumulate` the rows are added to `out`."""
+                 accumulate: bool = False, scale: float = 1.0) -> torch.Tensor:
+    """out[n, :] = scale * table[ids[n], :] as float32; with `accumulate` the rows are added to `out`."""
     _cuda(table, "table"); _cuda(ids, "ids", torch.int32)
     n, (vocab, hidden) = ids.numel(), table.shape
     if accumulate and out is None:
@@ -247,23 +279,26 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor | Non
     if out is None:
         out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
     _cuda(out, "out", torch.float32)
-    f = _fn("embed", "jv_embed_gather", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
-                                         c_void_p])
+    f = _fn("embed", "jv_embed_gather", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                                         c_void_p, c_void_p])
     _check(f(table.data_ptr(), _code(table, "table"), ids.data_ptr(), out.data_ptr(), n, hidden, vocab,
-             1 if accumulate else 0, _status_ptr(table.device), _stream()), "embed_gather")
+             1 if accumulate else 0, float(scale), _status_ptr(table.device), _stream()), "embed_gather")
     return out
 
 
 # ----------------------------------------------------------------------------- norm
 def rmsnorm(h: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
-            delta: torch.Tensor | None = None, rows: torch.Tensor | None = None) -> torch.Tensor:
-    """RMSNorm of rows of the float32 stream `h`, after adding `delta` (a tensor, a PartialSum or PickedRows, if given).
+            delta: torch.Tensor | None = None, rows: torch.Tensor | None = None, weight2: torch.Tensor | None = None):
+    """RMSNorm of rows of the float32 stream `h`, after adding `delta` (a tensor, a PartialSum, PickedRows or a BranchSum, if
+    given).
 
     Without `rows` every row is normalised and, when `delta` is given, `h` is updated
     in place with the sum.  With `rows` (int32) only those rows are produced and `h`
-    stays as it is.
+    stays as it is.  With `weight2` (not with `rows`) the result is a pair: the same normed rows with either weight.
     """
     _cuda(h, "h", torch.float32); _cuda(weight, "weight")
+    if weight2 is not None and (weight2.shape != weight.shape or weight2.dtype != weight.dtype or rows is not None):
+        raise KernelError("rmsnorm: the second weight is like the first, and not for picked rows of the stream")
     n_total, hidden = h.shape
     if weight.shape != (hidden,):
         raise KernelError(f"norm weight has shape {tuple(weight.shape)}, rows have {hidden} elements")
@@ -271,31 +306,40 @@ def rmsnorm(h: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.
         _cuda(rows, "rows", torch.int32)
     n_out = n_total if rows is None else rows.numel()
     y = torch.empty((n_out, hidden), dtype=out_dtype, device=h.device)
-    if isinstance(delta, PickedRows) and delta.pick.shape[1] <= 64 and hidden <= 12000:
-        picked, pick, coef = _cuda(delta.rows, "rows to pick"), _cuda(delta.pick, "pick", torch.int32), \
-            _cuda(delta.coef, "coef", torch.float32)
-        if delta.shape != h.shape or coef.shape != pick.shape:
+    y2 = torch.empty_like(y) if weight2 is not None else None
+    if weight2 is not None:
+        _cuda(weight2, "weight2")
+    result = y if y2 is None else (y, y2)
+    sum_of = delta.picked if isinstance(delta, BranchSum) else delta
+    if isinstance(sum_of, PickedRows) and sum_of.pick.shape[1] <= 64 and hidden <= 12000:
+        sum_of.check()
+        if sum_of.shape != h.shape:
             raise KernelError("the picked rows do not fit the stream")
-        f = _fn("norm", "jv_rmsnorm_pick", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
-                                            c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
-        _check(f(h.data_ptr(), picked.data_ptr(), _code(picked, "rows to pick"), pick.data_ptr(), coef.data_ptr(),
-                 pick.shape[1], picked.shape[0], _ptr(rows), weight.data_ptr(), _code(weight, "weight"), y.data_ptr(),
-                 _code(y, "out"), n_out, n_total, hidden, float(eps), _status_ptr(h.device), _stream()), "rmsnorm_pick")
-        return y
+        plus, n_parts, part_stride = _delta_parts(delta.delta if isinstance(delta, BranchSum) else None, h)
+        picked, pick = sum_of.rows, sum_of.pick
+        f = _fn("norm", "jv_rmsnorm_sum", [c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
+                                           c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                                           c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+        _check(f(h.data_ptr(), _ptr(plus), 0 if plus is None else _code(plus, "delta"), n_parts, part_stride,
+                 picked.data_ptr(), _code(picked, "rows to pick"), pick.data_ptr(), sum_of.coef.data_ptr(), pick.shape[1],
+                 picked.shape[0], _ptr(sum_of.own), _ptr(sum_of.own_coef), _ptr(rows), weight.data_ptr(),
+                 _code(weight, "weight"), y.data_ptr(), _code(y, "out"), _ptr(weight2), _ptr(y2), n_out, n_total, hidden,
+                 float(eps), _status_ptr(h.device), _stream()), "rmsnorm_sum")
+        return result
     delta, n_parts, part_stride = _delta_parts(delta, h)
-    f = _fn("norm", "jv_rmsnorm", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int,
+    f = _fn("norm", "jv_rmsnorm", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                    c_int, c_int, c_int, c_float, c_int, c_longlong, c_void_p, c_void_p])
     _check(f(h.data_ptr(), _ptr(delta), 0 if delta is None else _code(delta, "delta"), _ptr(rows),
-             weight.data_ptr(), _code(weight, "weight"), y.data_ptr(), _code(y, "out"), n_out, n_total, hidden,
-             float(eps), n_parts, part_stride, _status_ptr(h.device), _stream()), "rmsnorm")
-    return y
+             weight.data_ptr(), _code(weight, "weight"), y.data_ptr(), _code(y, "out"), _ptr(weight2), _ptr(y2), n_out,
+             n_total, hidden, float(eps), n_parts, part_stride, _status_ptr(h.device), _stream()), "rmsnorm")
+    return result
 
 
 def _delta_parts(delta, h: torch.Tensor):
     """(tensor, parts, elements between parts) for a `delta` that is a tensor, a PartialSum or None."""
     if delta is None:
         return None, 1, 0
-    if isinstance(delta, (PickedRows, GatedDelta)):
+    if isinstance(delta, (PickedRows, GatedDelta, BranchSum)):
         delta = delta.tensor()
     if isinstance(delta, PartialSum):
         parts = _cuda(delta.parts, "delta parts", torch.float32)
@@ -309,7 +353,7 @@ def _delta_parts(delta, h: torch.Tensor):
 
 
 def residual_add(h: torch.Tensor, delta) -> torch.Tensor:
-    """h += delta (a tensor, a PartialSum or a gated delta), the sum kept in float32."""
+    """h += delta (a tensor, a PartialSum, picked rows, a branch sum or a gated delta), the sum kept in float32."""
     _cuda(h, "h", torch.float32)
     if isinstance(delta, GatedDelta):
         gated_add_dyt(h, delta)
@@ -322,10 +366,11 @@ def residual_add(h: torch.Tensor, delta) -> torch.Tensor:
 
 
 # ----------------------------------------------------------------------- activation
-def swiglu(gate_up, block: int | None = None, out_dtype: torch.dtype | None = None) -> torch.Tensor:
+def swiglu(gate_up, block: int | None = None, out_dtype: torch.dtype | None = None,
+           out: torch.Tensor | None = None) -> torch.Tensor:
     """silu(gate) * up for a packed [n, 2*inter] tensor: blocks of `block` gate columns, each followed
     by the up columns of the same indices (default: all gate columns first).  The input may be a
-    PartialSum; the result then has `out_dtype`."""
+    PartialSum; the result then has `out_dtype`.  `out` [n, inter]: where to write, possibly a column range of wider rows."""
     n_parts, part_stride = 1, 0
     if isinstance(gate_up, PartialSum):
         if out_dtype is None:
@@ -343,9 +388,13 @@ def swiglu(gate_up, block: int | None = None, out_dtype: torch.dtype | None = No
     block = two_i // 2 if block is None else int(block)
     if block < 1 or (two_i // 2) % block:
         raise KernelError(f"gate|up block {block} does not divide {two_i // 2} columns")
-    act = torch.empty((n, two_i // 2), dtype=act_dtype, device=gate_up.device)
-    f = _fn("activation", "jv_swiglu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_longlong, c_void_p])
-    _check(f(gate_up.data_ptr(), act.data_ptr(), _code(act, "act"), n, two_i // 2, block, n_parts, part_stride, _stream()),
+    act = torch.empty((n, two_i // 2), dtype=act_dtype, device=gate_up.device) if out is None else \
+        _cuda(out, "out", act_dtype, contiguous=False)
+    if act.shape != (n, two_i // 2) or act.stride(1) != 1:
+        raise KernelError("swiglu: out is [n, columns / 2] with unit column stride")
+    f = _fn("activation", "jv_swiglu", [c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_longlong,
+                                        c_void_p])
+    _check(f(gate_up.data_ptr(), act.data_ptr(), act.stride(0), _code(act, "act"), n, two_i // 2, block, n_parts, part_stride, _stream()),
            "swiglu")
     return act
 
@@ -411,10 +460,11 @@ def attn_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.
               n_work: int, n_q_heads: int, n_kv_heads: int, head_dim: int, window: int, scale: float,
               split_size: int = 0, n_splits: int = 0, v_dim: int = 0, score_cap: float = 0.0, sigmoid: bool = False,
               bias: torch.Tensor | None = None, head_scale: torch.Tensor | None = None,
-              dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None, out_scale: float = 1.0) -> None:
+              dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None, out_scale: float = 1.0,
+              keep: int = 0) -> None:
     """Paged causal attention on CUDA cores (csrc/attn_simt.cu).  `work` is [n_work, 2] int32
     (entry, first token of the tile); with `n_splits` > 0 the work items are single tokens
-    whose keys are split into `n_splits` ranges of `split_size` positions.  `v_dim` > 0: only that many
+    whose visible keys are split into `n_splits` ranges of `split_size`.  `v_dim` > 0: only that many
     leading elements of a value row are used and `out` has v_dim elements per head (a cache whose values are
     the leading part of its keys is passed as both caches).
 
@@ -425,7 +475,7 @@ def attn_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.
     head]); `out` may be float32 whatever the type of q.  `head_scale` [query heads] multiplies the scaled scores of
     its head; `dist_bias` [query heads, distances] is added to the score of a key that lies so many positions back
     (the last column serves every larger distance); `sink` [query heads] adds exp(sink) once to the softmax's
-    denominator."""
+    denominator.  Under a window the first `keep` positions of a sequence stay visible."""
     n_dist = _score_extras("attn_simt", n_q_heads, head_scale, dist_bias, sink)
     for t, nm in ((q, "q"), (k_cache, "k_cache"), (v_cache, "v_cache")):
         _cuda(t, nm, q.dtype, contiguous=(nm != "q"))
@@ -454,14 +504,14 @@ def attn_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.
                                              c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                              c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int,
                                              c_int, c_float, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int,
-                                             c_void_p, c_int, c_float, c_void_p, c_void_p])
+                                             c_void_p, c_int, c_float, c_int, c_void_p, c_void_p])
     _check(f(q.data_ptr(), q_stride, out.data_ptr(), out.stride(0), _code(q, "q"), _ptr(part_o), _ptr(part_ml),
              k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), block_table.shape[1],
              cu_seqlens.data_ptr(), start_pos.data_ptr(), work.data_ptr(), n_work, n_q_heads, n_kv_heads, head_dim,
              k_cache.shape[1], k_cache.shape[0], int(window), float(scale), int(split_size), int(n_splits), v_dim,
              n_v_heads, v_row, float(score_cap), 1 if sigmoid else 0, _ptr(bias), 1 if out.dtype != q.dtype else 0,
              _ptr(head_scale), _ptr(dist_bias), n_dist, _ptr(sink), k_cache.shape[2], float(out_scale),
-             _status_ptr(q.device), _stream()), "attn_simt", launches=2 if n_splits > 0 else 1)
+             int(keep), _status_ptr(q.device), _stream()), "attn_simt", launches=2 if n_splits > 0 else 1)
 
 
 def _score_extras(who: str, n_q_heads: int, head_scale, dist_bias, sink) -> int:
@@ -503,7 +553,7 @@ def attn_general_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache:
                      n_work: int, n_q_heads: int, n_kv_heads: int, scale: float, split_size: int = 0, n_splits: int = 0,
                      score_cap: float = 0.0, sigmoid: bool = False, bias: torch.Tensor | None = None,
                      head_scale: torch.Tensor | None = None, dist_bias: torch.Tensor | None = None,
-                     sink: torch.Tensor | None = None, window: int = 0, out_scale: float = 1.0) -> None:
+                     sink: torch.Tensor | None = None, window: int = 0, out_scale: float = 1.0, keep: int = 0) -> None:
     """Paged causal attention on the tensor cores with the options of `attn_simt`: the key size and the key heads are the
     key cache's, the value size and the value heads the value cache's; bfloat16 in, bfloat16 or float32 out.
     `window`: the mask as one number (`mask_code`)."""
@@ -533,14 +583,14 @@ def attn_general_mma(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache:
     f = _fn(attn_general_mma_library(key_dim, value_dim), "jv_attn_general_mma",
             [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-             c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+             c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p])
     _check(f(q.data_ptr(), q_stride, out.data_ptr(), out.stride(0), 1 if out.dtype == torch.float32 else 0, _ptr(part_o),
              _ptr(part_ml), _ptr(counters), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(),
              block_table.shape[1], cu_seqlens.data_ptr(), start_pos.data_ptr(), work.data_ptr(), n_work, n_q_heads,
              n_kv_heads, n_v_heads, key_dim, value_dim, k_cache.shape[1], k_cache.shape[0], int(window), float(scale),
              float(score_cap), 1 if sigmoid else 0, _ptr(bias), _ptr(head_scale), _ptr(dist_bias), n_dist, _ptr(sink),
-             int(split_size), int(n_splits), k_cache.shape[2], float(out_scale), _status_ptr(q.device), _stream()),
-           "attn_general_mma")
+             int(split_size), int(n_splits), k_cache.shape[2], float(out_scale), int(keep), _status_ptr(q.device),
+             _stream()), "attn_general_mma")
 
 
 def attn_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: torch.Tensor, positions: torch.Tensor,
@@ -762,12 +812,13 @@ def attn_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: tor
                  n_work: int, n_q_heads: int, n_kv_heads: int, head_dim: int, scale: float, sigmoid: bool = False,
                  bias: torch.Tensor | None = None, head_scale: torch.Tensor | None = None,
                  dist_bias: torch.Tensor | None = None, sink: torch.Tensor | None = None, window: int = 0,
-                 out_scale: float = 1.0) -> None:
+                 out_scale: float = 1.0, keep: int = 0, score_cap: float = 0.0) -> None:
     """Paged causal attention of prompt portions on tcgen05 tensor cores with scores and output in tensor
     memory (csrc/attn_tcgen05.cu); `work` lists 128-row tiles of `attn_tcgen05_tokens_per_tile` tokens.  With
     `sigmoid` the weight of a visible key is sigmoid(score * scale + bias[query head]) instead of a softmax;
     `head_scale`, `dist_bias` and `sink` as for `attn_simt` (softmax only); `window`: the mask as one number
-    (`mask_code`).  `out_scale` multiplies the output."""
+    (`mask_code`), under which the first `keep` positions stay visible if it is a window.  `score_cap` > 0 (softmax only)
+    caps the scaled scores.  `out_scale` multiplies the output."""
     n_dist = _score_extras("attn_tcgen05", n_q_heads, head_scale, dist_bias, sink)
     for t, nm in ((q, "q"), (out, "out"), (k_cache, "k_cache"), (v_cache, "v_cache")):
         _cuda(t, nm, torch.bfloat16, contiguous=(nm not in ("q", "out")))     # q and out may be some heads of wider rows
@@ -784,12 +835,12 @@ def attn_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: tor
     f = _fn("attn_tcgen05", "jv_attn_tcgen05_ex", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                    c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                    c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
-                                                   c_int, c_float, c_void_p, c_void_p])
+                                                   c_int, c_int, c_float, c_float, c_void_p, c_void_p])
     _check(f(q.data_ptr(), q_stride, q.shape[0], out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
              block_table.data_ptr(), block_table.shape[1], cu_seqlens.data_ptr(), start_pos.data_ptr(), work.data_ptr(),
              n_work, n_q_heads, n_kv_heads, head_dim, k_cache.shape[1], k_cache.shape[0], float(scale),
              1 if sigmoid else 0, _ptr(bias), _ptr(head_scale), _ptr(dist_bias), n_dist, _ptr(sink), int(window),
-             float(out_scale), _status_ptr(q.device), _stream()), "attn_tcgen05")
+             int(keep), float(score_cap), float(out_scale), _status_ptr(q.device), _stream()), "attn_tcgen05")
 
 
 def attn_rows_tcgen05(q: torch.Tensor, q_stride: int, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
@@ -1074,21 +1125,21 @@ def _stream_ok(x: torch.Tensor, weight: torch.Tensor) -> bool:
 GEMM_EPILOGUES = {"bf16": 0, "f32": 1, "swiglu": 2, "gelu": 3}
 
 
-def gemm_tcgen05(x: torch.Tensor, weight: torch.Tensor, epilogue: str = "bf16") -> torch.Tensor:
+def gemm_tcgen05(x: torch.Tensor, weight: torch.Tensor, epilogue: str = "bf16", out: torch.Tensor | None = None) -> torch.Tensor:
     """x [M, K] times weight [N, K] transposed on tcgen05 tensor cores with the accumulator in
     tensor memory (csrc/gemm_tcgen05.cu).  epilogue "bf16" / "f32": the product in that type;
     "swiglu": silu(gate) * up as [M, N/2] bfloat16, for a weight whose every 256 rows are 128 gate rows
-    followed by the 128 up rows of the same indices."""
+    followed by the 128 up rows of the same indices.  `out`: where to write, possibly a column range of wider rows."""
     _cuda(x, "x", torch.bfloat16, contiguous=False); _cuda(weight, "weight", torch.bfloat16, contiguous=False)
     if x.dim() != 2 or weight.dim() != 2 or x.shape[1] != weight.shape[1] or x.stride(1) != 1 or weight.stride(1) != 1:
         raise KernelError(f"gemm shapes {tuple(x.shape)} x {tuple(weight.shape)}^T do not fit")
     m, k = x.shape
     n = weight.shape[0]
     code = GEMM_EPILOGUES[epilogue]
-    if epilogue == "swiglu":
-        y = torch.empty((m, n // 2), dtype=torch.bfloat16, device=x.device)
-    else:
-        y = torch.empty((m, n), dtype=torch.float32 if epilogue == "f32" else torch.bfloat16, device=x.device)
+    shape, dtype = (m, n // 2 if epilogue == "swiglu" else n), torch.float32 if epilogue == "f32" else torch.bfloat16
+    y = torch.empty(shape, dtype=dtype, device=x.device) if out is None else _cuda(out, "out", dtype, contiguous=False)
+    if tuple(y.shape) != shape or y.stride(1) != 1:
+        raise KernelError("gemm_tcgen05: out does not fit the product")
     f = _fn("gemm_tcgen05", "jv_gemm_tcgen05", [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
                                                 c_int, c_void_p, c_void_p])
     _check(f(x.data_ptr(), x.stride(0), weight.data_ptr(), weight.stride(0), y.data_ptr(), y.stride(0), m, n, k, code,
@@ -1153,6 +1204,8 @@ def branch_norm_add(h: torch.Tensor, branch, weight: torch.Tensor, eps: float, m
     PartialSum or a PickedRows; the latter two are added up as they are read."""
     _cuda(h, "h", torch.float32); _cuda(weight, "weight")
     pick = coef = None
+    if isinstance(branch, PickedRows) and branch.own is not None:
+        branch = branch.tensor()
     if isinstance(branch, PickedRows):
         branch, pick, coef = branch.rows, branch.pick, branch.coef
     n, hidden = h.shape
@@ -1290,29 +1343,38 @@ GROUP_SCORES = {"max": 0, "top2_sum": 1}
 
 
 def moe_route(logits: torch.Tensor, top: int, groups: int, keep: int, renorm: bool, scoring: str = "softmax",
-              group_score: str = "max", renorm_eps: float = 0.0, weight_scale: float = 1.0):
+              group_score: str = "max", renorm_eps: float = 0.0, weight_scale: float = 1.0,
+              correction: torch.Tensor | None = None, identity: int = 0):
     """(ids [n, top] int32, weights [n, top] float32) from the router logits [n, experts] float32: softmax over all
     experts or a sigmoid of each, group-limited choice of the `top` largest, largest first (csrc/moe_route.cu); a
     group scores as its best expert or as the sum of its two best; the chosen scores are divided by their sum
-    (+ `renorm_eps`) if `renorm`, and multiplied by `weight_scale`."""
+    (+ `renorm_eps`) if `renorm`, and multiplied by `weight_scale`.  `correction` [experts] float32 is added to the scores
+    for the choice only.  With `identity` > 0 the last so many experts are identity experts, and a third result [n] float32
+    holds the sum of the weights of those chosen."""
     _cuda(logits, "router logits", torch.float32, contiguous=False)
     n, experts = logits.shape
     if logits.stride(1) != 1:
         raise KernelError("router logits need unit column stride")
     ids = torch.empty((n, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=logits.device)
+    own = torch.empty(n, dtype=torch.float32, device=logits.device) if identity else None
+    if correction is not None:
+        _cuda(correction, "correction", torch.float32)
+        if correction.numel() != experts:
+            raise KernelError("moe_route: a correction per expert")
     f = _fn("moe_route", "jv_moe_route", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                          c_float, c_void_p, c_void_p, c_void_p])
+                                          c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
     _check(f(logits.data_ptr(), logits.stride(0), n, experts, top, groups, keep, 1 if renorm else 0,
-             ROUTER_SCORINGS[scoring], GROUP_SCORES[group_score], float(renorm_eps), float(weight_scale), ids.data_ptr(),
-             weights.data_ptr(), _stream()), "moe_route")
-    return ids, weights
+             ROUTER_SCORINGS[scoring], GROUP_SCORES[group_score], float(renorm_eps), float(weight_scale), _ptr(correction),
+             int(identity), ids.data_ptr(), weights.data_ptr(), _ptr(own), _stream()), "moe_route")
+    return (ids, weights, own) if identity else (ids, weights)
 
 
-def moe_align(ids: torch.Tensor, experts: int, tile: int):
+def moe_align(ids: torch.Tensor, experts: int, tile: int, identity: int = 0):
     """The (token, choice) pairs in the order of their experts, each expert's run padded to `tile` rows:
     (sorted_token [max_tiles * tile] (-1: padding), pos_of [n, top], tile_expert [max_tiles] (-1: unused), and
-    a one-element tensor: how many leading tiles are in use)."""
+    a one-element tensor: how many leading tiles are in use).  Choices from `experts` to `experts + identity` - 1 have no
+    rows: their pos_of is -1."""
     _cuda(ids, "ids", torch.int32)
     n, top = ids.shape
     pairs = n * top
@@ -1320,9 +1382,9 @@ def moe_align(ids: torch.Tensor, experts: int, tile: int):
     sorted_token = torch.empty(max_tiles * tile, dtype=torch.int32, device=ids.device)
     pos_of = torch.empty((n, top), dtype=torch.int32, device=ids.device)
     tile_expert = torch.empty(max_tiles + 1, dtype=torch.int32, device=ids.device)
-    f = _fn("moe_route", "jv_moe_align", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
+    f = _fn("moe_route", "jv_moe_align", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                           c_void_p, c_void_p])
-    _check(f(ids.data_ptr(), pairs, top, experts, tile, max_tiles, sorted_token.data_ptr(), pos_of.data_ptr(),
+    _check(f(ids.data_ptr(), pairs, top, experts, int(identity), tile, max_tiles, sorted_token.data_ptr(), pos_of.data_ptr(),
              tile_expert.data_ptr(), _status_ptr(ids.device), _stream()), "moe_align")
     return sorted_token, pos_of, tile_expert[:max_tiles], tile_expert[max_tiles:]
 
@@ -1591,6 +1653,24 @@ def delta_prepare(proj: torch.Tensor, r_off: int, k_off: int, a_off: int, zw: to
     return packed
 
 
+def gla_prepare(proj: torch.Tensor, q_off: int, k_off: int, low_off: int, w_up: torch.Tensor, bias: torch.Tensor, tau: float,
+                q_scale: float, heads: int, dim: int) -> torch.Tensor:
+    """Per token and head the vectors (r, k, w) of gated linear attention as float32 [n, heads, 3, dim]: r = q * q_scale,
+    w = sigmoid(z)^(1/tau) with z = w_up low + bias, `low` the `w_up.shape[1]` columns of `proj` from low_off on."""
+    _cuda(proj, "proj", contiguous=False); _cuda(w_up, "w_up"); _cuda(bias, "bias", w_up.dtype)
+    n, rank = proj.shape[0], w_up.shape[1]
+    if proj.stride(1) != 1 or w_up.shape[0] != heads * dim or bias.numel() != heads * dim or \
+            max(max(q_off, k_off) + heads * dim, low_off + rank) > proj.shape[1]:
+        raise KernelError("gla_prepare: shapes do not fit")
+    packed = torch.empty((n, heads, 3, dim), dtype=torch.float32, device=proj.device)
+    f = _fn("recurrent", "jv_gla_prepare", [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                                            c_float, c_float, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(f(proj.data_ptr(), _code(proj, "proj"), proj.stride(0), q_off, k_off, low_off, rank, w_up.data_ptr(),
+             bias.data_ptr(), _code(w_up, "w_up"), 1.0 / float(tau), float(q_scale), packed.data_ptr(), n, heads, dim,
+             _stream()), "gla_prepare")
+    return packed
+
+
 def memory_gates(proj: torch.Tensor, q_off: int, k_off: int, i_off: int, f_off: int, i_bias: torch.Tensor,
                  f_bias: torch.Tensor, cap: float, q_scale: float, state_m: torch.Tensor, cu_seqlens: torch.Tensor,
                  slots: torch.Tensor, n_entries: int, heads: int, dim: int):
@@ -1674,14 +1754,15 @@ def state_scan(packed: torch.Tensor, v: torch.Tensor, v_off: int, state: torch.T
 
 
 def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor, heads: int,
-                   value_dim: int, eps: float, gates: torch.Tensor | None = None) -> torch.Tensor:
+                   value_dim: int, eps: float, gates: torch.Tensor | None = None, gate_act: str = "sigmoid") -> torch.Tensor:
     """Each head of `o` [n, heads * value_dim] float32 divided by its root mean square, times `weight` [heads *
-    value_dim], times sigmoid(gate) (rows of `out`'s type, possibly a column range), written to `out` (possibly a
+    value_dim] or [value_dim] (shared by the heads), times sigmoid(gate), or silu(gate) by `gate_act` (rows of `out`'s type, possibly a column range), written to `out` (possibly a
     column range).  With `gates` [n, heads, 4] = (-, -, m, n . q) each head is first divided by
     max(|n . q|, exp(-m)) + 1e-6."""
     _cuda(o, "o", torch.float32); _cuda(weight, "weight"); _cuda(out, "out", contiguous=False)
     n = o.shape[0]
-    if o.shape[1] != heads * value_dim or out.shape != o.shape or out.stride(1) != 1 or weight.numel() != o.shape[1]:
+    if o.shape[1] != heads * value_dim or out.shape != o.shape or out.stride(1) != 1 or \
+            weight.numel() not in (o.shape[1], value_dim) or gate_act not in ("sigmoid", "silu"):
         raise KernelError("head_norm_gate: shapes do not fit")
     g_stride = 0
     if gate is not None:
@@ -1694,9 +1775,10 @@ def head_norm_gate(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor | N
         if tuple(gates.shape) != (n, heads, 4):
             raise KernelError("head_norm_gate: gates are [n, heads, 4]")
     f = _fn("recurrent", "jv_head_norm_gate", [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_longlong,
-                                               c_int, c_int, c_int, c_float, c_void_p, c_void_p])
+                                               c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p])
     _check(f(o.data_ptr(), weight.data_ptr(), _code(weight, "weight"), _ptr(gate), g_stride, out.data_ptr(),
-             _code(out, "out"), out.stride(0), n, heads, value_dim, float(eps), _ptr(gates), _stream()), "head_norm_gate")
+             _code(out, "out"), out.stride(0), n, heads, value_dim, float(eps), _ptr(gates),
+             1 if weight.numel() != o.shape[1] else 0, 1 if gate_act == "silu" else 0, _stream()), "head_norm_gate")
     return out
 
 
@@ -1748,10 +1830,10 @@ def head_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: 
                  token_entry: torch.Tensor, block_table: torch.Tensor, freq: torch.Tensor | None, interleaved: bool,
                  q_norm_w, k_norm_w, eps: float, value_norm: bool, value_freq: torch.Tensor | None, k_cache, v_cache,
                  n_q_heads: int, n_k_heads: int, n_v_heads: int, key_dim: int, value_dim: int,
-                 unit_heads: bool = False) -> None:
+                 unit_heads: bool = False, gain: float = 1.0) -> None:
     """Per head: RMSNorm of queries and keys with one weight vector [key_dim] shared by the heads (none: no norm, or with
     `unit_heads` a norm without a weight), rotation of
-    the first 2 * len(freq) elements (pairs in halves or `interleaved`); values divided by their root mean square
+    the first 2 * len(freq) elements (pairs in halves or `interleaved`; cos and sin times `gain`); values divided by their root mean square
     (`value_norm`) and rotated by their own position over 2 * len(value_freq) elements; keys and values written to
     their pages (both caches None: queries only).  32-bit arithmetic."""
     _cuda(proj, "proj", contiguous=False); _cuda(q_out, "q_out", proj.dtype)
@@ -1790,11 +1872,11 @@ def head_prepare(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_out: 
         raise KernelError("head_prepare: the projection row is too short")
     f = _fn("head_prepare", "jv_head_prepare",
             [c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
-             c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
+             c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
              c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
     _check(f(proj.data_ptr(), _code(proj, "proj"), proj.stride(0), q_off, k_off, v_off, q_out.data_ptr(),
              positions.data_ptr(), token_entry.data_ptr(), block_table.data_ptr(), block_table.shape[1], _ptr(freq), rot,
-             _ptr(value_freq), v_rot, 1 if interleaved else 0, _ptr(q_norm_w), _ptr(k_norm_w), w_code, float(eps),
+             float(gain), _ptr(value_freq), v_rot, 1 if interleaved else 0, _ptr(q_norm_w), _ptr(k_norm_w), w_code, float(eps),
              1 if value_norm else 0, 1 if unit_heads else 0, _ptr(k_cache) if writes else 0, _ptr(v_cache) if writes else 0,
              n, n_q_heads, n_k_heads, n_v_heads, key_dim, value_dim, page_size, num_pages, _status_ptr(proj.device),
              _stream()), "head_prepare")

@@ -14,12 +14,15 @@ which model it sits in.
                     tile_classes() -> work lists it wants for entries of several tokens: triples
                                       (tokens per tile, least new tokens, one more than the most)
     FeedForward     forward(x, step) -> y
+                    optional, for an arrangement that joins its output product with the mixer's: out_weight() [hidden,
+                    inner_size] (None: no such product), inner(x, step, out) writes what that product reads to `out`
+                    and returns what the feed-forward adds beside it (or None)
     Block           forward(h, delta, step, cache) -> (h, delta)   delta: not yet added to h
 """
 
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Optional
 
 import torch
@@ -53,6 +56,18 @@ class PagedKVNeed:
     v_heads: Optional[int] = None     # value heads and value size where they differ from the keys' (key head g
     v_head_dim: Optional[int] = None  # reads value head g % v_heads)
     chunk: Optional[int] = None       # keys are read only by the queries of their own chunk of this many positions
+    keep_first: int = 0               # under a window: the first so many positions stay readable
+
+    def for_reader(self, other: "PagedKVNeed") -> "PagedKVNeed":
+        """What the owner of a cache must keep when a layer with the need `other` reads it too."""
+        if (self.window, self.chunk) == (None, None) or (other.window, other.chunk) == (None, None):
+            return replace(self, window=None, chunk=None, keep_first=0)
+        keep = max(self.keep_first, other.keep_first)
+        if self.chunk is None and other.chunk is None:
+            return replace(self, window=max(self.window, other.window), keep_first=keep)
+        if self.chunk == other.chunk:
+            return self
+        return replace(self, window=None, chunk=None, keep_first=0)      # a window and chunks, or chunks of two sizes
 
 
 @dataclass(frozen=True)

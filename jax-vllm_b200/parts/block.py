@@ -254,14 +254,18 @@ register_block("branch_norm", BranchNormBlock)
 
 
 class ParallelBlock(Part):
-    """A layer whose two branches read ONE norm and are added together:
+    """A layer whose two branches read the same stream and are added together:
 
-        u = norm(h);   h <- h + (mixer(u) + feed_forward(u))          (the feed-forward is optional)
+        u = norm(h);   h <- h + (mixer(u) + feed_forward(u))                     one norm (`ffn_norm` None)
+        h <- h + (mixer(norm1(h)) + feed_forward(norm2(h)))                      two norms
 
-    Where both parts offer their products (`in_weight`, `from_projection`, `out_weight`) and agree in type, the
-    block runs two products a layer instead of four: u times the stacked input matrices [W_mixer_in; W_up], and
-    the two parts' activations side by side times the output matrices joined along k, [W_o | W_down], whose sum
-    over k IS mixer(u) + feed_forward(u).  The sum is handed on un-added, like every block's last branch."""
+    (the feed-forward is optional).  Where the parts offer their products and agree in type, the output products run as
+    one: the two parts' activations side by side times the output matrices joined along k, [W_o | W_down], whose sum
+    over k IS mixer + feed_forward.  With one norm the input products are one as well: u times the stacked matrices
+    [W_mixer_in; W_up] (`in_weight`, `from_projection`, `out_weight`).  With two norms the normed rows come from one pass
+    over the stream, which differ in the weight only, and the feed-forward makes its activation itself (`inner`); what it
+    adds beside the joint product (routed experts) is handed on with the product's result as an `ops.BranchSum`.  The sum
+    is handed on un-added, like every block's last branch."""
 
     def __init__(self, spec, prefix, ctx):
         p = spec.prefix
@@ -270,14 +274,17 @@ class ParallelBlock(Part):
         self.mixer = build(MIXERS, "mixer", spec.mixer, p, ctx)
         self.feed_forward = None if spec.feed_forward is None else \
             build(FEED_FORWARDS, "feed-forward", spec.feed_forward, p, ctx)
+        self.ffn_norm = None if spec.feed_forward is None or spec.ffn_norm is None else \
+            build(NORMS, "norm", spec.ffn_norm, p, ctx)
         if spec.cache_from is not None:
             if not hasattr(self.mixer, "writes_cache"):
                 raise ValueError(f"{p}: this mixer cannot read another layer's cache")
             self.mixer.writes_cache = False
         self.w_in = self.w_out = None
+        self.joint = self.one_pass = False
 
     def parts(self):
-        return tuple(part for part in (self.mixer_norm, self.mixer, self.feed_forward) if part is not None)
+        return tuple(part for part in (self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward) if part is not None)
 
     def tensor_specs(self):
         out = {}
@@ -290,25 +297,29 @@ class ParallelBlock(Part):
             part.bind(tensors)
         both = [part for part in (self.mixer, self.feed_forward) if part is not None]
         self.w_in = self.w_out = None
-        if all(hasattr(part, "from_projection") for part in both):
+        self.joint = False
+        if self.ffn_norm is None and all(hasattr(part, "from_projection") for part in both):
             ins, outs = [part.in_weight() for part in both], [part.out_weight() for part in both]
             if len({w.dtype for w in ins + outs}) == 1:
                 self.w_in = torch.cat(ins, dim=0).contiguous() if len(ins) > 1 else ins[0]
                 self.w_out = torch.cat(outs, dim=1).contiguous() if len(outs) > 1 else outs[0]
+        if self.ffn_norm is not None:
+            self.one_pass = hasattr(self.mixer_norm, "pairs_with") and self.mixer_norm.pairs_with(self.ffn_norm)
+            if hasattr(self.mixer, "from_projection") and hasattr(self.feed_forward, "inner"):
+                outs = [w for w in (self.mixer.out_weight(), self.feed_forward.out_weight()) if w is not None]
+                if len({w.dtype for w in outs}) == 1:
+                    self.joint = True
+                    self.w_out = torch.cat(outs, dim=1).contiguous() if len(outs) > 1 else outs[0]
 
     def forward(self, h, delta, step, cache):
         step.stream_copy = None
+        if self.ffn_norm is not None:
+            return self._two_norms(h, delta, step, cache)
         dt = self.ctx.dtype
         with trace_range("norm"):
             u = self.mixer_norm.norm(h, delta)
         if self.w_in is None:                       # parts without the packed interface: two branches, two sums
-            with trace_range("mixer"):
-                a = self.mixer.forward(u, step, cache)
-            if self.feed_forward is None:
-                return h, a
-            ops.residual_add(h, a)
-            with trace_range("feed_forward"):
-                return h, self.feed_forward.forward(u, step)
+            return self._two_branches(h, u, u, step, cache)
         with trace_range("in"):
             row = ops.linear(u, self.w_in, dt)
         rm, km = self.mixer.in_rows, self.mixer.heads_out
@@ -320,6 +331,35 @@ class ParallelBlock(Part):
                 self.feed_forward.from_projection(row[:, rm:], step, acts[:, km:])
         with trace_range("out"):
             return h, ops.linear(acts, self.w_out, dt, parts_ok=True)
+
+    def _two_branches(self, h, u, v, step, cache):
+        """The mixer on u and the feed-forward on v, each with products of its own."""
+        with trace_range("mixer"):
+            a = self.mixer.forward(u, step, cache)
+        if self.feed_forward is None:
+            return h, a
+        ops.residual_add(h, a)
+        with trace_range("feed_forward"):
+            return h, self.feed_forward.forward(v, step)
+
+    def _two_norms(self, h, delta, step, cache):
+        dt = self.ctx.dtype
+        with trace_range("norms"):
+            if self.one_pass:
+                u, v = self.mixer_norm.norm_pair(h, delta, self.ffn_norm)
+            else:
+                u, v = self.mixer_norm.norm(h, delta), self.ffn_norm.norm(h)
+        if not self.joint:
+            return self._two_branches(h, u, v, step, cache)
+        km = self.mixer.heads_out
+        acts = torch.empty((step.n_tokens, self.w_out.shape[1]), dtype=dt, device=u.device)
+        with trace_range("mixer"):
+            self.mixer.from_projection(ops.linear(u, self.mixer.in_weight(), dt), step, cache, acts[:, :km])
+        with trace_range("feed_forward"):
+            rest = self.feed_forward.inner(v, step, acts[:, km:])
+        with trace_range("out"):
+            y = ops.linear(acts, self.w_out, dt, parts_ok=True)
+        return h, (y if rest is None else ops.BranchSum(y, rest))
 
 
 register_block("parallel", ParallelBlock)

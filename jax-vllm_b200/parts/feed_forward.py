@@ -3,7 +3,8 @@
 the input once: in bfloat16 with an intermediate size that is a multiple of 128, as blocks of 128
 gate rows followed by the 128 up rows of the same indices, which lets the tcgen05 product of prompt
 steps apply the gate in its epilogue (the [tokens, 2*intermediate] product never reaches memory);
-otherwise all gate rows, then all up rows."""
+otherwise all gate rows, then all up rows.  An arrangement may join the down product with another part's
+(`out_weight`, `inner`)."""
 
 from __future__ import annotations
 
@@ -23,18 +24,22 @@ class GatedMLP(Part):
             raise ValueError(f"gated feed-forward: activation {spec.activation!r} is not built (silu is)")
         self.spec, self.ctx = spec, ctx
         self.prefix = f"{prefix}.{spec.prefix}" if spec.prefix else prefix
+        self.inner_size = spec.intermediate_size
         self.w_gate_up = self.w_down = self.block = None
 
+    def _names(self):
+        return tuple(f"{self.prefix}.{n}" for n in self.spec.names)
+
     def tensor_specs(self):
-        p, s = self.prefix, self.spec
-        return {f"{p}.gate_proj.weight": TensorSpec((s.intermediate_size, s.hidden_size)),
-                f"{p}.up_proj.weight": TensorSpec((s.intermediate_size, s.hidden_size)),
-                f"{p}.down_proj.weight": TensorSpec((s.hidden_size, s.intermediate_size))}
+        gate, up, down = self._names()
+        s = self.spec
+        return {gate: TensorSpec((s.intermediate_size, s.hidden_size)), up: TensorSpec((s.intermediate_size, s.hidden_size)),
+                down: TensorSpec((s.hidden_size, s.intermediate_size))}
 
     def bind(self, tensors):
-        p = self.prefix
-        g = self.compute_weight(tensors[f"{p}.gate_proj.weight"], self.ctx)
-        u = self.compute_weight(tensors[f"{p}.up_proj.weight"], self.ctx)
+        gate, up, down = self._names()
+        g = self.compute_weight(tensors[gate], self.ctx)
+        u = self.compute_weight(tensors[up], self.ctx)
         if g.dtype != u.dtype:
             g, u = g.float(), u.float()
         inter, hidden = g.shape
@@ -46,7 +51,7 @@ class GatedMLP(Part):
                                          dim=1).reshape(2 * inter, hidden).contiguous()
         else:
             self.w_gate_up = torch.cat([g, u], dim=0).contiguous()
-        self.w_down = self.compute_weight(tensors[f"{p}.down_proj.weight"], self.ctx).contiguous()
+        self.w_down = self.compute_weight(tensors[down], self.ctx).contiguous()
 
     # The gate is applied in the epilogue of the tcgen05 product once its 128 x 256 tiles are at least this many per
     # multiprocessor; with fewer, too many multiprocessors idle in the last round and the library product followed by
@@ -65,12 +70,24 @@ class GatedMLP(Part):
         tiles = -(-rows // 128) * -(-self.w_gate_up.shape[0] // 256)
         return tiles >= self.FUSED_GATE_TILES_PER_SM * ops.multiprocessors(self.w_gate_up.device)
 
+    def out_weight(self) -> torch.Tensor:
+        return self.w_down
+
+    def inner(self, x, step, out):
+        self._act(x, out)
+
+    def _act(self, x, out=None):
+        dt = self.ctx.dtype
+        wide = out is None or (out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)     # rows that the epilogue can write
+        if wide and self._fuse_gate(x.shape[0]):
+            return ops.gemm_tcgen05(x, self.w_gate_up, "swiglu", out=out)
+        # the parts of a sum are added four columns at a time
+        parts_ok = (self.block or self.spec.intermediate_size) % 4 == 0
+        return ops.swiglu(ops.linear(x, self.w_gate_up, dt, parts_ok=parts_ok), self.block, out_dtype=dt, out=out)
+
     def forward(self, x, step):
         dt = self.ctx.dtype
-        if self._fuse_gate(x.shape[0]):
-            act = ops.gemm_tcgen05(x, self.w_gate_up, "swiglu")
-        else:
-            act = ops.swiglu(ops.linear(x, self.w_gate_up, dt, parts_ok=True), self.block, out_dtype=dt)
+        act = self._act(x)
         # a few rows: the product may come as the parts of a sum, which the next norm adds as it reads them
         return ops.linear(act, self.w_down, dt, parts_ok=True)
 

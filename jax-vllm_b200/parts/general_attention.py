@@ -23,6 +23,10 @@ side, G * D elements) with a query that holds at key head c the mixture sum_{g o
 those queries once a token, and the attention kernels run H query heads on one key head of G * D elements under G value
 heads.  The cache holds what it would hold without the mixing.
 
+A layer that reads another layer's cache has queries (and a gate) of its own, and no projections of keys and values; its
+mask is its own too (the owner of the cache keeps what its readers see).  Under a window the first `keep_first` tokens of a
+sequence may stay visible.
+
 The part also offers its two products to an arrangement that packs them with another part's
 (`in_weight`, `from_projection`, `out_weight`): both then read the same normed input in one product and add
 their outputs in one product over the concatenated inputs.
@@ -81,22 +85,24 @@ class GeneralAttention(Part):
             if spec.position is not None else None
         if self.position is not None and self.position.dim > self.d:
             raise ValueError("rotary dim exceeds the key size")
-        self.writes_cache = True
         self.mask = ops.mask_code(spec.window, spec.chunk)
+        self.keep = int(spec.keep_first) if spec.window else 0
+        self.gain = 1.0 if self.position is None else getattr(self.position, "gain", 1.0)
         # heads prepared one by one (csrc/head_prepare.cu) where the layer asks for what only that kernel does
         interleaved = self.position is not None and getattr(self.position, "layout", "halves") == "interleaved"
         self.unit_heads = spec.head_norm_eps is not None and not spec.head_norm_weight
         self.talking = bool(spec.talk)
         self.by_head = (spec.head_norm_eps is not None or spec.value_norm_eps is not None or spec.rotate_values
-                        or interleaved or self.talking)
-        if self.talking and (spec.value_norm_eps is not None or spec.rotate_values or interleaved or spec.head_temperature
+                        or interleaved or self.gain != 1.0 or self.talking)
+        if self.talking and (spec.value_norm_eps is not None or spec.rotate_values or interleaved or self.gain != 1.0
+                             or self.keep or spec.head_temperature
                              or spec.distance_bias is not None or spec.weights != "softmax"
                              or (spec.head_norm_eps is not None and spec.head_norm_weight)):
             raise ValueError("scores mixed across heads are built for softmax weights, rotation in halves and heads normed "
                              "without a weight")
         if self.by_head and (spec.whole_norm_eps is not None or spec.query_temperature is not None
                              or spec.values_from_keys or spec.twin is not None):
-            raise ValueError("norms per head, normed or rotated values and interleaved pairs are built without a "
+            raise ValueError("norms per head, normed or rotated values, interleaved pairs and a rotation's gain are built without a "
                              "whole-projection norm, a query temperature, values taken from keys and two score maps")
         self.interleaved = interleaved
         self.value_freq = None
@@ -124,7 +130,7 @@ class GeneralAttention(Part):
         # the key row that the attention kernels see: with mixed scores the G key heads side by side, under one key head
         self.dk, self.nk = (self.hk * self.d, 1) if self.talking else (self.d, self.hk)
         plain = (spec.twin is None and spec.weights == "softmax" and not spec.score_cap and self.hv == self.hk
-                 and self.dv == self.d and not self.extras and not self.talking)
+                 and self.dv == self.d and not self.extras and not self.talking and not self.keep)
         self.plain = self.general = None
         if plain and ops.attn_mma_supports(ctx.dtype, self.d):
             self.plain = Attention(AttentionSpec(spec.hidden_size, self.hq, self.hk, self.d, spec.scale, prefix="",
@@ -133,10 +139,10 @@ class GeneralAttention(Part):
         elif ops.attn_general_mma_supports(ctx.dtype, self.dk, self.dv):
             self.general = ops.attn_general_mma_library(self.dk, self.dv)
             self.kernels += (self.general,)
-        # heads of 128 with sigmoid weights, or with a softmax that has a temperature per head, a bias by distance or a
-        # sink: prompt portions that fill a 128-row tile go to the tcgen05 kernel
-        self.big_tiles = (self.general is not None and not spec.score_cap and self.hv == self.hk and self.dv == self.d == 128
-                          and spec.twin is None and (spec.weights == "sigmoid") != bool(self.extras)
+        # heads of 128 with sigmoid weights, or with a softmax that has a cap, a temperature per head, a bias by distance, a
+        # sink or kept first tokens: prompt portions that fill a 128-row tile go to the tcgen05 kernel
+        self.big_tiles = (self.general is not None and self.hv == self.hk and self.dv == self.d == 128
+                          and spec.twin is None and not (spec.weights == "sigmoid" and (self.extras or spec.score_cap))
                           and self.out_scale == 1.0 and not self.talking)
         # scores mixed across heads: prompt portions on heads of 128 go to the tcgen05 kernel for whole key rows (of one key
         # head: to the ordinary one), portions of any length where no kernel with smaller tiles takes rows that long; single
@@ -152,13 +158,23 @@ class GeneralAttention(Part):
         self.w_in = self.w_o = self.q_norm = self.k_norm = self.bias = None
         self.head_scale = self.dist_bias = self.sink = self.talk = None
         self.lam = 0.0
+        self.heads_out = self.h * self.dv
+        self.writes_cache = True
+
+    @property
+    def writes_cache(self) -> bool:
+        """False for a layer that reads another layer's cache (set before the part is asked for its tensors)."""
+        return self._writes_cache
+
+    @writes_cache.setter
+    def writes_cache(self, value: bool) -> None:
+        self._writes_cache, s = bool(value), self.spec
         # columns of the packed projection
         self.k_off = self.hq * self.d
-        self.v_off = -1 if spec.values_from_keys else self.k_off + self.hk * self.d
-        self.g_off = self.k_off + self.hk * self.d + (0 if spec.values_from_keys else self.hv * self.dv)
-        self.g_rows = {None: 0, "head": self.h, "element": self.h * self.dv}[spec.gate]
+        self.v_off = -1 if s.values_from_keys else self.k_off + self.hk * self.d
+        self.g_off = self.k_off + (0 if not value else self.hk * self.d + (0 if s.values_from_keys else self.hv * self.dv))
+        self.g_rows = {None: 0, "head": self.h, "element": self.h * self.dv}[s.gate]
         self.in_rows = self.g_off + self.g_rows
-        self.heads_out = self.h * self.dv
 
     # -------------------------------------------------------------------- weights
     def _names(self):
@@ -167,19 +183,21 @@ class GeneralAttention(Part):
 
     def tensor_specs(self):
         n, s = self._names(), self.spec
-        specs = {n["q"]: TensorSpec((self.hq * self.d, s.hidden_size)),
-                 n["k"]: TensorSpec((self.hk * self.d, s.hidden_size)),
-                 n["o"]: TensorSpec((s.hidden_size, self.heads_out))}
-        if not s.values_from_keys:
+        specs = {n["q"]: TensorSpec((self.hq * self.d, s.hidden_size)), n["o"]: TensorSpec((s.hidden_size, self.heads_out))}
+        if self.writes_cache:
+            specs[n["k"]] = TensorSpec((self.hk * self.d, s.hidden_size))
+        if self.writes_cache and not s.values_from_keys:
             specs[n["v"]] = TensorSpec((self.hv * self.dv, s.hidden_size))
         if s.gate is not None:
             specs[n["g"]] = TensorSpec((self.g_rows, s.hidden_size))
         if s.whole_norm_eps is not None:
             specs[n["q_norm"]] = TensorSpec((self.hq * self.d,), kind="vector", init="ones_normal")
-            specs[n["k_norm"]] = TensorSpec((self.hk * self.d,), kind="vector", init="ones_normal")
+            if self.writes_cache:
+                specs[n["k_norm"]] = TensorSpec((self.hk * self.d,), kind="vector", init="ones_normal")
         if s.head_norm_eps is not None and s.head_norm_weight:
             specs[n["q_norm"]] = TensorSpec((self.d,), kind="vector", init="ones_normal")
-            specs[n["k_norm"]] = TensorSpec((self.d,), kind="vector", init="ones_normal")
+            if self.writes_cache:
+                specs[n["k_norm"]] = TensorSpec((self.d,), kind="vector", init="ones_normal")
         if s.score_bias:
             specs[n["bias"]] = TensorSpec((self.h,), kind="vector", init="normal")
         if s.twin is not None:
@@ -204,8 +222,10 @@ class GeneralAttention(Part):
 
     def bind(self, tensors):
         n, s = self._names(), self.spec
-        mats = [self._maps_first(tensors[n["q"]], self.h), self._maps_first(tensors[n["k"]], self.g)]
-        if not s.values_from_keys:
+        mats = [self._maps_first(tensors[n["q"]], self.h)]
+        if self.writes_cache:
+            mats.append(self._maps_first(tensors[n["k"]], self.g))
+        if self.writes_cache and not s.values_from_keys:
             mats.append(tensors[n["v"]])
         if s.gate is not None:
             mats.append(tensors[n["g"]])
@@ -215,8 +235,9 @@ class GeneralAttention(Part):
         self.w_in = torch.cat(mats, dim=0).contiguous()
         self.w_o = self.compute_weight(tensors[n["o"]], self.ctx).contiguous()
         if s.whole_norm_eps is not None or (s.head_norm_eps is not None and s.head_norm_weight):
-            self.q_norm, self.k_norm = tensors[n["q_norm"]].contiguous(), tensors[n["k_norm"]].contiguous()
-            if self.q_norm.dtype != self.k_norm.dtype:
+            self.q_norm = tensors[n["q_norm"]].contiguous()
+            self.k_norm = tensors[n["k_norm"]].contiguous() if self.writes_cache else None
+            if self.k_norm is not None and self.q_norm.dtype != self.k_norm.dtype:
                 self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
         if s.score_bias:
             self.bias = tensors[n["bias"]].to(torch.float32).contiguous()
@@ -241,8 +262,9 @@ class GeneralAttention(Part):
     def cache_need(self):
         s = self.spec
         if self.hv == self.hk and self.dv == self.d:
-            return PagedKVNeed(self.hk, self.d, s.window or None, chunk=s.chunk or None)
-        return PagedKVNeed(self.hk, self.d, s.window or None, v_heads=self.hv, v_head_dim=self.dv, chunk=s.chunk or None)
+            return PagedKVNeed(self.hk, self.d, s.window or None, chunk=s.chunk or None, keep_first=self.keep)
+        return PagedKVNeed(self.hk, self.d, s.window or None, v_heads=self.hv, v_head_dim=self.dv, chunk=s.chunk or None,
+                           keep_first=self.keep)
 
     def tile_classes(self, page_size: int):
         if self.plain is not None:
@@ -302,7 +324,7 @@ class GeneralAttention(Part):
                              self.interleaved, self.q_norm, self.k_norm, s.head_norm_eps or s.value_norm_eps or 0.0,
                              s.value_norm_eps is not None, self.value_freq, cache.k if writes else None,
                              cache.v if writes else None, self.hq, self.hk, self.hv, self.d, self.dv,
-                             unit_heads=self.unit_heads)
+                             unit_heads=self.unit_heads, gain=self.gain)
         else:
             ops.attn_prepare(row, 0, self.k_off, self.v_off, q, step.positions, step.token_entry, table, freq,
                              self.q_norm, self.k_norm, s.whole_norm_eps or 0.0, coef, every, cache.k if writes else None,
@@ -334,7 +356,7 @@ class GeneralAttention(Part):
             return self.plain.attend(q, a, step, cache, table)
         keys = cache.k.view(*cache.k.shape[:2], self.nk, self.dk) if self.talking else cache.k
         common = (keys, cache.v, table, step.cu_seqlens, step.start_pos)
-        extra = dict(score_cap=s.score_cap or 0.0, sigmoid=s.weights == "sigmoid", bias=self.bias)
+        extra = dict(score_cap=s.score_cap or 0.0, sigmoid=s.weights == "sigmoid", bias=self.bias, keep=self.keep)
         if self.extras:
             extra.update(head_scale=self.head_scale, dist_bias=self.dist_bias, sink=self.sink, out_scale=self.out_scale)
         if self.general is not None:
@@ -353,7 +375,8 @@ class GeneralAttention(Part):
             elif n_work and big:                           # 128-row tiles
                 ops.attn_tcgen05(q, q.stride(0), a, cache.k, cache.v, *common[2:], work, n_work, self.hq, self.hk, self.d,
                                  s.scale, sigmoid=s.weights == "sigmoid", bias=self.bias, head_scale=self.head_scale,
-                                 dist_bias=self.dist_bias, sink=self.sink, window=self.mask, out_scale=self.out_scale)
+                                 dist_bias=self.dist_bias, sink=self.sink, window=self.mask, out_scale=self.out_scale,
+                                 keep=self.keep, score_cap=s.score_cap or 0.0)
             elif n_work:
                 kernel(work, n_work)
         dwork, n_dec = step.decode_work
@@ -361,8 +384,10 @@ class GeneralAttention(Part):
             ops.attn_rows_decode(q, q.stride(0), a, *common, dwork, n_dec, self.hq, s.scale, step.max_seq_len,
                                  sink=self.sink, out_scale=self.out_scale)
         elif n_dec:
+            # the splits share what a query sees: at most its window with the kept tokens, or its chunk
             split = self.ctx.decode_split_size
-            kernel(dwork, n_dec, split_size=split, n_splits=max(1, -(-step.max_seq_len // split)))
+            most = s.window + self.keep if s.window else s.chunk or step.max_seq_len
+            kernel(dwork, n_dec, split_size=split, n_splits=max(1, -(-min(step.max_seq_len, most) // split)))
 
 
 register_mixer("general_attention", GeneralAttention)

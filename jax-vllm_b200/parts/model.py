@@ -7,7 +7,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .base import BuildContext, Part, TensorSpec
+from .base import BuildContext, PagedKVNeed, Part, TensorSpec
 from .block import build_block
 from .registry import NORMS, build
 
@@ -95,12 +95,18 @@ class Model(Part):
     # ---------------------------------------------------------------------- cache
     def cache_needs(self):
         """Per place in the run order: what the layer there needs to keep, or None (nothing, or
-        it reads another place's cache)."""
+        it reads another place's cache).  Pages are kept for every layer that reads them: the widest of the masks of the
+        owner and its readers."""
         def need(block):          # an arrangement that keeps something of its own says so; else it is the mixer's
             f = getattr(block, "cache_need", None)
             return f() if f is not None else block.mixer.cache_need()
 
-        return [need(self.layers[i]) if self.place_cache[k] == k else None for k, i in enumerate(self.order)]
+        needs = [need(self.layers[i]) if self.place_cache[k] == k else None for k, i in enumerate(self.order)]
+        for k, i in enumerate(self.order):
+            owner = self.place_cache[k]
+            if owner != k and isinstance(needs[owner], PagedKVNeed):
+                needs[owner] = needs[owner].for_reader(self.layers[i].mixer.cache_need())
+        return needs
 
     def tile_classes(self, page_size: int):
         """The attention work lists that the mixers of this model want (see BatchBuilder)."""
@@ -117,7 +123,7 @@ class Model(Part):
         if given, is called after every place of the run order with a copy of the stream as that layer leaves
         it (for comparing a model layer by layer; it costs a pass over the stream per layer)."""
         with ops.trace_range("embedding"):
-            h = ops.embed_gather(self.embedding, step.token_ids)
+            h = ops.embed_gather(self.embedding, step.token_ids, scale=self.spec.embedding_scale)
             if self.position_table is not None:      # a learned vector per position (a position beyond the table sets the
                 ops.embed_gather(self.position_table, step.positions, out=h, accumulate=True)   # status word)
         delta = None
@@ -129,7 +135,7 @@ class Model(Part):
                     ops.residual_add(h, delta)
                     delta = None
                 step.stream_copy = None
-                ops.embed_gather(self.embedding, step.token_ids, out=h, accumulate=True)
+                ops.embed_gather(self.embedding, step.token_ids, out=h, accumulate=True, scale=self.spec.embedding_scale)
             if k in self.pass_rows:
                 if delta is not None:
                     ops.residual_add(h, delta)

@@ -32,6 +32,14 @@ class RMSNorm(Part):
         by default; float32 for a reader that goes on in 32-bit)."""
         return ops.rmsnorm(h, self.weight, self.eps, out_dtype or self.ctx.dtype, delta=delta)
 
+    def norm_pair(self, h, delta, other):
+        """(norm(h + delta), other(h + delta)) in one pass, `other` a norm of this kind with the same eps; h is updated in
+        place with the sum."""
+        return ops.rmsnorm(h, self.weight, self.eps, self.ctx.dtype, delta=delta, weight2=other.weight)
+
+    def pairs_with(self, other) -> bool:
+        return isinstance(other, RMSNorm) and other.eps == self.eps and other.weight.dtype == self.weight.dtype
+
     def gather(self, h, delta, rows):
         """x[i] = norm(h[rows[i]] + delta[rows[i]]); h is left as it is."""
         return ops.rmsnorm(h, self.weight, self.eps, self.ctx.dtype, delta=delta, rows=rows)

@@ -4,8 +4,11 @@
                     terms read the old S; u the unit key; w a decay and a a removal rate per key channel)
     matrix_memory   S <- keep S + take k v^T, n <- keep n + take k, o = S^T q / (max(|n . q|, exp(-m)) + 1e-6)
                     with keep, take from a forget and an input gate in the log domain under a running maximum m
+    gated_linear_attention   S <- diag(a) S + k v^T,  o = S^T q            a = sigmoid(z)^(1/tau) per key channel, z from
+                    a low-rank pair of matrices (the second product is part of the preparation, in 32-bit)
 
-Both then divide each head's o by its root mean square, multiply by a weight and by sigmoid(W_g x), and project.
+All then divide each head's o by its root mean square, multiply by a weight and by a gate (sigmoid(W_g x), or silu for
+the linear attention), and project.
 The state is float32 and lives in the request's state slot (`FixedStateNeed`): a portion of a prompt starts from what
 the portion before left, a decoded token is a portion of one.  Everything that enters the recurrence besides the
 projections is formed in 32-bit by the prepare kernels.  The parts offer their products to an arrangement that packs
@@ -147,3 +150,54 @@ class MatrixMemory(_StateMixer):
 
 
 register_mixer("matrix_memory", MatrixMemory)
+
+
+class GatedLinearAttention(_StateMixer):
+    def __init__(self, spec, prefix, ctx):
+        self.spec, self.ctx = spec, ctx
+        self.prefix = f"{prefix}.{spec.prefix}" if spec.prefix else prefix
+        self.h, self.d, self.dv = int(spec.num_heads), int(spec.key_dim), int(spec.value_dim)
+        if self.h < 1 or not 1 <= self.d <= ops.SCAN_MAX_KEY or self.dv < 1:
+            raise ValueError(f"gated linear attention: keys of {self.d} are not built (1 .. {ops.SCAN_MAX_KEY})")
+        if not spec.tau > 0:
+            raise ValueError("gated linear attention: tau must be positive")
+        keys = ("q", "k", "v", "g", "a1", "a2", "a2_b", "norm", "o")
+        self.names = {k: f"{self.prefix}.{n}" for k, n in zip(keys, spec.names)}
+        self.hd, self.hv = self.h * self.d, self.h * self.dv
+        self.heads_out = self.hv
+        self.rank = self.in_rows = None               # known when the weights are bound
+        self.w_in = self.w_o = self.w_up = self.bias = self.norm = None
+
+    def tensor_specs(self):
+        n, W = self.names, self.spec.hidden_size
+        return {n["q"]: TensorSpec((self.hd, W)), n["k"]: TensorSpec((self.hd, W)), n["v"]: TensorSpec((self.hv, W)),
+                n["g"]: TensorSpec((self.hv, W)), n["a1"]: TensorSpec((-1, W)), n["a2"]: TensorSpec((self.hd, -1)),
+                n["a2_b"]: TensorSpec((self.hd,), kind="vector", init="normal"),
+                n["norm"]: TensorSpec((self.dv,), kind="vector", init="ones_normal"), n["o"]: TensorSpec((W, self.hv))}
+
+    def bind(self, tensors):
+        n = self.names
+        self.rank = int(tensors[n["a1"]].shape[0])
+        if tensors[n["a2"]].shape[1] != self.rank:
+            raise ValueError(f"{self.prefix}: the decay's two matrices differ in rank")
+        self.in_rows = 2 * self.hd + 2 * self.hv + self.rank
+        self._bind_in(tensors, ("q", "k", "v", "g", "a1"))
+        self.w_up = tensors[n["a2"]].contiguous()
+        self.bias = tensors[n["a2_b"]].contiguous()
+        if self.w_up.dtype != self.bias.dtype:
+            self.w_up, self.bias = self.w_up.float(), self.bias.float()
+        self.norm = tensors[n["norm"]].contiguous()
+
+    def cache_need(self):
+        return FixedStateNeed((self.hd * self.dv,), torch.float32)
+
+    def from_projection(self, row, step, cache, out):
+        hd, hv = self.hd, self.hv
+        packed = ops.gla_prepare(row, 0, hd, 2 * hd + 2 * hv, self.w_up, self.bias, self.spec.tau, self.spec.q_scale, self.h,
+                                 self.d)
+        o = ops.state_scan(packed, row, 2 * hd, cache.state, step.cu_seqlens, step.state_slots, step.n_entries, self.dv)
+        return ops.head_norm_gate(o, self.norm, row[:, 2 * hd + hv:2 * hd + 2 * hv], out, self.h, self.dv, self.spec.norm_eps,
+                                  gate_act="silu")
+
+
+register_mixer("gated_linear_attention", GatedLinearAttention)

@@ -66,6 +66,9 @@ def _register_builtin() -> None:
     from .models.tidarax import ARCHITECTURE as TIDARAX, TidaraxConfig
 
     register_architecture(TIDARAX, TidaraxConfig)
+    from .models.nasedra import ARCHITECTURE as NASEDRA, NasedraConfig
+
+    register_architecture(NASEDRA, NasedraConfig)
 
 
 _register_builtin()
