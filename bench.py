@@ -696,6 +696,8 @@ def design(name: str, layers, sizes, steps, warmup) -> int:
         return design_gogivik(layers or 3, sizes, steps, warmup)
     if name == "tidarax":
         return design_tidarax(layers or 2, sizes, steps, warmup)
+    if name == "nasedra":
+        return design_nasedra(layers or 4, sizes, steps, warmup)
     if name != "guronex":
         print(f"bench.py: no design {name!r}")
         return 2
@@ -1256,6 +1258,186 @@ def design_tidarax(layers, sizes, steps, warmup) -> int:
     return 0
 
 
+# ------------------------------------------------------------------ the Nasedra design beside Nufapel, Gogivik and Loselix
+# Layer sizes for `--design nasedra`: four layers (gated linear attention over a dense feed-forward; capped attention under
+# a window that keeps the first tokens, over routed experts with identity experts and a shared one; linear attention over
+# the same; attention that reads the second layer's keys, dense), beside Nufapel's layers (attention beside a matrix memory
+# of the same heads as the linear attention, dense and routed), Gogivik's chunked attention (chunks as long as the window)
+# and Loselix softmax attention, all of equal width, heads and dense feed-forward.  "w2k": the width of a 1B-class model;
+# "w4k": an 8B-class width; "small": heads of 64.
+NASEDRA_SIZES = {
+    "w2k": dict(width=2048, heads=16, kv=4, dim=128, vdim=128, window=1024, keep=4, mem=(8, 128, 256), ff=5632, experts=32,
+                identity=4, top=4, eff=1024, shared=1024),
+    "w4k": dict(width=4096, heads=32, kv=8, dim=128, vdim=128, window=1024, keep=4, mem=(8, 256, 512), ff=11008, experts=32,
+                identity=4, top=4, eff=2048, shared=2048),
+    "small": dict(width=1024, heads=16, kv=4, dim=64, vdim=64, window=512, keep=4, mem=(4, 64, 128), ff=2816, experts=16,
+                  identity=2, top=2, eff=1024, shared=512),
+}
+NASEDRA_KINDS = ("gla_dense", "attention_moe", "gla_moe", "reader_dense")
+
+
+def nasedra_configs(z, layers, vocab=32000):
+    copy = lambda x: json.loads(json.dumps(x))
+    mh, md, mv = z["mem"]
+    rot = {"base": 5e5, "dims": z["dim"], "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}
+    attention = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5, "rot": rot,
+                 "mask": {"size": z["window"], "keep_first": z["keep"]}, "softcap": 30.0}
+    linear = {"heads": mh, "dim": md, "vdim": mv, "tau": 16.0}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"]}, "shared": {"ff": z["shared"]},
+           "router": {"experts": z["experts"], "identity": z["identity"], "top": z["top"], "scale": 2.0}}
+    four = [{"type": "gla", "mixer": linear, "mlp": dense}, {"type": "attention", "mixer": attention, "mlp": moe},
+            {"type": "gla", "mixer": linear, "mlp": moe}, {"type": "attention", "mixer": dict(attention, kv_from=1), "mlp": dense}]
+    nasedra = {"architecture": "Nasedra", "embedding": {"scale": 1.0}, "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-5},
+               "layers": [copy(four[i % 4]) for i in range(layers)]}
+    nz = dict(z, delta=(1, 8), rank=8, buckets=32, bias_max=1024, groups=(4, 2))
+    nufapel, loselix = nufapel_configs(nz, 3, vocab)
+    pairs = (nufapel["layers"][0], nufapel["layers"][2])
+    nufapel = dict(nufapel, layers=[copy(pairs[i % 2]) for i in range(layers)])
+    loselix = dict(loselix, layers=[copy(loselix["layers"][0]) for _ in range(layers)])
+    gz = dict(z, chunk=z["window"], ssm=(4, 8, 8, 1), lat=(2, 8, 8, 8, 16, 16))
+    gogivik, _ = gogivik_configs(gz, 1, vocab)
+    return nasedra, nufapel, gogivik, loselix
+
+
+def nasedra_parts(model, z, layer_index, batch, tokens, reps, pk, sm_mhz):
+    """Layer `layer_index` of a Nasedra model in parts, each alone: the two norms, the attention kernel with the preparation
+    of its heads and its gate, or the recurrence whole (from the projected row to the gated heads) and its three kernels;
+    the whole mixer, the whole feed-forward, and the whole layer as the block runs it (two norms, joint output product).
+    One prompt of `tokens` tokens, then one decode step of `batch` requests at CONTEXT tokens.  Rooflines as for the other
+    designs: pairs and cache rows are those that the window and the kept tokens let a query see."""
+    import torch
+    from jax_vllm_b200 import make_driver, ops
+    from jax_vllm_b200.engine import StepEntry
+    W = z["width"]
+    flush = torch.zeros(160 << 20, dtype=torch.int16, device="cuda")
+    layer = model.layers[layer_index]
+    mixer, ff = layer.mixer, layer.feed_forward
+    out = {}
+    seen = lambda pos: min(pos + 1, z["window"] + z["keep"]) if pos >= z["window"] + z["keep"] else pos + 1
+    for phase in ("prefill", "decode"):
+        if phase == "prefill":
+            driver = make_driver(model, max_num_seqs=1, max_model_len=tokens + 16, block_size=PAGE, prefix_cache=False,
+                                 max_tokens_per_step=tokens, cuda_graphs=False)
+            rc = driver.cache.admit("p")
+            driver.cache.grow(rc, tokens)
+            entries = [StepEntry(rc, [(i * 7919 + 13) % 1000 for i in range(tokens)], (tokens - 1,))]
+            n, seqs, positions, keys = tokens, 1, range(tokens), tokens
+        else:
+            driver = make_driver(model, max_num_seqs=batch, max_model_len=CONTEXT + 64, block_size=PAGE, prefix_cache=False,
+                                 cuda_graphs=False)
+            rcs = fake_context(driver, batch, CONTEXT)
+            for rc in rcs:
+                driver.cache.grow(rc, rc.num_tokens + 1)
+            entries = [StepEntry(rc, [b], (0,)) for b, rc in enumerate(rcs)]
+            n, seqs, positions, keys = batch, batch, [CONTEXT] * batch, batch * seen(CONTEXT)
+        step = driver.runner.builder.build(entries)
+        cache = driver.runner.layer_caches[model.place_cache[layer_index]]
+        h = torch.randn((n, W), device="cuda")
+        delta = (torch.randn((n, W), device="cuda") * 0.1).to(torch.bfloat16)
+        x = (torch.randn((n, W), device="cuda") * 0.5).to(torch.bfloat16)
+        row = (torch.randn((n, mixer.in_rows), device="cuda") * 0.5).to(torch.bfloat16)
+        heads = torch.empty((n, mixer.heads_out), dtype=torch.bfloat16, device="cuda")
+        bw, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+        jobs = [("two norms", lambda: layer.mixer_norm.norm_pair(h, delta, layer.ffn_norm), (0.0, n * W * 14 / bw * 1e6, "flops"))]
+        if hasattr(mixer, "attend"):
+            pairs = sum(seen(p) for p in positions)
+            table = step.block_tables[cache.group]
+            q = torch.randn((n, mixer.hq * mixer.d), device="cuda").to(torch.bfloat16)
+            a = torch.empty((n, mixer.hq * mixer.dv), dtype=torch.bfloat16, device="cuda")
+            own = (cache.k, cache.v) if mixer.writes_cache else (None, None)
+            prep = lambda: ops.head_prepare(row, 0, mixer.k_off, mixer.v_off, q, step.positions, step.token_entry, table,
+                                            mixer.position.table(), True, None, None, 0.0, False, None, *own, mixer.hq, mixer.hk,
+                                            mixer.hv, mixer.d, mixer.dv, gain=mixer.gain)
+            flops = 2 * mixer.hq * (mixer.d + mixer.dv) * pairs
+            nbytes = keys * (mixer.hk * mixer.d + mixer.hv * mixer.dv) * 2 + n * mixer.hq * (mixer.d + mixer.dv) * 2
+            jobs += [("attention kernel", lambda: mixer.attend(q, a, step, cache, table), (flops / tf * 1e6, nbytes / bw * 1e6, "flops")),
+                     ("head preparation", prep, (0.0, n * mixer.g_off * 4 / bw * 1e6, "flops")),
+                     ("output gate", lambda: ops.attn_finish(a, heads, mixer.h, mixer.dv, gate=row[:, mixer.g_off:]),
+                      (0.0, n * mixer.heads_out * 6 / bw * 1e6, "flops"))]
+        else:
+            H, d, v = mixer.h, mixer.d, mixer.dv
+            hd, hv = mixer.hd, mixer.hv
+            fma = n * H * d * v * 3                                                # decay, write, read
+            nbytes = seqs * 2 * H * d * v * 4 + n * mixer.in_rows * 2 + n * mixer.heads_out * 2
+            roof = (fma / (FP32_LANES * sm_mhz * 1e6) * 1e6, nbytes / bw * 1e6, "fp32 lanes")
+            packed = ops.gla_prepare(row, 0, hd, 2 * hd + 2 * hv, mixer.w_up, mixer.bias, mixer.spec.tau, mixer.spec.q_scale, H, d)
+            o = torch.randn((n, hv), device="cuda")
+            jobs += [("recurrence", lambda: mixer.from_projection(row, step, cache, heads), roof),
+                     ("decay preparation", lambda: ops.gla_prepare(row, 0, hd, 2 * hd + 2 * hv, mixer.w_up, mixer.bias, mixer.spec.tau,
+                                                                   mixer.spec.q_scale, H, d), (0.0, n * hd * 16 / bw * 1e6, "flops")),
+                     ("state scan", lambda: ops.state_scan(packed, row, 2 * hd, cache.state, step.cu_seqlens, step.state_slots,
+                                                           step.n_entries, v), roof),
+                     ("gated norm", lambda: ops.head_norm_gate(o, mixer.norm, row[:, 2 * hd + hv:2 * hd + 2 * hv], heads, H, v, 1e-5,
+                                                               gate_act="silu"), (0.0, n * hv * 8 / bw * 1e6, "flops"))]
+        jobs.append(("mixer", lambda: mixer.forward(x, step, cache), None))
+        if NASEDRA_KINDS[layer_index % 4].endswith("dense"):
+            ff_flops, ff_bytes = 2 * n * 3 * z["ff"] * W, 3 * z["ff"] * W * 2
+        else:
+            # a choice falls on an expert with tensors as often as the random router says: on all alike
+            E, total = z["experts"], z["experts"] + z["identity"]
+            hit = E * (1 - (1 - z["top"] / total) ** n)
+            ff_flops = 2 * n * 3 * W * (z["top"] * E / total * z["eff"] + z["shared"])
+            ff_bytes = (hit * 3 * z["eff"] + 3 * z["shared"]) * W * 2
+        jobs.append(("feed-forward", lambda: ff.forward(x, step), (ff_flops / tf * 1e6, ff_bytes / bw * 1e6, "flops")))
+        jobs.append(("layer", lambda: layer.forward(h, delta, step, cache), None))
+        res = {}
+        for name, fn, roof in jobs:
+            us = time_part(fn, reps, flush)
+            res[name] = {"us": round(us, 1)}
+            if roof is not None:
+                t_math, t_bytes, unit = roof
+                ideal = max(t_math, t_bytes)
+                res[name].update(roofline_us=round(ideal, 1), bound=unit if t_math >= t_bytes else "bytes",
+                                 of_roofline=round(ideal / us, 3))
+        driver.runner.check_kernels()
+        out[phase] = res
+        del driver
+        torch.cuda.empty_cache()
+    return out
+
+
+def design_nasedra(layers, sizes, steps, warmup) -> int:
+    import torch
+    from jax_vllm_b200 import random_model, registry
+    pk, pk_src = peaks()
+    sizes = [t for t in sizes if t in NASEDRA_SIZES] or ["w2k", "w4k"]
+    out = {"design": "nasedra", "layers": layers, "prefill_tokens": PREFILL_TOKENS, "decode_batch": 8, "context": CONTEXT,
+           "dtype": "bf16", "data": "synthetic (random weights, seed 5)", "peaks": pk, "peak_source": pk_src, "sizes": {}}
+    for tag in sizes:
+        z = NASEDRA_SIZES[tag]
+        row = {}
+        for kind, cfg in zip(("nasedra", "nufapel", "gogivik", "loselix"), nasedra_configs(z, layers)):
+            model = random_model(registry.config_from_dict(cfg), seed=5, dtype="bf16", device="cuda:0")
+            row[kind], mhz = {}, 1965.0
+            if kind != "gogivik":                         # one layer beside the others': its parts only
+                with ClockSampler() as clocks:
+                    pms = time_prefill(model, PREFILL_TOKENS, warmup=2, reps=5)
+                    dms, launches, _, _ = time_decode(model, 8, steps, warmup)
+                row[kind] = dict(prefill_tok_s=round(PREFILL_TOKENS / (pms / 1e3), 1), prefill_ms=round(pms, 3),
+                                 decode_tok_s=round(8 / (dms / 1e3), 1), decode_ms_per_step=round(dms, 4),
+                                 decode_launches_per_step=launches, clocks=clocks.summary)
+                mhz = float(clocks.summary.get("sm_max_mhz") or 1965.0)
+            if kind == "loselix":
+                row[kind]["parts"] = design_parts(model, kind, dict(z, soft=(z["dim"], z["vdim"], z["dim"] // 2)), 0, 8,
+                                                  PREFILL_TOKENS, 7, pk)
+            elif kind == "gogivik":
+                row[kind]["parts"] = gogivik_parts(model, z, 0, 8, PREFILL_TOKENS, 7, pk, mhz)
+            elif kind == "nufapel":
+                # the parts' code tells dense from routed feed-forwards by the layer's number (0: dense, else routed)
+                row[kind]["parts"] = {TIDARAX_KINDS[i]: nufapel_parts(model, z, i, 8, PREFILL_TOKENS, 7, pk, mhz)
+                                      for i in range(min(2, layers))}
+            else:
+                row[kind]["config"] = dict(z)
+                row[kind]["parts"] = {NASEDRA_KINDS[i]: nasedra_parts(model, z, i, 8, PREFILL_TOKENS, 7, pk, mhz)
+                                      for i in range(min(4, layers))}
+            del model
+            torch.cuda.empty_cache()
+        out["sizes"][tag] = row
+    print(json.dumps(out))
+    return 0
+
+
 def reference_arm():
     why = ("the reference (jllm) needs jax, jaxlib and equinox and the hatchling build backend; none is installed "
            "and none is in the offline wheelhouse, so it can neither be installed nor run here")
@@ -1282,13 +1464,13 @@ def main():
     ap.add_argument("--with-workloads", action="store_true",
                     help="after the headline run, also run the two serving workloads and add their lines under `workloads`")
     ap.add_argument("--design", default=None, metavar="NAME",
-                    help="guronex, loselix, nufapel, gogivik or tidarax: that design's prefill and decode throughput at a few layer sizes "
+                    help="guronex, loselix, nufapel, gogivik, tidarax or nasedra: that design's prefill and decode throughput at a few layer sizes "
                          "beside its closest neighbours of equal size (Qwen3; later designs beside earlier ones), with the rooflines of "
                          "its kernels (see design())")
     ap.add_argument("--sizes", default="lite,mid,row576",
                     help="with --design: which of its layer sizes, comma-separated (guronex: lite,mid,row576; loselix: "
                          "w2k,w4k,mix, all by default; nufapel and gogivik: w2k,w4k,small, the first two by default; tidarax: w2k,w4k,w4k8,small, the "
-                         "first three by default)")
+                         "first three by default; nasedra: w2k,w4k,small, the first two by default)")
     ap.add_argument("--micro-eager", action="store_true",
                     help="with --micro: plain launches instead of replays of a CUDA graph (for a profiler)")
     args = ap.parse_args()
