@@ -57,7 +57,7 @@ struct Params {
   const float* head_scale; const float* dist_bias; int n_dist; const float* sink;
   int window;                  // the mask as one number (common.cuh, first_visible): 0, a window (> 0) or chunks (< 0)
   int keep;                    // positions below this one stay visible under a window
-  float score_cap_log2;        // > 0: the scaled score s (bias and head scale included) becomes cap * tanh(s / cap); times log2 e
+  float score_cap_log2;        // > 0: the scaled score s (bias and head scale included) becomes cap * tanh(s / cap); cap * log2 e
   float out_scale;             // multiplies the output
   int* status;
 };
@@ -72,6 +72,41 @@ struct Shared {
   int armed_q[Q_BUFFERS], armed_k[K_STAGES], armed_v[V_STAGES];   // parity of the phase a producer armed last; -1: never
   float xch[2][128];            // a row's two softmax threads exchange their maxima (and at the end their sums)
 };
+
+// x <- tanh(x) for a thread's 64 scores.  Where no score of the warp exceeds 0.75 in size, by x + x^3 q(x^2), q of degree 4,
+// the least largest relative error over that range among such polynomials (1.1e-7 in 32-bit; fitted for this kernel by
+// iteratively reweighted least squares), in packed pairs: the exponentials of the softmax are this role's scarce unit.
+// Elsewhere 1 - 2 / (1 + e^(2x)).
+__device__ __forceinline__ void tanh_scores(uint32_t (&sr)[2][32]) {
+  float size = 0.f;
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
+#pragma unroll
+    for (int i = 0; i < 32; i += 2)
+      size = max3(size, fabsf(__uint_as_float(sr[c][i])), fabsf(__uint_as_float(sr[c][i + 1])));
+  if (__all_sync(0xffffffffu, size <= 0.75f)) {
+    const uint64_t q0 = pack2(-0.333330691f, -0.333330691f), q1 = pack2(0.133265212f, 0.133265212f);
+    const uint64_t q2 = pack2(-0.0533902571f, -0.0533902571f), q3 = pack2(0.0196649097f, 0.0196649097f);
+    const uint64_t q4 = pack2(-0.00476948777f, -0.00476948777f);
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+      for (int i = 0; i < 32; i += 2) {
+        const uint64_t x = pack2(__uint_as_float(sr[c][i]), __uint_as_float(sr[c][i + 1]));
+        const uint64_t u = mul2(x, x);
+        const uint64_t q = fma2(fma2(fma2(fma2(q4, u, q3), u, q2), u, q1), u, q0);
+        float v0, v1;
+        unpack2(fma2(mul2(x, u), q, x), v0, v1);
+        sr[c][i] = __float_as_uint(v0); sr[c][i + 1] = __float_as_uint(v1);
+      }
+    return;
+  }
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      sr[c][i] = __float_as_uint(fmaf(-2.f, fast_rcp(1.f + fast_exp2(__uint_as_float(sr[c][i]) * (2.f * LOG2E))), 1.f));
+}
 
 // One work item as every role sees it.
 struct Item {
@@ -332,13 +367,13 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
       // With a head's own scale or a bias by distance the scores are first brought to the exponent's unit, s * scale *
       // head_scale * log2(e) + bias * log2(e), and the maximum, the reference and the exponentials work on that (`sc`,
       // what still multiplies a score in the exponent, is then 1).  The same for every thread of the block.
-      // So they are with a cap: cap * tanh(x / cap) * log2(e) = c - 2 c / (1 + 2^(2 y / cap)), c = cap * log2(e), y = x * log2(e).
+      // With a cap they become tanh(s / cap), and `sc` is the cap in the exponent's unit.
       const bool capped = p.score_cap_log2 > 0.f;
       const bool shaped = p.head_scale != nullptr || p.dist_bias != nullptr || capped;
-      const float cap_exp = capped ? 2.f * LOG2E / p.score_cap_log2 : 0.f, cap2 = -2.f * p.score_cap_log2;
       const int head = it.kv_head * G + min(hh, G - 1);
-      const float sc = shaped ? 1.f : p.scale_log2;
-      const float row_scale = p.scale_log2 * (p.head_scale != nullptr ? p.head_scale[head] : 1.f);
+      const float sc = capped ? p.score_cap_log2 : shaped ? 1.f : p.scale_log2;
+      const float unit = capped ? 1.f / p.score_cap_log2 : 1.f;
+      const float row_scale = p.scale_log2 * (p.head_scale != nullptr ? p.head_scale[head] : 1.f) * unit, bias_unit = LOG2E * unit;
       const float* dist_row = p.dist_bias != nullptr ? p.dist_bias + (size_t)head * p.n_dist : nullptr;
       // m_ref is the reference maximum that the exponentials are taken against.  It follows the true
       // maximum lazily: only when the maximum has grown by more than 2^8 (in the exponent) is O rescaled,
@@ -360,7 +395,17 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
           tmem_ld32_issue(s_addr, sr[0]);
           tmem_ld32_issue(s_addr + 32, sr[1]);
           tmem_ld_wait();
-          if (shaped) {
+          if (shaped && dist_row == nullptr) {
+            const uint64_t scale2 = pack2(row_scale, row_scale);
+#pragma unroll
+            for (int c = 0; c < 2; ++c)
+#pragma unroll
+              for (int i = 0; i < 32; i += 2) {
+                float v0, v1;
+                unpack2(mul2(pack2(__uint_as_float(sr[c][i]), __uint_as_float(sr[c][i + 1])), scale2), v0, v1);
+                sr[c][i] = __float_as_uint(v0); sr[c][i + 1] = __float_as_uint(v1);
+              }
+          } else if (shaped) {
             const int back0 = pos - key0;                        // how far back this thread's first key lies
             const int last_col = p.n_dist - 1;
 #pragma unroll
@@ -368,11 +413,11 @@ __global__ void __launch_bounds__(THREADS, 1) attn_tcgen05_kernel(const __grid_c
 #pragma unroll
               for (int i = 0; i < 32; ++i) {
                 float v = __uint_as_float(sr[c][i]) * row_scale;
-                if (dist_row != nullptr) v = fmaf(__ldg(dist_row + min(max(back0 - (c * 32 + i), 0), last_col)), LOG2E, v);
-                if (capped) v = fmaf(cap2, fast_rcp(1.f + fast_exp2(v * cap_exp)), p.score_cap_log2);
+                v = fmaf(__ldg(dist_row + min(max(back0 - (c * 32 + i), 0), last_col)), bias_unit, v);
                 sr[c][i] = __float_as_uint(v);
               }
           }
+          if (capped) tanh_scores(sr);
           // masking is a loop of its own behind a branch that the whole block takes or not: only the last
           // tile of an item has keys to hide
           if (need_mask) {

@@ -24,11 +24,13 @@
 //                                                                    at once)
 //
 // The columns of S evolve independently of one another, so the scan is parallel over (entry, head, value column) and
-// serial over an entry's tokens: a warp holds 8 columns x 4 lanes that share the key channels; a thread keeps its
-// KPT = ceil(key size / 4) state elements in registers from the entry's first token to its last, the per-token
-// vectors pass through shared memory in chunks that are fetched (cp.async) while the chunk before is computed, and
-// the two dot products of a token are two shuffles each.  A step of single tokens is the same kernel with one token
-// an entry: it then reads and writes the state once, which is all its traffic.
+// serial over an entry's tokens; a thread keeps its state elements in registers from the entry's first token to its last,
+// and the per-token vectors pass through shared memory in chunks that are fetched (cp.async) while the chunk before is
+// computed.  With the removal term (state_scan_kernel) a warp holds 8 columns x 4 lanes that share the key channels, and
+// the two dot products of a token are two shuffles each.  Without it (column_scan_kernel) a thread holds a block of the
+// state, a part of the key channels x 4 columns, so that what it reads of the vectors serves four columns, in packed
+// pairs of channels; 8 or 16 lanes share the channels and sum the four outputs in four or five shuffles.  A step of single tokens is the
+// same kernel with one token an entry: it then reads and writes the state once, which is all its traffic.
 //
 // jv_head_norm_gate finishes all: each head's output divided by its root mean square, times a weight per element (of all
 // heads, or one vector that the heads share), times sigmoid(gate) or silu(gate), rounded for the output product.
@@ -207,7 +209,8 @@ struct ScanParams {
   // blockIdx.x is a segment's number.  The columns of a segment's buffer, [D][v_tot] floats at (segment * heads +
   // head) * D * v_tot: the V value columns, the normaliser's (if any), then what the segment does to a state that
   // comes in: with the removal term D columns that start as the identity and take no value (the product of the
-  // tokens' transitions), without it one column that starts as ones (the product of the decays, channel by channel).
+  // tokens' transitions), without it one column that starts as ones (the product of the decays, channel by channel), and
+  // padding up to a multiple of four columns.
   //   mode 1  every segment but an entry's last runs from a zero state and writes its buffer in seg_local; no output
   //   (then scan_combine_kernel chains them: seg_start[s + 1] = transition(s) seg_start[s] + local(s))
   //   mode 2  every segment runs from seg_start (an entry's first: from the state) and writes the outputs; an entry's
@@ -230,7 +233,7 @@ __device__ __forceinline__ bool find_segment(const int* __restrict__ cu_seqlens,
   return false;
 }
 
-constexpr int SCAN_THREADS = 128;    // 4 warps of 8 columns x 4 key lanes
+constexpr int SCAN_THREADS = 128;    // with the removal term: 4 warps of 8 columns x 4 key lanes
 constexpr int SCAN_COLS = 32;
 
 template <int KPT> struct ScanShape {
@@ -249,9 +252,9 @@ __device__ __forceinline__ void cp_async_16(float* dst, const float* src) {
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-template <int KPT, bool REMOVAL, typename T>
+template <int KPT, typename T>
 __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanParams p) {
-  constexpr int NV = REMOVAL ? 5 : 3;
+  constexpr int NV = 5;
   constexpr int ROW = ScanShape<KPT>::ROW, CHUNK = ScanShape<KPT>::CHUNK;
   extern __shared__ __align__(16) float smem[];       // [2][CHUNK][NV][ROW]
   pdl_trigger();
@@ -275,15 +278,11 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanPara
     return;
   }
   if (t0 >= t1) return;
-  const bool is_n = !REMOVAL && p.state_n != nullptr && col == V;
-  const int v_n = V + ((!REMOVAL && p.state_n != nullptr) ? 1 : 0);   // columns that belong to the state
-  const int tcol = col - v_n;                          // mode 1: which column of the transition this thread carries
+  const int tcol = col - V;                            // mode 1: which column of the transition this thread carries
   const bool is_t = p.mode == 1 && tcol >= 0 && col < p.v_tot;
-  const bool live = col < V || is_n || is_t;
-  // element kk of this thread's column: S_g[kk * S_step] in the state, B_g[kk * v_tot] in a segment's buffer
-  float* S_g = is_n ? p.state_n + (size_t)slot * p.slot_stride + (size_t)h * D
-                    : p.state + (size_t)slot * p.slot_stride + (size_t)h * D * V + col;
-  const size_t S_step = is_n ? 1 : V;
+  const bool live = col < V || is_t;
+  // element kk of this thread's column: S_g[kk * V] in the state, B_g[kk * v_tot] in a segment's buffer
+  float* S_g = p.state + (size_t)slot * p.slot_stride + (size_t)h * D * V + col;
   const size_t B_off = ((size_t)blockIdx.x * p.heads + h) * D * p.v_tot + col;
   const bool from_state = p.mode == 0 || (p.mode == 2 && seg == 0);
   const bool to_state = p.mode == 0 || (p.mode == 2 && seg == n_seg - 1);
@@ -293,8 +292,8 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanPara
     const int kk = kl * KPT + i;
     float s0 = 0.f;
     if (live && kk < D) {
-      if (p.mode == 1) s0 = is_t ? ((REMOVAL ? kk == tcol : true) ? 1.f : 0.f) : 0.f;
-      else s0 = from_state ? S_g[(size_t)kk * S_step] : p.seg_start[B_off + (size_t)kk * p.v_tot];
+      if (p.mode == 1) s0 = is_t && kk == tcol ? 1.f : 0.f;
+      else s0 = from_state ? S_g[(size_t)kk * V] : p.seg_start[B_off + (size_t)kk * p.v_tot];
     }
     S[i] = s0;
   }
@@ -332,7 +331,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanPara
   auto fetch_v = [&](float* dst, int first) {
 #pragma unroll
     for (int t = 0; t < CHUNK; ++t)
-      dst[t] = is_n ? 1.f : (col < V && first + t < t1) ? to_f32(vsrc[(size_t)(first + t) * p.v_stride]) : 0.f;
+      dst[t] = (col < V && first + t < t1) ? to_f32(vsrc[(size_t)(first + t) * p.v_stride]) : 0.f;
   };
   stage(0, t0);
   fetch_v(vr, t0);
@@ -349,16 +348,14 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanPara
     auto token = [&](const int t, const float v) {
       const float* vec = smem + (size_t)(buf * CHUNK + t) * NV * ROW + kl * (KPT + 4);
       float dot = 0.f;
-      if (REMOVAL) {
 #pragma unroll
-        for (int i = 0; i < KPT; i += 4) {
-          const float4 u = *reinterpret_cast<const float4*>(vec + 3 * ROW + i);
-          dot = fmaf(u.x, S[i], dot); dot = fmaf(u.y, S[i + 1], dot);
-          dot = fmaf(u.z, S[i + 2], dot); dot = fmaf(u.w, S[i + 3], dot);
-        }
-        dot += __shfl_xor_sync(0xffffffffu, dot, 8);
-        dot += __shfl_xor_sync(0xffffffffu, dot, 16);
+      for (int i = 0; i < KPT; i += 4) {
+        const float4 u = *reinterpret_cast<const float4*>(vec + 3 * ROW + i);
+        dot = fmaf(u.x, S[i], dot); dot = fmaf(u.y, S[i + 1], dot);
+        dot = fmaf(u.z, S[i + 2], dot); dot = fmaf(u.w, S[i + 3], dot);
       }
+      dot += __shfl_xor_sync(0xffffffffu, dot, 8);
+      dot += __shfl_xor_sync(0xffffffffu, dot, 16);
       float o = 0.f;
 #pragma unroll
       for (int i = 0; i < KPT; i += 4) {
@@ -367,25 +364,19 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanPara
         const float4 w = *reinterpret_cast<const float4*>(vec + 2 * ROW + i);
         float s0 = fmaf(k.x, v, w.x * S[i]), s1 = fmaf(k.y, v, w.y * S[i + 1]);
         float s2 = fmaf(k.z, v, w.z * S[i + 2]), s3 = fmaf(k.w, v, w.w * S[i + 3]);
-        if (REMOVAL) {
-          const float4 b = *reinterpret_cast<const float4*>(vec + 4 * ROW + i);
-          s0 = fmaf(-b.x, dot, s0); s1 = fmaf(-b.y, dot, s1); s2 = fmaf(-b.z, dot, s2); s3 = fmaf(-b.w, dot, s3);
-        }
+        const float4 b = *reinterpret_cast<const float4*>(vec + 4 * ROW + i);
+        s0 = fmaf(-b.x, dot, s0); s1 = fmaf(-b.y, dot, s1); s2 = fmaf(-b.z, dot, s2); s3 = fmaf(-b.w, dot, s3);
         S[i] = s0; S[i + 1] = s1; S[i + 2] = s2; S[i + 3] = s3;
         o = fmaf(r.x, s0, o); o = fmaf(r.y, s1, o); o = fmaf(r.z, s2, o); o = fmaf(r.w, s3, o);
       }
       o += __shfl_xor_sync(0xffffffffu, o, 8);
       o += __shfl_xor_sync(0xffffffffu, o, 16);
-      if (kl == 0 && live && p.mode != 1) {
-        if (is_n) p.nq[((size_t)(first + t) * p.heads + h) * p.nq_stride] = o;
-        else p.out[(size_t)(first + t) * p.heads * V + (size_t)h * V + col] = o;
-      }
+      if (kl == 0 && live && p.mode != 1) p.out[(size_t)(first + t) * p.heads * V + (size_t)h * V + col] = o;
     };
-    if (REMOVAL && tokens == CHUNK) {
-      // with the removal term a token is a long chain of dependent steps (dot, two shuffles, update, dot, two shuffles):
+    if (tokens == CHUNK) {
+      // a token is a long chain of dependent steps (dot, two shuffles, update, dot, two shuffles):
       // a whole stage is unrolled, so that the reduction and the store of a token's output run under the next token's
-      // first dot product (measured: 1,024 -> 936 us for 2,048 tokens of 32 heads of 64).  Without the term the unrolled
-      // form needs 254 registers where the loop needs 168, and two blocks a multiprocessor are slower than three.
+      // first dot product (measured: 1,024 -> 936 us for 2,048 tokens of 32 heads of 64)
 #pragma unroll
       for (int t = 0; t < CHUNK; ++t) token(t, vr[t]);
     } else {
@@ -399,8 +390,209 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanPara
     const int kk = kl * KPT + i;
     if (live && kk < D) {
       if (p.mode == 1) p.seg_local[B_off + (size_t)kk * p.v_tot] = S[i];
-      else if (to_state) S_g[(size_t)kk * S_step] = S[i];
+      else if (to_state) S_g[(size_t)kk * V] = S[i];
     }
+  }
+}
+
+// Without the removal term.  A warp is LANES (8 or 16) key lanes, of KPT channels each, x 32 / LANES groups of 4 columns; a
+// block of 4 warps covers COLS columns; a warp whose columns are all unused only helps to stage.
+template <int LANES, int KPT> struct ColumnScanShape {
+  static constexpr int CHUNK = 8;                              // tokens per stage
+  static constexpr int WARP_COLS = 32 / LANES * 4, COLS = 4 * WARP_COLS;
+  static constexpr int ROW = LANES * (KPT + 4);                // floats of a vector in shared memory
+  static constexpr int SMEM = (int)sizeof(float) * 2 * CHUNK * (3 * ROW + COLS);
+};
+
+template <int LANES, int KPT, typename T>
+__global__ void __launch_bounds__(SCAN_THREADS) column_scan_kernel(const ScanParams p) {
+  using Shape = ColumnScanShape<LANES, KPT>;
+  constexpr int ROW = Shape::ROW, CHUNK = Shape::CHUNK, COLS = Shape::COLS, NV = 3;
+  extern __shared__ __align__(16) float smem[];       // [2][CHUNK][NV][ROW] vectors, [2][CHUNK][COLS] values
+  float* vals = smem + 2 * CHUNK * NV * ROW;
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int kl = lane % LANES, k0 = kl * KPT;          // this lane's key channels
+  const int base = blockIdx.z * COLS, lcol = warp * Shape::WARP_COLS + lane / LANES * 4, col = base + lcol;   // its first column
+  const int D = p.D, V = p.V;
+  int entry = blockIdx.x, seg = 0, n_seg = 1;
+  if (p.mode != 0 && !find_segment(p.cu_seqlens, p.n_entries, p.seg_len, blockIdx.x, entry, seg, n_seg)) return;
+  if (p.mode == 1 && seg == n_seg - 1) return;         // nothing follows an entry's last segment
+  int t0 = p.cu_seqlens[entry], t1 = p.cu_seqlens[entry + 1];
+  if (p.mode != 0) {
+    t0 += seg * p.seg_len;
+    t1 = min(t1, t0 + p.seg_len);
+  }
+  const int slot = p.slots[entry];
+  if (slot < 0 || slot >= p.n_slots) {
+    if (tid == 0) atomicOr(p.status, JV_STATUS_BAD_ROW);
+    return;
+  }
+  if (t0 >= t1) return;
+  const int v_n = V + (p.state_n != nullptr ? 1 : 0);  // columns that belong to the state; in mode 1 the next one carries
+  const int used = p.mode == 1 ? v_n + 1 : v_n;        // the product of the decays
+  const bool at_work = base + warp * Shape::WARP_COLS < used;        // some column of this warp is used (the same for the whole warp)
+  float* S_g = p.state + (size_t)slot * p.slot_stride + (size_t)h * D * V + col;
+  float* N_g = p.state_n != nullptr ? p.state_n + (size_t)slot * p.slot_stride + (size_t)h * D : nullptr;
+  const size_t B_off = ((size_t)blockIdx.x * p.heads + h) * D * p.v_tot + col;      // rows of v_tot, a multiple of 4
+  const bool state_vec = (V & 3) == 0 && ((uintptr_t)S_g & 15) == 0 && (p.slot_stride & 3) == 0;
+  const bool from_state = p.mode == 0 || (p.mode == 2 && seg == 0);
+  const bool to_state = p.mode == 0 || (p.mode == 2 && seg == n_seg - 1);
+  auto read4 = [&](int kk) -> float4 {                 // this thread's columns of channel kk before the first token
+    float e[4] = {0.f, 0.f, 0.f, 0.f};
+    if (kk < D && col < used) {
+      if (p.mode == 1) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) e[c] = col + c == v_n ? 1.f : 0.f;
+      } else if (!from_state) {
+        return *reinterpret_cast<const float4*>(p.seg_start + B_off + (size_t)kk * p.v_tot);
+      } else if (state_vec && col < V) {
+        return *reinterpret_cast<const float4*>(S_g + (size_t)kk * V);
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) e[c] = col + c < V ? S_g[(size_t)kk * V + c] : col + c < v_n ? N_g[kk] : 0.f;
+      }
+    }
+    return make_float4(e[0], e[1], e[2], e[3]);
+  };
+  auto write4 = [&](int kk, const float4& s) {
+    if (kk >= D || col >= used) return;
+    if (p.mode == 1) {
+      *reinterpret_cast<float4*>(p.seg_local + B_off + (size_t)kk * p.v_tot) = s;
+    } else if (to_state) {
+      if (state_vec && col < V) {
+        *reinterpret_cast<float4*>(S_g + (size_t)kk * V) = s;
+      } else {
+        const float e[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          if (col + c < V) S_g[(size_t)kk * V + c] = e[c];
+          else if (col + c < v_n) N_g[kk] = e[c];
+        }
+      }
+    }
+  };
+  uint64_t S[KPT / 2][4];                              // pairs of channels (k0 + 2 i, k0 + 2 i + 1) x columns
+#pragma unroll
+  for (int i = 0; i < KPT / 2; ++i) {
+    const float4 a = read4(k0 + 2 * i), b = read4(k0 + 2 * i + 1);
+    S[i][0] = pack2(a.x, b.x); S[i][1] = pack2(a.y, b.y); S[i][2] = pack2(a.z, b.z); S[i][3] = pack2(a.w, b.w);
+  }
+  for (int i = tid; i < 2 * CHUNK * NV * ROW; i += SCAN_THREADS) smem[i] = 0.f;     // the padding stays zero
+  __syncthreads();
+
+  auto stage = [&](int buf, int first) {
+    const int tokens = min(CHUNK, t1 - first), per_token = NV * D;
+    if ((D & 3) == 0) {                                // 16 bytes a copy: PIECES threads a vector, AT_ONCE vectors
+      constexpr int PIECES = LANES * KPT / 4, AT_ONCE = SCAN_THREADS / PIECES;
+      const int kk = (tid % PIECES) * 4, sub = tid / PIECES;
+      if (kk < D) {
+        float* dst = smem + (size_t)buf * CHUNK * NV * ROW + (kk / KPT) * (KPT + 4) + kk % KPT;
+        const float* src = p.packed + ((size_t)first * p.heads + h) * per_token + kk;
+        for (int tv = sub; tv < tokens * NV; tv += AT_ONCE)
+          cp_async_16(dst + tv * ROW, src + (size_t)(tv / NV) * p.heads * per_token + (tv % NV) * D);
+      }
+    } else {
+      for (int tv = 0; tv < tokens * NV; ++tv) {
+        float* row = smem + (size_t)(buf * CHUNK * NV + tv) * ROW;
+        const float* src = p.packed + ((size_t)(first + tv / NV) * p.heads + h) * per_token + (tv % NV) * D;
+        for (int kk = tid; kk < D; kk += SCAN_THREADS) cp_async_4(row + (kk / KPT) * (KPT + 4) + kk % KPT, src + kk);
+      }
+    }
+    cp_async_commit();
+  };
+  // the block's values of a chunk: asked for a chunk ahead, put into shared memory when the chunk begins
+  constexpr int VPT = CHUNK * COLS / SCAN_THREADS;
+  const int vcol = tid % COLS, vtok = tid / COLS;          // token vtok + 2 i
+  const T* vsrc = (const T*)p.v + p.v_off + (size_t)h * V + (base + vcol < V ? base + vcol : 0);
+  const float v_else = base + vcol == V && p.state_n != nullptr ? 1.f : 0.f;
+  float vr[VPT];
+  auto fetch_v = [&](int first) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int t = first + vtok + i * (SCAN_THREADS / COLS);
+      vr[i] = base + vcol < V && t < t1 ? to_f32(vsrc[(size_t)t * p.v_stride]) : v_else;
+    }
+  };
+  stage(0, t0);
+  fetch_v(t0);
+  int buf = 0;
+  for (int first = t0; first < t1; first += CHUNK, buf ^= 1) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i)
+      vals[(buf * CHUNK + vtok + i * (SCAN_THREADS / COLS)) * COLS + vcol] = vr[i];
+    cp_async_wait_all();
+    __syncthreads();                                   // this chunk has landed; the other buffers are free
+    if (first + CHUNK < t1) {
+      stage(buf ^ 1, first + CHUNK);
+      fetch_v(first + CHUNK);
+    }
+    if (!at_work) continue;
+    const int tokens = min(CHUNK, t1 - first);
+    if (p.mode == 1) {
+      for (int t = 0; t < tokens; ++t) {
+        const float* vec = smem + (size_t)(buf * CHUNK + t) * NV * ROW + kl * (KPT + 4);
+        const float4 v = *reinterpret_cast<const float4*>(vals + (buf * CHUNK + t) * COLS + lcol);
+        const uint64_t vv[4] = {pack2(v.x, v.x), pack2(v.y, v.y), pack2(v.z, v.z), pack2(v.w, v.w)};
+#pragma unroll
+        for (int i = 0; i < KPT; i += 4) {
+          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(vec + ROW + i);
+          const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(vec + 2 * ROW + i);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            S[i / 2][c] = fma2(k.x, vv[c], mul2(w.x, S[i / 2][c]));
+            S[i / 2 + 1][c] = fma2(k.y, vv[c], mul2(w.y, S[i / 2 + 1][c]));
+          }
+        }
+      }
+      continue;
+    }
+    for (int t = 0; t < tokens; ++t) {
+      const float* vec = smem + (size_t)(buf * CHUNK + t) * NV * ROW + kl * (KPT + 4);
+      const float4 v = *reinterpret_cast<const float4*>(vals + (buf * CHUNK + t) * COLS + lcol);
+      const uint64_t vv[4] = {pack2(v.x, v.x), pack2(v.y, v.y), pack2(v.z, v.z), pack2(v.w, v.w)};
+      uint64_t o2[4] = {0, 0, 0, 0};                   // pairs of zeros
+#pragma unroll
+      for (int i = 0; i < KPT; i += 4) {
+        const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(vec + i);
+        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(vec + ROW + i);
+        const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(vec + 2 * ROW + i);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          S[i / 2][c] = fma2(k.x, vv[c], mul2(w.x, S[i / 2][c]));
+          o2[c] = fma2(r.x, S[i / 2][c], o2[c]);
+          S[i / 2 + 1][c] = fma2(k.y, vv[c], mul2(w.y, S[i / 2 + 1][c]));
+          o2[c] = fma2(r.y, S[i / 2 + 1][c], o2[c]);
+        }
+      }
+      // the sums over the key lanes: in the first two steps a lane hands on the columns that it does not finish
+      float o[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        float lo, hi;
+        unpack2(o2[c], lo, hi);
+        o[c] = lo + hi;
+      }
+      const bool up = kl & (LANES / 2), up2 = kl & (LANES / 4);
+      const float a0 = (up ? o[2] : o[0]) + __shfl_xor_sync(0xffffffffu, up ? o[0] : o[2], LANES / 2);
+      const float a1 = (up ? o[3] : o[1]) + __shfl_xor_sync(0xffffffffu, up ? o[1] : o[3], LANES / 2);
+      float b = (up2 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, up2 ? a0 : a1, LANES / 4);
+#pragma unroll
+      for (int x = LANES / 8; x > 0; x >>= 1) b += __shfl_xor_sync(0xffffffffu, b, x);
+      const int mine = col + (up ? 2 : 0) + (up2 ? 1 : 0);
+      if (kl % (LANES / 4) == 0) {
+        if (mine < V) p.out[(size_t)(first + t) * p.heads * V + (size_t)h * V + mine] = b;
+        else if (mine < v_n) p.nq[((size_t)(first + t) * p.heads + h) * p.nq_stride] = b;
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < KPT / 2; ++i) {
+    float4 a, b;
+    unpack2(S[i][0], a.x, b.x); unpack2(S[i][1], a.y, b.y); unpack2(S[i][2], a.z, b.z); unpack2(S[i][3], a.w, b.w);
+    write4(k0 + 2 * i, a);
+    write4(k0 + 2 * i + 1, b);
   }
 }
 
@@ -517,49 +709,75 @@ __global__ void __launch_bounds__(128) scan_combine_kernel(const ScanParams p) {
   }
 }
 
-template <int KPT, bool REMOVAL, typename T>
-int launch_scan(const ScanParams& p, int entries, cudaStream_t stream) {
-  constexpr int NV = REMOVAL ? 5 : 3;
-  const size_t smem = sizeof(float) * 2 * ScanShape<KPT>::CHUNK * NV * ScanShape<KPT>::ROW;
-  auto kern = state_scan_kernel<KPT, REMOVAL, T>;
-  static bool done[JV_MAX_DEVICES] = {};
-  if (!jv_once_per_device(done, [&] {
-        return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess;
-      }))
-    return JV_ERR_UNSUPPORTED;
-  const int cols = p.V + ((!REMOVAL && p.state_n != nullptr) ? 1 : 0);
+// All three modes of a scan kernel: whole entries in one launch, or segments, the chain of their states, segments again.
+// `combine` launches the chain; `cols` are the columns of the state, `block_cols` those of a block.
+template <typename K, typename F>
+int launch_scan(K kern, size_t smem, int block_cols, int cols, int seg_cols, const ScanParams& p, int entries,
+                cudaStream_t stream, F&& combine) {
   if (p.mode == 0)
-    return jv_launch(kern, dim3(entries, p.heads, (cols + SCAN_COLS - 1) / SCAN_COLS), dim3(SCAN_THREADS), smem, stream, p);
+    return jv_launch(kern, dim3(entries, p.heads, (cols + block_cols - 1) / block_cols), dim3(SCAN_THREADS), smem, stream, p);
   // in segments: `entries` is then the largest number of segments there can be
   ScanParams q = p;
   q.mode = 1;
-  int rc = jv_launch(kern, dim3(entries, p.heads, (p.v_tot + SCAN_COLS - 1) / SCAN_COLS), dim3(SCAN_THREADS), smem, stream, q);
+  int rc = jv_launch(kern, dim3(entries, p.heads, (seg_cols + block_cols - 1) / block_cols), dim3(SCAN_THREADS), smem, stream, q);
   if (rc != JV_OK) return rc;
-  if (REMOVAL) {
+  rc = combine(q);
+  if (rc != JV_OK) return rc;
+  q.mode = 2;
+  return jv_launch(kern, dim3(entries, p.heads, (cols + block_cols - 1) / block_cols), dim3(SCAN_THREADS), smem, stream, q);
+}
+
+template <int KPT, typename T>
+int launch_removal_scan(const ScanParams& p, int entries, cudaStream_t stream) {
+  const size_t smem = sizeof(float) * 2 * ScanShape<KPT>::CHUNK * 5 * ScanShape<KPT>::ROW;
+  static bool done[JV_MAX_DEVICES] = {};
+  if (!jv_once_per_device(done, [&] {
+        return cudaFuncSetAttribute(state_scan_kernel<KPT, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) == cudaSuccess;
+      }))
+    return JV_ERR_UNSUPPORTED;
+  return launch_scan(state_scan_kernel<KPT, T>, smem, SCAN_COLS, p.V, p.v_tot, p, entries, stream, [&](const ScanParams& q) {
     const size_t csmem = sizeof(float) * ((size_t)p.D * 64 + (size_t)p.D * (((p.D + 3) & ~3) + 4));
-    if (csmem > 200 * 1024) return JV_ERR_UNSUPPORTED;
+    if (csmem > 200 * 1024) return (int)JV_ERR_UNSUPPORTED;
     static bool cdone[JV_MAX_DEVICES] = {};
     if (!jv_once_per_device(cdone, [&] {
           return cudaFuncSetAttribute(scan_combine_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) == cudaSuccess;
         }))
-      return JV_ERR_UNSUPPORTED;
-    rc = jv_launch(scan_combine_kernel, dim3(p.n_entries, p.heads, (cols + 31) / 32), dim3(128), csmem, stream, q);
-  } else {
-    rc = jv_launch(scan_combine_diag_kernel, dim3(p.n_entries, p.heads, (p.D * cols + 127) / 128), dim3(128), 0, stream, q);
-  }
-  if (rc != JV_OK) return rc;
-  q.mode = 2;
-  return jv_launch(kern, dim3(entries, p.heads, (cols + SCAN_COLS - 1) / SCAN_COLS), dim3(SCAN_THREADS), smem, stream, q);
+      return (int)JV_ERR_UNSUPPORTED;
+    return jv_launch(scan_combine_kernel, dim3(p.n_entries, p.heads, (p.V + 31) / 32), dim3(128), csmem, stream, q);
+  });
 }
 
-template <bool REMOVAL, typename T>
-int dispatch_scan(const ScanParams& p, int entries, cudaStream_t stream) {
-  const int kpt = (p.D + 3) / 4;
-  if (kpt <= 4) return launch_scan<4, REMOVAL, T>(p, entries, stream);
-  if (kpt <= 8) return launch_scan<8, REMOVAL, T>(p, entries, stream);
-  if (kpt <= 16) return launch_scan<16, REMOVAL, T>(p, entries, stream);
-  if (kpt <= 32) return launch_scan<32, REMOVAL, T>(p, entries, stream);
-  if (kpt <= 64) return launch_scan<64, REMOVAL, T>(p, entries, stream);
+template <int LANES, int KPT, typename T>
+int launch_column_scan(const ScanParams& p, int entries, cudaStream_t stream) {
+  using Shape = ColumnScanShape<LANES, KPT>;
+  constexpr int smem = Shape::SMEM;
+  auto kern = column_scan_kernel<LANES, KPT, T>;
+  static bool done[JV_MAX_DEVICES] = {};
+  if (!jv_once_per_device(done, [&] {
+        return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) == cudaSuccess;
+      }))
+    return JV_ERR_UNSUPPORTED;
+  const int cols = p.V + (p.state_n != nullptr ? 1 : 0);
+  return launch_scan(kern, smem, Shape::COLS, cols, cols + 1, p, entries, stream, [&](const ScanParams& q) {
+    return jv_launch(scan_combine_diag_kernel, dim3(p.n_entries, p.heads, (p.D * cols + 127) / 128), dim3(128), 0, stream, q);
+  });
+}
+
+template <typename T>
+int dispatch_scan(const ScanParams& p, bool removal, int entries, cudaStream_t stream) {
+  if (removal) {
+    const int kpt = (p.D + 3) / 4;
+    if (kpt <= 4) return launch_removal_scan<4, T>(p, entries, stream);
+    if (kpt <= 8) return launch_removal_scan<8, T>(p, entries, stream);
+    if (kpt <= 16) return launch_removal_scan<16, T>(p, entries, stream);
+    if (kpt <= 32) return launch_removal_scan<32, T>(p, entries, stream);
+    if (kpt <= 64) return launch_removal_scan<64, T>(p, entries, stream);
+    return JV_ERR_UNSUPPORTED;
+  }
+  if (p.D <= 32) return launch_column_scan<8, 4, T>(p, entries, stream);
+  if (p.D <= 64) return launch_column_scan<8, 8, T>(p, entries, stream);
+  if (p.D <= 128) return launch_column_scan<8, 16, T>(p, entries, stream);
+  if (p.D <= 256) return launch_column_scan<16, 16, T>(p, entries, stream);
   return JV_ERR_UNSUPPORTED;
 }
 
@@ -651,8 +869,8 @@ JV_EXPORT int jv_memory_gates(const void* proj, int dtype, long long stride, int
 // state_n (or null; without removal only): [slots][heads * D], rows `slot_stride` apart, the state of one more column
 // whose value is 1 at every token; its outputs go to nq[(token * heads + head) * nq_stride].
 // seg_len > 0: entries longer than seg_len tokens run in segments of that many, side by side (see ScanParams): three
-// launches; seg_local and seg_start hold max_segments * heads * D * (V + (state_n ? 1 : 0) + (removal ? D : 1)) floats
-// each, and max_segments is at least the number of segments of all entries together.
+// launches; seg_local and seg_start hold max_segments * heads * D * v_tot floats each (16-byte aligned), v_tot = V + D with
+// removal, else V + (state_n ? 1 : 0) + 1 rounded up to a multiple of 4, and max_segments is at least the number of segments of all entries together.
 JV_EXPORT int jv_state_scan(const float* packed, int removal, const void* v, int dtype, long long v_stride, int v_off,
                             float* out, float* state, long long slot_stride, const int* cu_seqlens, const int* slots,
                             int n_slots, int entries, int heads, int D, int V, float* state_n, float* nq, int nq_stride,
@@ -664,14 +882,14 @@ JV_EXPORT int jv_state_scan(const float* packed, int removal, const void* v, int
     return JV_ERR_UNSUPPORTED;
   ScanParams p;
   p.mode = seg_len > 0 ? 1 : 0; p.seg_len = seg_len; p.n_entries = entries; p.seg_local = seg_local; p.seg_start = seg_start;
-  p.v_tot = V + (state_n != nullptr ? 1 : 0) + (removal ? D : 1);
+  p.v_tot = removal ? V + D : (V + (state_n != nullptr ? 1 : 0) + 1 + 3) / 4 * 4;
   if (seg_len > 0) entries = max_segments;
   p.state_n = state_n; p.nq = nq; p.nq_stride = nq_stride;
   p.packed = packed; p.v = v; p.v_stride = v_stride; p.v_off = v_off; p.out = out; p.state = state;
   p.slot_stride = slot_stride; p.cu_seqlens = cu_seqlens; p.slots = slots; p.n_slots = n_slots; p.heads = heads;
   p.D = D; p.V = V; p.status = status;
   JV_DISPATCH_DTYPE(dtype, T, {
-    return removal ? dispatch_scan<true, T>(p, entries, stream) : dispatch_scan<false, T>(p, entries, stream);
+    return dispatch_scan<T>(p, removal != 0, entries, stream);
   });
   return JV_ERR_UNSUPPORTED;
 }

@@ -1740,7 +1740,7 @@ def state_scan(packed: torch.Tensor, v: torch.Tensor, v_off: int, state: torch.T
     max_segments, seg_local, seg_start = 0, None, None
     if segment > 0:
         max_segments = n // segment + n_entries
-        v_tot = value_dim + (1 if state_n is not None else 0) + (dim if nv == 5 else 1)
+        v_tot = value_dim + dim if nv == 5 else -(-(value_dim + (1 if state_n is not None else 0) + 1) // 4) * 4
         seg_local = torch.empty((2, max_segments, heads, dim, v_tot), dtype=torch.float32, device=packed.device)
         seg_start = seg_local[1]
     f = _fn("recurrent", "jv_state_scan", [c_void_p, c_int, c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p,
