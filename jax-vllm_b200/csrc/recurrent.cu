@@ -297,8 +297,10 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(const ScanPara
     }
     S[i] = s0;
   }
-  for (int i = tid; i < 2 * CHUNK * NV * ROW; i += SCAN_THREADS) smem[i] = 0.f;     // the padding stays zero
-  __syncthreads();
+  if (D != 4 * KPT) {                                  // channels beyond D stay zero
+    for (int i = tid; i < 2 * CHUNK * NV * ROW; i += SCAN_THREADS) smem[i] = 0.f;
+    __syncthreads();
+  }
 
   const T* vsrc = (const T*)p.v + p.v_off + (size_t)h * V + (col < V ? col : 0);
   auto stage = [&](int buf, int first) {
@@ -405,7 +407,7 @@ template <int LANES, int KPT> struct ColumnScanShape {
 };
 
 template <int LANES, int KPT, typename T>
-__global__ void __launch_bounds__(SCAN_THREADS) column_scan_kernel(const ScanParams p) {
+__global__ void __launch_bounds__(SCAN_THREADS, KPT >= 16 ? 3 : 4) column_scan_kernel(const ScanParams p) {
   using Shape = ColumnScanShape<LANES, KPT>;
   constexpr int ROW = Shape::ROW, CHUNK = Shape::CHUNK, COLS = Shape::COLS, NV = 3;
   extern __shared__ __align__(16) float smem[];       // [2][CHUNK][NV][ROW] vectors, [2][CHUNK][COLS] values
@@ -473,15 +475,6 @@ __global__ void __launch_bounds__(SCAN_THREADS) column_scan_kernel(const ScanPar
       }
     }
   };
-  uint64_t S[KPT / 2][4];                              // pairs of channels (k0 + 2 i, k0 + 2 i + 1) x columns
-#pragma unroll
-  for (int i = 0; i < KPT / 2; ++i) {
-    const float4 a = read4(k0 + 2 * i), b = read4(k0 + 2 * i + 1);
-    S[i][0] = pack2(a.x, b.x); S[i][1] = pack2(a.y, b.y); S[i][2] = pack2(a.z, b.z); S[i][3] = pack2(a.w, b.w);
-  }
-  for (int i = tid; i < 2 * CHUNK * NV * ROW; i += SCAN_THREADS) smem[i] = 0.f;     // the padding stays zero
-  __syncthreads();
-
   auto stage = [&](int buf, int first) {
     const int tokens = min(CHUNK, t1 - first), per_token = NV * D;
     if ((D & 3) == 0) {                                // 16 bytes a copy: PIECES threads a vector, AT_ONCE vectors
@@ -515,8 +508,18 @@ __global__ void __launch_bounds__(SCAN_THREADS) column_scan_kernel(const ScanPar
       vr[i] = base + vcol < V && t < t1 ? to_f32(vsrc[(size_t)t * p.v_stride]) : v_else;
     }
   };
+  if (D != LANES * KPT) {                              // channels beyond D stay zero in the places that are used
+    for (int i = tid; i < min(2 * CHUNK, t1 - t0) * NV * ROW; i += SCAN_THREADS) smem[i] = 0.f;
+    __syncthreads();
+  }
   stage(0, t0);
   fetch_v(t0);
+  uint64_t S[KPT / 2][4];                              // pairs of channels (k0 + 2 i, k0 + 2 i + 1) x columns
+#pragma unroll
+  for (int i = 0; i < KPT / 2; ++i) {
+    const float4 a = read4(k0 + 2 * i), b = read4(k0 + 2 * i + 1);
+    S[i][0] = pack2(a.x, b.x); S[i][1] = pack2(a.y, b.y); S[i][2] = pack2(a.z, b.z); S[i][3] = pack2(a.w, b.w);
+  }
   int buf = 0;
   for (int first = t0; first < t1; first += CHUNK, buf ^= 1) {
 #pragma unroll

@@ -1697,8 +1697,24 @@ def memory_gates(proj: torch.Tensor, q_off: int, k_off: int, i_off: int, f_off: 
     return packed, gates
 
 
-SCAN_SEGMENT = 64          # tokens of a segment when long entries are scanned in segments side by side
-SCAN_SEGMENT_MEAN = 32     # ... which happens when the entries of a step have this many tokens on average, at least
+# Long entries are scanned in segments side by side (without the removal term) when a step has SCAN_MIN_TOKENS tokens and
+# SCAN_SEGMENT_MEAN an entry on average: in the longest segments that still give the device SCAN_WARPS warps, or in none
+# where whole long entries alone give it SCAN_WHOLE_WARPS (a segment's tokens are gone through twice).  Measured on 148
+# multiprocessors, 32-bit state, microseconds whole / best segment: 2,048 tokens of 8 heads of 128 x 256 (128 warps) 972 /
+# 256 (64 tokens), of 8 heads of 256 x 512 (512) 1,051 / 826 (256), of 64 heads of 128 x 64 (256) 978 / 491 (128); eight
+# such entries of the first size (1,024) 1,293 / 1,507.
+SCAN_SEGMENTS = (256, 128, 64, 32)
+SCAN_MIN_TOKENS, SCAN_SEGMENT_MEAN, SCAN_WARPS, SCAN_WHOLE_WARPS, SCAN_LONG_MEAN = 256, 32, 4096, 700, 256
+
+
+def scan_segment(n: int, n_entries: int, heads: int, dim: int, columns: int) -> int:
+    """Tokens a segment for `state_scan` without the removal term (0: whole entries)."""
+    if n < SCAN_MIN_TOKENS or n < SCAN_SEGMENT_MEAN * n_entries:
+        return 0
+    warps = heads * -(-columns // (16 if dim <= 128 else 8))          # of one entry, or of one segment
+    if n >= SCAN_LONG_MEAN * n_entries and warps * n_entries >= SCAN_WHOLE_WARPS:
+        return 0
+    return next((seg for seg in SCAN_SEGMENTS if warps * n >= SCAN_WARPS * seg), SCAN_SEGMENTS[-1])
 
 
 def state_scan(packed: torch.Tensor, v: torch.Tensor, v_off: int, state: torch.Tensor, cu_seqlens: torch.Tensor,
@@ -1711,8 +1727,8 @@ def state_scan(packed: torch.Tensor, v: torch.Tensor, v_off: int, state: torch.T
     state has one more column whose value is 1 at every token (a normaliser n <- w n + k); its output n . r goes to
     the fourth place of `gates` [n, heads, 4].
 
-    A step whose entries are long runs them in segments of `segment` tokens side by side (None: `SCAN_SEGMENT` when
-    the step has 4 segments' tokens and `SCAN_SEGMENT_MEAN` tokens an entry; 0: never): every segment first runs from
+    A step whose entries are long runs them in segments of `segment` tokens side by side (None: by `scan_segment` without
+    the removal term, never with it; 0: never): every segment first runs from
     a zero state and records what it does to a state that comes in, the segments of an entry are chained, and every
     segment runs again from its true start for the outputs.  The result differs from the token-by-token order by
     32-bit rounding only."""
@@ -1734,7 +1750,7 @@ def state_scan(packed: torch.Tensor, v: torch.Tensor, v_off: int, state: torch.T
     if segment is None:
         # with the removal term a segment carries `dim` more columns and the chain is a matrix product a segment: at
         # the sizes measured (32 heads of 64, 2,048 tokens) the three launches take longer than the one
-        segment = SCAN_SEGMENT if nv == 3 and n >= 4 * SCAN_SEGMENT and n >= SCAN_SEGMENT_MEAN * n_entries else 0
+        segment = scan_segment(n, n_entries, heads, dim, value_dim + (state_n is not None)) if nv == 3 else 0
     if nv == 5 and 4 * dim * (64 + (dim + 3) // 4 * 4 + 4) > 200 * 1024:
         segment = 0          # the kernel that chains segments keeps a [dim][dim] transition in shared memory
     max_segments, seg_local, seg_start = 0, None, None
