@@ -242,13 +242,13 @@ def test_a_window_that_keeps_the_first_tokens_on_the_attention_kernels(name, win
     assert matters >= 4, "the mask does not matter here"
 
 
-@pytest.mark.parametrize("cap", [None, 6.0])
+@pytest.mark.parametrize("cap", [None, 6.0, 60.0])
 @pytest.mark.parametrize("window,keep", [(1, 1), (72, 4), (200, 0), (200, 128), (100, 129), (150, 300), (64, 40)])
 @pytest.mark.parametrize("Hq,Hk", [(4, 2), (3, 3), (8, 1)])
 def test_a_window_that_keeps_the_first_tokens_on_the_tcgen05_prompt_kernel(Hq, Hk, window, keep, cap):
     """Whole 128-row tiles of a prompt portion on heads of 128: context whose pages before the window have been given back
     except those of the kept tokens (which end within, at and past a tile, and past the window's start), a last tile that
-    is not full, an entry of one tile from position 0; with and without a cap."""
+    is not full, an entry of one tile from position 0; without a cap, with one that scores exceed, with one far above them."""
     from jax_vllm_b200 import ops
     D, P, scale = 128, 16, 1.3 * 128 ** -0.5
     tpt = ops.attn_tcgen05_tokens_per_tile(Hq, Hk)
